@@ -640,6 +640,7 @@ PYBIND11_MODULE(_ovcore, mod) {
         .def_readwrite("tok_src", &DescLayout::tok_src).def_readwrite("tok_dst", &DescLayout::tok_dst).def_readwrite("logit_idx", &DescLayout::logit_idx)
         .def_readwrite("past_lens", &DescLayout::past_lens).def_readwrite("subsequence_begins", &DescLayout::subsequence_begins)
         .def_readwrite("block_indices_begins", &DescLayout::block_indices_begins).def_readwrite("block_indices", &DescLayout::block_indices)
+        .def_readwrite("state_slots", &DescLayout::state_slots)
         .def_readwrite("Tcap", &DescLayout::Tcap).def_readwrite("Bcap", &DescLayout::Bcap).def_readwrite("blocks_cap", &DescLayout::blocks_cap);
     py::class_<ScheduledStep>(mod, "ScheduledStep")
         .def_readonly("seqs", &ScheduledStep::seqs)

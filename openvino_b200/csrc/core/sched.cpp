@@ -239,6 +239,7 @@ void Scheduler::fill(const ScheduledStep& st, int32_t* d, const DescLayout& lay,
         if (!host_ids && !s.generated.empty() && ends_on_last) d[lay.tok_src + t + n - 1] = (int32_t)s.slot;
         d[lay.tok_dst + (int64_t)i] = ends_on_last ? (int32_t)s.slot : -1;
         d[lay.past_lens + (int64_t)i] = (int32_t)c0;
+        if (lay.state_slots >= 0) d[lay.state_slots + (int64_t)i] = (int32_t)s.slot;
         d[lay.logit_idx + (int64_t)i] = (int32_t)(t + n - 1);
         const int64_t k = (c0 + n + bs - 1) / bs;
         if (nb + k > lay.blocks_cap) throw std::length_error("block table does not fit the descriptor buffer");

@@ -67,7 +67,7 @@ struct ScheduledStep {
 // Offsets (in int32 words) of the descriptor fields inside one packed step buffer.
 struct DescLayout {
     int64_t ids = 0, positions = 0, slot_map = 0, tok_src = 0, tok_dst = 0, logit_idx = 0, past_lens = 0, subsequence_begins = 0,
-            block_indices_begins = 0, block_indices = 0;
+            block_indices_begins = 0, block_indices = 0, state_slots = -1;   // state_slots: slot of every sequence (-1: no such field)
     int64_t Tcap = 0, Bcap = 0, blocks_cap = 0;
 };
 

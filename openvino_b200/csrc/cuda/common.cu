@@ -118,6 +118,8 @@ unsigned ovb_set_peer_spin_limit(unsigned polls) {
 #ifdef OVB_DEBUG_BOUNDS
 int ovb_debug_set_limits_attention(const ovb::DebugLimits* l);
 int ovb_debug_set_limits_elementwise(const ovb::DebugLimits* l);
+int ovb_debug_set_limits_heads(const ovb::DebugLimits* l);
+int ovb_debug_set_limits_exact(const ovb::DebugLimits* l);
 #endif
 
 int ovb_debug_bounds_enabled(void) {
@@ -135,6 +137,8 @@ int ovb_debug_set_limits(int kv_blocks, int vocab) {
     l.vocab = vocab;
     l.status = ovb::status_word();
     if (int rc = ovb_debug_set_limits_attention(&l)) return rc;
+    if (int rc = ovb_debug_set_limits_heads(&l)) return rc;
+    if (int rc = ovb_debug_set_limits_exact(&l)) return rc;
     return ovb_debug_set_limits_elementwise(&l);
 #else
     (void)kv_blocks; (void)vocab;

@@ -10,6 +10,7 @@
 #include <cuda_fp8.h>
 
 #include "common.cuh"
+#include "store_types.cuh"
 #include "debug_bounds.cuh"
 #include "sm100_ptx.cuh"
 
@@ -295,19 +296,19 @@ __global__ void scatter_tokens_kernel(const int* __restrict__ tokens, const int*
 }
 
 // ------------------------------------------------------------------------------------ argmax
-template <int THREADS>
+template <int THREADS, class E>
 __global__ void __launch_bounds__(THREADS)
-argmax_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int vocab, void* __restrict__ out_ids, int ids_i32,
+argmax_kernel(const E* __restrict__ logits, int ld, int vocab, void* __restrict__ out_ids, int ids_i32,
               float* __restrict__ out_max) {
     pdl_enter();
     __shared__ float sv[THREADS / 32];
     __shared__ int si[THREADS / 32];
     const size_t row = blockIdx.x;
-    const __nv_bfloat16* lr = logits + row * ld;
+    const E* lr = logits + row * ld;
     float best = -CUDART_INF_F;
     int bi = 0x7fffffff;
     const int nvec = vocab >> 3;
-    const bool aligned = ((reinterpret_cast<uintptr_t>(lr) & 15) == 0);
+    const bool aligned = sizeof(E) == 2 && ((reinterpret_cast<uintptr_t>(lr) & 15) == 0);
     if (aligned) {
         for (int v = threadIdx.x; v < nvec; v += THREADS) {
             Pack8 a;
@@ -319,12 +320,12 @@ argmax_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int vocab, void*
             }
         }
         for (int i = nvec * 8 + threadIdx.x; i < vocab; i += THREADS) {
-            const float f = __bfloat162float(lr[i]);
+            const float f = ld_f32(lr + i);
             if (f > best) { best = f; bi = i; }
         }
     } else {
         for (int i = threadIdx.x; i < vocab; i += THREADS) {
-            const float f = __bfloat162float(lr[i]);
+            const float f = ld_f32(lr + i);
             if (f > best) { best = f; bi = i; }
         }
     }
@@ -977,8 +978,14 @@ int ovb_argmax(const void* logits, int ld, int rows, int vocab, void* out_ids, i
                ovb_stream_t stream_) {
     cudaStream_t stream = static_cast<cudaStream_t>(stream_);
     OVB_REQUIRE(logits && out_ids && rows > 0 && vocab > 0, "ovb_argmax: bad arguments");
-    OVB_CHECK_CUDA(launch_pdl(argmax_kernel<1024>, dim3(rows), dim3(1024), 0, stream, (const __nv_bfloat16*)logits, ld, vocab, out_ids, ids_i32, out_max));
+    OVB_CHECK_CUDA(launch_pdl(argmax_kernel<1024, __nv_bfloat16>, dim3(rows), dim3(1024), 0, stream, (const __nv_bfloat16*)logits, ld, vocab, out_ids, ids_i32, out_max));
     OVB_CHECK_CUDA(cudaGetLastError());
+    return 0;
+}
+
+int ovb_argmax_f32(const float* logits, int ld, int rows, int vocab, void* out_ids, int ids_i32, float* out_max, ovb_stream_t stream) {
+    OVB_REQUIRE(logits && out_ids && rows > 0 && vocab > 0, "ovb_argmax_f32: bad arguments");
+    OVB_CHECK_CUDA(launch_pdl(argmax_kernel<1024, float>, dim3(rows), dim3(1024), 0, static_cast<cudaStream_t>(stream), logits, ld, vocab, out_ids, ids_i32, out_max));
     return 0;
 }
 

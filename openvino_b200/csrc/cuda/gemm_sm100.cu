@@ -91,7 +91,9 @@ struct GemmKParams {
     int nvls_reducers;        // in-switch all-reduce: the first CTAs of the grid only reduce (0: every tile CTA reduces its own tile)
     const int* group_off;
     int num_groups;
-    int group_mode;
+    int group_mode;           // 3: block-diagonal, no offsets (group g reads x at column g * group_ldx and writes out at column g * group_ldo)
+    int group_ldx, group_ldo;
+    float act_limit, act_slope, act_shift;   // OVB_ACT_GLU_LIMITED
 };
 
 // polls of a peer flag (~0.25 us apart) before a wait gives up: GemmKParams::spin_limit, set per launch from peer_spin_limit()
@@ -129,6 +131,13 @@ __device__ __forceinline__ float apply_act(float v, int act) {
         }
         default: return v;
     }
+}
+
+// Clamped gate and up values with a sigmoid of adjustable slope (OVB_ACT_GLU_LIMITED).
+__device__ __forceinline__ float glu_limited(const GemmKParams& p, float g, float u) {
+    g = fminf(g, p.act_limit);
+    u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
+    return g / (1.0f + __expf(-p.act_slope * g)) * (u + p.act_shift);
 }
 
 // Expand one u32 (8 packed u4 in the plugin nibble order) to 8 bf16: (q - zp) * scale.
@@ -329,6 +338,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
     }
     int n_tile, t_tile;
     int w_tile, w_kb0 = 0;          // weight tile and first k-block inside the (possibly stacked) weight
+    int x_col = 0, out_col = 0;     // first column of x / out of this CTA's group (block-diagonal product)
     int t0, T_end = p.T;            // first row of the tile, one past the last valid row
     if (p.group_off != nullptr) {
         // the offsets come from an earlier kernel of the stream: nothing of this CTA may run before that kernel is done
@@ -349,6 +359,13 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         T_end = min(end, p.T);
         w_tile = p.group_mode == 1 ? g * tiles_n + n_tile : n_tile;
         w_kb0 = p.group_mode == 2 ? g * ((p.K + TILE_K - 1) / TILE_K) : 0;
+    } else if (!QUANT && p.group_mode == 3) {
+        const int tiles_n = (p.N + TILE_N - 1) / TILE_N, per_group = tiles_n * ((p.T + BT - 1) / BT), g = cta / per_group;
+        tile_coords(cta - g * per_group, p.N, p.T, BT, n_tile, t_tile);
+        w_tile = g * tiles_n + n_tile;
+        t0 = t_tile * BT;
+        x_col = g * p.group_ldx;
+        out_col = g * p.group_ldo;
     } else {
         tile_coords(cta, p.N, p.T, BT, n_tile, t_tile);
         w_tile = n_tile;
@@ -443,14 +460,14 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 }
                 pdl_wait();
                 if (OVB_PDL_GEMM == 2) pdl_trigger();
-                for (int i = 0; i < pre; ++i) tma_load_2d(smem + i * STAGE_BYTES, &tmX, &full_x[i], (kb_begin + i) * TILE_K, t0);
+                for (int i = 0; i < pre; ++i) tma_load_2d(smem + i * STAGE_BYTES, &tmX, &full_x[i], (kb_begin + i) * TILE_K + x_col, t0);
                 uint32_t phase = pre == stages ? 1 : 0;
                 int s = pre == stages ? 0 : pre;
                 for (int i = pre; i < num_kb; ++i) {
                     if (!mbar_wait(&empty[s], phase ^ 1, abort_flag, p.status)) break;
                     const int kb = kb_begin + i;
                     mbar_arrive_expect_tx(&full_x[s], X_BYTES + W_BYTES);
-                    tma_load_2d(smem + s * STAGE_BYTES, &tmX, &full_x[s], kb * TILE_K, t0);
+                    tma_load_2d(smem + s * STAGE_BYTES, &tmX, &full_x[s], kb * TILE_K + x_col, t0);
                     load_w(s, kb);
                     if (++s == stages) { s = 0; phase ^= 1; }
                 }
@@ -629,7 +646,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         // stores that cover 256 contiguous bytes per token row.
         const bool fast = p.world <= 1 && p.splits == 1 && !p.out_f32 && (n0 + TILE_N <= p.N) && (p.ldo % 8 == 0) &&
                           ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0) &&
-                          (p.residual == nullptr || ((p.ldr % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.residual) & 15) == 0)));
+                          out_col % 8 == 0 && (p.residual == nullptr || ((p.ldr % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.residual) & 15) == 0)));
         // fp32 staging keeps a single rounding (after the residual add): BT x 128 x 4 bytes <= 2 * STAGE_BYTES
         float* stage_out = reinterpret_cast<float*>(smem);
 
@@ -1050,9 +1067,9 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 v = apply_act(v, p.act);
                 if (p.residual) v += to_float(reinterpret_cast<const E*>(p.residual)[(size_t)tok * p.ldr + oc]);
                 if (p.out_f32)
-                    reinterpret_cast<float*>(p.out)[(size_t)tok * p.ldo + oc] = v;
+                    reinterpret_cast<float*>(p.out)[(size_t)tok * p.ldo + out_col + oc] = v;
                 else
-                    reinterpret_cast<E*>(p.out)[(size_t)tok * p.ldo + oc] = from_float<E>(v);
+                    reinterpret_cast<E*>(p.out)[(size_t)tok * p.ldo + out_col + oc] = from_float<E>(v);
             }
         };
 
@@ -1090,7 +1107,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         if (comm && p.splits == 1) {
             run_comm = true;
             comm_tile_ok = acc_ok;   // acc_ok is uniform over the epilogue threads
-        } else if (fast && p.act == OVB_ACT_SWIGLU) {
+        } else if (fast && (p.act == OVB_ACT_SWIGLU || p.act == OVB_ACT_GLU_LIMITED)) {
             // Gated MLP: the tile holds 64 "gate" rows followed by the 64 "up" rows of the same channels (the packer
             // interleaves them per tile), so out[tok, 64 * tile + c] = silu(gate_c) * up_c needs this tile only.
             asm volatile("bar.sync 1, %0;" ::"n"(DQ_THREADS));
@@ -1105,7 +1122,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                         uint4 v;
                         E* ve = reinterpret_cast<E*>(&v);
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) ve[j] = from_float<E>(g[j] / (1.0f + __expf(-g[j])) * u[j]);
+                        for (int j = 0; j < 8; ++j) ve[j] = from_float<E>(p.act == OVB_ACT_SWIGLU ? g[j] / (1.0f + __expf(-g[j])) * u[j] : glu_limited(p, g[j], u[j]));
                         *reinterpret_cast<uint4*>(reinterpret_cast<E*>(p.out) + (size_t)(t0 + col) * p.ldo + n_tile * (TILE_N / 2) + pc * 8) = v;
                     }
                 }
@@ -1132,7 +1149,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                         E* ve = reinterpret_cast<E*>(&v);
 #pragma unroll
                         for (int j = 0; j < 8; ++j) ve[j] = from_float<E>(f[j]);
-                        *reinterpret_cast<uint4*>(reinterpret_cast<E*>(p.out) + tok * p.ldo + n0 + pc * 8) = v;
+                        *reinterpret_cast<uint4*>(reinterpret_cast<E*>(p.out) + tok * p.ldo + out_col + n0 + pc * 8) = v;
                     }
                 }
             }
@@ -1385,7 +1402,8 @@ static int launch(const ovb_gemm_args* a, const CUtensorMap& tmW, const CUtensor
     if (p.splits > kMaxSplits) p.splits = kMaxSplits;
     p.kblocks_per_split = ceil_div(total_kb, p.splits);
     cfg.gridDim = dim3(ceil_div(a->N, TILE_N) * ceil_div(a->T, BT), 1, p.splits);
-    if (p.group_off != nullptr)     // every group may end with a partial row tile: num_groups extra tiles cover the worst case
+    if (p.group_mode == 3) cfg.gridDim = dim3(ceil_div(a->N, TILE_N) * ceil_div(a->T, BT) * p.num_groups, 1, 1);
+    else if (p.group_off != nullptr)     // every group may end with a partial row tile: num_groups extra tiles cover the worst case
         cfg.gridDim = dim3(ceil_div(a->N, TILE_N) * (ceil_div(a->T, BT) + p.num_groups), 1, 1);
     p.nvls_reducers = 0;
     if (p.nvls && p.splits == 1 && p.group_off == nullptr && (int)cfg.gridDim.x > resident[1]) {
@@ -1514,7 +1532,7 @@ int ovb_gemm(const ovb_gemm_args* a, ovb_stream_t stream_) {
         OVB_REQUIRE(a->N % 4 == 0 && (reinterpret_cast<uintptr_t>(a->scales) & 15) == 0,
                     "ovb_gemm: quantised weights need N %% 4 == 0 and a 16-byte aligned (scale, zero point) table");
     }
-    const bool swiglu = a->act == OVB_ACT_SWIGLU;
+    const bool swiglu = a->act == OVB_ACT_SWIGLU || a->act == OVB_ACT_GLU_LIMITED;   // gated: two rows of W make one output column
     if (swiglu) {
         // fused gated MLP: W rows are interleaved per 128-row tile (64 gate rows, then the 64 up rows of the same channels)
         OVB_REQUIRE(a->N % TILE_N == 0 && !a->out_f32 && a->residual == nullptr && a->comm == nullptr && a->bias == nullptr,
@@ -1523,8 +1541,13 @@ int ovb_gemm(const ovb_gemm_args* a, ovb_stream_t stream_) {
                     "ovb_gemm: the SWIGLU epilogue needs a 16-byte aligned output with a row pitch that is a multiple of 8");
     }
 
-    const bool grouped = a->group_offsets != nullptr;
-    if (grouped) {
+    const bool diag = a->group_mode == 3;
+    const bool grouped = a->group_offsets != nullptr || diag;
+    if (diag) {
+        OVB_REQUIRE(a->group_offsets == nullptr && a->num_groups >= 1 && a->w_tiled && !quant && a->comm == nullptr && a->K % TILE_K == 0 && a->act == OVB_ACT_NONE &&
+                        a->bias == nullptr && a->residual == nullptr && a->group_ldx % 8 == 0 && a->w_kb_stride == 0,
+                    "ovb_gemm: the block-diagonal product needs tile-packed 16-bit weights, K %% 64 == 0, column pitches that are multiples of 8 and a plain epilogue");
+    } else if (grouped) {
         OVB_REQUIRE(a->num_groups >= 1 && a->num_groups <= 256 && (a->group_mode == 1 || a->group_mode == 2), "ovb_gemm: grouped GEMM needs 1..256 groups and group_mode 1 or 2");
         OVB_REQUIRE((a->wmode == OVB_W_U4 || (a->w_tiled && !quant)) && a->comm == nullptr && a->N % TILE_N == 0 && a->K % TILE_K == 0,
                     "ovb_gemm: grouped GEMM needs tile-packed weights (u4 or 16-bit), N %% 128 == 0, K %% 64 == 0 and no communicator");
@@ -1554,6 +1577,11 @@ int ovb_gemm(const ovb_gemm_args* a, ovb_stream_t stream_) {
     p.group_off = a->group_offsets;
     p.num_groups = a->num_groups;
     p.group_mode = a->group_mode;
+    p.group_ldx = a->group_ldx;
+    p.group_ldo = a->group_ldo;
+    p.act_limit = a->act_limit;
+    p.act_slope = a->act_slope;
+    p.act_shift = a->act_shift;
     if (a->comm != nullptr && static_cast<const ovb_comm*>(a->comm)->world > 1) {
         const ovb_comm* c = static_cast<const ovb_comm*>(a->comm);
         OVB_REQUIRE(c->world <= 8 && c->rank >= 0 && c->rank < c->world, "ovb_gemm: bad communicator (rank %d of %d)", c->rank, c->world);
@@ -1608,7 +1636,9 @@ int ovb_gemm(const ovb_gemm_args* a, ovb_stream_t stream_) {
     CUtensorMap tmW, tmX;
     const int ldx = a->ldx ? a->ldx : a->K;
     const CUtensorMapDataType dt16 = f16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-    if (int rc = make_tmap_2d(&tmX, a->x, dt16, 2, a->T, a->K, (uint64_t)ldx * 2, bt, TILE_K, true)) return rc;
+    // (block-diagonal: the columns of all groups; what a group's last k-block reads behind them is filled with zeros)
+    const int xcols = diag ? (a->x_cols > 0 ? a->x_cols : ldx) : a->K;
+    if (int rc = make_tmap_2d(&tmX, a->x, dt16, 2, a->T, xcols, (uint64_t)ldx * 2, bt, TILE_K, true)) return rc;
     int rc = 0;
     if (a->wmode == OVB_W_U4 || (a->w_tiled && !quant)) {
         OVB_REQUIRE(a->K % TILE_K == 0, "ovb_gemm: tile-packed weights need K to be a multiple of 64");

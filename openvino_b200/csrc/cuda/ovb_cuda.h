@@ -50,6 +50,8 @@ enum {
     OVB_ACT_SWIGLU = 4,   // gated MLP: every 128-row tile of W holds 64 "gate" rows, then the 64 "up" rows of the same channels;
                           // out [T, N/2] = silu(gate) * up
     OVB_ACT_GELU_TANH = 5,
+    OVB_ACT_GLU_LIMITED = 6,   // rows of W as for SWIGLU; g = min(gate, act_limit), u = clamp(up, -act_limit, act_limit);
+                               // out [T, N/2] = g * sigmoid(act_slope * g) * (u + act_shift)
 };
 
 typedef struct {
@@ -85,6 +87,12 @@ typedef struct {
     const int* group_offsets;
     int num_groups;
     int group_mode;
+    // group_mode 3, block-diagonal (group_offsets is NULL): for every group g, out[:, g * group_ldo + (0 .. N)] =
+    // x[:, g * group_ldx + (0 .. K)] * W_g^T over all T rows. W stacks the groups along N, each padded to whole 128-row tiles; N is the
+    // number of columns written per group, K (a multiple of 64) may reach into the next group's columns of x where W_g is zero.
+    int group_ldx, group_ldo;
+    int x_cols;             // columns of x that may be read (0: the row pitch)
+    float act_limit, act_slope, act_shift;
 } ovb_gemm_args;
 
 int ovb_gemm(const ovb_gemm_args* a, ovb_stream_t stream);
@@ -305,6 +313,103 @@ int ovb_comm_argmax_combine(const ovb_comm* c, int* ids, const float* max_vals, 
 int ovb_comm_allreduce_bf16(const ovb_comm* c, void* data, int64_t n, ovb_stream_t stream);
 /* The same for fp32 / fp16 / bf16 tensors (dtype: OVB_DT_*); n elements, a multiple of 16 bytes. */
 int ovb_comm_allreduce(const ovb_comm* c, void* data, int64_t n, int dtype, ovb_stream_t stream);
+
+// ---------------------------------------------------------------------------------------------
+// Layered decoders (fp32 residual stream; storage type OVB_DT_F32 or OVB_DT_BF16 everywhere below, arithmetic in fp32).
+// Row pitches (ld*) and offsets are in elements.
+
+// h[r] = table[ids[r]] (fp32), x[r] = the same in the storage type (may be NULL).
+int ovb_stream_embed(const int* ids, const void* table, float* h, void* x, int rows, int cols, int vocab, int ldt, int ldh, int ldx, int dtype,
+                     ovb_stream_t stream);
+// s = alpha * h[row_idx ? row_idx[r] : r] (+ y[r], fp32, may be NULL); out = s / sqrt(mean(s^2) + eps) * (w_offset + w) to h_out (fp32)
+// and / or x_out (storage type). h_out may be h when row_idx is NULL.
+int ovb_sum_rmsnorm(const float* h, const int* row_idx, const float* y, const float* w, float* h_out, void* x_out, int rows, int cols, int ldh, int ldy,
+                    int ldho, int ldx, float alpha, float w_offset, float eps, int dtype, ovb_stream_t stream);
+// g = min(gate, limit), u = clamp(up, -limit, limit); out = g * sigmoid(slope * g) * (u + shift); up starts up_off columns after gate.
+int ovb_glu_limited(const void* gu, void* out, int rows, int F, int up_off, int ldg, int ldo, float limit, float slope, float shift, int dtype,
+                    ovb_stream_t stream);
+// fp32 products without tensor cores: out[b] = act(x[b] w[b]^T + bias[b]); s* = elements between batch members.
+int ovb_gemm_f32(const float* x, const float* w, const float* bias, float* out, int batch, long long sx, long long sw, long long sb, long long so, int T, int N,
+                 int K, int ldx, int ldw, int ldo, int act, ovb_stream_t stream);
+int ovb_argmax_f32(const float* logits, int ld, int rows, int vocab, void* out_ids, int ids_i32, float* out_max, ovb_stream_t stream);
+int ovb_sample_f32(const float* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed, const int* step, int* out_ids,
+                   ovb_stream_t stream);
+
+// Query / key norms, rotary positions and cache rows of grouped-query attention (attention_heads.cu).
+typedef struct {
+    void* proj;              // [T, ldp]: H query heads (pitch dk_pad), G key heads at k_off (pitch dk_pad), G value heads at v_off (pitch dv_pad)
+    void* k_cache;           // [blocks, G, block_size, dk_pad]
+    void* v_cache;           // [blocks, G, block_size, dv_pad]
+    const float* q_norm;     // [D] or NULL
+    const float* k_norm;
+    const float* inv_freq;   // [rot_dims / 2] or NULL
+    const int* positions;
+    const int* slot_map;
+    int T, H, G, D, Dv, dk_pad, dv_pad, ldp, k_off, v_off, block_size, rot_dims, dtype;
+    float rot_mult, eps;
+} ovb_heads_args;
+int ovb_heads_prepare(const ovb_heads_args* a, ovb_stream_t stream);
+
+// Latent attention: the normed low-rank row and the turned shared key part of every token go to the cache, the turned query
+// parts to q_rot (which may be their own place in proj).
+typedef struct {
+    void* proj;              // [T, ldp]: H query heads (pitch q_pitch, turned part at q_rot_off), low-rank row at c_off, shared key part at kr_off
+    void* q_rot;             // + t * ld_qr + head * qr_pitch
+    void* cache;             // [blocks, block_size, row_pitch]: low-rank row at 0, key part at key_off
+    const float* c_norm;     // [C]
+    const float* inv_freq;
+    const int* positions;
+    const int* slot_map;
+    int T, H, C, R, q_pitch, q_rot_off, c_off, kr_off, ldp, ld_qr, qr_pitch, row_pitch, key_off, block_size, rot_dims, dtype;
+    float rot_mult, eps;
+} ovb_latent_args;
+int ovb_latent_prepare(const ovb_latent_args* a, ovb_stream_t stream);
+
+// Causal attention over a paged cache with key and value sizes of their own, an optional sliding window (a position sees itself and
+// the window - 1 positions before it; 0 = off) and an optional sigmoid gate on the output. Key rows: ((block * Hkv + kv head) *
+// block_size + slot) * k_row, value rows likewise with v_row (v may point into the key rows).
+typedef struct {
+    const void* q;            // + t * ldq + head * q_head
+    const void* k;
+    const void* v;
+    void* out;                // + t * ldo + head * o_head
+    const void* gate;         // + t * ld_gate + head * gate_head, or NULL
+    const int* past_lens;
+    const int* subsequence_begins;
+    const int* block_indices;
+    const int* block_indices_begins;
+    float* scratch;           // split-KV partials or NULL
+    long long scratch_bytes;
+    int B, T, Hq, Hkv, Dk, Dv;          // Dk: padded key size (zeros behind the true size), Dv: true value size
+    int ldq, q_head, k_row, v_row, ldo, o_head, ld_gate, gate_head;
+    int block_size, window, max_context_len, max_q_len, dtype;
+    float scale;
+    int exact;                // 1: fp32 arithmetic throughout (no tensor cores)
+} ovb_wattn_args;
+int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream);
+
+// Griffin's recurrent block between its projections (recurrent.cu). ovb_causal_conv: u = conv(x); then the caller computes the gate
+// pre-activations gates = [ra u | ri u] block by block; ovb_lru_scan: r, i = sigmoid(gates + gate_b), a = exp(-r * log_decay),
+// S <- a S + sqrt(1 - a^2) i u, out = S * gelu_tanh(y), and both states are brought up to date.
+typedef struct {
+    const void* x;            // [T, ldx] convolution input (projection, bias added)
+    const void* y;            // [T, ldy] other branch before its activation
+    void* u;                  // [T, ldu] convolution output, blocks of bw channels at a pitch of ub_pitch
+    void* out;                // [T, ldo]
+    const float* gates;       // [T, ldg]: block b at b * gb_pitch, r part at 0, i part at gi_off
+    const float* gate_b;      // [2, N] biases of r and i
+    const float* log_decay;   // [N] positive: log a = -r * log_decay
+    const float* conv_w;      // [taps, N]
+    const float* conv_b;      // [N]
+    float* state;             // [slots, N]
+    float* conv_state;        // [slots, taps - 1, N]
+    const int* subsequence_begins;
+    const int* past_lens;
+    const int* slots;         // [B]
+    int B, T, N, taps, bw, ub_pitch, gb_pitch, gi_off, ldx, ldy, ldu, ldg, ldo, max_q_len, dtype;
+} ovb_rglru_args;
+int ovb_causal_conv(const ovb_rglru_args* a, ovb_stream_t stream);
+int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -1,5 +1,6 @@
-// Linear-recurrence layers of hybrid LLMs: the selective state-space scan (Mamba-2 form) and the gated delta rule
-// (Gated DeltaNet / Qwen3-Next linear attention). Both walk the tokens of a sequence in order with the recurrent state
+// Linear-recurrence layers of hybrid LLMs: the selective state-space scan (Mamba-2 form), the gated delta rule
+// (Gated DeltaNet / Qwen3-Next linear attention) and, at the end of the file, the real-gated linear recurrent unit with its
+// short convolution (Griffin's recurrent block). The first two walk the tokens of a sequence in order with the recurrent state
 // of one head resident in registers: one warp owns four rows (state-space) or four columns (delta rule) of the state
 // matrix, its 32 lanes hold the rows' elements, and the dot products of a token are warp shuffles (four sums share six
 // shuffles). The state is read from and written to HBM once per launch; the token vectors every row of a head shares are
@@ -12,6 +13,8 @@
 #include <type_traits>
 
 #include "common.cuh"
+#include "sm100_ptx.cuh"
+#include "store_types.cuh"
 
 namespace ovb {
 
@@ -218,6 +221,121 @@ gated_delta_rule_kernel(const float* __restrict__ q, const float* __restrict__ k
             if (cw + c < Dv && lane + 32 * i < Dk) sbase[(size_t)(lane + 32 * i) * Dv + cw + c] = st[c][i];
 }
 
+// ------------------------------------------------------------------------------ real-gated linear recurrent unit
+// Ragged batches: tokens subsequence_begins[b] .. of sequence b continue from the state in slot slots[b], or from zeros when
+// past_lens[b] == 0 (a slot that another request used before needs no clearing). The state of a channel is S (fp32) and the
+// last taps - 1 inputs of the convolution.
+
+// u[t, c] = bias[c] + sum_j w[j, c] * x[t - (taps - 1) + j, c]. u is laid out block by block with a pitch of ub_pitch columns per
+// block of bw channels, as the block-diagonal gate product reads it.
+template <class E>
+__global__ void __launch_bounds__(256) causal_conv_kernel(ovb_rglru_args p) {
+    pdl_enter();
+    __shared__ int s_b;
+    const int t = blockIdx.x;
+    if (threadIdx.x == 0) {
+        int b = 0;
+        while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
+        s_b = b;
+    }
+    __syncthreads();
+    const int b = s_b, begin = p.subsequence_begins[b], keep = p.taps - 1;
+    const bool fresh = p.past_lens[b] == 0;
+    const E* x = reinterpret_cast<const E*>(p.x);
+    const float* old = p.conv_state + (size_t)p.slots[b] * keep * p.N;
+    E* u = reinterpret_cast<E*>(p.u) + (size_t)t * p.ldu;
+    for (int c = blockIdx.y * 256 + threadIdx.x; c < p.N; c += gridDim.y * 256) {
+        float acc = p.conv_b[c];
+        for (int j = 0; j < p.taps; ++j) {
+            const int s = t - keep + j - begin;          // token of the chunk; negative: before it
+            float v = 0.f;
+            if (s >= 0) v = ld_f32(x + (size_t)(begin + s) * p.ldx + c);
+            else if (!fresh) v = old[(size_t)(s + keep) * p.N + c];
+            acc = fmaf(p.conv_w[(size_t)j * p.N + c], v, acc);
+        }
+        st_f32(u + (c / p.bw) * p.ub_pitch + c % p.bw, acc);
+    }
+}
+
+// gelu (tanh form) of the other branch
+__device__ __forceinline__ float rec_gelu_tanh(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+constexpr int LRU_L = 8;    // tokens per warp and round
+
+// One group of 32 channels (a lane each) of one sequence. The NW warps of the group take consecutive pieces of LRU_L tokens: each
+// composes the affine maps S -> a S + b of its piece, the pieces' maps are chained through shared memory, and the piece is then
+// replayed from its true starting state. NW = 1 (decode): a CTA holds four independent groups.
+template <class E, int NW>
+__global__ void __launch_bounds__(NW == 1 ? 128 : NW * 32) lru_scan_kernel(ovb_rglru_args p) {
+    pdl_enter();
+    __shared__ float sA[NW][32], sB[NW][32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int b = blockIdx.y, w = NW == 1 ? 0 : warp;
+    const int c = (NW == 1 ? blockIdx.x * 4 + warp : blockIdx.x) * 32 + lane;
+    const bool live = c < p.N;
+    const int begin = p.subsequence_begins[b], len = p.subsequence_begins[b + 1] - begin, slot = p.slots[b];
+    const bool fresh = p.past_lens[b] == 0;
+    const int cc = live ? c : 0, blk = cc / p.bw, cb = cc % p.bw;
+    const float lam = p.log_decay[cc], br = p.gate_b[cc], bi = p.gate_b[p.N + cc];
+    float* state = p.state + (size_t)slot * p.N + cc;
+    float carry = (fresh || !live) ? 0.f : *state;
+    for (int t0 = 0; t0 < len; t0 += NW * LRU_L) {
+        const int tw = t0 + w * LRU_L;
+        float a[LRU_L], x[LRU_L], A = 1.f, S = 0.f;
+#pragma unroll
+        for (int i = 0; i < LRU_L; ++i) {
+            a[i] = 1.f;
+            x[i] = 0.f;
+            if (live && tw + i < len) {
+                const size_t t = (size_t)(begin + tw + i);
+                const float* g = p.gates + t * p.ldg + blk * p.gb_pitch;
+                const float r = 1.f / (1.f + expf(-(g[cb] + br))), in = 1.f / (1.f + expf(-(g[p.gi_off + cb] + bi)));
+                const float log_a = -r * lam;
+                const float u = ld_f32(reinterpret_cast<const E*>(p.u) + t * p.ldu + blk * p.ub_pitch + cb);
+                a[i] = expf(log_a);
+                x[i] = sqrtf(-expm1f(2.f * log_a)) * in * u;
+            }
+            S = fmaf(a[i], S, x[i]);
+            A *= a[i];
+        }
+        float s = carry;
+        if (NW > 1) {
+            sA[w][lane] = A;
+            sB[w][lane] = S;
+            __syncthreads();
+            float all = carry;
+#pragma unroll
+            for (int k = 0; k < NW; ++k) {
+                if (k == w) s = all;
+                all = fmaf(sA[k][lane], all, sB[k][lane]);
+            }
+            carry = all;
+        }
+#pragma unroll
+        for (int i = 0; i < LRU_L; ++i) {
+            s = fmaf(a[i], s, x[i]);
+            if (live && tw + i < len) {
+                const size_t t = (size_t)(begin + tw + i);
+                const float y = rec_gelu_tanh(ld_f32(reinterpret_cast<const E*>(p.y) + t * p.ldy + c));
+                st_f32(reinterpret_cast<E*>(p.out) + t * p.ldo + c, s * y);
+            }
+        }
+        if (NW == 1) carry = s;
+        else __syncthreads();
+    }
+    if (!live || w != 0) return;
+    *state = carry;
+    const int keep = p.taps - 1;
+    float* old = p.conv_state + (size_t)slot * keep * p.N + c;
+    for (int j = 0; j < keep; ++j) {
+        const int s = len - keep + j;                     // ascending j only reads rows that are not overwritten yet
+        float v = 0.f;
+        if (s >= 0) v = ld_f32(reinterpret_cast<const E*>(p.x) + (size_t)(begin + s) * p.ldx + c);
+        else if (!fresh) v = old[(size_t)(s + keep) * p.N];
+        old[(size_t)j * p.N] = v;
+    }
+}
+
 // OVB_SSM_ROWS_PER_WARP = 4 keeps the four-row (four-column) form of both kernels for every shape (8 by default where it applies)
 int env_rows_per_warp() {
     const char* e = getenv("OVB_SSM_ROWS_PER_WARP");
@@ -281,6 +399,38 @@ int ovb_gated_delta_rule(const float* q, const float* k, const float* v, const f
         else
             gated_delta_rule_kernel<NV, 4><<<dim3(ceil_div(Dv, REC_WARPS * 4), B * Hv), REC_WARPS * 32, 0, stream>>>(q, k, v, gate, beta, state, y, L, Hq, Hv, Dk, Dv);
         OVB_CHECK_CUDA(cudaGetLastError());
+        return 0;
+    });
+}
+
+static int check_rglru(const ovb_rglru_args* a, const char* what) {
+    using namespace ovb;
+    OVB_REQUIRE(a && a->x && a->u && a->conv_w && a->conv_b && a->subsequence_begins && a->past_lens && a->slots && a->conv_state, "%s: null operand", what);
+    OVB_REQUIRE(a->B > 0 && a->B <= 65535 && a->T > 0 && a->N > 0 && a->taps > 0 && a->bw > 0 && a->N % a->bw == 0 && a->ub_pitch >= a->bw, "%s: bad sizes", what);
+    return 0;
+}
+
+int ovb_causal_conv(const ovb_rglru_args* a, ovb_stream_t stream) {
+    using namespace ovb;
+    if (int rc = check_rglru(a, "ovb_causal_conv")) return rc;
+    return dispatch_store(a->dtype, "ovb_causal_conv", [&](auto e) -> int {
+        using E = decltype(e);
+        const int cy = ceil_div(a->N, 256);
+        OVB_CHECK_CUDA(launch_pdl(causal_conv_kernel<E>, dim3(a->T, cy < 65535 ? cy : 65535), dim3(256), 0, (cudaStream_t)stream, *a));
+        return 0;
+    });
+}
+
+int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream) {
+    using namespace ovb;
+    if (int rc = check_rglru(a, "ovb_lru_scan")) return rc;
+    OVB_REQUIRE(a->y && a->gates && a->gate_b && a->log_decay && a->state && a->out, "ovb_lru_scan: null operand");
+    return dispatch_store(a->dtype, "ovb_lru_scan", [&](auto e) -> int {
+        using E = decltype(e);
+        if (a->max_q_len <= LRU_L)
+            OVB_CHECK_CUDA(launch_pdl(lru_scan_kernel<E, 1>, dim3(ceil_div(a->N, 128), a->B), dim3(128), 0, (cudaStream_t)stream, *a));
+        else
+            OVB_CHECK_CUDA(launch_pdl(lru_scan_kernel<E, 16>, dim3(ceil_div(a->N, 32), a->B), dim3(512), 0, (cudaStream_t)stream, *a));
         return 0;
     });
 }

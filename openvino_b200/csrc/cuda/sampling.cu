@@ -8,6 +8,7 @@
 #include "common.cuh"
 #include "sm100_ptx.cuh"
 #include <cuda_bf16.h>
+#include "store_types.cuh"
 
 namespace ovb {
 
@@ -41,22 +42,23 @@ __device__ __forceinline__ uint64_t mix64(uint64_t z) {
     return z ^ (z >> 31);
 }
 
-__global__ void __launch_bounds__(kSampleThreads) sample_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int V, float inv_temp,
+template <class E>
+__global__ void __launch_bounds__(kSampleThreads) sample_kernel(const E* __restrict__ logits, int ld, int V, float inv_temp,
                                                                 int top_k, float top_p, uint64_t seed, const int* __restrict__ step_ptr,
                                                                 int* __restrict__ out_ids) {
     pdl_enter();
     __shared__ float sh[33];
     __shared__ float scan[kSampleThreads];
     const int row = blockIdx.x;
-    const __nv_bfloat16* l = logits + (size_t)row * ld;
+    const E* l = logits + (size_t)row * ld;
     const int per = (V + kSampleThreads - 1) / kSampleThreads;          // contiguous chunk per thread (index order matters for the draw)
     const int v0 = threadIdx.x * per, v1 = min(V, v0 + per);
     float mx = -INFINITY, mn = INFINITY;
-    for (int v = v0; v < v1; ++v) { const float x = __bfloat162float(l[v]); mx = fmaxf(mx, x); mn = fminf(mn, x); }
+    for (int v = v0; v < v1; ++v) { const float x = ld_f32(l + v); mx = fmaxf(mx, x); mn = fminf(mn, x); }
     mx = block_reduce(mx, sh, true);
     mn = -block_reduce(-mn, sh, true);
     float z = 0.f;
-    for (int v = v0; v < v1; ++v) z += __expf((__bfloat162float(l[v]) - mx) * inv_temp);
+    for (int v = v0; v < v1; ++v) z += __expf((ld_f32(l + v) - mx) * inv_temp);
     z = block_reduce(z, sh, false);
     // bisection on the threshold: keep(lo) is never smaller than the wanted set, keep(hi) may be
     float lo = mn, hi = mx;
@@ -66,7 +68,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_kernel(const __nv_bfloa
             const float mid = 0.5f * (lo + hi);
             float cnt = 0.f, mass = 0.f;
             for (int v = v0; v < v1; ++v) {
-                const float x = __bfloat162float(l[v]);
+                const float x = ld_f32(l + v);
                 if (x >= mid) { cnt += 1.f; mass += __expf((x - mx) * inv_temp); }
             }
             cnt = block_reduce(cnt, sh, false);
@@ -80,7 +82,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_kernel(const __nv_bfloa
     const float thr = (restrict_k || restrict_p) ? lo : -INFINITY;
     float local = 0.f;
     for (int v = v0; v < v1; ++v) {
-        const float x = __bfloat162float(l[v]);
+        const float x = ld_f32(l + v);
         if (x >= thr) local += __expf((x - mx) * inv_temp);
     }
     scan[threadIdx.x] = local;
@@ -101,7 +103,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_kernel(const __nv_bfloa
         float acc = before;
         int pick = -1;
         for (int v = v0; v < v1; ++v) {
-            const float x = __bfloat162float(l[v]);
+            const float x = ld_f32(l + v);
             if (x >= thr) {
                 acc += __expf((x - mx) * inv_temp);
                 pick = v;
@@ -181,14 +183,28 @@ using namespace ovb;
 // out_ids[row] ~ softmax(logits[row] / temperature) restricted to the top_k most likely tokens and to the smallest
 // set of probability mass >= top_p. top_k <= 0 and top_p >= 1 switch the restrictions off. `step` (device int, may be
 // NULL) is mixed into the random stream, so replays of a captured graph draw fresh numbers when the word is bumped.
-int ovb_sample(const void* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed,
-               const int* step, int* out_ids, ovb_stream_t stream_) {
-    cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+}  // extern "C"
+
+template <class E>
+static int sample_rows(const E* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed, const int* step, int* out_ids,
+                       cudaStream_t stream) {
     OVB_REQUIRE(logits && out_ids && rows > 0 && vocab > 0 && temperature > 0.f, "ovb_sample: bad arguments (temperature must be > 0)");
-    OVB_CHECK_CUDA(launch_pdl(sample_kernel, dim3(rows), dim3(kSampleThreads), 0, stream, (const __nv_bfloat16*)logits, ld, vocab, 1.0f / temperature, top_k,
+    OVB_CHECK_CUDA(launch_pdl(sample_kernel<E>, dim3(rows), dim3(kSampleThreads), 0, stream, logits, ld, vocab, 1.0f / temperature, top_k,
                                                        top_p <= 0.f ? 1e-6f : top_p, seed, step, out_ids));
     OVB_CHECK_CUDA(cudaGetLastError());
     return 0;
+}
+
+extern "C" {
+
+int ovb_sample(const void* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed,
+               const int* step, int* out_ids, ovb_stream_t stream_) {
+    return sample_rows((const __nv_bfloat16*)logits, ld, rows, vocab, temperature, top_k, top_p, seed, step, out_ids, static_cast<cudaStream_t>(stream_));
+}
+
+int ovb_sample_f32(const float* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed, const int* step, int* out_ids,
+                   ovb_stream_t stream_) {
+    return sample_rows(logits, ld, rows, vocab, temperature, top_k, top_p, seed, step, out_ids, static_cast<cudaStream_t>(stream_));
 }
 
 int ovb_sample_gumbel(const void* logits, int ld, int rows, int vocab, int vocab_offset, float temperature, uint64_t seed, const int* step,

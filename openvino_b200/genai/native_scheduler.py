@@ -36,6 +36,8 @@ def make_layout(offsets: Dict[str, tuple], Tcap: int, Bcap: int, max_blocks: int
     for name in ("ids", "positions", "slot_map", "tok_src", "tok_dst", "logit_idx", "past_lens", "subsequence_begins",
                  "block_indices_begins", "block_indices"):
         setattr(lay, name, offsets[name][0])
+    if "state_slots" in offsets:
+        lay.state_slots = offsets["state_slots"][0]
     lay.Tcap, lay.Bcap, lay.blocks_cap = Tcap, Bcap, Bcap * max_blocks
     return lay
 

@@ -13,7 +13,7 @@ from typing import Dict, List, Optional, Sequence as Seq
 import numpy as np
 import torch
 
-from ..runtime.cuda_llm import CudaLlmExecutor, StepBuffers, StepShape
+from ..runtime.cuda_llm import LlmExecutor, StepShape
 from .native_scheduler import NativeScheduler, make_layout
 from .scheduler import ScheduledStep, Scheduler, SchedulerConfig, Sequence
 
@@ -77,8 +77,16 @@ class StepPlan:
 
 from ..utils import trace as _trace
 
+
+def step_shape(st: ScheduledStep) -> StepShape:
+    """What the executor has to know on the host about a scheduled step."""
+    return StepShape(st.T, len(st.seqs), st.max_q_len, st.max_ctx)
+
+
 class ContinuousBatchingPipeline:
-    def __init__(self, executor: CudaLlmExecutor, scheduler_config: SchedulerConfig):
+    def __init__(self, executor: LlmExecutor, scheduler_config: SchedulerConfig):
+        if executor.has_recurrent_state and getattr(scheduler_config, "enable_prefix_caching", False):
+            raise ValueError("prefix caching shares attention blocks; the state of recurrent layers after a cached prefix is not kept")
         self.ex = executor
         self.cfg = scheduler_config
         self.scheduler = self._make_scheduler(scheduler_config)
@@ -135,7 +143,7 @@ class ContinuousBatchingPipeline:
         self.metrics.h2d_bytes += ex.upload(sb, k)
         B = len(st.seqs)
         with _trace.scope("ov::genai", "decode_step" if decode else "prefill_step"):
-            ex.run(sb, StepShape(st.T, B, st.max_q_len, st.max_ctx))
+            ex.run(sb, step_shape(st))
         ev = ex.download_tokens_async(sb, B, k)
         self.metrics.d2h_bytes += B * 4
         m = self.metrics
@@ -185,7 +193,7 @@ class ContinuousBatchingPipeline:
             else:
                 sched.fill(st, {name: arr[off:off + n] for name, (off, n) in sb.offsets.items()})
             descs[id(sb)].append(torch.from_numpy(arr))
-            steps.append((sb, len(descs[id(sb)]) - 1, StepShape(st.T, len(st.seqs), st.max_q_len, st.max_ctx)))
+            steps.append((sb, len(descs[id(sb)]) - 1, step_shape(st)))
             sched.commit(st, None)
         dev = {k: (torch.stack(v).to(ex.device) if v else None) for k, v in descs.items()}
         return StepPlan(steps, dev, sum(len(p) for p in prompts), len(prompts) * gen.max_new_tokens)

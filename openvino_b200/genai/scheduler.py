@@ -208,6 +208,25 @@ class Scheduler:
         max_ctx = max(s.num_computed + n for s, n in zip(seqs, num_new))
         return ScheduledStep(seqs, num_new, T, max(num_new), max_ctx)
 
+    # -- steps of given tokens: the caller names the batch, nothing is sampled (genai/replay.py)
+    def admit(self, seq: Sequence) -> None:
+        seq.slot = self._free_slots.popleft()
+        self.running.append(seq)
+
+    def place(self, seqs: List[Sequence], num_new: List[int]) -> ScheduledStep:
+        """A step of ``num_new[i]`` further known tokens of every sequence; takes the blocks they need."""
+        for s, n in zip(seqs, num_new):
+            if not self.blocks.grow(s, s.num_computed + n):
+                raise RuntimeError("the KV cache (%d blocks of %d tokens) is too small" % (self.cfg.num_kv_blocks, self.cfg.block_size))
+        return ScheduledStep(list(seqs), list(num_new), sum(num_new), max(num_new), max(s.num_computed + n for s, n in zip(seqs, num_new)))
+
+    def advance(self, step: ScheduledStep) -> None:
+        for s, n in zip(step.seqs, step.num_new):
+            s.num_computed += n
+
+    def retire(self, seq: Sequence) -> None:
+        self._finish(seq)
+
     # -- descriptor of a scheduled step, written into numpy views of the pinned mirror --------
     def fill(self, step: ScheduledStep, views: Dict[str, np.ndarray]) -> None:
         bs = self.cfg.block_size
@@ -236,6 +255,8 @@ class Scheduler:
                 src[n - 1] = s.slot
             views["tok_dst"][i] = s.slot if c0 + n == s.total_len else -1
             views["past_lens"][i] = c0
+            if "state_slots" in views:
+                views["state_slots"][i] = s.slot
             views["logit_idx"][i] = t + n - 1
             k = (c0 + n + bs - 1) // bs
             views["block_indices"][nb:nb + k] = tbl[:k]

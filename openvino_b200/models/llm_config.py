@@ -3,7 +3,9 @@ benchmarks. The named configurations are the ones of the serving benchmarks (Lla
 Llama-3-70B, Mixtral-8x7B); ``tiny`` variants keep tests fast."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, replace
+from typing import List, Optional, Tuple, Union
 
 
 @dataclass(frozen=True)
@@ -48,3 +50,104 @@ TINY_MOE = LlmConfig(name="tiny-moe", vocab_size=512, hidden_size=256, num_layer
                      head_dim=128, ffn_size=256, num_experts=4, experts_top_k=2, weight_format="bf16")
 
 NAMED = {c.name: c for c in (LLAMA3_8B, LLAMA3_70B, MIXTRAL_8X7B, TINY_LLAMA, TINY_MOE)}
+
+
+# ----------------------------------------------------------------------------------------- layered decoders
+# A decoder whose layers are listed one by one: every layer names its token mixer and its feed-forward, each with sizes of its
+# own. The residual stream is fp32. The serving program of these configurations is runtime/layered_llm.py.
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of the first ``dims`` dimensions by the position (dimension i paired with i + dims / 2). ``yarn`` = (factor,
+    original length, fast, slow): frequencies that turn less than ``slow`` times over the original length are divided by the
+    factor, those that turn more than ``fast`` times are kept, with a linear ramp over the dimensions in between."""
+    dims: int
+    base: float
+    yarn: Optional[Tuple[float, float, float, float]] = None
+
+    def inv_freq(self) -> List[float]:
+        freq = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.yarn is None:
+            return freq
+        factor, original, fast, slow = self.yarn
+        turns_at = lambda t: self.dims * math.log(original / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
+        first = max(math.floor(turns_at(fast)), 0)
+        last = min(math.ceil(turns_at(slow)), self.dims - 1)
+        width = max(last - first, 0.001)
+        keep = [1.0 - min(max((i - first) / width, 0.0), 1.0) for i in range(self.dims // 2)]
+        return [f * k + f / factor * (1.0 - k) for f, k in zip(freq, keep)]
+
+    def multiplier(self) -> float:
+        """Factor of cos and sin."""
+        return 1.0 if self.yarn is None else 0.1 * math.log(self.yarn[0]) + 1.0
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Grouped-query attention; ``window`` 0 = full causal attention, else a position sees itself and window - 1 before it."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+    qk_norm: bool = False          # RMS norm of every query / key head, one weight of size dim for all heads
+    gated: bool = False            # heads times sigmoid(W_g x) before the output projection
+    rotary: Optional[RotarySpec] = None
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention whose keys and values are projections of one normed low-rank row per token, plus a rotated key part that all
+    heads share; those two are what is cached."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rotary: RotarySpec
+    window: int = 0
+
+
+@dataclass(frozen=True)
+class RgLruSpec:
+    """Griffin's recurrent block: short causal convolution, block-diagonal gates, real-gated linear recurrent unit."""
+    width: int
+    blocks: int
+    taps: int
+    decay: float = 8.0             # log a = -decay * r * softplus(lambda)
+
+
+@dataclass(frozen=True)
+class LimitedGluSpec:
+    """g = min(gate, limit), u = clamp(up, -limit, limit); g * sigmoid(slope * g) * (u + shift)."""
+    ff: int
+    limit: float
+    slope: float = 1.702
+    shift: float = 1.0
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Union[AttentionSpec, LatentAttentionSpec, RgLruSpec]
+    mlp: Optional[LimitedGluSpec] = None
+
+
+@dataclass(frozen=True)
+class LayeredConfig:
+    """Layers with the norm after each sum: x <- norm(residual_scale * x + sublayer(x)), norm weight = norm_offset + stored."""
+    name: str
+    vocab_size: int
+    hidden_size: int
+    layers: Tuple[LayerSpec, ...]
+    norm_eps: float = 1e-5
+    residual_scale: float = 1.0
+    norm_offset: float = 0.0
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        return any(isinstance(l.mixer, RgLruSpec) for l in self.layers)

@@ -1,0 +1,57 @@
+"""Checkpoint folders (``config.json`` + ``model.safetensors``): the architecture that ``config.json`` names selects the reader of
+its configuration and the names of its tensors; everything else (weights in kernel layout, cache, scheduling, sampling) is the
+serving program's. Graph models (IR, ONNX, ...) do not pass through here: see frontend/ and runtime/llm_import.py.
+"""
+from __future__ import annotations
+
+import json
+import os
+from dataclasses import dataclass
+from typing import Callable, Dict
+
+from ..utils.safetensors import SafetensorsFile
+from . import busatar
+from .llm_config import LayeredConfig
+
+
+@dataclass(frozen=True)
+class Architecture:
+    read_config: Callable[[dict], LayeredConfig]
+    tensor_name: Callable[[int, str, str], str]
+
+
+ARCHITECTURES: Dict[str, Architecture] = {"Busatar": Architecture(busatar.read_config, busatar.tensor_name)}
+
+
+def register(name: str, arch: Architecture) -> None:
+    ARCHITECTURES[name] = arch
+
+
+@dataclass
+class Checkpoint:
+    """A configuration and where its tensors come from."""
+    config: LayeredConfig
+    arch: Architecture
+    tensors: object            # mapping name -> torch.Tensor
+
+    def __call__(self, layer: int, part: str, key: str):
+        return self.tensors[self.arch.tensor_name(layer, part, key)]
+
+
+def is_checkpoint_dir(path: str) -> bool:
+    return os.path.isfile(os.path.join(path, "config.json")) and os.path.isfile(os.path.join(path, "model.safetensors"))
+
+
+def load_checkpoint(path: str) -> Checkpoint:
+    with open(os.path.join(path, "config.json")) as f:
+        cfg = json.load(f)
+    return from_dict(cfg, SafetensorsFile(os.path.join(path, "model.safetensors")))
+
+
+def from_dict(cfg: dict, tensors) -> Checkpoint:
+    """The same from a parsed configuration and any name -> tensor mapping."""
+    name = cfg.get("architecture")
+    if name not in ARCHITECTURES:
+        raise ValueError("unknown architecture '%s' (known: %s)" % (name, ", ".join(sorted(ARCHITECTURES))))
+    arch = ARCHITECTURES[name]
+    return Checkpoint(arch.read_config(cfg), arch, tensors)

@@ -20,7 +20,9 @@ _PKG = Path(__file__).resolve().parent.parent
 _LIB_PATH = Path(os.environ["OVB_CUDA_LIB"]) if os.environ.get("OVB_CUDA_LIB") else _PKG / "lib" / "libovb_cuda.so"
 
 W_BF16, W_U4, W_U8, W_F16, W_F8 = 0, 1, 2, 3, 4
-ACT_NONE, ACT_GELU_ERF, ACT_RELU, ACT_SILU, ACT_SWIGLU, ACT_GELU_TANH = 0, 1, 2, 3, 4, 5
+W_F32 = 16                     # fp32 weights: products without tensor cores (ovb_gemm_f32)
+DT_F32, DT_BF16 = 0, 2         # storage types of the layered decoders' kernels
+ACT_NONE, ACT_GELU_ERF, ACT_RELU, ACT_SILU, ACT_SWIGLU, ACT_GELU_TANH, ACT_GLU_LIMITED = 0, 1, 2, 3, 4, 5, 6
 
 STATUS_NAMES = {0: "ok", 1: "mbarrier wait timed out", 2: "peer flag wait timed out", 3: "bad argument seen on device",
                 4: "local flag wait timed out", 5: "index out of range (debug build; the access was skipped)"}
@@ -37,6 +39,8 @@ class GemmArgs(C.Structure):
         ("splits", C.c_int), ("block_t", C.c_int), ("w_tiled", C.c_int),
         ("comm", C.c_void_p), ("w_kb_stride", C.c_int),
         ("group_offsets", C.c_void_p), ("num_groups", C.c_int), ("group_mode", C.c_int),
+        ("group_ldx", C.c_int), ("group_ldo", C.c_int), ("x_cols", C.c_int),
+        ("act_limit", C.c_float), ("act_slope", C.c_float), ("act_shift", C.c_float),
     ]
 
 
@@ -50,6 +54,34 @@ class PaArgs(C.Structure):
         ("sliding_window", C.c_int), ("scale", C.c_float),
         ("kv_u8", C.c_int), ("k_meta", C.c_void_p), ("v_meta", C.c_void_p),
     ]
+
+
+def _fields(pointers, ints, floats=()):
+    return ([(n, C.c_void_p) for n in pointers] + [(n, C.c_int) for n in ints] + [(n, C.c_float) for n in floats])
+
+
+class HeadsArgs(C.Structure):
+    _fields_ = _fields(("proj", "k_cache", "v_cache", "q_norm", "k_norm", "inv_freq", "positions", "slot_map"),
+                       ("T", "H", "G", "D", "Dv", "dk_pad", "dv_pad", "ldp", "k_off", "v_off", "block_size", "rot_dims", "dtype"), ("rot_mult", "eps"))
+
+
+class LatentArgs(C.Structure):
+    _fields_ = _fields(("proj", "q_rot", "cache", "c_norm", "inv_freq", "positions", "slot_map"),
+                       ("T", "H", "C", "R", "q_pitch", "q_rot_off", "c_off", "kr_off", "ldp", "ld_qr", "qr_pitch", "row_pitch", "key_off", "block_size",
+                        "rot_dims", "dtype"), ("rot_mult", "eps"))
+
+
+class WindowAttnArgs(C.Structure):
+    _fields_ = (_fields(("q", "k", "v", "out", "gate", "past_lens", "subsequence_begins", "block_indices", "block_indices_begins", "scratch"), ())
+                + [("scratch_bytes", C.c_longlong)]
+                + _fields((), ("B", "T", "Hq", "Hkv", "Dk", "Dv", "ldq", "q_head", "k_row", "v_row", "ldo", "o_head", "ld_gate", "gate_head", "block_size",
+                               "window", "max_context_len", "max_q_len", "dtype"), ("scale",)) + [("exact", C.c_int)])
+
+
+class RgLruArgs(C.Structure):
+    _fields_ = _fields(("x", "y", "u", "out", "gates", "gate_b", "log_decay", "conv_w", "conv_b", "state", "conv_state", "subsequence_begins", "past_lens",
+                        "slots"),
+                       ("B", "T", "N", "taps", "bw", "ub_pitch", "gb_pitch", "gi_off", "ldx", "ldy", "ldu", "ldg", "ldo", "max_q_len", "dtype"))
 
 
 _lib = None
@@ -246,15 +278,20 @@ class PackedWeight:
 # ------------------------------------------------------------------------------------------ ops
 def gemm(x: torch.Tensor, w: PackedWeight, out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None,
          act: int = ACT_NONE, out_f32: bool = False, ws: Optional[Workspace] = None, splits: int = 0,
-         block_t: int = 0, comm=None) -> torch.Tensor:
+         block_t: int = 0, comm=None, glu=None) -> torch.Tensor:
     """out[T, N] = act(x[T, K] @ dequant(W)^T + bias) + residual  on the tcgen05 GEMM.
 
-    ``comm`` (a ``parallel.comm.CommStruct``): sum the product over the tensor-parallel ranks inside the epilogue."""
+    ``comm`` (a ``parallel.comm.CommStruct``): sum the product over the tensor-parallel ranks inside the epilogue.
+    ``glu`` (limit, slope, shift): parameters of ``ACT_GLU_LIMITED``. fp32 weights (``W_F32``) take the product without
+    tensor cores; ``x`` and ``out`` are then fp32."""
     assert x.dim() == 2 and x.stride(1) == 1
     T, K = x.shape
     assert K == w.K, (K, w.K)
+    if w.mode == W_F32:
+        assert residual is None and comm is None
+        return _gemm_f32(x, w, out, act)
     if out is None:
-        out = torch.empty((T, w.N // 2 if act == ACT_SWIGLU else w.N), dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
+        out = torch.empty((T, w.N // 2 if act in (ACT_SWIGLU, ACT_GLU_LIMITED) else w.N), dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
     if ws is None:
         ws = default_workspace(x.device)
     a = GemmArgs()
@@ -272,8 +309,120 @@ def gemm(x: torch.Tensor, w: PackedWeight, out: Optional[torch.Tensor] = None, r
     a.w_kb_stride = int(getattr(w, "kb_stride", 0) or 0)
     a.w_tiled = 1 if (w.tiled and w.mode in (W_BF16, W_F16)) else 0
     a.comm = C.addressof(comm) if comm is not None else None
+    if act == ACT_GLU_LIMITED:
+        a.act_limit, a.act_slope, a.act_shift = glu
     _check(lib().ovb_gemm(C.byref(a), C.c_void_p(_stream())), "ovb_gemm")
     return out
+
+
+def _gemm_f32(x: torch.Tensor, w: "PackedWeight", out: Optional[torch.Tensor], act: int = ACT_NONE) -> torch.Tensor:
+    T, K = x.shape
+    if out is None:
+        out = torch.empty((T, w.N), dtype=torch.float32, device=x.device)
+    _check(lib().ovb_gemm_f32(C.c_void_p(x.data_ptr()), C.c_void_p(w.w.data_ptr()), C.c_void_p(_ptr(w.bias)), C.c_void_p(out.data_ptr()), C.c_int(1),
+                              C.c_longlong(0), C.c_longlong(0), C.c_longlong(0), C.c_longlong(0), C.c_int(T), C.c_int(w.N), C.c_int(K), C.c_int(x.stride(0)),
+                              C.c_int(K), C.c_int(out.stride(0)), C.c_int(act), C.c_void_p(_stream())), "ovb_gemm_f32")
+    return out
+
+
+class BlockDiagWeight:
+    """Independent products side by side: group g maps K columns of x (starting at column g * pitch) to N columns of out.
+
+    ``w`` is [G, N, K]. 16-bit weights are tile-packed, every group padded to whole 128-row tiles and K to 64 columns with zeros;
+    what the last k-block of a group reads of its neighbour's columns is multiplied by those zeros (and must be finite)."""
+
+    def __init__(self, w: torch.Tensor):
+        self.G, self.N, self.K = w.shape
+        if w.dtype == torch.float32:
+            self.mode, self.w, self.packed = W_F32, w.contiguous(), None
+            return
+        Np, Kp = (self.N + 127) // 128 * 128, (self.K + 63) // 64 * 64
+        full = torch.zeros((self.G, Np, Kp), dtype=w.dtype, device=w.device)
+        full[:, :self.N, :self.K] = w
+        self.mode, self.packed = W_BF16, PackedWeight.from_dense(full.reshape(self.G * Np, Kp))
+
+
+def gemm_block_diag(x: torch.Tensor, w: BlockDiagWeight, out: torch.Tensor, x_pitch: int, out_pitch: int, ws: Optional[Workspace] = None) -> torch.Tensor:
+    """out[:, g * out_pitch + n] = sum_k x[:, g * x_pitch + k] * w[g, n, k] for all groups in one launch."""
+    T = x.shape[0]
+    if w.mode == W_F32:
+        _check(lib().ovb_gemm_f32(C.c_void_p(x.data_ptr()), C.c_void_p(w.w.data_ptr()), C.c_void_p(None), C.c_void_p(out.data_ptr()), C.c_int(w.G),
+                                  C.c_longlong(x_pitch), C.c_longlong(w.N * w.K), C.c_longlong(0), C.c_longlong(out_pitch), C.c_int(T), C.c_int(w.N),
+                                  C.c_int(w.K), C.c_int(x.stride(0)), C.c_int(w.K), C.c_int(out.stride(0)), C.c_int(ACT_NONE), C.c_void_p(_stream())),
+               "ovb_gemm_f32 (block-diagonal)")
+        return out
+    if ws is None:
+        ws = default_workspace(x.device)
+    a = GemmArgs()
+    a.x, a.w, a.out = x.data_ptr(), w.packed.w.data_ptr(), out.data_ptr()
+    a.ws, a.counters, a.ws_bytes = ws.gemm_ws.data_ptr(), ws.counters.data_ptr(), ws.gemm_ws.numel() * 4
+    a.T, a.N, a.K = T, w.N, w.packed.K
+    a.ldx, a.ldo, a.x_cols = x.stride(0), out.stride(0), x.shape[1]
+    a.wmode, a.act, a.out_f32, a.splits, a.w_tiled = W_BF16, ACT_NONE, 1 if out.dtype == torch.float32 else 0, 1, 1
+    a.num_groups, a.group_mode, a.group_ldx, a.group_ldo = w.G, 3, x_pitch, out_pitch
+    _check(lib().ovb_gemm(C.byref(a), C.c_void_p(_stream())), "ovb_gemm (block-diagonal)")
+    return out
+
+
+def storage_type(dtype: torch.dtype) -> int:
+    return {torch.float32: DT_F32, torch.bfloat16: DT_BF16}[dtype]
+
+
+def stream_embed(ids, table, h, x=None):
+    """h[r] = table[ids[r]] in fp32; ``x`` (optional) gets the row in the table's type."""
+    vocab, cols = table.shape
+    _check(lib().ovb_stream_embed(C.c_void_p(ids.data_ptr()), C.c_void_p(table.data_ptr()), C.c_void_p(h.data_ptr()), C.c_void_p(_ptr(x)), C.c_int(ids.numel()),
+                                  C.c_int(cols), C.c_int(vocab), C.c_int(table.stride(0)), C.c_int(h.stride(0)), C.c_int(x.stride(0) if x is not None else 0),
+                                  C.c_int(storage_type(table.dtype)), C.c_void_p(_stream())), "ovb_stream_embed")
+
+
+def sum_rmsnorm(h, w, eps, cols, rows=None, y=None, alpha=1.0, w_offset=0.0, h_out=None, x_out=None, row_idx=None):
+    """s = alpha * h (+ y); s / sqrt(mean(s^2) + eps) * (w_offset + w) to ``h_out`` (fp32) and / or ``x_out``. ``w`` is padded with
+    zeros to a multiple of four; ``row_idx`` gathers rows of h."""
+    rows = (row_idx if row_idx is not None else h).shape[0] if rows is None else rows
+    ld = lambda t: C.c_int(t.stride(0) if t is not None else 0)
+    _check(lib().ovb_sum_rmsnorm(C.c_void_p(h.data_ptr()), C.c_void_p(_ptr(row_idx)), C.c_void_p(_ptr(y)), C.c_void_p(w.data_ptr()), C.c_void_p(_ptr(h_out)),
+                                 C.c_void_p(_ptr(x_out)), C.c_int(rows), C.c_int(cols), ld(h), ld(y), ld(h_out), ld(x_out), C.c_float(alpha), C.c_float(w_offset),
+                                 C.c_float(eps), C.c_int(storage_type(x_out.dtype if x_out is not None else torch.float32)), C.c_void_p(_stream())),
+           "ovb_sum_rmsnorm")
+
+
+def glu_limited(gu, out, F, up_off, limit, slope=1.702, shift=1.0):
+    _check(lib().ovb_glu_limited(C.c_void_p(gu.data_ptr()), C.c_void_p(out.data_ptr()), C.c_int(gu.shape[0]), C.c_int(F), C.c_int(up_off), C.c_int(gu.stride(0)),
+                                 C.c_int(out.stride(0)), C.c_float(limit), C.c_float(slope), C.c_float(shift), C.c_int(storage_type(gu.dtype)),
+                                 C.c_void_p(_stream())), "ovb_glu_limited")
+    return out
+
+
+def _fill(args, values):
+    for k, v in values.items():
+        setattr(args, k, v.data_ptr() if isinstance(v, torch.Tensor) else v)
+    return args
+
+
+def heads_prepare(**kw) -> None:
+    """Head norms, rotation and cache rows of grouped-query attention; fields of ``ovb_heads_args``."""
+    _check(lib().ovb_heads_prepare(C.byref(_fill(HeadsArgs(), kw)), C.c_void_p(_stream())), "ovb_heads_prepare")
+
+
+def latent_prepare(**kw) -> None:
+    """Cache row and turned query parts of latent attention; fields of ``ovb_latent_args``."""
+    _check(lib().ovb_latent_prepare(C.byref(_fill(LatentArgs(), kw)), C.c_void_p(_stream())), "ovb_latent_prepare")
+
+
+def window_attention(**kw) -> None:
+    """Paged attention with separate key / value sizes, window and output gate; fields of ``ovb_wattn_args``."""
+    _check(lib().ovb_window_attention(C.byref(_fill(WindowAttnArgs(), kw)), C.c_void_p(_stream())), "ovb_window_attention")
+
+
+def causal_conv(**kw) -> None:
+    """Short causal convolution of a ragged batch; fields of ``ovb_rglru_args``."""
+    _check(lib().ovb_causal_conv(C.byref(_fill(RgLruArgs(), kw)), C.c_void_p(_stream())), "ovb_causal_conv")
+
+
+def lru_scan(**kw) -> None:
+    """Real-gated linear recurrent unit of a ragged batch; fields of ``ovb_rglru_args``."""
+    _check(lib().ovb_lru_scan(C.byref(_fill(RgLruArgs(), kw)), C.c_void_p(_stream())), "ovb_lru_scan")
 
 
 def rmsnorm(x, gamma, eps, residual=None, out=None, residual_out=None):
@@ -425,11 +574,12 @@ def pack_conv_weight(w: torch.Tensor, bias=None) -> "PackedWeight":
 
 def sample(logits: torch.Tensor, temperature: float, top_k: int = 0, top_p: float = 1.0, seed: int = 0, step: Optional[torch.Tensor] = None,
            out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Draw one token per row of bf16 ``logits`` [rows, V]; ``step``: device int32 word mixed into the random stream."""
+    """Draw one token per row of bf16 or fp32 ``logits`` [rows, V]; ``step``: device int32 word mixed into the random stream."""
     rows, V = logits.shape
     if out is None:
         out = torch.empty(rows, dtype=torch.int32, device=logits.device)
-    _check(lib().ovb_sample(C.c_void_p(logits.data_ptr()), C.c_int(logits.stride(0)), C.c_int(rows), C.c_int(V), C.c_float(temperature),
+    fn = lib().ovb_sample_f32 if logits.dtype == torch.float32 else lib().ovb_sample
+    _check(fn(C.c_void_p(logits.data_ptr()), C.c_int(logits.stride(0)), C.c_int(rows), C.c_int(V), C.c_float(temperature),
                             C.c_int(top_k), C.c_float(top_p), C.c_uint64(seed & 0xFFFFFFFFFFFFFFFF), C.c_void_p(_ptr(step)),
                             C.c_void_p(out.data_ptr()), C.c_void_p(_stream())), "ovb_sample")
     return out
@@ -556,7 +706,8 @@ def argmax(logits, out=None, out_max=None):
     rows, vocab = logits.shape
     if out is None:
         out = torch.empty(rows, dtype=torch.int64, device=logits.device)
-    _check(lib().ovb_argmax(C.c_void_p(logits.data_ptr()), C.c_int(logits.stride(0)), C.c_int(rows), C.c_int(vocab),
+    fn = lib().ovb_argmax_f32 if logits.dtype == torch.float32 else lib().ovb_argmax
+    _check(fn(C.c_void_p(logits.data_ptr()), C.c_int(logits.stride(0)), C.c_int(rows), C.c_int(vocab),
                             C.c_void_p(out.data_ptr()), C.c_int(1 if out.dtype == torch.int32 else 0),
                             C.c_void_p(_ptr(out_max)), C.c_void_p(_stream())), "ovb_argmax")
     return out

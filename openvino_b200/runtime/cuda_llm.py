@@ -171,15 +171,18 @@ class StepBuffers:
 
     Descriptor layout (int32 words): ids[Tcap] positions[Tcap] slot_map[Tcap] tok_src[Tcap] tok_dst[Bcap] logit_idx[Bcap]
     past_lens[Bcap] subsequence_begins[Bcap+1] block_indices_begins[Bcap+1] block_indices[Bcap*max_blocks].
-    The host fills a pinned mirror and uploads it with ONE copy per step.
+    ``state_slots`` adds state_slots[Bcap], the slot of every sequence's recurrent state. The host fills a pinned mirror and
+    uploads it with ONE copy per step. The activations are the subclass's.
     """
 
-    def __init__(self, cfg: LlmConfig, Tcap: int, Bcap: int, max_blocks_per_seq: int, device, tp_size: int = 1, comm=None):
+    def __init__(self, Tcap: int, Bcap: int, max_blocks_per_seq: int, device, vocab: int, logits_dtype=torch.bfloat16, state_slots: bool = False):
         self.Tcap, self.Bcap, self.max_blocks = Tcap, Bcap, max_blocks_per_seq
         sizes = [("ids", Tcap), ("positions", Tcap), ("slot_map", Tcap), ("tok_src", Tcap), ("tok_dst", Bcap),
                  ("logit_idx", Bcap), ("past_lens", Bcap),
                  ("subsequence_begins", Bcap + 1), ("block_indices_begins", Bcap + 1),
                  ("block_indices", Bcap * max_blocks_per_seq)]
+        if state_slots:
+            sizes.append(("state_slots", Bcap))
         self.offsets, off = {}, 0
         for name, n in sizes:
             self.offsets[name] = (off, n)
@@ -189,6 +192,22 @@ class StepBuffers:
         pin = (lambda t: t.pin_memory()) if torch.cuda.is_available() else (lambda t: t)
         # two pinned mirrors: the host fills one while the upload of the other may still be in flight
         self.desc_hosts = [pin(torch.zeros(off, dtype=torch.int32)) for _ in range(2)]
+        self.logits = torch.empty((Bcap, vocab), dtype=logits_dtype, device=device)
+        self.tokens = torch.zeros(Bcap, dtype=torch.int32, device=device)
+        self.tokens_host = [pin(torch.zeros(Bcap, dtype=torch.int32)) for _ in range(2)]
+        self.logit_max = torch.empty(Bcap, dtype=torch.float32, device=device)
+
+    def view(self, name: str, host=None) -> torch.Tensor:
+        """Field of the device descriptor (host=None) or of pinned mirror ``host`` (0 or 1)."""
+        off, n = self.offsets[name]
+        return (self.desc if host is None else self.desc_hosts[int(host)])[off:off + n]
+
+
+class LlamaStepBuffers(StepBuffers):
+    """Step buffers of a Llama-family decoder: descriptor plus bf16 activations."""
+
+    def __init__(self, cfg: LlmConfig, Tcap: int, Bcap: int, max_blocks_per_seq: int, device, tp_size: int = 1, comm=None):
+        super().__init__(Tcap, Bcap, max_blocks_per_seq, device, cfg.vocab_size // tp_size)
         H, D = cfg.hidden_size, cfg.head_dim
         hq, hkv, ffn = cfg.num_heads // tp_size, cfg.num_kv_heads // tp_size, cfg.ffn_size // tp_size
         bf = dict(dtype=torch.bfloat16, device=device)
@@ -221,15 +240,6 @@ class StepBuffers:
             self.act = torch.empty((Tcap, ffn), **bf)
         self.last_h = torch.empty((Bcap, H), **bf)
         self.last_x = torch.empty((Bcap, H), **bf)
-        self.logits = torch.empty((Bcap, cfg.vocab_size // tp_size), **bf)
-        self.tokens = torch.zeros(Bcap, dtype=torch.int32, device=device)
-        self.tokens_host = [pin(torch.zeros(Bcap, dtype=torch.int32)) for _ in range(2)]
-        self.logit_max = torch.empty(Bcap, dtype=torch.float32, device=device)
-
-    def view(self, name: str, host=None) -> torch.Tensor:
-        """Field of the device descriptor (host=None) or of pinned mirror ``host`` (0 or 1)."""
-        off, n = self.offsets[name]
-        return (self.desc if host is None else self.desc_hosts[int(host)])[off:off + n]
 
 
 @dataclass
@@ -241,58 +251,43 @@ class StepShape:
 
 
 # ----------------------------------------------------------------------------------------- executor
-class CudaLlmExecutor:
-    """Runs steps of a decoder-only model on one GPU (one tensor-parallel rank)."""
+class LlmExecutor:
+    """What every serving program shares: the step buffers' life cycle, CUDA graphs of decode steps, sampling and the device-side
+    token feedback. A subclass allocates its cache and step buffers (``prefill``, ``decode``) and runs its layers in
+    ``_forward``, which ends with ``_sample``."""
 
-    def __init__(self, cfg: LlmConfig, weights: LlmWeights, num_kv_blocks: int, block_size: int = 16,
-                 max_batch_tokens: int = 8192, max_seqs: int = 64, max_blocks_per_seq: int = 0, device="cuda",
-                 comm=None, use_cuda_graphs: bool = True, kv_cache_precision: str = "bf16"):
-        self.cfg, self.w = cfg, weights
-        self.kv_u8 = str(kv_cache_precision).lower() == "u8"
-        if self.kv_u8 and (cfg.head_dim != 128 or block_size != 16):
-            raise ValueError("the u8 KV cache is served for head size 128 and 16-token blocks")
+    has_recurrent_state = False
+
+    def __init__(self, cfg, num_kv_blocks: int, block_size: int, max_seqs: int, max_blocks_per_seq: int, device, use_cuda_graphs: bool = True,
+                 tp_size: int = 1, tp_rank: int = 0, comm=None):
+        self.cfg = cfg
         self.device = torch.device(device)
         self.block_size = block_size
         self.num_kv_blocks = num_kv_blocks
-        self.tp_size, self.tp_rank = weights.tp_size, weights.tp_rank
+        self.tp_size, self.tp_rank = tp_size, tp_rank
         self.comm = comm
         self.use_cuda_graphs = use_cuda_graphs
-        self.hq = cfg.num_heads // self.tp_size
-        self.hkv = cfg.num_kv_heads // self.tp_size
         self.max_seqs = max_seqs
         if max_blocks_per_seq <= 0:
             max_blocks_per_seq = max(1, num_kv_blocks // max(1, max_seqs)) + 1
         self.max_blocks_per_seq = max_blocks_per_seq
-        # KV_CACHE_PRECISION = u8: rows are stored as bytes with one fp16 (scale, zero point) pair per (block, head, slot):
-        # half the cache memory and half the decode traffic of the 16-bit cache
-        self.k_cache = [torch.zeros((num_kv_blocks, self.hkv, block_size, cfg.head_dim), dtype=torch.uint8 if self.kv_u8 else torch.bfloat16,
-                                    device=self.device) for _ in range(cfg.num_layers)]
-        self.v_cache = [torch.zeros_like(k) for k in self.k_cache]
-        self.k_meta = [torch.zeros((num_kv_blocks, self.hkv, block_size, 2), dtype=torch.float16, device=self.device) if self.kv_u8 else None
-                       for _ in range(cfg.num_layers)]
-        self.v_meta = [torch.zeros_like(m) if m is not None else None for m in self.k_meta]
         self.ws = K.Workspace(self.device)
-        if self.tp_size > 1:
-            if comm is None:
-                raise ValueError("tensor-parallel weights need a communicator")
-            moe_rows = max_batch_tokens + 1 if (cfg.num_experts and max_batch_tokens >= MOE_GATHER_MIN_TOKENS) else 0
-            comm.setup(cfg.hidden_size, max_batch_tokens, cfg.num_layers,
-                       tensor_bytes=(max_batch_tokens + max_seqs + 2 + moe_rows) * cfg.hidden_size * 2 + 8192
-                       + max_seqs * cfg.vocab_size * 2 + 4096)
-        self.prefill = StepBuffers(cfg, max_batch_tokens, max_seqs, max_blocks_per_seq, self.device, self.tp_size, comm if self.tp_size > 1 else None)
-        self.decode = StepBuffers(cfg, max_seqs, max_seqs, max_blocks_per_seq, self.device, self.tp_size, comm if self.tp_size > 1 else None)
-        # top-k / top-p under tensor parallelism need the whole row: every rank places its vocabulary shard into a zeroed
-        # full-width buffer in the symmetric heap and the ranks sum the buffers (adding zeros is exact in bf16)
-        self.full_logits = comm.alloc((max(max_seqs, 1), cfg.vocab_size)) if self.tp_size > 1 else None
-        # token sampled last for every request slot (device-side feedback between chained steps)
-        self.last_token = torch.zeros(max(max_seqs, 1) * 4, dtype=torch.int32, device=self.device)
+        # request slots of the scheduler; token sampled last for every slot (device-side feedback between chained steps)
+        self.num_slots = max(max_seqs, 1) * 4
+        self.last_token = torch.zeros(self.num_slots, dtype=torch.int32, device=self.device)
         self._graphs = {}
-        self._expert_windows = {}
         self.kernel_launches = 0
         # sampling: None = greedy; (temperature, top_k, top_p, seed) = stochastic. The step word is
         # bumped on the device before every draw, so replays of a captured decode graph keep drawing fresh numbers.
         self.sampling = None
         self.sample_step = torch.zeros(1, dtype=torch.int32, device=self.device)
+
+    def _forward(self, sb: StepBuffers, shp: "StepShape") -> None:
+        raise NotImplementedError
+
+    def _recurrent_state(self) -> List[torch.Tensor]:
+        """Tensors that a step advances in place (running the same step twice would advance them twice)."""
+        return []
 
     def set_sampling(self, temperature: float = 0.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> None:
         new = None if temperature <= 0 else (float(temperature), int(top_k), float(top_p), int(seed))
@@ -302,6 +297,131 @@ class CudaLlmExecutor:
         if new != self.sampling:
             self._graphs.clear()       # captured decode graphs embed the sampling kernel
         self.sampling = new
+
+    def _sample(self, sb: StepBuffers, B: int) -> None:
+        if self.sampling is not None:
+            temp, top_k, top_p, seed = self.sampling
+            K.bump(self.sample_step)
+            if self.tp_size > 1 and (top_k > 0 or top_p < 1.0):
+                # truncated sampling needs the whole row: gather the shards (sum of zero-padded rows over the ranks), then
+                # every rank runs the same draw with the same seed and step, so all ranks get the same tokens
+                shard = self.cfg.vocab_size // self.tp_size
+                full = self.full_logits[:B]
+                full.zero_()
+                full[:, self.w.tp_rank * shard:(self.w.tp_rank + 1) * shard].copy_(sb.logits[:B])
+                self.kernel_launches += 2 + self.comm.all_reduce_large(full)
+                K.sample(full, temp, top_k, top_p, seed, self.sample_step, out=sb.tokens[:B])
+            elif self.tp_size > 1:
+                # every rank perturbs its vocabulary shard with noise that depends on the global token index, then the
+                # ranks exchange (best value, index): a draw from the full softmax without gathering the logits
+                shard = self.cfg.vocab_size // self.tp_size
+                K.sample_gumbel(sb.logits[:B], temp, seed, self.sample_step, vocab_offset=self.w.tp_rank * shard, out=sb.tokens[:B],
+                                out_max=sb.logit_max[:B])
+                self.comm.argmax_combine(sb.tokens[:B], sb.logit_max[:B], shard)
+            else:
+                K.sample(sb.logits[:B], temp, top_k, top_p, seed, self.sample_step, out=sb.tokens[:B])
+            self.kernel_launches += 1
+        elif self.tp_size == 1:
+            K.argmax(sb.logits[:B], out=sb.tokens[:B])
+        else:
+            K.argmax(sb.logits[:B], out=sb.tokens[:B], out_max=sb.logit_max[:B])
+            self.comm.argmax_combine(sb.tokens[:B], sb.logit_max[:B], self.cfg.vocab_size // self.tp_size)
+        K.scatter_tokens(sb.tokens[:B], sb.view("tok_dst")[:B], self.last_token)
+
+    # -- public: run one step whose descriptor already sits in sb.desc (device)
+    def run(self, sb: StepBuffers, shp: StepShape) -> torch.Tensor:
+        decode = sb is self.decode and shp.max_q_len == 1
+        if decode and self.use_cuda_graphs:
+            ctx_bucket = max(256, 1 << (max(1, shp.max_ctx) - 1).bit_length())
+            key = (shp.B, ctx_bucket)
+            g = self._graphs.get(key)
+            if g is None:
+                g = self._capture(sb, StepShape(shp.T, shp.B, 1, ctx_bucket))
+                self._graphs[key] = g
+            g.replay()
+            self.kernel_launches += self._graph_launches
+        else:
+            self._forward(sb, shp)
+        return sb.tokens[:shp.B]
+
+    def _capture(self, sb: StepBuffers, shp: StepShape):
+        # warm-up outside capture (first-use setup such as function attributes), then capture
+        s = torch.cuda.Stream(device=self.device)
+        s.wait_stream(torch.cuda.current_stream())
+        saved, saved_last = sb.desc.clone(), self.last_token.clone()
+        saved_state = [t.clone() for t in self._recurrent_state()]
+        with torch.cuda.stream(s):
+            self._forward(sb, shp)
+        torch.cuda.current_stream().wait_stream(s)
+        torch.cuda.synchronize()
+        # undo the warm-up's side effects on the feedback state; the KV rows it wrote are rewritten with
+        # the same values by the real step
+        sb.desc.copy_(saved)
+        self.last_token.copy_(saved_last)
+        for t, v in zip(self._recurrent_state(), saved_state):
+            t.copy_(v)
+        before = self.kernel_launches
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self._forward(sb, shp)
+        self._graph_launches = self.kernel_launches - before
+        self.kernel_launches = before
+        return g
+
+    # -- host side helpers -------------------------------------------------------------------
+    def upload(self, sb: StepBuffers, mirror: int = 0) -> int:
+        """One H2D copy of a pinned descriptor mirror. Returns bytes copied."""
+        sb.desc.copy_(sb.desc_hosts[mirror], non_blocking=True)
+        return sb.desc_words * 4
+
+    def download_tokens_async(self, sb: StepBuffers, B: int, mirror: int = 0) -> "torch.cuda.Event":
+        """Queue the D2H copy of the sampled tokens into pinned buffer ``mirror``; the returned event
+        completes when the values are readable on the host."""
+        sb.tokens_host[mirror][:B].copy_(sb.tokens[:B], non_blocking=True)
+        ev = torch.cuda.Event()
+        ev.record()
+        return ev
+
+    def download_tokens(self, sb: StepBuffers, B: int, mirror: int = 0) -> torch.Tensor:
+        self.download_tokens_async(sb, B, mirror).synchronize()
+        return sb.tokens_host[mirror][:B]
+
+
+class CudaLlmExecutor(LlmExecutor):
+    """Runs steps of a decoder-only model on one GPU (one tensor-parallel rank)."""
+
+    def __init__(self, cfg: LlmConfig, weights: LlmWeights, num_kv_blocks: int, block_size: int = 16,
+                 max_batch_tokens: int = 8192, max_seqs: int = 64, max_blocks_per_seq: int = 0, device="cuda",
+                 comm=None, use_cuda_graphs: bool = True, kv_cache_precision: str = "bf16"):
+        self.w = weights
+        self.kv_u8 = str(kv_cache_precision).lower() == "u8"
+        if self.kv_u8 and (cfg.head_dim != 128 or block_size != 16):
+            raise ValueError("the u8 KV cache is served for head size 128 and 16-token blocks")
+        super().__init__(cfg, num_kv_blocks, block_size, max_seqs, max_blocks_per_seq, device, use_cuda_graphs, weights.tp_size, weights.tp_rank, comm)
+        max_blocks_per_seq = self.max_blocks_per_seq
+        self.hq = cfg.num_heads // self.tp_size
+        self.hkv = cfg.num_kv_heads // self.tp_size
+        # KV_CACHE_PRECISION = u8: rows are stored as bytes with one fp16 (scale, zero point) pair per (block, head, slot):
+        # half the cache memory and half the decode traffic of the 16-bit cache
+        self.k_cache = [torch.zeros((num_kv_blocks, self.hkv, block_size, cfg.head_dim), dtype=torch.uint8 if self.kv_u8 else torch.bfloat16,
+                                    device=self.device) for _ in range(cfg.num_layers)]
+        self.v_cache = [torch.zeros_like(k) for k in self.k_cache]
+        self.k_meta = [torch.zeros((num_kv_blocks, self.hkv, block_size, 2), dtype=torch.float16, device=self.device) if self.kv_u8 else None
+                       for _ in range(cfg.num_layers)]
+        self.v_meta = [torch.zeros_like(m) if m is not None else None for m in self.k_meta]
+        if self.tp_size > 1:
+            if comm is None:
+                raise ValueError("tensor-parallel weights need a communicator")
+            moe_rows = max_batch_tokens + 1 if (cfg.num_experts and max_batch_tokens >= MOE_GATHER_MIN_TOKENS) else 0
+            comm.setup(cfg.hidden_size, max_batch_tokens, cfg.num_layers,
+                       tensor_bytes=(max_batch_tokens + max_seqs + 2 + moe_rows) * cfg.hidden_size * 2 + 8192
+                       + max_seqs * cfg.vocab_size * 2 + 4096)
+        self.prefill = LlamaStepBuffers(cfg, max_batch_tokens, max_seqs, max_blocks_per_seq, self.device, self.tp_size, comm if self.tp_size > 1 else None)
+        self.decode = LlamaStepBuffers(cfg, max_seqs, max_seqs, max_blocks_per_seq, self.device, self.tp_size, comm if self.tp_size > 1 else None)
+        # top-k / top-p under tensor parallelism need the whole row: every rank places its vocabulary shard into a zeroed
+        # full-width buffer in the symmetric heap and the ranks sum the buffers (adding zeros is exact in bf16)
+        self.full_logits = comm.alloc((max(max_seqs, 1), cfg.vocab_size)) if self.tp_size > 1 else None
+        self._expert_windows = {}
 
     # -- one forward pass over the buffers of `sb`
     def _forward(self, sb: StepBuffers, shp: StepShape) -> None:
@@ -404,91 +524,6 @@ class CudaLlmExecutor:
             K.gemm(x, wt, out=h, residual=h, ws=self.ws)
         else:
             self.comm.gemm_allreduce(x, wt, h, self.ws, site)
-
-    def _sample(self, sb: StepBuffers, B: int) -> None:
-        if self.sampling is not None:
-            temp, top_k, top_p, seed = self.sampling
-            K.bump(self.sample_step)
-            if self.tp_size > 1 and (top_k > 0 or top_p < 1.0):
-                # truncated sampling needs the whole row: gather the shards (sum of zero-padded rows over the ranks), then
-                # every rank runs the same draw with the same seed and step, so all ranks get the same tokens
-                shard = self.cfg.vocab_size // self.tp_size
-                full = self.full_logits[:B]
-                full.zero_()
-                full[:, self.w.tp_rank * shard:(self.w.tp_rank + 1) * shard].copy_(sb.logits[:B])
-                self.kernel_launches += 2 + self.comm.all_reduce_large(full)
-                K.sample(full, temp, top_k, top_p, seed, self.sample_step, out=sb.tokens[:B])
-            elif self.tp_size > 1:
-                # every rank perturbs its vocabulary shard with noise that depends on the global token index, then the
-                # ranks exchange (best value, index): a draw from the full softmax without gathering the logits
-                shard = self.cfg.vocab_size // self.tp_size
-                K.sample_gumbel(sb.logits[:B], temp, seed, self.sample_step, vocab_offset=self.w.tp_rank * shard, out=sb.tokens[:B],
-                                out_max=sb.logit_max[:B])
-                self.comm.argmax_combine(sb.tokens[:B], sb.logit_max[:B], shard)
-            else:
-                K.sample(sb.logits[:B], temp, top_k, top_p, seed, self.sample_step, out=sb.tokens[:B])
-            self.kernel_launches += 1
-        elif self.tp_size == 1:
-            K.argmax(sb.logits[:B], out=sb.tokens[:B])
-        else:
-            K.argmax(sb.logits[:B], out=sb.tokens[:B], out_max=sb.logit_max[:B])
-            self.comm.argmax_combine(sb.tokens[:B], sb.logit_max[:B], self.cfg.vocab_size // self.tp_size)
-        K.scatter_tokens(sb.tokens[:B], sb.view("tok_dst")[:B], self.last_token)
-
-    # -- public: run one step whose descriptor already sits in sb.desc (device)
-    def run(self, sb: StepBuffers, shp: StepShape) -> torch.Tensor:
-        decode = sb is self.decode and shp.max_q_len == 1
-        if decode and self.use_cuda_graphs:
-            ctx_bucket = max(256, 1 << (max(1, shp.max_ctx) - 1).bit_length())
-            key = (shp.B, ctx_bucket)
-            g = self._graphs.get(key)
-            if g is None:
-                g = self._capture(sb, StepShape(shp.T, shp.B, 1, ctx_bucket))
-                self._graphs[key] = g
-            g.replay()
-            self.kernel_launches += self._graph_launches
-        else:
-            self._forward(sb, shp)
-        return sb.tokens[:shp.B]
-
-    def _capture(self, sb: StepBuffers, shp: StepShape):
-        # warm-up outside capture (first-use setup such as function attributes), then capture
-        s = torch.cuda.Stream(device=self.device)
-        s.wait_stream(torch.cuda.current_stream())
-        saved, saved_last = sb.desc.clone(), self.last_token.clone()
-        with torch.cuda.stream(s):
-            self._forward(sb, shp)
-        torch.cuda.current_stream().wait_stream(s)
-        torch.cuda.synchronize()
-        # undo the warm-up's side effects on the feedback state; the KV rows it wrote are rewritten with
-        # the same values by the real step
-        sb.desc.copy_(saved)
-        self.last_token.copy_(saved_last)
-        before = self.kernel_launches
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._forward(sb, shp)
-        self._graph_launches = self.kernel_launches - before
-        self.kernel_launches = before
-        return g
-
-    # -- host side helpers -------------------------------------------------------------------
-    def upload(self, sb: StepBuffers, mirror: int = 0) -> int:
-        """One H2D copy of a pinned descriptor mirror. Returns bytes copied."""
-        sb.desc.copy_(sb.desc_hosts[mirror], non_blocking=True)
-        return sb.desc_words * 4
-
-    def download_tokens_async(self, sb: StepBuffers, B: int, mirror: int = 0) -> "torch.cuda.Event":
-        """Queue the D2H copy of the sampled tokens into pinned buffer ``mirror``; the returned event
-        completes when the values are readable on the host."""
-        sb.tokens_host[mirror][:B].copy_(sb.tokens[:B], non_blocking=True)
-        ev = torch.cuda.Event()
-        ev.record()
-        return ev
-
-    def download_tokens(self, sb: StepBuffers, B: int, mirror: int = 0) -> torch.Tensor:
-        self.download_tokens_async(sb, B, mirror).synchronize()
-        return sb.tokens_host[mirror][:B]
 
     def kv_cache_bytes(self) -> int:
         return sum(2 * k.numel() * k.element_size() + (2 * m.numel() * 2 if m is not None else 0) for k, m in zip(self.k_cache, self.k_meta))

@@ -1,0 +1,352 @@
+"""Serving program of layered decoders (``LayeredConfig``): every layer is a token mixer and an optional feed-forward with sizes of
+their own, the residual stream is fp32 and each sum is followed by a norm.
+
+The executor shares step descriptors, paging, CUDA graphs, sampling and token feedback with the other programs (``LlmExecutor``)
+and adds per-layer caches: key / value pages of grouped-query attention, one row per token of latent attention, and fp32
+recurrent state per request slot. Matrix products and activations are bf16 (fp32 accumulation), or everything is fp32 with
+``dtype=torch.float32``.
+
+Layout rules. Row pitches are multiples of 64 elements and heads are padded to 16, so that the tensor-core kernels read whole
+fragments; weights carry zeros at the padding and every buffer starts out as zeros, so padding never contributes.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Optional
+
+import torch
+
+from ..models.llm_config import AttentionSpec, LatentAttentionSpec, LayeredConfig, LimitedGluSpec, RgLruSpec, RotarySpec
+from ..models.registry import Checkpoint
+from ..ops import cuda as K
+from .cuda_llm import LlmExecutor, StepBuffers, StepShape
+
+
+def _up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+def _pad_rows(w: torch.Tensor, groups: int, pitch: int) -> torch.Tensor:
+    """[groups * n, K] -> [groups * pitch, K] with zero rows behind every group's n."""
+    n = w.shape[0] // groups
+    return torch.nn.functional.pad(w.reshape(groups, n, -1), (0, 0, 0, pitch - n)).reshape(groups * pitch, -1)
+
+
+def _pad_cols(w: torch.Tensor, groups: int, pitch: int) -> torch.Tensor:
+    N, n = w.shape[0], w.shape[1] // groups
+    return torch.nn.functional.pad(w.reshape(N, groups, n), (0, pitch - n)).reshape(N, groups * pitch)
+
+
+class _Packer:
+    """Checkpoint tensors of one layer -> device tensors in kernel layout, in the compute type."""
+
+    def __init__(self, ckpt: Checkpoint, layer: int, device, dtype: torch.dtype):
+        self.ckpt, self.layer, self.device, self.dtype = ckpt, layer, device, dtype
+
+    def raw(self, part: str, key: str) -> torch.Tensor:
+        return self.ckpt(self.layer, part, key).to(self.device)
+
+    def f32(self, part: str, key: str, pad_to: int = 1) -> torch.Tensor:
+        t = self.raw(part, key).float().reshape(-1)
+        return torch.nn.functional.pad(t, (0, _up(t.numel(), pad_to) - t.numel())).contiguous()
+
+    def linear(self, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> K.PackedWeight:
+        """[N, K] with K padded to the pitch of its input."""
+        w = torch.nn.functional.pad(w.to(self.dtype), (0, _up(w.shape[1], 64) - w.shape[1])).contiguous()
+        bias = bias.to(self.dtype).contiguous() if bias is not None else None
+        if self.dtype == torch.float32:
+            return K.PackedWeight(K.W_F32, w, w.shape[0], w.shape[1], bias=bias)
+        return K.PackedWeight.from_dense(w, bias=bias)
+
+    def block_diag(self, w: torch.Tensor) -> K.BlockDiagWeight:
+        return K.BlockDiagWeight(w.to(self.dtype).contiguous())
+
+
+class _Rotation:
+    def __init__(self, rot: Optional[RotarySpec], device):
+        self.dims = rot.dims if rot else 0
+        self.mult = rot.multiplier() if rot else 1.0
+        self.inv_freq = torch.tensor(rot.inv_freq(), dtype=torch.float64).float().to(device) if rot else None
+
+    def args(self) -> dict:
+        return dict(rot_dims=self.dims, rot_mult=self.mult, inv_freq=self.inv_freq)
+
+
+class AttentionMixer:
+    """Grouped-query attention: one product for q, k, v and the gate, norms + rotation + cache write, attention with the gate in
+    its epilogue, output projection."""
+
+    def __init__(self, s: AttentionSpec, pk: _Packer):
+        self.s, self.rot = s, _Rotation(s.rotary, pk.device)
+        self.dk, self.dv = _up(s.dim, 16), _up(s.vdim, 16)
+        parts = [_pad_rows(pk.raw("mix", "q"), s.heads, self.dk), _pad_rows(pk.raw("mix", "k"), s.kv_heads, self.dk),
+                 _pad_rows(pk.raw("mix", "v"), s.kv_heads, self.dv)]
+        if s.gated:
+            parts.append(_pad_rows(pk.raw("mix", "g"), s.heads, self.dv))
+        self.k_off = s.heads * self.dk
+        self.v_off = self.k_off + s.kv_heads * self.dk
+        self.g_off = self.v_off + s.kv_heads * self.dv
+        self.proj = pk.linear(torch.cat(parts, 0))
+        self.o = pk.linear(_pad_cols(pk.raw("mix", "o"), s.heads, self.dv))
+        self.q_norm = pk.f32("mix", "q.norm") if s.qk_norm else None
+        self.k_norm = pk.f32("mix", "k.norm") if s.qk_norm else None
+
+    def allocate(self, ex: "LayeredExecutor") -> None:
+        shape = (ex.num_kv_blocks, self.s.kv_heads, ex.block_size)
+        self.k_cache = torch.zeros(shape + (self.dk,), dtype=ex.dtype, device=ex.device)
+        self.v_cache = torch.zeros(shape + (self.dv,), dtype=ex.dtype, device=ex.device)
+
+    def state(self) -> List[torch.Tensor]:
+        return []
+
+    def cache_bytes(self) -> int:
+        return self.k_cache.nbytes + self.v_cache.nbytes
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+        s, T = self.s, shp.T
+        proj = sb.scratch("proj", T, self.proj.N)
+        K.gemm(x, self.proj, out=proj, ws=ex.ws)
+        K.heads_prepare(proj=proj, k_cache=self.k_cache, v_cache=self.v_cache, q_norm=self.q_norm, k_norm=self.k_norm, positions=sb.view("positions"),
+                        slot_map=sb.view("slot_map"), T=T, H=s.heads, G=s.kv_heads, D=s.dim, Dv=s.vdim, dk_pad=self.dk, dv_pad=self.dv, ldp=proj.stride(0),
+                        k_off=self.k_off, v_off=self.v_off, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **self.rot.args())
+        attn = sb.scratch("attn", T, self.o.K)
+        gate = dict(gate=proj[:, self.g_off:], ld_gate=proj.stride(0), gate_head=self.dv) if s.gated else {}
+        ex.attention(sb, shp, q=proj, k=self.k_cache, v=self.v_cache, out=attn, Hq=s.heads, Hkv=s.kv_heads, Dk=self.dk, Dv=s.vdim, ldq=proj.stride(0),
+                     q_head=self.dk, k_row=self.dk, v_row=self.dv, ldo=attn.stride(0), o_head=self.dv, window=s.window, scale=s.scale, **gate)
+        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
+        ex.kernel_launches += 4
+
+
+class LatentAttentionMixer:
+    """Latent attention over the cached low-rank rows. The key projection is moved to the query (q W_uk) and the value projection
+    behind the weighted sum, so that all heads attend to the one cached row per token."""
+
+    def __init__(self, s: LatentAttentionSpec, pk: _Packer):
+        self.s, self.rot = s, _Rotation(s.rotary, pk.device)
+        H, D, R, C, Dv = s.heads, s.dim, s.rot_dim, s.kv_rank, s.vdim
+        self.dp, self.rp, self.cp, self.dv = _up(D, 16), _up(R, 16), _up(C, 16), _up(Dv, 16)
+        self.q_pitch, self.row = self.dp + self.rp, self.cp + self.rp
+        q = pk.raw("mix", "q").reshape(H, D + R, -1)
+        q = torch.cat([_pad_rows(q[:, :D].reshape(H * D, -1), H, self.dp).reshape(H, self.dp, -1),
+                       _pad_rows(q[:, D:].reshape(H * R, -1), H, self.rp).reshape(H, self.rp, -1)], 1).reshape(H * self.q_pitch, -1)
+        dkv = pk.raw("mix", "dkv")
+        self.c_off = H * self.q_pitch
+        self.kr_off = self.c_off + self.cp
+        self.proj = pk.linear(torch.cat([q, _pad_rows(dkv[:C], 1, self.cp), _pad_rows(dkv[C:], 1, self.rp)], 0))
+        self.c_norm = pk.f32("mix", "dkv.norm")
+        self.uk = pk.block_diag(pk.raw("mix", "uk").reshape(H, D, C).transpose(1, 2))
+        self.uv = pk.block_diag(pk.raw("mix", "uv").reshape(H, Dv, C))
+        self.o = pk.linear(_pad_cols(pk.raw("mix", "o"), H, self.dv))
+
+    def allocate(self, ex: "LayeredExecutor") -> None:
+        self.cache = torch.zeros((ex.num_kv_blocks, ex.block_size, self.row), dtype=ex.dtype, device=ex.device)
+
+    def state(self) -> List[torch.Tensor]:
+        return []
+
+    def cache_bytes(self) -> int:
+        return self.cache.nbytes
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+        s, T, H = self.s, shp.T, self.s.heads
+        proj = sb.scratch("proj", T, self.proj.N)
+        K.gemm(x, self.proj, out=proj, ws=ex.ws)
+        q = sb.scratch("latent_q", T, H * self.row)
+        K.latent_prepare(proj=proj, q_rot=q[:, self.cp:], cache=self.cache, c_norm=self.c_norm, positions=sb.view("positions"), slot_map=sb.view("slot_map"), T=T,
+                         H=H, C=s.kv_rank, R=s.rot_dim, q_pitch=self.q_pitch, q_rot_off=self.dp, c_off=self.c_off, kr_off=self.kr_off, ldp=proj.stride(0),
+                         ld_qr=q.stride(0), qr_pitch=self.row, row_pitch=self.row, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage,
+                         eps=ex.cfg.norm_eps, **self.rot.args())
+        K.gemm_block_diag(proj[:, :self.c_off], self.uk, q, self.q_pitch, self.row, ws=ex.ws)
+        lat = sb.scratch("latent_o", T, H * self.cp)
+        ex.attention(sb, shp, q=q, k=self.cache, v=self.cache, out=lat, Hq=H, Hkv=1, Dk=self.row, Dv=s.kv_rank, ldq=q.stride(0), q_head=self.row,
+                     k_row=self.row, v_row=self.row, ldo=lat.stride(0), o_head=self.cp, window=s.window, scale=s.scale)
+        attn = sb.scratch("attn", T, self.o.K)
+        K.gemm_block_diag(lat[:, :H * self.cp], self.uv, attn, self.cp, self.dv, ws=ex.ws)
+        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
+        ex.kernel_launches += 6
+
+
+class RgLruMixer:
+    """Griffin's recurrent block: one product for both branches, convolution, block-diagonal gate product, recurrence with the
+    other branch's activation in its epilogue, output projection. State per request slot, fp32."""
+
+    def __init__(self, s: RgLruSpec, pk: _Packer):
+        self.s = s
+        N, B = s.width, s.blocks
+        if N % B:
+            raise ValueError("recurrent width %d is not a multiple of its %d blocks" % (N, B))
+        self.bw = N // B
+        self.bp, self.np = _up(self.bw, 16), _up(N, 8)
+        pad = lambda t: torch.nn.functional.pad(t, (0, self.np - N))
+        self.proj = pk.linear(torch.cat([_pad_rows(pk.raw("mix", "y"), 1, self.np), _pad_rows(pk.raw("mix", "x"), 1, self.np)], 0),
+                              torch.cat([pad(pk.raw("mix", "y.b")), pad(pk.raw("mix", "x.b"))]))
+        self.conv_w = pk.raw("mix", "conv").float().t().contiguous()          # [taps, N]
+        self.conv_b = pk.f32("mix", "conv.b")
+        ra, ri = pk.raw("mix", "ra"), pk.raw("mix", "ri")
+        grow = lambda w: torch.nn.functional.pad(w, (0, 0, 0, self.bp - self.bw))
+        self.gates = pk.block_diag(torch.cat([grow(ra), grow(ri)], 1))        # [B, 2 * bp, bw]
+        self.gate_b = torch.stack([pk.f32("mix", "ra.b"), pk.f32("mix", "ri.b")]).contiguous()
+        self.log_decay = (s.decay * torch.nn.functional.softplus(pk.raw("mix", "lam").double())).float().contiguous()
+        self.o = pk.linear(pk.raw("mix", "o"))
+
+    def allocate(self, ex: "LayeredExecutor") -> None:
+        self.lru_state = torch.zeros((ex.num_slots, self.s.width), dtype=torch.float32, device=ex.device)
+        self.conv_state = torch.zeros((ex.num_slots, max(self.s.taps - 1, 1), self.s.width), dtype=torch.float32, device=ex.device)
+
+    def state(self) -> List[torch.Tensor]:
+        return [self.lru_state, self.conv_state]
+
+    def cache_bytes(self) -> int:
+        return self.lru_state.nbytes + self.conv_state.nbytes
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+        s, T = self.s, shp.T
+        proj = sb.scratch("proj", T, self.proj.N)
+        K.gemm(x, self.proj, out=proj, ws=ex.ws)
+        u = sb.scratch("lru_u", T, s.blocks * self.bp)
+        gates = sb.scratch("lru_gates", T, s.blocks * 2 * self.bp, torch.float32)
+        out = sb.scratch("lru_out", T, self.o.K)
+        args = dict(x=proj[:, self.np:], y=proj, u=u, out=out, gates=gates, gate_b=self.gate_b, log_decay=self.log_decay, conv_w=self.conv_w,
+                    conv_b=self.conv_b, state=self.lru_state, conv_state=self.conv_state, subsequence_begins=sb.view("subsequence_begins"),
+                    past_lens=sb.view("past_lens"), slots=sb.view("state_slots"), B=shp.B, T=T, N=s.width, taps=s.taps, bw=self.bw, ub_pitch=self.bp,
+                    gb_pitch=2 * self.bp, gi_off=self.bp, ldx=proj.stride(0), ldy=proj.stride(0), ldu=u.stride(0), ldg=gates.stride(0), ldo=out.stride(0),
+                    max_q_len=shp.max_q_len, dtype=ex.storage)
+        K.causal_conv(**args)
+        K.gemm_block_diag(u, self.gates, gates, self.bp, 2 * self.bp, ws=ex.ws)
+        K.lru_scan(**args)
+        K.gemm(out, self.o, out=y, out_f32=True, ws=ex.ws)
+        ex.kernel_launches += 5
+
+
+class LimitedGlu:
+    """Gated MLP with clamped halves; in bf16 the activation runs in the epilogue of the gate / up product."""
+
+    def __init__(self, s: LimitedGluSpec, pk: _Packer):
+        self.s, self.fp = s, _up(s.ff, 64)
+        gate, up = _pad_rows(pk.raw("mlp", "gate"), 1, self.fp), _pad_rows(pk.raw("mlp", "up"), 1, self.fp)
+        self.fused = pk.dtype == torch.bfloat16
+        self.gate_up = pk.linear(K.interleave_gate_up(gate, up) if self.fused else torch.cat([gate, up], 0))
+        self.down = pk.linear(pk.raw("mlp", "down"))
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+        s, act = self.s, sb.scratch("mlp_act", shp.T, self.fp)
+        if self.fused:
+            K.gemm(x, self.gate_up, out=act, act=K.ACT_GLU_LIMITED, glu=(s.limit, s.slope, s.shift), ws=ex.ws)
+        else:
+            gu = sb.scratch("mlp_gu", shp.T, 2 * self.fp)
+            K.gemm(x, self.gate_up, out=gu, ws=ex.ws)
+            K.glu_limited(gu, act, s.ff, self.fp, s.limit, s.slope, s.shift)
+            ex.kernel_launches += 1
+        K.gemm(act, self.down, out=y, out_f32=True, ws=ex.ws)
+        ex.kernel_launches += 2
+
+
+MIXERS = {AttentionSpec: AttentionMixer, LatentAttentionSpec: LatentAttentionMixer, RgLruSpec: RgLruMixer}
+
+
+class _Layer:
+    def __init__(self, spec, pk: _Packer):
+        self.mixer = MIXERS[type(spec.mixer)](spec.mixer, pk)
+        self.norm1 = pk.f32("norm", "1", 4)
+        self.mlp = LimitedGlu(spec.mlp, pk) if spec.mlp is not None else None
+        self.norm2 = pk.f32("norm", "2", 4) if spec.mlp is not None else None
+
+
+class LayeredWeights:
+    """All weights of a layered decoder on the device, in kernel layout."""
+
+    def __init__(self, ckpt: Checkpoint, device, dtype: torch.dtype = torch.bfloat16):
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError("layered decoders are served in bfloat16 or float32")
+        self.config, self.dtype = ckpt.config, dtype
+        self.layers = [_Layer(spec, _Packer(ckpt, i, device, dtype)) for i, spec in enumerate(ckpt.config.layers)]
+        pk = _Packer(ckpt, -1, device, dtype)
+        self.embed = pk.raw("", "embed").to(dtype).contiguous()
+        self.final_norm = pk.f32("", "final.norm", 4)
+        self.head = pk.linear(pk.raw("", "head"))
+
+
+class LayeredStepBuffers(StepBuffers):
+    """Descriptor, fp32 residual stream ``h``, its copy ``x`` in the compute type (``h`` itself in fp32), sublayer output ``y`` and
+    named scratch that layers share."""
+
+    def __init__(self, cfg: LayeredConfig, dtype: torch.dtype, Tcap: int, Bcap: int, max_blocks_per_seq: int, device):
+        super().__init__(Tcap, Bcap, max_blocks_per_seq, device, cfg.vocab_size, logits_dtype=torch.float32, state_slots=True)
+        width = _up(cfg.hidden_size, 64)
+        zeros = lambda rows, dt: torch.zeros((rows, width), dtype=dt, device=device)
+        self.h, self.y = zeros(Tcap, torch.float32), zeros(Tcap, torch.float32)
+        self.x = self.h if dtype == torch.float32 else zeros(Tcap, dtype)
+        self.last_x = zeros(Bcap, dtype)
+        self.device, self.dtype = device, dtype
+        self._scratch: Dict[tuple, torch.Tensor] = {}
+
+    def scratch(self, name: str, rows: int, cols: int, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        """[rows, cols] view of a buffer that starts out as zeros; its row pitch is a multiple of 64."""
+        dtype = dtype or self.dtype
+        key = (name, cols, dtype)
+        if key not in self._scratch:
+            self._scratch[key] = torch.zeros((self.Tcap, _up(cols, 64)), dtype=dtype, device=self.device)
+        return self._scratch[key][:rows, :cols]
+
+
+class LayeredExecutor(LlmExecutor):
+    """Runs steps of a layered decoder on one GPU."""
+
+    def __init__(self, weights: LayeredWeights, num_kv_blocks: int, block_size: int = 16, max_batch_tokens: int = 8192, max_seqs: int = 64,
+                 max_blocks_per_seq: int = 0, device="cuda", use_cuda_graphs: bool = True):
+        cfg = weights.config
+        super().__init__(cfg, num_kv_blocks, block_size, max_seqs, max_blocks_per_seq, device, use_cuda_graphs)
+        self.w, self.dtype, self.storage = weights, weights.dtype, K.storage_type(weights.dtype)
+        self.has_recurrent_state = cfg.has_recurrent_state
+        for layer in weights.layers:
+            layer.mixer.allocate(self)
+        make = lambda Tcap: LayeredStepBuffers(cfg, self.dtype, Tcap, max_seqs, self.max_blocks_per_seq, self.device)
+        self.prefill, self.decode = make(max_batch_tokens), make(max_seqs)
+
+    def _recurrent_state(self) -> List[torch.Tensor]:
+        return [t for layer in self.w.layers for t in layer.mixer.state()]
+
+    def kv_cache_bytes(self) -> int:
+        return sum(layer.mixer.cache_bytes() for layer in self.w.layers)
+
+    def attention(self, sb: LayeredStepBuffers, shp: StepShape, **kw) -> None:
+        """Paged attention of this step's tokens (``K.window_attention``) with the batch description filled in."""
+        K.window_attention(past_lens=sb.view("past_lens"), subsequence_begins=sb.view("subsequence_begins"), block_indices=sb.view("block_indices"),
+                           block_indices_begins=sb.view("block_indices_begins"), B=shp.B, T=shp.T, block_size=self.block_size,
+                           max_context_len=shp.max_ctx, max_q_len=shp.max_q_len, dtype=self.storage, scratch=self.ws.pa_scratch,
+                           scratch_bytes=self.ws.pa_scratch.nbytes, exact=1 if self.dtype == torch.float32 else 0, **kw)
+
+    def _norm(self, sb: LayeredStepBuffers, T: int, w: torch.Tensor) -> None:
+        """x <- norm(residual_scale * x + y), in fp32, plus the copy that the next products read."""
+        cfg = self.cfg
+        K.sum_rmsnorm(sb.h[:T], w, cfg.norm_eps, cfg.hidden_size, y=sb.y[:T], alpha=cfg.residual_scale, w_offset=cfg.norm_offset, h_out=sb.h[:T],
+                      x_out=None if sb.x is sb.h else sb.x[:T])
+
+    def _forward(self, sb: LayeredStepBuffers, shp: StepShape) -> None:
+        T, B = shp.T, shp.B
+        ids = sb.view("ids")[:T]
+        K.resolve_ids(ids, sb.view("tok_src")[:T], self.last_token)
+        K.stream_embed(ids, self.w.embed, sb.h, None if sb.x is sb.h else sb.x)
+        x, y = sb.x[:T], sb.y[:T]
+        for i, layer in enumerate(self.w.layers):
+            layer.mixer.run(self, sb, shp, x, y)
+            self._norm(sb, T, layer.norm1)
+            if layer.mlp is not None:
+                layer.mlp.run(self, sb, shp, x, y)
+                self._norm(sb, T, layer.norm2)
+                self.kernel_launches += 1
+        self._logits(sb, sb.view("logit_idx")[:B], sb.logits[:B])
+        self.kernel_launches += 2 + len(self.w.layers) + 3
+        self._sample(sb, B)
+
+    def _logits(self, sb: LayeredStepBuffers, rows: torch.Tensor, out: torch.Tensor) -> None:
+        cfg, x = self.cfg, sb.last_x[:rows.shape[0]]
+        K.sum_rmsnorm(sb.h, self.w.final_norm, cfg.norm_eps, cfg.hidden_size, w_offset=cfg.norm_offset, x_out=x, row_idx=rows)
+        K.gemm(x, self.w.head, out=out, out_f32=True, ws=self.ws)
+
+    def logits_at(self, sb: LayeredStepBuffers, rows: List[int]) -> torch.Tensor:
+        """Logits (fp32) after the step that ``sb`` holds, at the given token rows of its batch."""
+        idx = torch.tensor(rows, dtype=torch.int32, device=self.device)
+        out = torch.empty((len(rows), self.cfg.vocab_size), dtype=torch.float32, device=self.device)
+        for i in range(0, len(rows), sb.Bcap):
+            self._logits(sb, idx[i:i + sb.Bcap], out[i:i + sb.Bcap])
+        return out
