@@ -21,53 +21,12 @@
 #include "attention.cuh"
 #include "common.cuh"
 #include "debug_bounds.cuh"
+#include "mma_sync.cuh"
 #include "sm100_ptx.cuh"
 
 namespace ovb {
 
 OVB_DEBUG_LIMITS_DEFINE
-
-// ------------------------------------------------------------------------------ small PTX helpers
-__device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc, bool valid) {
-    const int sz = valid ? 16 : 0;   // src-size 0 => 16 zero bytes are written
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void cp_async4(void* smem_dst, const void* gsrc, bool valid) {
-    const int sz = valid ? 4 : 0;
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-template <bool F16>
-__device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-    if (F16)
-        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                     : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                     : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-    else
-        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                     : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                     : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-template <bool F16>
-__device__ __forceinline__ uint32_t pack2(float lo, float hi) {
-    if (F16) {
-        __half2 v = __floats2half2_rn(lo, hi);
-        return *reinterpret_cast<uint32_t*>(&v);
-    }
-    return pack_bf16x2(lo, hi);
-}
 
 // Shared tiles are [rows][D] 16-bit with the 16-byte chunk index XOR-ed with (row & 7): ldmatrix of
 // 8 consecutive rows at one chunk column then touches 8 different bank groups.
@@ -350,6 +309,13 @@ __global__ void __launch_bounds__(256, 1) pa_prefill_kernel(PaKParams p) {
 }
 
 // ------------------------------------------------------------------------------ decode (q_len == 1)
+// One value of a decoded token's output, through the optional gate.
+__device__ __forceinline__ void store_decoded(const PaKParams& p, int tok, int hq, int d, float v) {
+    if (p.gate != nullptr)
+        v /= 1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)tok * p.ld_gate + (size_t)hq * p.gate_head + d]));
+    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.ldo + (size_t)hq * p.o_head + d] = __float2bfloat16_rn(v);
+}
+
 // CTA = 4 warps for one (sequence, kv head, kv split). Each warp walks pages w, w+4, ... of the
 // split with its own double-buffered page stage (no CTA-wide barriers in the loop), keeping
 // online-softmax state for the G query heads (padded to the 16-row MMA tile); the 4 warps merge
@@ -357,39 +323,50 @@ __global__ void __launch_bounds__(256, 1) pa_prefill_kernel(PaKParams p) {
 // pa_decode_combine_kernel finishes.
 // KVU8: the cache holds bytes with a (scale, zero point) pair per row (half the traffic of a 16-bit cache): a page is staged
 // as bytes and the warp expands it into its one bf16 page pair right before the MMAs.
-template <int D, int G, int PAGE, bool KVU8 = false>
+// DK / DV: key and value sizes, multiples of 64; cache rows may be shorter (p.k_row, p.v_row: the rest is filled with zeros).
+// GT: query heads per KV head, or 0: any number (p.group), up to eight of them per CTA.
+template <int DK, int DV, int GT, int PAGE, bool KVU8, int NST>
 __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
     pdl_enter_attn();
-    constexpr int CH = D / 8;
-    constexpr int NST = 3;   // page stages per warp
+    constexpr int CHK = DK / 8, CHV = DV / 8;
+    constexpr int GMAX = GT > 0 ? GT : 8;
+    static_assert(!KVU8 || (DK == DV && GT > 0), "byte cache: one head size");
+    constexpr int D = DK;                                              // (byte cache)
     constexpr int U8_PAGE = PAGE * D + PAGE * 4;                       // bytes of one staged u8 page (rows, then the pairs)
-    constexpr int STAGE = KVU8 ? 2 * U8_PAGE : 2 * PAGE * D * 2;       // K and V of one stage
+    constexpr int STAGE = KVU8 ? 2 * U8_PAGE : PAGE * (DK + DV) * 2;   // K and V of one stage (NST page stages per warp)
     constexpr int WARP_BYTES = NST * STAGE + (KVU8 ? 2 * PAGE * D * 2 : 0);
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int b = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
+    const int b = blockIdx.x, split = blockIdx.z;
+    const int parts = GT > 0 ? 1 : (p.group + 7) / 8;     // CTAs that share the query heads of a KV head
+    const int h = GT > 0 ? (int)blockIdx.y : (int)blockIdx.y / parts;
+    const int hq0 = GT > 0 ? h * GT : h * p.group + ((int)blockIdx.y % parts) * 8;
+    const int G = GT > 0 ? GT : min(8, (h + 1) * p.group - hq0);
     uint8_t* sQ = smem;                                   // 16 x D
-    uint8_t* sKV = smem + 16 * D * 2 + warp * WARP_BYTES;
+    uint8_t* sKV = smem + 16 * DK * 2 + warp * WARP_BYTES;
     uint8_t* sExp = sKV + NST * STAGE;                    // KVU8: the warp's expanded bf16 K and V pages
-    float* sMerge = reinterpret_cast<float*>(smem + 16 * D * 2 + 4 * WARP_BYTES);   // [4][G][D+2]
+    // after its last page a warp leaves its [GMAX][DV + 2] partials at the start of its own stages
+    auto merge_row = [&](int w, int r) { return reinterpret_cast<float*>(smem + 16 * DK * 2 + w * WARP_BYTES) + r * (DV + 2); };
+    static_assert(GMAX * (DV + 2) * 4 <= WARP_BYTES, "partials fit the page stages");
 
     const int tok = p.subsequence_begins[b];
     const int ctx = p.past_lens[b] + 1;
     const int blk_begin = p.block_indices_begins[b];
-    int k_lo = split * p.keys_per_split;
-    int k_hi = min(ctx, k_lo + p.keys_per_split);
-    if (p.sliding_window > 0) k_lo = max(k_lo, ((ctx - p.sliding_window) / PAGE) * PAGE);
+    // the splits share the keys from the first page that the window touches
+    const int k_first = p.sliding_window > 0 ? max(0, (ctx - p.sliding_window) / PAGE * PAGE) : 0;
+    const int k_lo = k_first + split * p.keys_per_split;
+    const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int page_lo = k_lo / PAGE;
     const int page_hi = (k_hi + PAGE - 1) / PAGE;         // exclusive
     const int win_lo = p.sliding_window > 0 ? ctx - p.sliding_window : 0;
 
     // Q: G real rows, the rest zero
-    for (int i = threadIdx.x; i < 16 * CH; i += 128) {
-        const int r = i / CH, c = i % CH;
-        const bool valid = r < G;
-        const uint8_t* src = reinterpret_cast<const uint8_t*>(p.q) + ((size_t)tok * p.ldq + (size_t)(h * G + (valid ? r : 0)) * D) * 2 + c * 16;
-        cp_async16(sQ + tile_off<D>(r, c), src, valid);
+    for (int i = threadIdx.x; i < 16 * CHK; i += 128) {
+        const int r = i / CHK, c = i % CHK;
+        const bool valid = r < G && (GT > 0 || c * 8 < p.k_row);
+        const uint8_t* src = reinterpret_cast<const uint8_t*>(p.q) + ((size_t)tok * p.ldq + (size_t)(hq0 + (valid ? r : 0)) * p.q_head) * 2 + (valid ? c : 0) * 16;
+        cp_async16(sQ + tile_off<DK>(r, c), src, valid);
     }
     cp_async_commit();
 
@@ -413,14 +390,29 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
             }
             return;
         }
-        const uint8_t* kb = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk * p.Hkv + h) * PAGE * D) * 2;
-        const uint8_t* vb = reinterpret_cast<const uint8_t*>(p.v_cache) + (((size_t)blk * p.Hkv + h) * PAGE * D) * 2;
-        uint8_t* dk = sKV + st * (2 * PAGE * D * 2);
-        uint8_t* dv = dk + PAGE * D * 2;
-        for (int i = lane; i < PAGE * CH; i += 32) {
-            const int r = i / CH, c = i % CH;
-            cp_async16(dk + tile_off<D>(r, c), kb + (size_t)r * D * 2 + c * 16, pv);
-            cp_async16(dv + tile_off<D>(r, c), vb + (size_t)r * D * 2 + c * 16, pv);
+        const int k_row = GT > 0 ? DK : p.k_row, v_row = GT > 0 ? DV : p.v_row;
+        const uint8_t* kb = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk * p.Hkv + h) * PAGE * k_row) * 2;
+        const uint8_t* vb = reinterpret_cast<const uint8_t*>(p.v_cache) + (((size_t)blk * p.Hkv + h) * PAGE * v_row) * 2;
+        uint8_t* dk = sKV + st * STAGE;
+        uint8_t* dv = dk + PAGE * DK * 2;
+        if (DK == DV) {
+            for (int i = lane; i < PAGE * CHK; i += 32) {
+                const int r = i / CHK, c = i % CHK;
+                const bool ck = GT > 0 || c * 8 < k_row, cv = GT > 0 || c * 8 < v_row;
+                cp_async16(dk + tile_off<DK>(r, c), kb + (ck ? (size_t)r * k_row * 2 + c * 16 : 0), pv && ck);
+                cp_async16(dv + tile_off<DV>(r, c), vb + (cv ? (size_t)r * v_row * 2 + c * 16 : 0), pv && cv);
+            }
+        } else {
+            for (int i = lane; i < PAGE * CHK; i += 32) {
+                const int r = i / CHK, c = i % CHK;
+                const bool ck = GT > 0 || c * 8 < k_row;
+                cp_async16(dk + tile_off<DK>(r, c), kb + (ck ? (size_t)r * k_row * 2 + c * 16 : 0), pv && ck);
+            }
+            for (int i = lane; i < PAGE * CHV; i += 32) {
+                const int r = i / CHV, c = i % CHV;
+                const bool cv = GT > 0 || c * 8 < v_row;
+                cp_async16(dv + tile_off<DV>(r, c), vb + (cv ? (size_t)r * v_row * 2 + c * 16 : 0), pv && cv);
+            }
         }
     };
     // prologue: NST-1 pages in flight
@@ -432,17 +424,17 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
     }
     cp_async_wait<NST - 1>();   // Q landed (oldest group)
     __syncthreads();
-    uint32_t qf[D / 16][4];
+    uint32_t qf[DK / 16][4];
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks) {
+    for (int ks = 0; ks < DK / 16; ++ks) {
         const int r = (lane & 7) + 8 * ((lane >> 3) & 1);
         const int c = ks * 2 + (lane >> 4);
-        ldsm_x4(smem_u32(sQ + tile_off<D>(r, c)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+        ldsm_x4(smem_u32(sQ + tile_off<DK>(r, c)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
     }
 
-    float o_acc[D / 8][4];
+    float o_acc[DV / 8][4];
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+    for (int i = 0; i < DV / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
     float m_run = -CUDART_INF_F, l_run = 0.f;   // rows >= 8 are padding: only row (lane>>2) state is kept
 
     int st = 0;
@@ -451,8 +443,8 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
         cp_async_commit();
         cp_async_wait<NST - 1>();
         __syncwarp();
-        const uint8_t* kS = sKV + st * (2 * PAGE * D * 2);
-        const uint8_t* vS = kS + PAGE * D * 2;
+        const uint8_t* kS = sKV + st * STAGE;
+        const uint8_t* vS = kS + PAGE * DK * 2;
         if (KVU8) {
             const uint8_t* uk = sKV + st * STAGE;
             expand_u8_tile<D>(uk, uk + PAGE * D, sExp, PAGE, lane, 32);
@@ -465,14 +457,14 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
 #pragma unroll
         for (int i = 0; i < PAGE / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
 #pragma unroll
             for (int nt = 0; nt < PAGE / 8; nt += 2) {
                 uint32_t b0, b1, b2, b3;
                 const int m = lane >> 3;
                 const int kr = nt * 8 + (m >> 1) * 8 + (lane & 7);
                 const int kc = ks * 2 + (m & 1);
-                ldsm_x4(smem_u32(kS + tile_off<D>(kr, kc)), b0, b1, b2, b3);
+                ldsm_x4(smem_u32(kS + tile_off<DK>(kr, kc)), b0, b1, b2, b3);
                 mma16816<false>(s[nt], qf[ks], b0, b1);
                 mma16816<false>(s[nt + 1], qf[ks], b2, b3);
             }
@@ -496,7 +488,7 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
         m_run = mx;
         l_run *= corr;
 #pragma unroll
-        for (int i = 0; i < D / 8; ++i) { o_acc[i][0] *= corr; o_acc[i][1] *= corr; }
+        for (int i = 0; i < DV / 8; ++i) { o_acc[i][0] *= corr; o_acc[i][1] *= corr; }
         uint32_t pf[PAGE / 16][4];
 #pragma unroll
         for (int nt = 0; nt < PAGE / 8; ++nt) {
@@ -509,12 +501,12 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
 #pragma unroll
         for (int kk = 0; kk < PAGE / 16; ++kk) {
 #pragma unroll
-            for (int dn = 0; dn < D / 8; dn += 2) {
+            for (int dn = 0; dn < DV / 8; dn += 2) {
                 uint32_t b0, b1, b2, b3;
                 const int m = lane >> 3;
                 const int vr = kk * 16 + (m & 1) * 8 + (lane & 7);
                 const int vc = dn + (m >> 1);
-                ldsm_x4_t(smem_u32(vS + tile_off<D>(vr, vc)), b0, b1, b2, b3);
+                ldsm_x4_t(smem_u32(vS + tile_off<DV>(vr, vc)), b0, b1, b2, b3);
                 mma16816<false>(o_acc[dn], pf[kk], b0, b1);
                 mma16816<false>(o_acc[dn + 1], pf[kk], b2, b3);
             }
@@ -523,65 +515,64 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
         st = (st + 1) % NST;
     }
     cp_async_wait<0>();
+    __syncwarp();
 
     // ---- merge the 4 warps (rows 0..G-1 only)
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 1);
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
     const int r = lane >> 2;
     if (r < G) {
-        float* dst = sMerge + ((size_t)warp * G + r) * (D + 2);
+        float* dst = merge_row(warp, r);
 #pragma unroll
-        for (int dn = 0; dn < D / 8; ++dn) {
+        for (int dn = 0; dn < DV / 8; ++dn) {
             const int d = dn * 8 + (lane & 3) * 2;
             dst[d] = o_acc[dn][0];
             dst[d + 1] = o_acc[dn][1];
         }
-        if ((lane & 3) == 0) { dst[D] = m_run; dst[D + 1] = l_run; }
+        if ((lane & 3) == 0) { dst[DV] = m_run; dst[DV + 1] = l_run; }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < G * D; i += 128) {
-        const int rr = i / D, d = i % D;
+    for (int i = threadIdx.x; i < G * DV; i += 128) {
+        const int rr = i / DV, d = i % DV;
         float m = -CUDART_INF_F;
 #pragma unroll
-        for (int w = 0; w < 4; ++w) m = fmaxf(m, sMerge[((size_t)w * G + rr) * (D + 2) + D]);
+        for (int w = 0; w < 4; ++w) m = fmaxf(m, merge_row(w, rr)[DV]);
         float l = 0.f, o = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) {
-            const float* src = sMerge + ((size_t)w * G + rr) * (D + 2);
-            const float sc = (src[D] == -CUDART_INF_F) ? 0.f : exp2f(src[D] - m);
-            l += src[D + 1] * sc;
+            const float* src = merge_row(w, rr);
+            const float sc = (src[DV] == -CUDART_INF_F) ? 0.f : exp2f(src[DV] - m);
+            l += src[DV + 1] * sc;
             o += src[d] * sc;
         }
-        const int hq = h * G + rr;
+        const int hq = hq0 + rr;
         if (p.nsplit == 1) {
-            reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.Hq * D + (size_t)hq * D + d] =
-                __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
+            if (GT > 0 || d < p.dv_store) store_decoded(p, tok, hq, d, l > 0.f ? o / l : 0.f);
         } else {
-            float* sc = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit + split) * (D + 2);
+            float* sc = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit + split) * (DV + 2);
             sc[d] = o;
-            if (d == 0) { sc[D] = m; sc[D + 1] = l; }
+            if (d == 0) { sc[DV] = m; sc[DV + 1] = l; }
         }
     }
 }
 
-template <int D>
-__global__ void pa_decode_combine_kernel(PaKParams p) {
+// Split-KV partials [Hq, nsplit, dv + 2] of every sequence (sums, then maximum and denominator) -> output rows.
+__global__ void pa_decode_combine_kernel(PaKParams p, int dv) {
     pdl_enter_attn();
     const int b = blockIdx.x, hq = blockIdx.y;
     const int tok = p.subsequence_begins[b];
-    const float* base = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit) * (D + 2);
-    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float* base = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit) * (dv + 2);
+    for (int d = threadIdx.x; d < p.dv_store; d += blockDim.x) {
         float m = -CUDART_INF_F;
-        for (int s = 0; s < p.nsplit; ++s) m = fmaxf(m, base[(size_t)s * (D + 2) + D]);
+        for (int s = 0; s < p.nsplit; ++s) m = fmaxf(m, base[(size_t)s * (dv + 2) + dv]);
         float l = 0.f, o = 0.f;
         for (int s = 0; s < p.nsplit; ++s) {
-            const float* src = base + (size_t)s * (D + 2);
-            const float sc = (src[D] == -CUDART_INF_F) ? 0.f : exp2f(src[D] - m);
-            l += src[D + 1] * sc;
+            const float* src = base + (size_t)s * (dv + 2);
+            const float sc = (src[dv] == -CUDART_INF_F) ? 0.f : exp2f(src[dv] - m);
+            l += src[dv + 1] * sc;
             o += src[d] * sc;
         }
-        reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.Hq * D + (size_t)hq * D + d] =
-            __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
+        store_decoded(p, tok, hq, d, l > 0.f ? o / l : 0.f);
     }
 }
 
@@ -609,22 +600,32 @@ static int launch_prefill(const PaKParams& p, int num_q_tiles, cudaStream_t stre
     return 0;
 }
 
-template <int D, int G, bool KVU8 = false>
-static int launch_decode(const PaKParams& p, cudaStream_t stream) {
+int launch_decode_combine(const PaKParams& p, int dv, cudaStream_t stream) {
+    OVB_CHECK_CUDA(launch_pdl(pa_decode_combine_kernel, dim3(p.B, p.Hq), dim3(128), 0, stream, p, dv));
+    OVB_CHECK_CUDA(cudaGetLastError());
+    return 0;
+}
+
+template <int DK, int DV, int G, bool KVU8, int NST>
+static int launch_decode_sizes(const PaKParams& p, cudaStream_t stream) {
     constexpr int PAGE = 16;
-    const int warp_bytes = KVU8 ? 3 * 2 * (PAGE * D + PAGE * 4) + 2 * PAGE * D * 2 : 3 * 2 * PAGE * D * 2;
-    const int smem = 16 * D * 2 + 4 * warp_bytes + 4 * G * (D + 2) * 4 + 128;
-    auto kern = pa_decode_kernel<D, G, PAGE, KVU8>;
+    const int warp_bytes = KVU8 ? NST * 2 * (PAGE * DK + PAGE * 4) + 2 * PAGE * DK * 2 : NST * PAGE * (DK + DV) * 2;
+    const int smem = 16 * DK * 2 + 4 * warp_bytes + 128;
+    auto kern = pa_decode_kernel<DK, DV, G, PAGE, KVU8, NST>;
     static std::atomic<uint64_t> configured{0};
     if (int rc = set_smem_once(configured, reinterpret_cast<const void*>(kern), smem)) return rc;
-    dim3 grid(p.B, p.Hkv, p.nsplit);
+    dim3 grid(p.B, p.Hkv * (G > 0 ? 1 : (p.group + 7) / 8), p.nsplit);
     OVB_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(128), smem, stream, p));
     OVB_CHECK_CUDA(cudaGetLastError());
-    if (p.nsplit > 1) {
-        OVB_CHECK_CUDA(launch_pdl(pa_decode_combine_kernel<D>, dim3(p.B, p.Hq), dim3(128), 0, stream, p));
-        OVB_CHECK_CUDA(cudaGetLastError());
-    }
-    return 0;
+    return p.nsplit > 1 ? launch_decode_combine(p, DV, stream) : 0;
+}
+
+// Heads of one size D packed without gaps.
+template <int D, int G, bool KVU8 = false>
+static int launch_decode(PaKParams p, cudaStream_t stream) {
+    p.q_head = p.o_head = p.dv_store = p.k_row = p.v_row = D;
+    p.ldo = p.Hq * D;
+    return launch_decode_sizes<D, D, G, KVU8, 3>(p, stream);
 }
 
 // OVB_ATTN_TC=0 in the environment keeps prefill and dense attention on the mma.sync kernel (for comparisons).
@@ -646,6 +647,30 @@ static int decode_nsplit(int B, int Hkv, int max_ctx) {
     if (n < 1) n = 1;
     if (n > 32) n = 32;
     return n;
+}
+
+int launch_window_decode(PaKParams p, int dk, int dv, int max_ctx, long long scratch_bytes, cudaStream_t stream) {
+    auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    if (p.block_size != 16 || dk > 256 || dv > 256 || p.k_row % 8 || p.v_row % 8 || p.ldq % 8 || p.q_head % 8 || !aligned(p.q) || !aligned(p.k_cache) ||
+        !aligned(p.v_cache))
+        return ERR_UNSUPPORTED;
+    const int ck = dk <= 64 ? 64 : dk <= 128 ? 128 : 256, cv = dv <= 64 ? 64 : dv <= 128 ? 128 : 256;
+    const int keys = p.sliding_window > 0 && p.sliding_window + 15 < max_ctx ? p.sliding_window + 15 : max_ctx;   // a window may start inside a page
+    p.dv_store = dv;
+    p.nsplit = decode_nsplit(p.B, p.Hkv * ((p.group + 7) / 8), keys);
+    const long long per_split = (long long)p.B * p.Hq * (cv + 2) * 4;
+    if (p.scratch == nullptr || per_split * p.nsplit > scratch_bytes) p.nsplit = p.scratch == nullptr || scratch_bytes < per_split ? 1 : (int)(scratch_bytes / per_split);
+    p.keys_per_split = ((keys + p.nsplit - 1) / p.nsplit + 63) / 64 * 64;
+    if (ck == 64) {
+        if (cv == 64) return launch_decode_sizes<64, 64, 0, false, 3>(p, stream);
+        return cv == 128 ? launch_decode_sizes<64, 128, 0, false, 3>(p, stream) : launch_decode_sizes<64, 256, 0, false, 3>(p, stream);
+    }
+    if (ck == 128) {
+        if (cv == 64) return launch_decode_sizes<128, 64, 0, false, 3>(p, stream);
+        return cv == 128 ? launch_decode_sizes<128, 128, 0, false, 3>(p, stream) : launch_decode_sizes<128, 256, 0, false, 2>(p, stream);
+    }
+    if (cv == 64) return launch_decode_sizes<256, 64, 0, false, 3>(p, stream);
+    return cv == 128 ? launch_decode_sizes<256, 128, 0, false, 2>(p, stream) : launch_decode_sizes<256, 256, 0, false, 2>(p, stream);
 }
 
 }  // namespace ovb

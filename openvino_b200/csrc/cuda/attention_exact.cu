@@ -6,6 +6,7 @@
 // and uses its first part as the value).
 #include <math_constants.h>
 
+#include "attention.cuh"
 #include "debug_bounds.cuh"
 #include "sm100_ptx.cuh"
 #include "store_types.cuh"
@@ -129,5 +130,24 @@ extern "C" int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream
     OVB_REQUIRE(a->past_lens && a->subsequence_begins && a->block_indices && a->block_indices_begins, "ovb_window_attention: null batch descriptor");
     OVB_REQUIRE(a->B > 0 && a->T > 0 && a->Hkv > 0 && a->Hq > 0 && a->Hq % a->Hkv == 0 && a->Dk > 0 && a->Dv > 0 && a->block_size > 0,
                 "ovb_window_attention: bad sizes");
+    if (a->dtype == OVB_DT_BF16 && !a->exact) {      // the tensor-core kernels, where they serve the sizes
+        PaKParams p;
+        memset(&p, 0, sizeof(p));
+        p.q = a->q; p.out = a->out; p.k_cache = a->k; p.v_cache = a->v; p.gate = a->gate;
+        p.past_lens = a->past_lens; p.subsequence_begins = a->subsequence_begins;
+        p.block_indices = a->block_indices; p.block_indices_begins = a->block_indices_begins;
+        p.scratch = a->scratch;
+        p.B = a->B; p.T = a->T; p.Hq = a->Hq; p.Hkv = a->Hkv; p.group = a->Hq / a->Hkv;
+        p.ldq = a->ldq; p.q_head = a->q_head; p.ldo = a->ldo; p.o_head = a->o_head; p.k_row = a->k_row; p.v_row = a->v_row;
+        p.ld_gate = a->ld_gate; p.gate_head = a->gate_head;
+        p.block_size = a->block_size; p.sliding_window = a->window; p.causal = 1;
+        p.scale_log2 = a->scale * 1.4426950408889634f;
+        const bool decode = a->max_q_len == 1 && a->T == a->B;
+        const int rc = a->k == a->v ? (a->Hkv == 1 && a->gate == nullptr ? launch_latent_attention(p, a->Dk, (a->Dv + 15) / 16 * 16, a->max_q_len, a->max_context_len,
+                                                                                                   a->scratch_bytes, (cudaStream_t)stream) : ERR_UNSUPPORTED)
+                     : decode ? launch_window_decode(p, a->Dk, a->Dv, a->max_context_len, a->scratch_bytes, (cudaStream_t)stream)
+                              : a->scale > 0.f ? launch_window_tc(p, a->Dk, 0, (a->Dv + 15) / 16 * 16, (cudaStream_t)stream) : ERR_UNSUPPORTED;
+        if (rc != ERR_UNSUPPORTED) return rc;
+    }
     return launch_attention_exact(*a, (cudaStream_t)stream);
 }

@@ -20,7 +20,7 @@
 //                        of 256): the accumulator O, which lives in tensor memory, then has to be rescaled only a few
 //                        times per row instead of once per tile. Epilogue: O / l -> 16-bit -> global.
 //
-// Tensor memory (512 columns): S0 0..127, S1 128..255, O 256..256+D-1, P0 and P1 (64 columns each) behind it.
+// Tensor memory (512 columns): S0 0..127, S1 128..255, O 256..256+DV-1, P0 and P1 (64 columns each) behind it.
 // Every wait is bounded (mbar_wait) and reports through the status word.
 #include <math_constants.h>
 
@@ -65,23 +65,34 @@ __device__ __forceinline__ uint32_t pack16(float lo, float hi) {
     return pack_bf16x2(lo, hi);
 }
 
-template <int D, int G, bool PAGED, bool F16>
+// Where keys and values come from: pages of the cache, dense tensors, or rows expanded from a latent cache (PaKParams::kv_rows).
+enum : int { SRC_PAGED = 0, SRC_DENSE = 1, SRC_LATENT = 2 };
+
+// Tokens per tile for a group of g query heads: whole 8-row groups, so that every head's rows start on a swizzle boundary.
+__host__ __device__ constexpr int tile_tokens(int g) { return kBM / g / 8 * 8; }
+
+// KH / RH / VH: 64-column (128-byte) parts of a key row, of its shared second part, and of a value row. A part that reaches past
+// the end of a cache row is filled with zeros by the copy, so any size that is a multiple of 8 is served; what the query tile
+// holds behind a head's columns meets those zeros. GT: query heads per KV head, 0 = at run time (p.group).
+template <int KH, int RH, int VH, int GT, int SRC, bool F16>
 __global__ void __launch_bounds__(192, 1)
 pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                     PaKParams p, int* status) {
-    constexpr int TOK = kBM / G;               // tokens per tile
-    constexpr int HALVES = D / 64;             // 64-column (128-byte) halves of a row
-    constexpr int Q_BYTES = kBM * D * 2, KV_BYTES = kBK * D * 2;
-    constexpr uint32_t TM_S = 0, TM_O = 256, TM_P = 256 + D;   // tensor-memory columns
+                     const __grid_constant__ CUtensorMap tmR, PaKParams p, int* status) {
+    constexpr bool PAGED = SRC != SRC_DENSE;                   // ragged batch with a descriptor
+    constexpr int DK = (KH + RH) * 64, DV = VH * 64;
+    const int G = GT > 0 ? GT : p.group;
+    const int TOK = tile_tokens(G);            // tokens per tile
+    constexpr int Q_BYTES = kBM * DK * 2, K_BYTES = kBK * DK * 2, V_BYTES = kBK * DV * 2;
+    constexpr uint32_t TM_S = 0, TM_O = 256, TM_P = 256 + DV;   // tensor-memory columns
     constexpr uint32_t IDESC_QK = umma_idesc_f16(kBM, kBK, !F16);
-    constexpr uint32_t IDESC_PV = umma_idesc_f16(kBM, D, !F16) | (1u << 16);   // B operand MN-major
+    constexpr uint32_t IDESC_PV = umma_idesc_f16(kBM, DV, !F16) | (1u << 16);   // B operand MN-major
 
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* sQ = smem;
     uint8_t* sK = sQ + Q_BYTES;                // two stages
-    uint8_t* sV = sK + 2 * KV_BYTES;           // two stages
-    uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * KV_BYTES);
+    uint8_t* sV = sK + 2 * K_BYTES;            // two stages
+    uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * V_BYTES);
     uint64_t* q_full = bars;
     uint64_t* k_full = bars + 1;               // [2]
     uint64_t* v_full = bars + 3;               // [2]
@@ -157,34 +168,36 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         // One lane posts the byte counts; then every lane issues the boxes of its own (page, half): a single thread that
         // issues the 64 small copies of a tile one after the other is slower than the tensor core consumes them.
         if (lane == 0) {
-            mbar_arrive_expect_tx(q_full, Q_BYTES);
+            mbar_arrive_expect_tx(q_full, G * TOK * DK * 2);
             for (int g = 0; g < G; ++g)
-                for (int hf = 0; hf < HALVES; ++hf)
-                    tma_load_2d(sQ + hf * (kBM * 128) + g * (TOK * 128), &tmQ, q_full, (h * G + g) * D + hf * 64, tok_begin + tq0);
+                for (int hf = 0; hf < KH + RH; ++hf)
+                    tma_load_2d(sQ + hf * (kBM * 128) + g * (TOK * 128), &tmQ, q_full,
+                                (h * G + g) * p.q_head + (hf < KH ? hf * 64 : p.q_shared + (hf - KH) * 64), tok_begin + tq0);
         }
+        // row of key 0 of this sequence in contiguous key / value rows
+        const int row_base = SRC == SRC_DENSE ? b * p.dense_S : SRC == SRC_LATENT ? p.kv_rows[b] - latent_first_key(past, p.sliding_window) : 0;
         for (int j = 0; j < ntiles; ++j) {
             const int st = j & 1;
             if (j >= 2 && !mbar_wait(&kv_empty[st], ((j >> 1) - 1) & 1, abort_flag, status)) break;
             const int j0 = kv_start + j * kBK;
             const int npages = (min(kv_end, j0 + kBK) - j0 + kPage - 1) / kPage;
             if (lane == 0) {
-                mbar_arrive_expect_tx(&k_full[st], npages * kPage * D * 2);
-                mbar_arrive_expect_tx(&v_full[st], npages * kPage * D * 2);
+                mbar_arrive_expect_tx(&k_full[st], npages * kPage * DK * 2);
+                mbar_arrive_expect_tx(&v_full[st], npages * kPage * DV * 2);
             }
             __syncwarp();
-            for (int u = lane; u < npages * HALVES; u += 32) {
-                const int pg = u / HALVES, hf = u % HALVES;
-                int row, col;
-                if (PAGED) {
+            for (int u = lane; u < npages * (KH + RH + VH); u += 32) {      // keys first
+                const int part = u / npages, pg = u % npages;
+                int row = row_base + j0 + pg * kPage, col_k = h * p.k_head, col_v = h * p.v_head;
+                if (SRC == SRC_PAGED || (RH > 0 && part >= KH && part < KH + RH)) {
                     const int blk = p.block_indices[blk_begin + j0 / kPage + pg];
-                    row = (blk * p.Hkv + h) * kPage;
-                    col = 0;
-                } else {
-                    row = b * p.dense_S + j0 + pg * kPage;
-                    col = h * D;
+                    row = SRC == SRC_PAGED ? (blk * p.Hkv + h) * kPage : blk * kPage;
+                    col_k = col_v = 0;
                 }
-                tma_load_2d(sK + st * KV_BYTES + hf * (kBK * 128) + pg * (kPage * 128), &tmK, &k_full[st], col + hf * 64, row);
-                tma_load_2d(sV + st * KV_BYTES + hf * (kBK * 128) + pg * (kPage * 128), &tmV, &v_full[st], col + hf * 64, row);
+                uint8_t* dk = sK + st * K_BYTES + part * (kBK * 128) + pg * (kPage * 128);
+                if (part < KH) tma_load_2d(dk, &tmK, &k_full[st], col_k + part * 64, row);
+                else if (RH > 0 && part < KH + RH) tma_load_2d(dk, &tmR, &k_full[st], p.shared_col + (part - KH) * 64, row);
+                else tma_load_2d(sV + st * V_BYTES + (part - KH - RH) * (kBK * 128) + pg * (kPage * 128), &tmV, &v_full[st], col_v + (part - KH - RH) * 64, row);
             }
         }
         __syncwarp();
@@ -199,9 +212,9 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                 if (j >= 2) ok = ok && mbar_wait(&s_free[st], ((j >> 1) - 1) & 1, abort_flag, status);
                 if (!ok) break;
                 tc_fence_after_sync();
-                const uint64_t dk = umma_desc_k_sw128(smem_u32(sK + st * KV_BYTES), 1024);
+                const uint64_t dk = umma_desc_k_sw128(smem_u32(sK + st * K_BYTES), 1024);
 #pragma unroll
-                for (int ks = 0; ks < D / 16; ++ks) {
+                for (int ks = 0; ks < DK / 16; ++ks) {
                     const uint64_t off = (uint64_t)(((ks >> 2) * (kBM * 128) + (ks & 3) * 32) >> 4);
                     umma_f16_ss_elect(tmem + TM_S + st * kBK, dq + off, dk + off, IDESC_QK, ks > 0 ? 1u : 0u);
                 }
@@ -215,7 +228,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                 tc_fence_after_sync();
                 const int keys = min(kBK, kv_end - (kv_start + i * kBK));
                 const int ksteps = (keys + 15) / 16;
-                const uint64_t dv = umma_desc_mn_sw128(smem_u32(sV + st * KV_BYTES), kBK * 128, 1024);
+                const uint64_t dv = umma_desc_mn_sw128(smem_u32(sV + st * V_BYTES), kBK * 128, 1024);
                 for (int kk = 0; kk < ksteps; ++kk)
                     umma_f16_ts_elect(tmem + TM_O, tmem + TM_P + st * 64 + kk * 8, dv + (uint64_t)((kk * 16 * 128) >> 4), IDESC_PV,
                                       (i > 0 || kk > 0) ? 1u : 0u);
@@ -229,7 +242,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         const int r = threadIdx.x;                       // 0..127 = tensor-memory lane
         const int g = r / TOK, tl = r % TOK;
         const int qpos = past + tq0 + tl;
-        const bool row_valid = (tq0 + tl) < q_len;
+        const bool row_valid = (tq0 + tl) < q_len && (GT > 0 || g < G);
         const uint32_t lane_base = tmem + (uint32_t(warp * 32) << 16);
         float m_used = -CUDART_INF_F, l_sum = 0.f;
         bool ok = true;
@@ -280,7 +293,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                     if (!ok) break;
                     tc_fence_after_sync();
 #pragma unroll 1
-                    for (int c = 0; c < D; c += 32) {
+                    for (int c = 0; c < DV; c += 32) {
                         uint32_t o[32];
                         tmem_ld_x16(lane_base + TM_O + c, o);
                         tmem_ld_x16(lane_base + TM_O + c + 16, o + 16);
@@ -324,9 +337,11 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (ok) {
             tc_fence_after_sync();
             const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-            uint8_t* dst = reinterpret_cast<uint8_t*>(p.out) + ((size_t)(tok_begin + tq0 + tl) * p.Hq * D + (size_t)(h * G + g) * D) * 2;
+            uint8_t* dst = reinterpret_cast<uint8_t*>(p.out) + ((size_t)(tok_begin + tq0 + tl) * p.ldo + (size_t)(h * G + g) * p.o_head) * 2;
+            const uint8_t* gate = p.gate == nullptr ? nullptr : reinterpret_cast<const uint8_t*>(p.gate) +
+                                  ((size_t)(tok_begin + tq0 + tl) * p.ld_gate + (size_t)(h * G + g) * p.gate_head) * 2;
 #pragma unroll 1
-            for (int c = 0; c < D; c += 16) {
+            for (int c = 0; c < p.dv_store; c += 16) {
                 uint32_t o[16];
                 if (ntiles > 0) {
                     tmem_ld_x16(lane_base + TM_O + c, o);
@@ -334,6 +349,12 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                 } else {
 #pragma unroll
                     for (int i = 0; i < 16; ++i) o[i] = 0u;
+                }
+                if (gate != nullptr && row_valid) {
+                    uint4 gw[2] = {*reinterpret_cast<const uint4*>(gate + c * 2), *reinterpret_cast<const uint4*>(gate + c * 2 + 16)};
+                    const __nv_bfloat16* gv = reinterpret_cast<const __nv_bfloat16*>(gw);
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) / (1.f + __expf(-__bfloat162float(gv[i]))));
                 }
                 if (row_valid) {
                     uint4 w0, w1;
@@ -365,11 +386,11 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     }
 }
 
-template <int D, int G, bool PAGED, bool F16>
-int launch_tc(const PaKParams& p, int num_q_tiles, cudaStream_t stream) {
-    constexpr int TOK = kBM / G;
-    const int smem = kBM * D * 2 + 4 * kBK * D * 2 + 256 + 1024;
-    auto kern = pa_prefill_tc_kernel<D, G, PAGED, F16>;
+template <int KH, int RH, int VH, int G, int SRC, bool F16>
+int launch_tc_parts(const PaKParams& p, int num_q_tiles, cudaStream_t stream) {
+    const int TOK = tile_tokens(G > 0 ? G : p.group);
+    const int smem = kBM * (KH + RH) * 128 + 2 * kBK * (KH + RH + VH) * 128 + 256 + 1024;
+    auto kern = pa_prefill_tc_kernel<KH, RH, VH, G, SRC, F16>;
     static std::atomic<uint64_t> configured{0};
     int dev = 0;
     OVB_CHECK_CUDA(cudaGetDevice(&dev));
@@ -379,21 +400,36 @@ int launch_tc(const PaKParams& p, int num_q_tiles, cudaStream_t stream) {
         configured.fetch_or(bit, std::memory_order_release);
     }
     const CUtensorMapDataType dt = F16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-    CUtensorMap tmQ, tmK, tmV;
+    CUtensorMap tmQ, tmK, tmV, tmR;
     // Q rows are tokens; a box is the TOK tokens of a tile x 64 columns of one head (rows past T read as zeros)
     if (int rc = make_tmap_2d(&tmQ, p.q, dt, 2, (uint64_t)p.T, (uint64_t)p.ldq, (uint64_t)p.ldq * 2, TOK, 64, true)) return rc;
-    if (PAGED) {
-        // the cache seen as rows of D elements: row = (block * Hkv + head) * 16 + slot; the row count only bounds coordinates
+    if (SRC == SRC_PAGED) {
+        // the cache seen as rows of one head: row = (block * Hkv + head) * 16 + slot; the row count only bounds coordinates
         const uint64_t rows = 1ull << 30;
-        if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, rows, D, (uint64_t)D * 2, kPage, 64, true)) return rc;
-        if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, rows, D, (uint64_t)D * 2, kPage, 64, true)) return rc;
+        if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, rows, p.k_row, (uint64_t)p.k_row * 2, kPage, 64, true)) return rc;
+        if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, rows, p.v_row, (uint64_t)p.v_row * 2, kPage, 64, true)) return rc;
+    } else if (SRC == SRC_LATENT) {
+        // pages of 16 rows that reach past a sequence's last key read the next sequence's rows (masked) or zeros behind the last
+        const uint64_t rows = 1ull << 30;
+        if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.kv_ld, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
+        if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.kv_ld, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
+        if (int rc = make_tmap_2d(&tmR, p.shared, dt, 2, rows, p.shared_row, (uint64_t)p.shared_row * 2, kPage, 64, true)) return rc;
     } else {
         const uint64_t rows = (uint64_t)p.B * p.dense_S;
         if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, rows, (uint64_t)p.ld_kv, (uint64_t)p.ld_kv * 2, kPage, 64, true)) return rc;
         if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, rows, (uint64_t)p.ld_kv, (uint64_t)p.ld_kv * 2, kPage, 64, true)) return rc;
     }
-    OVB_CHECK_CUDA(launch_pdl(kern, dim3(num_q_tiles, p.Hkv), dim3(192), (size_t)smem, stream, tmQ, tmK, tmV, p, status_word()));
+    if (SRC != SRC_LATENT) tmR = tmK;      // unused
+    OVB_CHECK_CUDA(launch_pdl(kern, dim3(num_q_tiles, p.Hkv), dim3(192), (size_t)smem, stream, tmQ, tmK, tmV, tmR, p, status_word()));
     return 0;
+}
+
+// Heads of one size D packed without gaps.
+template <int D, int G, bool PAGED, bool F16>
+int launch_tc(PaKParams p, int num_q_tiles, cudaStream_t stream) {
+    p.q_head = p.o_head = p.dv_store = p.k_row = p.v_row = p.k_head = p.v_head = D;
+    p.ldo = p.Hq * D;
+    return launch_tc_parts<D / 64, 0, D / 64, G, PAGED ? SRC_PAGED : SRC_DENSE, F16>(p, num_q_tiles, stream);
 }
 
 }  // namespace
@@ -420,6 +456,29 @@ int launch_prefill_tc(const PaKParams& p, int D, int G, bool paged, bool f16, in
     } else if (!paged && G == 1) {
         if (D == 64) return f16 ? launch_tc<64, 1, false, true>(p, num_q_tiles, stream) : launch_tc<64, 1, false, false>(p, num_q_tiles, stream);
         if (D == 128) return f16 ? launch_tc<128, 1, false, true>(p, num_q_tiles, stream) : launch_tc<128, 1, false, false>(p, num_q_tiles, stream);
+    }
+    return ERR_UNSUPPORTED;
+}
+
+int launch_window_tc(PaKParams p, int dk, int dshared, int dv, cudaStream_t stream) {
+    const int kh = ceil_div(dk, 64), rh = ceil_div(dshared, 64), vh = ceil_div(dv, 64);
+    if (p.block_size != kPage || p.group < 1 || p.group > 16 || kh + rh > 3 || rh > 1 || vh > 2) return ERR_UNSUPPORTED;
+    auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    if (!aligned(p.q) || !aligned(p.k_cache) || !aligned(p.v_cache) || !aligned(p.out) || !aligned(p.gate) || !aligned(p.shared)) return ERR_UNSUPPORTED;
+    if (p.ldq % 8 || p.q_head % 8 || p.ldo % 8 || p.o_head % 8 || p.ld_gate % 8 || p.gate_head % 8 || dv % 16 || p.k_row % 8 || p.v_row % 8) return ERR_UNSUPPORTED;
+    p.dv_store = dv;
+    const int tiles = p.T / tile_tokens(p.group) + p.B;      // upper bound of the tiles of all sequences
+    if (rh > 0) {
+        if (kh == 1) return vh == 1 ? launch_tc_parts<1, 1, 1, 1, SRC_LATENT, false>(p, tiles, stream) : launch_tc_parts<1, 1, 2, 1, SRC_LATENT, false>(p, tiles, stream);
+        return vh == 1 ? launch_tc_parts<2, 1, 1, 1, SRC_LATENT, false>(p, tiles, stream) : launch_tc_parts<2, 1, 2, 1, SRC_LATENT, false>(p, tiles, stream);
+    }
+    switch (kh * 2 + vh) {
+        case 3: return launch_tc_parts<1, 0, 1, 0, SRC_PAGED, false>(p, tiles, stream);
+        case 4: return launch_tc_parts<1, 0, 2, 0, SRC_PAGED, false>(p, tiles, stream);
+        case 5: return launch_tc_parts<2, 0, 1, 0, SRC_PAGED, false>(p, tiles, stream);
+        case 6: return launch_tc_parts<2, 0, 2, 0, SRC_PAGED, false>(p, tiles, stream);
+        case 7: return launch_tc_parts<3, 0, 1, 0, SRC_PAGED, false>(p, tiles, stream);
+        case 8: return launch_tc_parts<3, 0, 2, 0, SRC_PAGED, false>(p, tiles, stream);
     }
     return ERR_UNSUPPORTED;
 }

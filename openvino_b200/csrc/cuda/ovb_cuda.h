@@ -388,6 +388,27 @@ typedef struct {
 } ovb_wattn_args;
 int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream);
 
+// Latent attention over expanded rows (prefill). ovb_latent_gather copies the first `cols` elements of the cached rows that the windows
+// of the batch's new tokens reach (from a multiple of 128 on) to out [rows, out_pitch], sequence by sequence, and writes the sequences'
+// first rows to kv_rows [B + 1]; rows = their total as the host computes it. The caller expands them: kv = out * [W_k | W_v]^T with key
+// heads of k_head columns (a multiple of 64, zeros behind the true size) and, from v_off on, value heads of v_head columns.
+int ovb_latent_gather(const void* cache, void* out, int* kv_rows, const int* past_lens, const int* subsequence_begins, const int* block_indices,
+                      const int* block_indices_begins, int B, int rows, int cols, int row_pitch, int out_pitch, int window, int block_size, ovb_stream_t stream);
+typedef struct {
+    const void* q;            // [T, ldq]: query heads at a pitch of q_head, their turned part at q_rot_off
+    const void* kv;           // [rows, ld_kv]
+    const void* cache;        // [blocks, block_size, row_pitch]: shared key part at key_off
+    void* out;                // [T, ldo]: heads of Dv columns (a multiple of 16) at a pitch of o_head
+    const int* kv_rows;
+    const int* past_lens;
+    const int* subsequence_begins;
+    const int* block_indices;
+    const int* block_indices_begins;
+    int B, T, H, rows, R, Dv, ldq, q_head, q_rot_off, ld_kv, k_head, v_off, v_head, row_pitch, key_off, ldo, o_head, block_size, window;
+    float scale;
+} ovb_latent_prefill_args;
+int ovb_latent_prefill(const ovb_latent_prefill_args* a, ovb_stream_t stream);
+
 // Griffin's recurrent block between its projections (recurrent.cu). ovb_causal_conv: u = conv(x); then the caller computes the gate
 // pre-activations gates = [ra u | ri u] block by block; ovb_lru_scan: r, i = sigmoid(gates + gate_b), a = exp(-r * log_decay),
 // S <- a S + sqrt(1 - a^2) i u, out = S * gelu_tanh(y), and both states are brought up to date.

@@ -80,7 +80,11 @@ from ..utils import trace as _trace
 
 def step_shape(st: ScheduledStep) -> StepShape:
     """What the executor has to know on the host about a scheduled step."""
-    return StepShape(st.T, len(st.seqs), st.max_q_len, st.max_ctx)
+    spans = None
+    if st.max_q_len > 1:
+        seqs = st.native.seqs if hasattr(st, "native") else st.seqs
+        spans = tuple((int(s.num_computed), int(n)) for s, n in zip(seqs, st.num_new))
+    return StepShape(st.T, len(st.seqs), st.max_q_len, st.max_ctx, spans)
 
 
 class ContinuousBatchingPipeline:

@@ -78,6 +78,12 @@ class WindowAttnArgs(C.Structure):
                                "window", "max_context_len", "max_q_len", "dtype"), ("scale",)) + [("exact", C.c_int)])
 
 
+class LatentPrefillArgs(C.Structure):
+    _fields_ = _fields(("q", "kv", "cache", "out", "kv_rows", "past_lens", "subsequence_begins", "block_indices", "block_indices_begins"),
+                       ("B", "T", "H", "rows", "R", "Dv", "ldq", "q_head", "q_rot_off", "ld_kv", "k_head", "v_off", "v_head", "row_pitch", "key_off", "ldo",
+                        "o_head", "block_size", "window"), ("scale",))
+
+
 class RgLruArgs(C.Structure):
     _fields_ = _fields(("x", "y", "u", "out", "gates", "gate_b", "log_decay", "conv_w", "conv_b", "state", "conv_state", "subsequence_begins", "past_lens",
                         "slots"),
@@ -413,6 +419,19 @@ def latent_prepare(**kw) -> None:
 def window_attention(**kw) -> None:
     """Paged attention with separate key / value sizes, window and output gate; fields of ``ovb_wattn_args``."""
     _check(lib().ovb_window_attention(C.byref(_fill(WindowAttnArgs(), kw)), C.c_void_p(_stream())), "ovb_window_attention")
+
+
+def latent_gather(cache, out, kv_rows, past_lens, subsequence_begins, block_indices, block_indices_begins, B, rows, cols, row_pitch, out_pitch, window,
+                  block_size) -> None:
+    """Cached rows that the windows of a batch reach -> contiguous ``out``; ``kv_rows`` [B + 1] gets the sequences' first rows."""
+    ptrs = [C.c_void_p(t.data_ptr()) for t in (cache, out, kv_rows, past_lens, subsequence_begins, block_indices, block_indices_begins)]
+    _check(lib().ovb_latent_gather(*ptrs, C.c_int(B), C.c_int(rows), C.c_int(cols), C.c_int(row_pitch), C.c_int(out_pitch), C.c_int(window), C.c_int(block_size),
+                                   C.c_void_p(_stream())), "ovb_latent_gather")
+
+
+def latent_prefill(**kw) -> None:
+    """Latent attention over expanded rows; fields of ``ovb_latent_prefill_args``."""
+    _check(lib().ovb_latent_prefill(C.byref(_fill(LatentPrefillArgs(), kw)), C.c_void_p(_stream())), "ovb_latent_prefill")
 
 
 def causal_conv(**kw) -> None:

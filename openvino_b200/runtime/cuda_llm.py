@@ -248,6 +248,7 @@ class StepShape:
     B: int            # sequences in the step
     max_q_len: int    # longest sub-sequence (1 = pure decode)
     max_ctx: int      # longest context after this step
+    spans: Optional[tuple] = None     # (tokens before this step, tokens of this step) of every sequence; None: not known to the host
 
 
 # ----------------------------------------------------------------------------------------- executor

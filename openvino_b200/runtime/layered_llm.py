@@ -117,8 +117,10 @@ class AttentionMixer:
 
 
 class LatentAttentionMixer:
-    """Latent attention over the cached low-rank rows. The key projection is moved to the query (q W_uk) and the value projection
-    behind the weighted sum, so that all heads attend to the one cached row per token."""
+    """Latent attention over the cached low-rank rows, in one of two forms of the same sums. Absorbed: the key projection moves to the
+    query (q W_uk) and the value projection behind the weighted sum, so that all heads attend to the one cached row per token; the
+    form of decoding, of fp32 and of head sizes that the prefill kernel does not serve. Expanded: the rows that the step's windows
+    reach become per-head keys and values; fewer operations when many new tokens share them (prefill)."""
 
     def __init__(self, s: LatentAttentionSpec, pk: _Packer):
         self.s, self.rot = s, _Rotation(s.rotary, pk.device)
@@ -136,6 +138,18 @@ class LatentAttentionMixer:
         self.uk = pk.block_diag(pk.raw("mix", "uk").reshape(H, D, C).transpose(1, 2))
         self.uv = pk.block_diag(pk.raw("mix", "uv").reshape(H, Dv, C))
         self.o = pk.linear(_pad_cols(pk.raw("mix", "o"), H, self.dv))
+        self.k_head, self.v_head = _up(D, 64), _up(Dv, 64)
+        self.ukv = None
+        if pk.dtype == torch.bfloat16 and self.k_head <= 128 and R <= 64 and self.v_head <= 128 and s.scale > 0:
+            self.ukv = pk.linear(torch.cat([_pad_rows(pk.raw("mix", "uk"), H, self.k_head), _pad_rows(pk.raw("mix", "uv"), H, self.v_head)], 0))
+
+    def _expanded_rows(self, sb: "LayeredStepBuffers", shp: StepShape) -> int:
+        """Cached rows that this step's windows reach (as csrc/cuda/attention.cuh counts them), or 0: run the absorbed form."""
+        if self.ukv is None or shp.spans is None:
+            return 0
+        first = lambda past: max(0, past - self.s.window + 1) // 128 * 128 if self.s.window > 0 else 0
+        rows = sum(past + new - first(past) for past, new in shp.spans)
+        return rows if rows <= 2 * sb.Tcap else 0
 
     def allocate(self, ex: "LayeredExecutor") -> None:
         self.cache = torch.zeros((ex.num_kv_blocks, ex.block_size, self.row), dtype=ex.dtype, device=ex.device)
@@ -150,19 +164,42 @@ class LatentAttentionMixer:
         s, T, H = self.s, shp.T, self.s.heads
         proj = sb.scratch("proj", T, self.proj.N)
         K.gemm(x, self.proj, out=proj, ws=ex.ws)
-        q = sb.scratch("latent_q", T, H * self.row)
-        K.latent_prepare(proj=proj, q_rot=q[:, self.cp:], cache=self.cache, c_norm=self.c_norm, positions=sb.view("positions"), slot_map=sb.view("slot_map"), T=T,
+        rows = self._expanded_rows(sb, shp)
+        q = proj if rows else sb.scratch("latent_q", T, H * self.row)
+        q_rot = dict(q_rot=proj[:, self.dp:], ld_qr=proj.stride(0), qr_pitch=self.q_pitch) if rows else \
+            dict(q_rot=q[:, self.cp:], ld_qr=q.stride(0), qr_pitch=self.row)
+        K.latent_prepare(proj=proj, cache=self.cache, c_norm=self.c_norm, positions=sb.view("positions"), slot_map=sb.view("slot_map"), T=T,
                          H=H, C=s.kv_rank, R=s.rot_dim, q_pitch=self.q_pitch, q_rot_off=self.dp, c_off=self.c_off, kr_off=self.kr_off, ldp=proj.stride(0),
-                         ld_qr=q.stride(0), qr_pitch=self.row, row_pitch=self.row, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage,
-                         eps=ex.cfg.norm_eps, **self.rot.args())
+                         row_pitch=self.row, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **q_rot, **self.rot.args())
+        attn = sb.scratch("attn", T, self.o.K)
+        if rows:
+            self._attend_expanded(ex, sb, shp, rows, proj, attn)
+        else:
+            self._attend_absorbed(ex, sb, shp, proj, q, attn)
+        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
+        ex.kernel_launches += 3
+
+    def _attend_expanded(self, ex, sb, shp: StepShape, rows: int, proj: torch.Tensor, attn: torch.Tensor) -> None:
+        s, H = self.s, self.s.heads
+        batch = dict(past_lens=sb.view("past_lens"), subsequence_begins=sb.view("subsequence_begins"), block_indices=sb.view("block_indices"),
+                     block_indices_begins=sb.view("block_indices_begins"), B=shp.B, window=s.window, block_size=ex.block_size)
+        lat = sb.scratch("latent_rows", rows, self.ukv.K, cap=2 * sb.Tcap)
+        kv = sb.scratch("latent_kv", rows, self.ukv.N, cap=2 * sb.Tcap)
+        K.latent_gather(cache=self.cache, out=lat, kv_rows=sb.kv_rows, rows=rows, cols=self.cp, row_pitch=self.row, out_pitch=lat.stride(0), **batch)
+        K.gemm(lat, self.ukv, out=kv, ws=ex.ws)
+        K.latent_prefill(q=proj, kv=kv, cache=self.cache, out=attn, kv_rows=sb.kv_rows, T=shp.T, H=H, rows=rows, R=s.rot_dim, Dv=self.dv, ldq=proj.stride(0),
+                         q_head=self.q_pitch, q_rot_off=self.dp, ld_kv=kv.stride(0), k_head=self.k_head, v_off=H * self.k_head, v_head=self.v_head,
+                         row_pitch=self.row, key_off=self.cp, ldo=attn.stride(0), o_head=self.dv, scale=s.scale, **batch)
+        ex.kernel_launches += 3
+
+    def _attend_absorbed(self, ex, sb, shp: StepShape, proj: torch.Tensor, q: torch.Tensor, attn: torch.Tensor) -> None:
+        s, T, H = self.s, shp.T, self.s.heads
         K.gemm_block_diag(proj[:, :self.c_off], self.uk, q, self.q_pitch, self.row, ws=ex.ws)
         lat = sb.scratch("latent_o", T, H * self.cp)
         ex.attention(sb, shp, q=q, k=self.cache, v=self.cache, out=lat, Hq=H, Hkv=1, Dk=self.row, Dv=s.kv_rank, ldq=q.stride(0), q_head=self.row,
                      k_row=self.row, v_row=self.row, ldo=lat.stride(0), o_head=self.cp, window=s.window, scale=s.scale)
-        attn = sb.scratch("attn", T, self.o.K)
         K.gemm_block_diag(lat[:, :H * self.cp], self.uv, attn, self.cp, self.dv, ws=ex.ws)
-        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
-        ex.kernel_launches += 6
+        ex.kernel_launches += 3
 
 
 class RgLruMixer:
@@ -276,15 +313,16 @@ class LayeredStepBuffers(StepBuffers):
         self.h, self.y = zeros(Tcap, torch.float32), zeros(Tcap, torch.float32)
         self.x = self.h if dtype == torch.float32 else zeros(Tcap, dtype)
         self.last_x = zeros(Bcap, dtype)
+        self.kv_rows = torch.zeros(Bcap + 1, dtype=torch.int32, device=device)
         self.device, self.dtype = device, dtype
         self._scratch: Dict[tuple, torch.Tensor] = {}
 
-    def scratch(self, name: str, rows: int, cols: int, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-        """[rows, cols] view of a buffer that starts out as zeros; its row pitch is a multiple of 64."""
+    def scratch(self, name: str, rows: int, cols: int, dtype: Optional[torch.dtype] = None, cap: int = 0) -> torch.Tensor:
+        """[rows, cols] view of a buffer of ``cap`` (default: Tcap) rows that starts out as zeros; its row pitch is a multiple of 64."""
         dtype = dtype or self.dtype
         key = (name, cols, dtype)
         if key not in self._scratch:
-            self._scratch[key] = torch.zeros((self.Tcap, _up(cols, 64)), dtype=dtype, device=self.device)
+            self._scratch[key] = torch.zeros((cap or self.Tcap, _up(cols, 64)), dtype=dtype, device=self.device)
         return self._scratch[key][:rows, :cols]
 
 
