@@ -1,11 +1,13 @@
-"""``LLMPipeline``: text generation from a model object or an IR directory, the way ``openvino_genai.LLMPipeline`` is used.
+"""``LLMPipeline``: text generation from a model object, an IR directory or a checkpoint directory, the way
+``openvino_genai.LLMPipeline`` is used.
 
     pipe = LLMPipeline("model_dir_or_xml", "CUDA")            # or LLMPipeline(ov_model, "CUDA")
     out = pipe.generate([[1, 15043, 29892]], max_new_tokens=32)
 
 The model graph is analysed and lifted into the device's serving program (paged KV cache, continuous batching, CUDA
 graphs; see runtime/llm_import.py); under tensor parallelism every rank constructs the pipeline with its communicator.
-Prompts are token-id lists; a tokenizer object with ``encode`` / ``decode`` may be supplied for text in, text out (a
+A directory with ``config.json`` and ``model.safetensors`` is loaded by the architecture that its configuration names
+(models/registry.py) and served by the layered program (runtime/layered_llm.py). Prompts are token-id lists; a tokenizer object with ``encode`` / ``decode`` may be supplied for text in, text out (a
 byte-level one ships here for tests; real vocabularies come from the model's own tokenizer files).
 """
 from __future__ import annotations
@@ -17,6 +19,7 @@ import torch
 
 from .._graph import Model
 from ..frontend import read_model
+from ..models.registry import is_checkpoint_dir, load_checkpoint
 from .pipeline import ContinuousBatchingPipeline, GenerationConfig, GenerationResult
 from .scheduler import SchedulerConfig
 
@@ -33,13 +36,30 @@ class ByteTokenizer:
         return bytes(i - 3 for i in ids if 3 <= i < 259).decode("utf-8", errors="replace")
 
 
+def _cuda_index(device: str) -> int:
+    return int(device.split(".")[1]) if "." in device else (torch.cuda.current_device() if torch.cuda.is_available() else 0)
+
+
 class LLMPipeline:
     def __init__(self, model: Union[str, Model], device: str = "CUDA", tokenizer=None, comm=None, tp_rank: int = 0, tp_size: int = 1,
                  max_num_seqs: int = 64, max_num_batched_tokens: int = 8192, max_model_len: int = 4096, block_size: int = 16,
                  kv_cache_blocks: int = 0, **properties):
-        """``properties``: further device properties for ``compile_model`` (e.g. ``KV_CACHE_PRECISION="u8"``)."""
+        """``properties``: further device properties for ``compile_model`` (e.g. ``KV_CACHE_PRECISION="u8"``). A checkpoint directory
+        takes ``INFERENCE_PRECISION_HINT`` (bf16, the default, or f32), ``CUDA_USE_GRAPHS`` and a scheduler's ``dynamic_split_fuse``."""
         if device.split(".")[0] not in ("CUDA", "GPU"):
             raise RuntimeError("LLMPipeline runs on the CUDA device; use compile_model for '%s'" % device)
+        self.tokenizer = tokenizer
+        if not isinstance(model, Model) and is_checkpoint_dir(str(model)):
+            if tp_size > 1:
+                raise NotImplementedError("checkpoint directories are served on one GPU")
+            from ..runtime.layered_llm import create_executor
+            self.compiled_model = None
+            self.executor, self.scheduler_config = create_executor(
+                load_checkpoint(str(model)), _cuda_index(device), max_num_seqs=max_num_seqs, max_num_batched_tokens=max_num_batched_tokens,
+                max_model_len=max_model_len, block_size=block_size, kv_cache_blocks=kv_cache_blocks, properties=properties)
+            self.config = self.executor.cfg
+            self.pipeline = ContinuousBatchingPipeline(self.executor, self.scheduler_config)
+            return
         if not isinstance(model, Model):
             path = str(model)
             if os.path.isdir(path):
@@ -53,7 +73,7 @@ class LLMPipeline:
             mgr = passes.Manager()
             mgr.register_pass(passes.SDPAToPagedAttention())
             mgr.run_passes(model)
-        dev_index = int(device.split(".")[1]) if "." in device else (torch.cuda.current_device() if torch.cuda.is_available() else 0)
+        dev_index = _cuda_index(device)
         config = {props.cuda.serving_program: True}
         config.update(properties)
         if tp_size > 1:
@@ -67,7 +87,6 @@ class LLMPipeline:
             max_num_seqs=max_num_seqs, max_num_batched_tokens=max_num_batched_tokens, max_model_len=max_model_len, block_size=block_size,
             kv_cache_blocks=kv_cache_blocks, comm=comm)
         self.pipeline = ContinuousBatchingPipeline(self.executor, self.scheduler_config)
-        self.tokenizer = tokenizer
 
     def get_tokenizer(self):
         return self.tokenizer

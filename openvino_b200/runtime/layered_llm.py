@@ -388,3 +388,29 @@ class LayeredExecutor(LlmExecutor):
         for i in range(0, len(rows), sb.Bcap):
             self._logits(sb, idx[i:i + sb.Bcap], out[i:i + sb.Bcap])
         return out
+
+
+def create_executor(ckpt: Checkpoint, device_index: int = 0, max_num_seqs: int = 64, max_num_batched_tokens: int = 8192, max_model_len: int = 4096,
+                    block_size: int = 16, kv_cache_blocks: int = 0, properties: Optional[dict] = None):
+    """Executor of a checkpoint and the scheduler limits that fit it: ``(executor, SchedulerConfig)``. ``properties``:
+    INFERENCE_PRECISION_HINT (bf16 / f32), CUDA_USE_GRAPHS, dynamic_split_fuse; others are refused."""
+    from .. import properties as props
+    from ..genai.scheduler import SchedulerConfig
+    opts = {str(k): v for k, v in (properties or {}).items()}
+    precision = str(opts.pop(str(props.hint.inference_precision), "bf16")).lower()
+    dtypes = {"bf16": torch.bfloat16, "bfloat16": torch.bfloat16, "f32": torch.float32, "float32": torch.float32}
+    if precision not in dtypes:
+        raise ValueError("a checkpoint is served in bf16 or f32, not '%s'" % precision)
+    graphs = str(opts.pop(str(props.cuda.use_cuda_graphs), True)).upper() not in ("FALSE", "NO", "0")
+    fuse = bool(opts.pop("dynamic_split_fuse", False))
+    if opts:
+        raise ValueError("unknown properties for a checkpoint: %s" % ", ".join(sorted(opts)))
+    device = torch.device("cuda", device_index)
+    blocks_per_seq = (max_model_len + block_size - 1) // block_size + 1
+    num_blocks = kv_cache_blocks or max_num_seqs * blocks_per_seq + 8
+    with torch.cuda.device(device), torch.no_grad():
+        ex = LayeredExecutor(LayeredWeights(ckpt, device, dtypes[precision]), num_kv_blocks=num_blocks, block_size=block_size,
+                             max_batch_tokens=max_num_batched_tokens, max_seqs=max_num_seqs, max_blocks_per_seq=blocks_per_seq, device=device,
+                             use_cuda_graphs=graphs)
+    return ex, SchedulerConfig(max_num_batched_tokens=max_num_batched_tokens, max_num_seqs=max_num_seqs, num_kv_blocks=num_blocks, block_size=block_size,
+                               max_blocks_per_seq=blocks_per_seq, dynamic_split_fuse=fuse)

@@ -28,16 +28,15 @@ def main(argv=None) -> int:
     from ..genai.replay import Replay
     from ..models.registry import load_checkpoint
     from ..ops import cuda as K
-    from ..runtime.layered_llm import LayeredExecutor, LayeredWeights
+    from ..runtime.layered_llm import create_executor
 
-    device = torch.device("cuda", torch.cuda.current_device())
     block = 16
     seqs = max(1, min(args.max_tokens, 128))
     longest = (args.max_tokens + block - 1) // block + 1
     with torch.no_grad():
-        weights = LayeredWeights(load_checkpoint(args.model), device, getattr(torch, args.dtype))
-        ex = LayeredExecutor(weights, num_kv_blocks=longest + seqs, block_size=block, max_batch_tokens=max(seqs, min(args.max_tokens, 8192)), max_seqs=seqs,
-                             max_blocks_per_seq=longest, device=device)
+        ex, _ = create_executor(load_checkpoint(args.model), torch.cuda.current_device(), max_num_seqs=seqs,
+                                max_num_batched_tokens=max(seqs, min(args.max_tokens, 8192)), max_model_len=args.max_tokens, block_size=block,
+                                kv_cache_blocks=longest + seqs, properties={"INFERENCE_PRECISION_HINT": args.dtype})
         replay = Replay(ex)
         for line in sys.stdin:
             if not line.strip():
