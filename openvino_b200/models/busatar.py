@@ -48,3 +48,28 @@ def tensor_name(layer: int, part: str, key: str) -> str:
     if layer < 0:
         return key
     return "l%d.norm%s" % (layer, key) if part == "norm" else "l%d.%s.%s" % (layer, part, key)
+
+
+def tensor_shapes(cfg: LayeredConfig) -> dict:
+    """Name -> shape of every tensor of a checkpoint."""
+    W = cfg.hidden_size
+    out = {"embed": (cfg.vocab_size, W), "final.norm": (W,), "head": (cfg.vocab_size, W)}
+    for i, layer in enumerate(cfg.layers):
+        m, mix = layer.mixer, {}
+        if isinstance(m, AttentionSpec):
+            mix = {"q": (m.heads * m.dim, W), "k": (m.kv_heads * m.dim, W), "v": (m.kv_heads * m.vdim, W), "q.norm": (m.dim,), "k.norm": (m.dim,),
+                   "g": (m.heads * m.vdim, W), "o": (W, m.heads * m.vdim)}
+        elif isinstance(m, LatentAttentionSpec):
+            mix = {"q": (m.heads * (m.dim + m.rot_dim), W), "dkv": (m.kv_rank + m.rot_dim, W), "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank),
+                   "uv": (m.heads * m.vdim, m.kv_rank), "o": (W, m.heads * m.vdim)}
+        elif isinstance(m, RgLruSpec):
+            N, B = m.width, m.blocks
+            mix = {"y": (N, W), "y.b": (N,), "x": (N, W), "x.b": (N,), "conv": (N, m.taps), "conv.b": (N,), "ra": (B, N // B, N // B), "ra.b": (B, N // B),
+                   "ri": (B, N // B, N // B), "ri.b": (B, N // B), "lam": (N,), "o": (W, N)}
+        out.update({tensor_name(i, "mix", k): v for k, v in mix.items()})
+        out[tensor_name(i, "norm", "1")] = (W,)
+        if layer.mlp is not None:
+            F = layer.mlp.ff
+            out[tensor_name(i, "norm", "2")] = (W,)
+            out.update({tensor_name(i, "mlp", "gate"): (F, W), tensor_name(i, "mlp", "up"): (F, W), tensor_name(i, "mlp", "down"): (W, F)})
+    return out

@@ -18,9 +18,10 @@ from .llm_config import LayeredConfig
 class Architecture:
     read_config: Callable[[dict], LayeredConfig]
     tensor_name: Callable[[int, str, str], str]
+    tensor_shapes: Callable[[LayeredConfig], dict]
 
 
-ARCHITECTURES: Dict[str, Architecture] = {"Busatar": Architecture(busatar.read_config, busatar.tensor_name)}
+ARCHITECTURES: Dict[str, Architecture] = {"Busatar": Architecture(busatar.read_config, busatar.tensor_name, busatar.tensor_shapes)}
 
 
 def register(name: str, arch: Architecture) -> None:
@@ -34,8 +35,18 @@ class Checkpoint:
     arch: Architecture
     tensors: object            # mapping name -> torch.Tensor
 
+    def __post_init__(self):
+        self._shapes = self.arch.tensor_shapes(self.config)
+
     def __call__(self, layer: int, part: str, key: str):
-        return self.tensors[self.arch.tensor_name(layer, part, key)]
+        name = self.arch.tensor_name(layer, part, key)
+        try:
+            t = self.tensors[name]
+        except KeyError:
+            raise KeyError("the checkpoint has no tensor '%s'" % name) from None
+        if tuple(t.shape) != tuple(self._shapes[name]):
+            raise ValueError("tensor '%s' has the shape %s, its configuration asks for %s" % (name, tuple(t.shape), tuple(self._shapes[name])))
+        return t
 
 
 def is_checkpoint_dir(path: str) -> bool:

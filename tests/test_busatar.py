@@ -22,7 +22,7 @@ def tokens(n, vocab, seed):
 # ------------------------------------------------------------------------------------------------ host side
 def test_configuration_is_read_from_the_file(tmp_path):
     from openvino_b200.models.llm_config import AttentionSpec, LatentAttentionSpec, LimitedGluSpec, RgLruSpec
-    from openvino_b200.models.registry import load_checkpoint
+    from openvino_b200.models.registry import from_dict, load_checkpoint
     cfg = CONFIGS["mixed"]
     weights = oracle.random_weights(cfg, 1)
     oracle.write_model(tmp_path, cfg, weights)
@@ -38,6 +38,12 @@ def test_configuration_is_read_from_the_file(tmp_path):
     for name, t in weights.items():
         assert torch.equal(ck.tensors[name].float(), t)
     assert torch.equal(ck(2, "mix", "conv").float(), weights["l2.mix.conv"]) and torch.equal(ck(-1, "", "head").float(), weights["head"])
+    with pytest.raises(KeyError, match="no tensor 'l9.mix.q'"):
+        ck(9, "mix", "q")
+    assert ck.arch.tensor_shapes(c) == {n: tuple(t.shape) for n, t in weights.items()}
+    wrong = dict(weights, head=weights["head"][:-1])
+    with pytest.raises(ValueError, match="'head' has the shape"):
+        from_dict(cfg, wrong)(-1, "", "head")
     with pytest.raises(ValueError, match="unknown architecture"):
         (tmp_path / "config.json").write_text(json.dumps(dict(cfg, architecture="Nobody")))
         load_checkpoint(str(tmp_path))
