@@ -124,13 +124,21 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatentParams p) {
         if (slot < 0) return;
         E* row = reinterpret_cast<E*>(p.cache) + (size_t)slot * p.row_pitch;
         const E* c = proj + p.c_off;
+        const int nvec = p.C / 4;             // (rows and offsets are multiples of 16 elements)
         float ss = 0.f;
-        for (int i = lane; i < p.C; i += 32) {
-            const float v = ld_f32(c + i);
-            ss += v * v;
+#pragma unroll 4
+        for (int i = lane; i < nvec; i += 32) {
+            const float4 v = ld4_f32(c + i * 4);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
+        for (int i = nvec * 4 + lane; i < p.C; i += 32) ss += ld_f32(c + i) * ld_f32(c + i);
         const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.C + p.eps);
-        for (int i = lane; i < p.C; i += 32) st_f32(row + i, ld_f32(c + i) * inv * p.c_norm[i]);
+#pragma unroll 4
+        for (int i = lane; i < nvec; i += 32) {
+            const float4 v = ld4_f32(c + i * 4), g = ld4_f32(p.c_norm + i * 4);
+            st4_f32(row + i * 4, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+        }
+        for (int i = nvec * 4 + lane; i < p.C; i += 32) st_f32(row + i, ld_f32(c + i) * inv * p.c_norm[i]);
         const E* kr = proj + p.kr_off;
         for (int i = lane; i < half; i += 32) {
             float u = ld_f32(kr + i), v = ld_f32(kr + i + half);
@@ -190,6 +198,8 @@ int ovb_latent_prepare(const ovb_latent_args* a, ovb_stream_t stream) {
     OVB_REQUIRE(a->T > 0 && a->H > 0 && a->C > 0 && a->R > 0 && a->block_size > 0 && a->key_off >= a->C && a->key_off + a->R <= a->row_pitch,
                 "ovb_latent_prepare: bad sizes");
     OVB_REQUIRE(a->rot_dims > 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->R && a->inv_freq, "ovb_latent_prepare: bad rotation");
+    OVB_REQUIRE(a->ldp % 4 == 0 && a->c_off % 4 == 0 && a->row_pitch % 4 == 0 && (reinterpret_cast<uintptr_t>(a->c_norm) & 15) == 0,
+                "ovb_latent_prepare: rows must be aligned to 4 elements");
     LatentParams p = {a->proj, a->q_rot, a->cache, a->c_norm, a->positions, a->slot_map, {a->inv_freq, a->rot_dims, a->rot_mult},
                       a->T, a->H, a->C, a->R, a->q_pitch, a->q_rot_off, a->c_off, a->kr_off, a->ldp, a->ld_qr, a->qr_pitch, a->row_pitch, a->key_off,
                       a->block_size, a->eps};

@@ -2,10 +2,12 @@
 //
 // latent_attention_kernel: every query head attends to the same cached row per token; the first part of that row is also the value.
 // One CTA serves one token (decode: one sequence), 16 or 32 of its heads and one share of the visible keys. Key tiles of 64 rows
-// pass through two shared-memory stages (cp.async), once for both products:
-//   scores   warp w multiplies the heads' queries with keys 8w .. 8w + 7 of the tile,
-//   softmax  running maximum over the CTA (per-warp maxima through shared memory), P as bf16 in shared memory,
-//   sums     warp w owns its own slice of the value columns for all 64 keys, so the accumulator needs no merge.
+// pass through two shared-memory stages, one bulk copy per row, and are read for both products:
+//   scores   the 8 warps split the row's columns in quarters and the tile's keys in halves; the queries' fragments of a warp's
+//            quarter stay in registers for the whole loop. The four partial sums meet in shared memory.
+//   softmax  8 or 16 neighbouring threads per head add the partials, mask, keep running maximum and sum; P as bf16.
+//   sums     every warp owns its own slice of the value columns for all 64 keys, so the accumulator needs no merge.
+// Rows are 16 bytes longer in shared memory than in the cache, which spreads ldmatrix over all banks.
 // With split keys the partial sums go to scratch and the decode kernels' merge finishes.
 //
 // latent_gather_kernel: the rows that the windows of a batch's new tokens reach, made contiguous, so that a plain product expands
@@ -27,215 +29,259 @@ namespace {
 
 constexpr int kWarps = 8, kKeys = 64;
 
+constexpr int kScorePitch = kKeys + 8;    // floats per row of partial scores
+
 struct LatentKParams {
     PaKParams p;
-    int row, pitch, cpad;     // elements of a cached row that take part, its pitch in shared memory (whole 128 bytes), value columns
+    int row, cpad;            // elements of a cached row that take part, value columns (multiples of 16)
+    int* status;
 };
 
-__device__ __forceinline__ uint32_t row_off(int r, int chunk, int pitch) { return uint32_t(r * pitch * 2 + ((chunk ^ (r & 7)) << 4)); }
+__device__ __forceinline__ uint32_t p_off(int r, int chunk) { return uint32_t(r * kKeys * 2 + ((chunk ^ (r & 7)) << 4)); }
 
-template <int MT, int VT>
+// MT: 16-head tiles; VT: 16-column pieces of the value per warp; KQ: most 16-column steps in a quarter of the row.
+template <int MT, int VT, int KQ>
 __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(LatentKParams a) {
-    pdl_enter_attn();
+    constexpr int R = MT * 16, TPR = kWarps * 32 / R, NQ = kKeys / (TPR * 4);    // rows, threads per row, quads of keys per thread
     const PaKParams& p = a.p;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
-    const int pitch = a.pitch, nch = a.row / 8, ksteps = a.row / 16;
-    const int stage = kKeys * pitch * 2;
-    uint8_t* sQ = smem;
-    uint8_t* sK = sQ + MT * 16 * pitch * 2;                              // two stages
-    uint8_t* sP = sK + 2 * stage;                                        // [MT * 16][64] bf16
-    float* sMax = reinterpret_cast<float*>(sP + MT * 16 * kKeys * 2);    // [MT * 16][8]
-    __shared__ int s_b;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x, h0 = blockIdx.y * MT * 16, split = blockIdx.z;
-    if (threadIdx.x == 0) {
+    const int row_bytes = a.row * 2, pitch = row_bytes + 16, ksteps = a.row / 16;
+    const int stage = kKeys * pitch;
+    const int shared_part = max(R * pitch, 4 * R * kScorePitch * 4);
+    uint8_t* sK = smem;                                                  // two stages
+    uint8_t* sQ = sK + 2 * stage;                                        // queries, then partial scores [4][R][kScorePitch]
+    float* sS = reinterpret_cast<float*>(sQ);
+    uint8_t* sP = sQ + shared_part;                                      // [R][64] bf16
+    float* sCorr = reinterpret_cast<float*>(sP + R * kKeys * 2);         // [R]
+    float* sMax = sCorr + R;                                             // [R]
+    uint64_t* full = reinterpret_cast<uint64_t*>(sMax + R);              // [2]
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(full + 2);
+    int* s_b = const_cast<int*>(abort_flag) + 1;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int t = blockIdx.x, h0 = blockIdx.y * R, split = blockIdx.z;
+    if (tid == 0) {
+        mbar_init(&full[0], 1);
+        mbar_init(&full[1], 1);
+        mbar_fence_init();
+        *abort_flag = 0;
+    }
+    pdl_enter_attn();
+    if (tid == 0) {
         int b = 0;
         while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
-        s_b = b;
+        *s_b = b;
     }
-    for (int r = warp; r < MT * 16; r += kWarps) {
+    for (int r = warp; r < R; r += kWarps) {
         const bool valid = h0 + r < p.Hq;
         const uint8_t* src = reinterpret_cast<const uint8_t*>(p.q) + ((size_t)t * p.ldq + (size_t)(valid ? h0 + r : 0) * p.q_head) * 2;
-        for (int c = lane; c < nch; c += 32) cp_async16(sQ + row_off(r, c, pitch), src + c * 16, valid);
+        for (int c = lane; c < a.row / 8; c += 32) cp_async16(sQ + r * pitch + c * 16, src + c * 16, valid);
     }
+    cp_async_commit();
     __syncthreads();
-    const int b = s_b;
+    const int b = *s_b;
     const int ctx = p.past_lens[b] + t - p.subsequence_begins[b] + 1;    // keys that exist for this token
     const int lo = p.sliding_window > 0 ? max(0, ctx - p.sliding_window) : 0;
     const int k_lo = lo / kKeys * kKeys + split * p.keys_per_split;
     const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int ntiles = k_hi > k_lo ? (k_hi - k_lo + kKeys - 1) / kKeys : 0;
     const int* blocks = p.block_indices + p.block_indices_begins[b];
-    auto load = [&](int tile, int st) {
-        const int j0 = k_lo + tile * kKeys + warp * 8;                   // a warp's eight rows lie in one page
-        const bool any = j0 < k_hi;
-        const int blk = any ? OVB_DBG_BLOCK(blocks[j0 / p.block_size]) : 0;
-        const uint8_t* src = reinterpret_cast<const uint8_t*>(p.k_cache) + ((size_t)blk * p.block_size + (any ? j0 % p.block_size : 0)) * p.k_row * 2;
-        uint8_t* dst = sK + st * stage;
-#pragma unroll
-        for (int r = 0; r < 8; ++r)
-            for (int c = lane; c < nch; c += 32) cp_async16(dst + row_off(warp * 8 + r, c, pitch), src + ((size_t)r * p.k_row) * 2 + c * 16, j0 + r < k_hi);
+    auto load = [&](int tile, int st) {      // warp 0; keys past the end repeat the last one (finite, and masked)
+        if (lane == 0) mbar_arrive_expect_tx(&full[st], kKeys * row_bytes);
+        __syncwarp();
+        for (int r = lane; r < kKeys; r += 32) {
+            const int j = min(k_lo + tile * kKeys + r, k_hi - 1);
+            const int blk = OVB_DBG_BLOCK(blocks[j / p.block_size]);
+            bulk_load_1d(sK + st * stage + r * pitch, reinterpret_cast<const uint8_t*>(p.k_cache) + ((size_t)blk * p.block_size + j % p.block_size) * p.k_row * 2,
+                         row_bytes, &full[st]);
+        }
     };
-    if (ntiles > 0) load(0, 0);
-    cp_async_commit();
-
-    float o[MT][VT * 2][4];
-    float m_run[MT][2], l_run[MT][2];
+    if (warp == 0 && ntiles > 0) load(0, 0);
+    cp_async_wait<0>();
+    __syncthreads();
+    // ---- this warp's quarter of the queries, in registers
+    const int kq = warp & 3, kg = warp >> 2, per = (ksteps + 3) / 4;
+    const int k0 = kq * per, kn = max(0, min(per, ksteps - k0));
+    uint32_t qf[MT][KQ][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < KQ; ++i) {
+            const int ks = k0 + min(i, max(kn - 1, 0));                  // (steps past the end are not used)
+            ldsm_x4(smem_u32(sQ + (m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * pitch + ks * 32 + (lane >> 4) * 16), qf[m][i][0], qf[m][i][1], qf[m][i][2],
+                    qf[m][i][3]);
+        }
+    float o[MT][VT * 2][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int i = 0; i < VT * 2; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
-        m_run[m][0] = m_run[m][1] = -CUDART_INF_F;
-        l_run[m][0] = l_run[m][1] = 0.f;
-    }
+    const int srow = tid / TPR, sc = tid % TPR;                          // softmax: this thread's row and place in it
+    float m_run = -CUDART_INF_F, l_run = 0.f;
+    const int gm = lane >> 3;
+    bool ok = true;
     for (int tile = 0; tile < ntiles; ++tile) {
         const int st = tile & 1;
-        cp_async_wait<0>();
-        __syncthreads();                                                 // the tile has landed; the other stage and sP are free
-        if (tile + 1 < ntiles) load(tile + 1, st ^ 1);
-        cp_async_commit();
+        __syncthreads();                                                 // the other stage, the partials and P are free
+        if (warp == 0 && tile + 1 < ntiles) load(tile + 1, st ^ 1);
+        ok = mbar_wait(&full[st], (tile >> 1) & 1, abort_flag, a.status);
         const uint8_t* kS = sK + st * stage;
-        // ---- scores of keys 8 * warp .. + 7 (two accumulators: even and odd steps)
-        float s[MT][2][4];
+        // ---- partial scores: 32 keys of half kg over the columns of quarter kq
+        float s[MT][4][4];
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) s[m][0][i] = s[m][1][i] = 0.f;
-#pragma unroll 2
-        for (int ks = 0; ks < ksteps; ks += 2) {
-            uint32_t k0, k1, k2, k3;
-            ldsm_x4(smem_u32(kS + row_off(warp * 8 + (lane & 7), ks * 2 + (lane >> 3), pitch)), k0, k1, k2, k3);
+            for (int n = 0; n < 4; ++n) s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f;
 #pragma unroll
-            for (int m = 0; m < MT; ++m) {
-                uint32_t q[4];
-                const int r = m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1);
-                ldsm_x4(smem_u32(sQ + row_off(r, ks * 2 + (lane >> 4), pitch)), q[0], q[1], q[2], q[3]);
-                mma16816<false>(s[m][0], q, k0, k1);
-                if (ks + 1 < ksteps) {
-                    ldsm_x4(smem_u32(sQ + row_off(r, ks * 2 + 2 + (lane >> 4), pitch)), q[0], q[1], q[2], q[3]);
-                    mma16816<false>(s[m][1], q, k2, k3);
-                }
+        for (int i = 0; i < KQ; ++i) {
+            if (i < kn) {
+                uint32_t kf[8];
+#pragma unroll
+                for (int g = 0; g < 2; ++g)
+                    ldsm_x4(smem_u32(kS + (kg * 32 + g * 16 + (gm >> 1) * 8 + (lane & 7)) * pitch + (k0 + i) * 32 + (gm & 1) * 16), kf[g * 4], kf[g * 4 + 1],
+                            kf[g * 4 + 2], kf[g * 4 + 3]);
+#pragma unroll
+                for (int m = 0; m < MT; ++m)
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) mma16816<false>(s[m][n], qf[m][i], kf[n * 2], kf[n * 2 + 1]);
             }
         }
-        // ---- mask, maximum over the tile
-        const int j = k_lo + tile * kKeys + warp * 8 + (lane & 3) * 2;
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int ri = 0; ri < 2; ++ri) {
-                float mx = -CUDART_INF_F;
+            for (int n = 0; n < 4; ++n)
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const bool ok = j + e >= lo && j + e < k_hi;
-                    const float v = ok ? (s[m][0][ri * 2 + e] + s[m][1][ri * 2 + e]) * p.scale_log2 : -CUDART_INF_F;
-                    s[m][0][ri * 2 + e] = v;
-                    mx = fmaxf(mx, v);
-                }
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                if ((lane & 3) == 0) sMax[(m * 16 + ri * 8 + (lane >> 2)) * kWarps + warp] = mx;
-            }
+                for (int ri = 0; ri < 2; ++ri)
+                    *reinterpret_cast<float2*>(sS + (kq * R + m * 16 + ri * 8 + (lane >> 2)) * kScorePitch + kg * 32 + n * 8 + (lane & 3) * 2) =
+                        make_float2(s[m][n][ri * 2], s[m][n][ri * 2 + 1]);
         __syncthreads();
+        // ---- softmax of a row by TPR neighbouring threads
+        float v[NQ][4];
+        float mx = m_run;
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+        for (int g = 0; g < NQ; ++g) {
+            const int key = (g * TPR + sc) * 4;
+            float4 x = *reinterpret_cast<const float4*>(sS + srow * kScorePitch + key);
 #pragma unroll
-            for (int ri = 0; ri < 2; ++ri) {
-                const int r = m * 16 + ri * 8 + (lane >> 2);
-                const float4 x = *reinterpret_cast<const float4*>(sMax + r * kWarps), y = *reinterpret_cast<const float4*>(sMax + r * kWarps + 4);
-                const float mnew = fmaxf(m_run[m][ri], fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(y.x, y.y), fmaxf(y.z, y.w))));
-                const float base = mnew == -CUDART_INF_F ? 0.f : mnew;
-                const float corr = exp2f(m_run[m][ri] - base);
-                const float e0 = exp2f(s[m][0][ri * 2] - base), e1 = exp2f(s[m][0][ri * 2 + 1] - base);
-                m_run[m][ri] = mnew;
-                l_run[m][ri] = l_run[m][ri] * corr + e0 + e1;
-                *reinterpret_cast<uint32_t*>(sP + row_off(r, warp, kKeys) + (lane & 3) * 4) = pack_bf16x2(e0, e1);
-#pragma unroll
-                for (int i = 0; i < VT * 2; ++i) {
-                    o[m][i][ri * 2] *= corr;
-                    o[m][i][ri * 2 + 1] *= corr;
-                }
+            for (int q = 1; q < 4; ++q) {
+                const float4 y = *reinterpret_cast<const float4*>(sS + (q * R + srow) * kScorePitch + key);
+                x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
             }
+            const float xs[4] = {x.x, x.y, x.z, x.w};
+            const int j = k_lo + tile * kKeys + key;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                v[g][e] = j + e >= lo && j + e < k_hi ? xs[e] * p.scale_log2 : -CUDART_INF_F;
+                mx = fmaxf(mx, v[g][e]);
+            }
+        }
+#pragma unroll
+        for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+        const float base = mx == -CUDART_INF_F ? 0.f : mx;
+        const float corr = exp2f(m_run - base);
+        m_run = mx;
+        l_run *= corr;
+#pragma unroll
+        for (int g = 0; g < NQ; ++g) {
+            float e[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                e[k] = exp2f(v[g][k] - base);
+                l_run += e[k];
+            }
+            const int key = (g * TPR + sc) * 4;
+            *reinterpret_cast<uint2*>(sP + p_off(srow, key / 8) + (key & 4) * 2) = make_uint2(pack_bf16x2(e[0], e[1]), pack_bf16x2(e[2], e[3]));
+        }
+        if (sc == 0) sCorr[srow] = corr;
         __syncthreads();
         // ---- O += P V for this warp's value columns
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int ri = 0; ri < 2; ++ri) {
+                const float c = sCorr[m * 16 + ri * 8 + (lane >> 2)];
+#pragma unroll
+                for (int i = 0; i < VT * 2; ++i) {
+                    o[m][i][ri * 2] *= c;
+                    o[m][i][ri * 2 + 1] *= c;
+                }
+            }
 #pragma unroll
         for (int kk = 0; kk < kKeys / 16; ++kk) {
             uint32_t pf[MT][4];
 #pragma unroll
             for (int m = 0; m < MT; ++m)
-                ldsm_x4(smem_u32(sP + row_off(m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1), kk * 2 + (lane >> 4), kKeys)), pf[m][0], pf[m][1], pf[m][2], pf[m][3]);
+                ldsm_x4(smem_u32(sP + p_off(m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1), kk * 2 + (lane >> 4))), pf[m][0], pf[m][1], pf[m][2], pf[m][3]);
 #pragma unroll
-            for (int v = 0; v < VT; ++v) {
-                const int col = (warp * VT + v) * 16;
-                if (col >= a.cpad) break;
-                uint32_t b0, b1, b2, b3;
-                const int q = lane >> 3;
-                ldsm_x4_t(smem_u32(kS + row_off(kk * 16 + (q & 1) * 8 + (lane & 7), col / 8 + (q >> 1), pitch)), b0, b1, b2, b3);
+            for (int w = 0; w < VT; ++w) {
+                const int col = (warp * VT + w) * 16;
+                if (col < a.cpad) {
+                    uint32_t b0, b1, b2, b3;
+                    ldsm_x4_t(smem_u32(kS + (kk * 16 + (gm & 1) * 8 + (lane & 7)) * pitch + col * 2 + (gm >> 1) * 16), b0, b1, b2, b3);
 #pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    mma16816<false>(o[m][2 * v], pf[m], b0, b1);
-                    mma16816<false>(o[m][2 * v + 1], pf[m], b2, b3);
+                    for (int m = 0; m < MT; ++m) {
+                        mma16816<false>(o[m][2 * w], pf[m], b0, b1);
+                        mma16816<false>(o[m][2 * w + 1], pf[m], b2, b3);
+                    }
                 }
             }
         }
     }
-    cp_async_wait<0>();
-    // ---- denominators: every warp holds the sums over its own keys
-    __syncthreads();
+    // ---- denominators
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int ri = 0; ri < 2; ++ri) {
-            float l = l_run[m][ri];
-            l += __shfl_xor_sync(0xffffffffu, l, 1);
-            l += __shfl_xor_sync(0xffffffffu, l, 2);
-            if ((lane & 3) == 0) sMax[(m * 16 + ri * 8 + (lane >> 2)) * kWarps + warp] = l;
-        }
+    for (int d = 1; d < TPR; d <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, d);
     __syncthreads();
+    if (sc == 0) {
+        sCorr[srow] = l_run;
+        sMax[srow] = m_run;
+    }
+    __syncthreads();
+    if (!ok) {                                                           // a copy did not arrive: reported, nothing is stored
+        for (int i = 0; i < 200; ++i) __nanosleep(1000);                 // copies still in flight land before the shared memory is reused
+        return;
+    }
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int ri = 0; ri < 2; ++ri) {
             const int r = m * 16 + ri * 8 + (lane >> 2), h = h0 + r;
             if (h >= p.Hq) continue;
-            float l = 0.f;
-#pragma unroll
-            for (int w = 0; w < kWarps; ++w) l += sMax[r * kWarps + w];
-            const float inv = p.nsplit > 1 ? 1.f : (l > 0.f ? 1.f / l : 0.f);
-            float* sc = p.scratch + (((size_t)t * p.Hq + h) * p.nsplit + split) * (a.cpad + 2);
+            const float l = sCorr[r], inv = l > 0.f ? 1.f / l : 0.f;
+            float* scr = p.scratch + (((size_t)t * p.Hq + h) * p.nsplit + split) * (a.cpad + 2);
 #pragma unroll
             for (int i = 0; i < VT * 2; ++i) {
                 const int col = warp * VT * 16 + i * 8 + (lane & 3) * 2;
-                if (col >= a.cpad) break;
-                if (p.nsplit > 1) {
-                    sc[col] = o[m][i][ri * 2];
-                    sc[col + 1] = o[m][i][ri * 2 + 1];
-                } else {
-                    *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.o_head + col) =
-                        pack_bf16x2(o[m][i][ri * 2] * inv, o[m][i][ri * 2 + 1] * inv);
+                if (col < a.cpad) {
+                    if (p.nsplit > 1)
+                        *reinterpret_cast<float2*>(scr + col) = make_float2(o[m][i][ri * 2], o[m][i][ri * 2 + 1]);
+                    else
+                        *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.o_head + col) =
+                            pack_bf16x2(o[m][i][ri * 2] * inv, o[m][i][ri * 2 + 1] * inv);
                 }
             }
             if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
-                sc[a.cpad] = m_run[m][ri];
-                sc[a.cpad + 1] = l;
+                scr[a.cpad] = sMax[r];
+                scr[a.cpad + 1] = l;
             }
         }
 }
 
-template <int MT, int VT>
+template <int MT, int VT, int KQ>
 int launch_latent(const LatentKParams& a, cudaStream_t stream) {
-    const int smem = (MT * 16 + 2 * kKeys) * a.pitch * 2 + MT * 16 * kKeys * 2 + MT * 16 * kWarps * 4 + 128;
-    if (smem > 227 * 1024 - 64) return ERR_UNSUPPORTED;
-    auto kern = latent_attention_kernel<MT, VT>;
+    constexpr int R = MT * 16;
+    const int pitch = a.row * 2 + 16, shared_part = R * pitch > 4 * R * kScorePitch * 4 ? R * pitch : 4 * R * kScorePitch * 4;
+    const int smem = 2 * kKeys * pitch + shared_part + R * kKeys * 2 + 2 * R * 4 + 64 + 128;
+    if (smem > 227 * 1024 || a.row / 16 > 4 * KQ) return ERR_UNSUPPORTED;
+    auto kern = latent_attention_kernel<MT, VT, KQ>;
     static std::atomic<uint64_t> configured{0};   // one bit per device; raised to the whole limit once
     int dev = 0;
     OVB_CHECK_CUDA(cudaGetDevice(&dev));
     const uint64_t bit = 1ull << (dev & 63);
     if (!(configured.load(std::memory_order_acquire) & bit)) {
-        OVB_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 64));
+        OVB_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         configured.fetch_or(bit, std::memory_order_release);
     }
-    OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.p.T, ceil_div(a.p.Hq, MT * 16), a.p.nsplit), dim3(kWarps * 32), (size_t)smem, stream, a));
+    OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.p.T, ceil_div(a.p.Hq, R), a.p.nsplit), dim3(kWarps * 32), (size_t)smem, stream, a));
     return a.p.nsplit > 1 ? launch_decode_combine(a.p, a.cpad, stream) : 0;
 }
 
@@ -284,14 +330,14 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __res
 }  // namespace
 
 int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int max_ctx, long long scratch_bytes, cudaStream_t stream) {
-    if (p.block_size % 8 || row % 16 || cpad > 512 || row > 1024 || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
+    if (row % 16 || cpad > 512 || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
         (reinterpret_cast<uintptr_t>(p.q) & 15) || (reinterpret_cast<uintptr_t>(p.k_cache) & 15) || (reinterpret_cast<uintptr_t>(p.out) & 3) || p.T > (1 << 30))
         return ERR_UNSUPPORTED;
     LatentKParams a;
     a.p = p;
     a.row = row;
-    a.pitch = (row + 63) / 64 * 64;
     a.cpad = cpad;
+    a.status = status_word();
     a.p.dv_store = cpad;
     const int mt = p.Hq <= 16 ? 1 : 2;
     const int keys = p.sliding_window > 0 && p.sliding_window + kKeys - 1 < max_ctx ? p.sliding_window + kKeys - 1 : max_ctx;
@@ -312,8 +358,8 @@ int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int m
     a.p.nsplit = best;
     a.p.keys_per_split = ceil_div(tiles, best) * kKeys;
     const int vt = cpad <= 128 ? 1 : cpad <= 256 ? 2 : 4;
-    if (mt == 1) return vt == 1 ? launch_latent<1, 1>(a, stream) : vt == 2 ? launch_latent<1, 2>(a, stream) : launch_latent<1, 4>(a, stream);
-    return vt == 1 ? launch_latent<2, 1>(a, stream) : vt == 2 ? launch_latent<2, 2>(a, stream) : launch_latent<2, 4>(a, stream);
+    if (mt == 1) return vt == 1 ? launch_latent<1, 1, 3>(a, stream) : vt == 2 ? launch_latent<1, 2, 5>(a, stream) : launch_latent<1, 4, 9>(a, stream);
+    return vt == 1 ? launch_latent<2, 1, 3>(a, stream) : vt == 2 ? launch_latent<2, 2, 5>(a, stream) : launch_latent<2, 4, 9>(a, stream);
 }
 
 }  // namespace ovb

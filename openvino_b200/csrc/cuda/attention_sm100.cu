@@ -332,16 +332,24 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
             tc_fence_before_sync();
             mbar_arrive(&p_full[st]);
         }
-        // ---- epilogue: O / l
+        // ---- epilogue: O / l. The gate's row is requested before the last product is waited for.
+        uint4 gw[DV / 8];
+        const bool gated = p.gate != nullptr && row_valid;
+        if (gated) {
+            const uint4* gate = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.gate) + (size_t)(tok_begin + tq0 + tl) * p.ld_gate +
+                                                               (size_t)(h * G + g) * p.gate_head);
+#pragma unroll
+            for (int c = 0; c < DV / 8; ++c)
+                if (c * 8 < p.dv_store) gw[c] = gate[c];
+        }
         if (ok && ntiles > 0) ok = mbar_wait(&pv_done[(ntiles - 1) & 1], ((ntiles - 1) >> 1) & 1, abort_flag, status);
         if (ok) {
             tc_fence_after_sync();
             const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
             uint8_t* dst = reinterpret_cast<uint8_t*>(p.out) + ((size_t)(tok_begin + tq0 + tl) * p.ldo + (size_t)(h * G + g) * p.o_head) * 2;
-            const uint8_t* gate = p.gate == nullptr ? nullptr : reinterpret_cast<const uint8_t*>(p.gate) +
-                                  ((size_t)(tok_begin + tq0 + tl) * p.ld_gate + (size_t)(h * G + g) * p.gate_head) * 2;
-#pragma unroll 1
-            for (int c = 0; c < p.dv_store; c += 16) {
+#pragma unroll
+            for (int c = 0; c < DV; c += 16) {
+                if (c >= p.dv_store) break;
                 uint32_t o[16];
                 if (ntiles > 0) {
                     tmem_ld_x16(lane_base + TM_O + c, o);
@@ -350,9 +358,8 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
 #pragma unroll
                     for (int i = 0; i < 16; ++i) o[i] = 0u;
                 }
-                if (gate != nullptr && row_valid) {
-                    uint4 gw[2] = {*reinterpret_cast<const uint4*>(gate + c * 2), *reinterpret_cast<const uint4*>(gate + c * 2 + 16)};
-                    const __nv_bfloat16* gv = reinterpret_cast<const __nv_bfloat16*>(gw);
+                if (gated) {
+                    const __nv_bfloat16* gv = reinterpret_cast<const __nv_bfloat16*>(gw + c / 8);
 #pragma unroll
                     for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) / (1.f + __expf(-__bfloat162float(gv[i]))));
                 }

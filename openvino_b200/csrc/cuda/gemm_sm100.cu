@@ -647,6 +647,8 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         const bool fast = p.world <= 1 && p.splits == 1 && !p.out_f32 && (n0 + TILE_N <= p.N) && (p.ldo % 8 == 0) &&
                           ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0) &&
                           out_col % 8 == 0 && (p.residual == nullptr || ((p.ldr % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.residual) & 15) == 0)));
+        // fp32 output of a tile inside N: the lanes of a warp hold 32 consecutive columns of a token, stored as they are
+        const bool plain32 = !QUANT && p.world <= 1 && p.splits == 1 && p.out_f32 && n0 + TILE_N <= p.N && p.residual == nullptr && p.act == OVB_ACT_NONE;
         // fp32 staging keeps a single rounding (after the residual add): BT x 128 x 4 bytes <= 2 * STAGE_BYTES
         float* stage_out = reinterpret_cast<float*>(smem);
 
@@ -1092,6 +1094,11 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
                         stage_out[(c0 + j) * TILE_N + row] = apply_act(__uint_as_float(r[j]) + bias_v, p.act);
+                } else if (plain32) {
+                    float* o = reinterpret_cast<float*>(p.out) + (size_t)(t0 + c0) * p.ldo + out_col + oc;
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        if (t0 + c0 + j < T_end) o[(size_t)j * p.ldo] = __uint_as_float(r[j]) + bias_v;
                 } else if (p.splits == 1) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j) finish(c0 + j, __uint_as_float(r[j]));

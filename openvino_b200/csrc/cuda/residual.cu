@@ -20,7 +20,13 @@ __global__ void stream_embed_kernel(const int* __restrict__ ids, const E* __rest
     int id = ids[row];
     if ((unsigned)id >= (unsigned)vocab) id = 0;
     const E* src = table + (size_t)id * ldt;
-    for (int c = threadIdx.x; c < cols; c += blockDim.x) {
+    const int nvec = (cols % 4 == 0 && ldt % 4 == 0) ? cols / 4 : 0;
+    for (int k = threadIdx.x; k < nvec; k += blockDim.x) {
+        const float4 v = ld4_f32(src + k * 4);
+        st4_f32(h + (size_t)row * ldh + k * 4, v);
+        if (x) st4_f32(x + (size_t)row * ldx + k * 4, v);
+    }
+    for (int c = nvec * 4 + threadIdx.x; c < cols; c += blockDim.x) {
         const float v = ld_f32(src + c);
         h[(size_t)row * ldh + c] = v;
         if (x) st_f32(x + (size_t)row * ldx + c, v);
@@ -115,7 +121,7 @@ using namespace ovb;
 
 int ovb_stream_embed(const int* ids, const void* table, float* h, void* x, int rows, int cols, int vocab, int ldt, int ldh, int ldx, int dtype,
                      ovb_stream_t stream) {
-    OVB_REQUIRE(ids && table && h && rows > 0 && cols > 0 && vocab > 0, "ovb_stream_embed: bad arguments");
+    OVB_REQUIRE(ids && table && h && rows > 0 && cols > 0 && vocab > 0 && ldh % 4 == 0 && ldx % 4 == 0, "ovb_stream_embed: bad arguments");
     return dispatch_store(dtype, "ovb_stream_embed", [&](auto e) -> int {
         using E = decltype(e);
         OVB_CHECK_CUDA(launch_pdl(stream_embed_kernel<E>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, ids, (const E*)table, h, (E*)x, cols, vocab, ldt,
