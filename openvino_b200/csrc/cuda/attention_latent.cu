@@ -34,6 +34,7 @@ constexpr int kScorePitch = kKeys + 8;    // floats per row of partial scores
 struct LatentKParams {
     PaKParams p;
     int row, cpad;            // elements of a cached row that take part, value columns (multiples of 16)
+    int block_shift;          // log2 of the block size
     int* status;
 };
 
@@ -86,17 +87,23 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
     const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int ntiles = k_hi > k_lo ? (k_hi - k_lo + kKeys - 1) / kKeys : 0;
     const int* blocks = p.block_indices + p.block_indices_begins[b];
-    auto load = [&](int tile, int st) {      // warp 0; keys past the end repeat the last one (finite, and masked)
-        if (lane == 0) mbar_arrive_expect_tx(&full[st], kKeys * row_bytes);
-        __syncwarp();
-        for (int r = lane; r < kKeys; r += 32) {
-            const int j = min(k_lo + tile * kKeys + r, k_hi - 1);
-            const int blk = OVB_DBG_BLOCK(blocks[j / p.block_size]);
-            bulk_load_1d(sK + st * stage + r * pitch, reinterpret_cast<const uint8_t*>(p.k_cache) + ((size_t)blk * p.block_size + j % p.block_size) * p.k_row * 2,
-                         row_bytes, &full[st]);
+    // Eight lanes of every warp copy one row of a tile each; the row's place is looked up a tile ahead. Keys past the end repeat
+    // the last one (finite, and masked).
+    const uint8_t* next_row = nullptr;
+    auto look_up = [&](int tile) {
+        if (lane < 8 && tile < ntiles) {
+            const int j = min(k_lo + tile * kKeys + warp * 8 + lane, k_hi - 1);
+            const int blk = OVB_DBG_BLOCK(blocks[j >> a.block_shift]);
+            next_row = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk << a.block_shift) + (j & (p.block_size - 1))) * p.k_row * 2;
         }
     };
-    if (warp == 0 && ntiles > 0) load(0, 0);
+    auto load = [&](int tile, int st) {
+        if (tid == 0) mbar_arrive_expect_tx(&full[st], kKeys * row_bytes);
+        if (lane < 8) bulk_load_1d(sK + st * stage + (warp * 8 + lane) * pitch, next_row, row_bytes, &full[st]);
+        look_up(tile + 1);
+    };
+    look_up(0);
+    if (ntiles > 0) load(0, 0);
     cp_async_wait<0>();
     __syncthreads();
     // ---- this warp's quarter of the queries, in registers
@@ -123,7 +130,7 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
     for (int tile = 0; tile < ntiles; ++tile) {
         const int st = tile & 1;
         __syncthreads();                                                 // the other stage, the partials and P are free
-        if (warp == 0 && tile + 1 < ntiles) load(tile + 1, st ^ 1);
+        if (tile + 1 < ntiles) load(tile + 1, st ^ 1);
         ok = mbar_wait(&full[st], (tile >> 1) & 1, abort_flag, a.status);
         const uint8_t* kS = sK + st * stage;
         // ---- partial scores: 32 keys of half kg over the columns of quarter kq
@@ -312,7 +319,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __res
     if (blockIdx.x == 0)
         for (int b = threadIdx.x; b <= B; b += 256) kv_rows[b] = s_begin[b];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int r = blockIdx.x * 64 + warp; r < min(rows, (int)blockIdx.x * 64 + 64); r += 8) {
+    for (int r = blockIdx.x * 16 + warp; r < min(rows, (int)blockIdx.x * 16 + 16); r += 8) {
         int lo = 0, hi = B;                  // last b with s_begin[b] <= r
         while (lo + 1 < hi) {
             const int mid = (lo + hi) / 2;
@@ -330,13 +337,15 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __res
 }  // namespace
 
 int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int max_ctx, long long scratch_bytes, cudaStream_t stream) {
-    if (row % 16 || cpad > 512 || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
+    if (row % 16 || cpad > 512 || (p.block_size & (p.block_size - 1)) || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
         (reinterpret_cast<uintptr_t>(p.q) & 15) || (reinterpret_cast<uintptr_t>(p.k_cache) & 15) || (reinterpret_cast<uintptr_t>(p.out) & 3) || p.T > (1 << 30))
         return ERR_UNSUPPORTED;
     LatentKParams a;
     a.p = p;
     a.row = row;
     a.cpad = cpad;
+    a.block_shift = 0;
+    while ((1 << a.block_shift) < p.block_size) ++a.block_shift;
     a.status = status_word();
     a.p.dv_store = cpad;
     const int mt = p.Hq <= 16 ? 1 : 2;
@@ -380,7 +389,7 @@ int ovb_latent_gather(const void* cache, void* out, int* kv_rows, const int* pas
                 "ovb_latent_gather: bad arguments");
     OVB_REQUIRE(cols % 8 == 0 && row_pitch % 8 == 0 && out_pitch % 8 == 0 && cols <= row_pitch && cols <= out_pitch,
                 "ovb_latent_gather: rows must be multiples of 8 elements");
-    OVB_CHECK_CUDA(launch_pdl(latent_gather_kernel, dim3(ceil_div(rows, 64)), dim3(256), (size_t)(B + 1) * 4, (cudaStream_t)stream, (const uint8_t*)cache,
+    OVB_CHECK_CUDA(launch_pdl(latent_gather_kernel, dim3(ceil_div(rows, 16)), dim3(256), (size_t)(B + 1) * 4, (cudaStream_t)stream, (const uint8_t*)cache,
                               (uint8_t*)out, kv_rows, past_lens, subsequence_begins, block_indices, block_indices_begins, B, rows, cols * 2, row_pitch * 2,
                               out_pitch * 2, window, block_size));
     return 0;

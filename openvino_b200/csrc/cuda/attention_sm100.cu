@@ -361,7 +361,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                 if (gated) {
                     const __nv_bfloat16* gv = reinterpret_cast<const __nv_bfloat16*>(gw + c / 8);
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) / (1.f + __expf(-__bfloat162float(gv[i]))));
+                    for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__fdividef(__uint_as_float(o[i]), 1.f + __expf(-__bfloat162float(gv[i]))));
                 }
                 if (row_valid) {
                     uint4 w0, w1;

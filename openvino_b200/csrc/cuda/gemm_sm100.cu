@@ -42,6 +42,9 @@ constexpr int TILE_K = 64;       // bf16 elements per k-block = one 128-byte swi
 // a CTA there (its instructions issue several times slower while the dequant warps run), and two CTAs bring two issuers.
 constexpr int num_dq_warps(int bt, int wmode) { (void)bt; (void)wmode; return 8; }
 constexpr int gemm_threads(int bt, int wmode) { return (3 + num_dq_warps(bt, wmode)) * 32; }
+#ifndef OVB_GEMM_DIRECT
+#define OVB_GEMM_DIRECT 1        // 16-bit epilogue of the larger tiles without a stop in shared memory
+#endif
 constexpr int MAX_STAGES = 8;    // MMA stages
 constexpr int MAX_PSLOTS = 16;   // packed-weight ring slots
 constexpr int kBandN = 16;       // weight tiles per rasterisation band
@@ -647,6 +650,8 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         const bool fast = p.world <= 1 && p.splits == 1 && !p.out_f32 && (n0 + TILE_N <= p.N) && (p.ldo % 8 == 0) &&
                           ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0) &&
                           out_col % 8 == 0 && (p.residual == nullptr || ((p.ldr % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.residual) & 15) == 0)));
+        // plain 16-bit output of the larger tiles: straight from the accumulator's registers
+        const bool direct16 = OVB_GEMM_DIRECT && BT >= 128 && fast && p.act == OVB_ACT_NONE && p.residual == nullptr;
         // fp32 output of a tile inside N: the lanes of a warp hold 32 consecutive columns of a token, stored as they are
         const bool plain32 = !QUANT && p.world <= 1 && p.splits == 1 && p.out_f32 && n0 + TILE_N <= p.N && p.residual == nullptr && p.act == OVB_ACT_NONE;
         // fp32 staging keeps a single rounding (after the residual add): BT x 128 x 4 bytes <= 2 * STAGE_BYTES
@@ -1090,6 +1095,17 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 if (comm && p.splits == 1) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j) stage_out[(c0 + j) * TILE_N + row] = __uint_as_float(r[j]);
+                } else if (direct16) {
+                    // two tokens at a time: neighbouring lanes exchange a value, so that each stores two adjacent columns of one token
+                    const int odd = lane & 1;
+                    E* o = reinterpret_cast<E*>(p.out) + (size_t)(t0 + c0 + odd) * p.ldo + out_col + (oc & ~1);
+#pragma unroll
+                    for (int j = 0; j < 16; j += 2) {
+                        const float v0 = __uint_as_float(r[j]) + bias_v, v1 = __uint_as_float(r[j + 1]) + bias_v;
+                        const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
+                        E pair[2] = {from_float<E>(odd ? got : v0), from_float<E>(odd ? v1 : got)};
+                        if (t0 + c0 + j + odd < T_end) *reinterpret_cast<uint32_t*>(o + (size_t)j * p.ldo) = *reinterpret_cast<uint32_t*>(pair);
+                    }
                 } else if (fast) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
@@ -1134,7 +1150,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                     }
                 }
             }
-        } else if (fast) {
+        } else if (fast && !direct16) {
             asm volatile("bar.sync 1, %0;" ::"n"(DQ_THREADS));
             if (acc_ok) {
                 constexpr int PIECES = BT * (TILE_N / 8);     // 16-byte pieces in the tile

@@ -228,7 +228,29 @@ gated_delta_rule_kernel(const float* __restrict__ q, const float* __restrict__ k
 
 // u[t, c] = bias[c] + sum_j w[j, c] * x[t - (taps - 1) + j, c]. u is laid out block by block with a pitch of ub_pitch columns per
 // block of bw channels, as the block-diagonal gate product reads it. A thread owns V consecutive channels of a strip of tokens.
-template <class E, int V>
+template <int V>
+__device__ __forceinline__ void conv_load(const float* src, float (&v)[V]) {
+    if constexpr (V == 4) {
+        const float4 q = ld4_f32(src);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    } else {
+        v[0] = *src;
+    }
+}
+template <int V>
+__device__ __forceinline__ void conv_load(const __nv_bfloat16* src, float (&v)[V]) {
+    if constexpr (V == 4) {
+        const float4 q = ld4_f32(src);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    } else {
+        v[0] = __bfloat162float(*src);
+    }
+}
+
+constexpr int CONV_STRIP = 8;    // tokens per thread of a prompt
+
+// TAPS > 0: the number of taps at compile time; a strip whose inputs all lie in one sequence's chunk then reads each of them once.
+template <class E, int V, int TAPS>
 __global__ void __launch_bounds__(128) causal_conv_kernel(ovb_rglru_args p, int strip) {
     pdl_enter();
     const int c = (blockIdx.y * 128 + threadIdx.x) * V, keep = p.taps - 1;
@@ -237,16 +259,33 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ovb_rglru_args p, int 
     const int t_end = min(p.T, t + strip);
     while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
     const E* x = reinterpret_cast<const E*>(p.x) + c;
-    auto load = [&](const auto* src, float (&v)[V]) {
-        if constexpr (V == 4) {
-            const float4 q = ld4_f32(src);
-            v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
-        } else {
-            v[0] = ld_f32(src);
-        }
+    E* u = reinterpret_cast<E*>(p.u) + (c / p.bw) * p.ub_pitch + c % p.bw;
+    auto put = [&](int tok, const float (&acc)[V]) {
+        if constexpr (V == 4) st4_f32(u + (size_t)tok * p.ldu, make_float4(acc[0], acc[1], acc[2], acc[3]));
+        else st_f32(u + (size_t)tok * p.ldu, acc[0]);
     };
     float bias[V];
-    load(p.conv_b + c, bias);
+    conv_load<V>(p.conv_b + c, bias);
+    if (TAPS > 0 && strip == CONV_STRIP && t - (TAPS - 1) >= p.subsequence_begins[b] && t + CONV_STRIP <= p.subsequence_begins[b + 1]) {
+        constexpr int KEEP = TAPS > 0 ? TAPS - 1 : 0, TW = TAPS > 0 ? TAPS : 1;
+        float in[CONV_STRIP + KEEP][V], w[TW][V];
+#pragma unroll
+        for (int j = 0; j < CONV_STRIP + KEEP; ++j) conv_load<V>(x + (size_t)(t - KEEP + j) * p.ldx, in[j]);
+#pragma unroll
+        for (int j = 0; j < TW; ++j) conv_load<V>(p.conv_w + (size_t)j * p.N + c, w[j]);
+#pragma unroll
+        for (int k = 0; k < CONV_STRIP; ++k) {
+            float acc[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                acc[i] = bias[i];
+#pragma unroll
+                for (int j = 0; j < TW; ++j) acc[i] = fmaf(w[j][i], in[k + j][i], acc[i]);
+            }
+            put(t + k, acc);
+        }
+        return;
+    }
     for (; t < t_end; ++t) {
         while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
         const int begin = p.subsequence_begins[b];
@@ -256,157 +295,101 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ovb_rglru_args p, int 
         for (int j = 0; j < p.taps; ++j) {
             const int s = t - keep + j;                  // token; before the chunk of the sequence: from its state
             float v[V] = {}, w[V];
-            if (s >= begin) load(x + (size_t)s * p.ldx, v);
-            else if (p.past_lens[b] != 0) load(p.conv_state + ((size_t)p.slots[b] * keep + s - begin + keep) * p.N + c, v);
-            load(p.conv_w + (size_t)j * p.N + c, w);
+            if (s >= begin) conv_load<V>(x + (size_t)s * p.ldx, v);
+            else if (p.past_lens[b] != 0) conv_load<V>(p.conv_state + ((size_t)p.slots[b] * keep + s - begin + keep) * p.N + c, v);
+            conv_load<V>(p.conv_w + (size_t)j * p.N + c, w);
 #pragma unroll
             for (int i = 0; i < V; ++i) acc[i] = fmaf(w[i], v[i], acc[i]);
         }
-        E* u = reinterpret_cast<E*>(p.u) + (size_t)t * p.ldu + (c / p.bw) * p.ub_pitch + c % p.bw;
-        if constexpr (V == 4) st4_f32(u, make_float4(acc[0], acc[1], acc[2], acc[3]));
-        else st_f32(u, acc[0]);
+        put(t, acc);
     }
 }
 
 __device__ __forceinline__ float rec_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 // gelu of the other branch: 0.5 z (1 + tanh(v)) = z * sigmoid(2 v)
 __device__ __forceinline__ float rec_gelu_tanh(float z) { return z * rec_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
+__device__ __forceinline__ float rec_sqrt(float z) {
+    float r;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(z));
+    return r;
+}
 
 constexpr int LRU_L = 8;    // tokens per warp and round
 
-template <int V>
-__device__ __forceinline__ void rec_load(const float* src, float (&v)[V]) {
-    if constexpr (V == 2) {
-        const float2 q = *reinterpret_cast<const float2*>(src);
-        v[0] = q.x; v[1] = q.y;
-    } else {
-        v[0] = *src;
-    }
-}
-template <int V>
-__device__ __forceinline__ void rec_load(const __nv_bfloat16* src, float (&v)[V]) {
-    if constexpr (V == 2) {
-        const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
-        v[0] = q.x; v[1] = q.y;
-    } else {
-        v[0] = __bfloat162float(*src);
-    }
-}
-template <int V>
-__device__ __forceinline__ void rec_store(float* dst, const float (&v)[V]) {
-    if constexpr (V == 2) *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
-    else *dst = v[0];
-}
-template <int V>
-__device__ __forceinline__ void rec_store(__nv_bfloat16* dst, const float (&v)[V]) {
-    if constexpr (V == 2) *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v[0], v[1]);
-    else *dst = __float2bfloat16_rn(v[0]);
-}
-
-// One group of 32 * V channels (V a lane) of one sequence. The NW warps of the group take consecutive pieces of LRU_L tokens: each
+// One group of 32 channels (a lane each) of one sequence. The NW warps of the group take consecutive pieces of LRU_L tokens: each
 // composes the affine maps S -> a S + b of its piece, the pieces' maps are chained through shared memory, and the piece is then
 // replayed from its true starting state. NW = 1 (decode): a CTA holds four independent groups.
-template <class E, int NW, int V>
+template <class E, int NW>
 __global__ void __launch_bounds__(NW == 1 ? 128 : NW * 32) lru_scan_kernel(ovb_rglru_args p) {
     pdl_enter();
-    __shared__ float sA[NW][32 * V], sB[NW][32 * V];
+    __shared__ float sA[2][NW][32], sB[2][NW][32];        // (two sets: one barrier per round)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int b = blockIdx.y, w = NW == 1 ? 0 : warp;
-    const int c = ((NW == 1 ? blockIdx.x * 4 + warp : blockIdx.x) * 32 + lane) * V;
-    const bool live = c < p.N;                            // (V channels lie in one block: bw is a multiple of V)
+    const int c = (NW == 1 ? blockIdx.x * 4 + warp : blockIdx.x) * 32 + lane;
+    const bool live = c < p.N;
     const int begin = p.subsequence_begins[b], len = p.subsequence_begins[b + 1] - begin, slot = p.slots[b];
     const bool fresh = p.past_lens[b] == 0;
     const int cc = live ? c : 0, blk = cc / p.bw, cb = cc % p.bw;
-    float lam[V], br[V], bi[V], carry[V] = {};
-    rec_load<V>(p.log_decay + cc, lam);
-    rec_load<V>(p.gate_b + cc, br);
-    rec_load<V>(p.gate_b + p.N + cc, bi);
+    const float lam = p.log_decay[cc], br = p.gate_b[cc], bi = p.gate_b[p.N + cc];
+    const float* gates = p.gates + (size_t)begin * p.ldg + blk * p.gb_pitch + cb;
+    const E* us = reinterpret_cast<const E*>(p.u) + (size_t)begin * p.ldu + blk * p.ub_pitch + cb;
+    const E* ys = reinterpret_cast<const E*>(p.y) + (size_t)begin * p.ldy + cc;
+    E* out = reinterpret_cast<E*>(p.out) + (size_t)begin * p.ldo + cc;
     float* state = p.state + (size_t)slot * p.N + cc;
-    if (!fresh && live) rec_load<V>(state, carry);
-    for (int t0 = 0; t0 < len; t0 += NW * LRU_L) {
-        const int tw = t0 + w * LRU_L;
-        float a[LRU_L][V], x[LRU_L][V], A[V], S[V];
+    float carry = fresh ? 0.f : *state;
+    int set = 0;
+    for (int t0 = 0; t0 < len; t0 += NW * LRU_L, set ^= 1) {
+        const int tw = t0 + w * LRU_L, n = min(LRU_L, len - tw);
+        float a[LRU_L], x[LRU_L], y[LRU_L], A = 1.f, S = 0.f;
+        {
+            float gr[LRU_L], gi[LRU_L];
 #pragma unroll
-        for (int i = 0; i < V; ++i) {
-            A[i] = 1.f;
-            S[i] = 0.f;
-        }
-#pragma unroll
-        for (int k = 0; k < LRU_L; ++k) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) {
-                a[k][i] = 1.f;
-                x[k][i] = 0.f;
-            }
-            if (live && tw + k < len) {
-                const size_t t = (size_t)(begin + tw + k);
-                const float* g = p.gates + t * p.ldg + blk * p.gb_pitch + cb;
-                float gr[V], gi[V], u[V];
-                rec_load<V>(g, gr);
-                rec_load<V>(g + p.gi_off, gi);
-                rec_load<V>(reinterpret_cast<const E*>(p.u) + t * p.ldu + blk * p.ub_pitch + cb, u);
-#pragma unroll
-                for (int i = 0; i < V; ++i) {
-                    // e = a - 1, exact for a close to one; 1 - a^2 = -e (2 + e)
-                    const float e = expm1f(-rec_sigmoid(gr[i] + br[i]) * lam[i]);
-                    a[k][i] = 1.f + e;
-                    x[k][i] = sqrtf(-e * (2.f + e)) * rec_sigmoid(gi[i] + bi[i]) * u[i];
-                }
+            for (int k = 0; k < LRU_L; ++k) {             // all loads of the piece at once; past its end the last token again
+                const size_t t = (size_t)min(tw + k, len - 1);
+                gr[k] = gates[t * p.ldg];
+                gi[k] = gates[t * p.ldg + p.gi_off];
+                x[k] = ld_f32(us + t * p.ldu);
+                y[k] = ld_f32(ys + t * p.ldy);
             }
 #pragma unroll
-            for (int i = 0; i < V; ++i) {
-                S[i] = fmaf(a[k][i], S[i], x[k][i]);
-                A[i] *= a[k][i];
+            for (int k = 0; k < LRU_L; ++k) {
+                // e = a - 1, exact for a close to one; 1 - a^2 = -e (2 + e)
+                const float e = expm1f(-rec_sigmoid(gr[k] + br) * lam);
+                a[k] = k < n ? 1.f + e : 1.f;
+                x[k] = k < n ? rec_sqrt(-e * (2.f + e)) * rec_sigmoid(gi[k] + bi) * x[k] : 0.f;
+                y[k] = rec_gelu_tanh(y[k]);
+                S = fmaf(a[k], S, x[k]);
+                A *= a[k];
             }
         }
-        float s[V];
-#pragma unroll
-        for (int i = 0; i < V; ++i) s[i] = carry[i];
+        float s = carry;
         if (NW > 1) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) {
-                sA[w][i * 32 + lane] = A[i];
-                sB[w][i * 32 + lane] = S[i];
-            }
+            sA[set][w][lane] = A;
+            sB[set][w][lane] = S;
             __syncthreads();
 #pragma unroll
-            for (int k = 0; k < NW; ++k)
-#pragma unroll
-                for (int i = 0; i < V; ++i) {
-                    if (k == w) s[i] = carry[i];
-                    carry[i] = fmaf(sA[k][i * 32 + lane], carry[i], sB[k][i * 32 + lane]);
-                }
+            for (int k = 0; k < NW; ++k) {
+                if (k == w) s = carry;
+                carry = fmaf(sA[set][k][lane], carry, sB[set][k][lane]);
+            }
         }
 #pragma unroll
         for (int k = 0; k < LRU_L; ++k) {
-            float o[V] = {};
-            const size_t t = (size_t)(begin + tw + k);
-            const bool ok = live && tw + k < len;
-            if (ok) rec_load<V>(reinterpret_cast<const E*>(p.y) + t * p.ldy + c, o);
-#pragma unroll
-            for (int i = 0; i < V; ++i) {
-                s[i] = fmaf(a[k][i], s[i], x[k][i]);
-                o[i] = s[i] * rec_gelu_tanh(o[i]);
-            }
-            if (ok) rec_store<V>(reinterpret_cast<E*>(p.out) + t * p.ldo + c, o);
+            s = fmaf(a[k], s, x[k]);
+            if (live && k < n) st_f32(out + (size_t)(tw + k) * p.ldo, s * y[k]);
         }
-        if (NW == 1) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) carry[i] = s[i];
-        } else {
-            __syncthreads();
-        }
+        if (NW == 1) carry = s;
     }
     if (!live || w != 0) return;
-    rec_store<V>(state, carry);
+    *state = carry;
     const int keep = p.taps - 1;
     float* old = p.conv_state + (size_t)slot * keep * p.N + c;
     for (int j = 0; j < keep; ++j) {
         const int s = len - keep + j;                     // ascending j only reads rows that are not overwritten yet
-        float v[V] = {};
-        if (s >= 0) rec_load<V>(reinterpret_cast<const E*>(p.x) + (size_t)(begin + s) * p.ldx + c, v);
-        else if (!fresh) rec_load<V>(old + (size_t)(s + keep) * p.N, v);
-        rec_store<V>(old + (size_t)j * p.N, v);
+        float v = 0.f;
+        if (s >= 0) v = ld_f32(reinterpret_cast<const E*>(p.x) + (size_t)(begin + s) * p.ldx + c);
+        else if (!fresh) v = old[(size_t)(s + keep) * p.N];
+        old[(size_t)j * p.N] = v;
     }
 }
 
@@ -491,12 +474,16 @@ int ovb_causal_conv(const ovb_rglru_args* a, ovb_stream_t stream) {
     if (int rc = check_rglru(a, "ovb_causal_conv")) return rc;
     return dispatch_store(a->dtype, "ovb_causal_conv", [&](auto e) -> int {
         using E = decltype(e);
-        const int strip = a->max_q_len <= 4 ? 1 : 8;      // (a new sequence for every token: no strip to walk)
+        const int strip = a->max_q_len <= 4 ? 1 : CONV_STRIP;      // (a new sequence for every token: no strip to walk)
         const bool vec = a->bw % 4 == 0 && a->ldx % 4 == 0 && a->ldu % 4 == 0 && a->ub_pitch % 4 == 0 && rec_aligned(a->x) && rec_aligned(a->u);
         const dim3 grid(ceil_div(a->T, strip), ceil_div(a->N, vec ? 512 : 128));
-        if (vec) OVB_CHECK_CUDA(launch_pdl(causal_conv_kernel<E, 4>, grid, dim3(128), 0, (cudaStream_t)stream, *a, strip));
-        else OVB_CHECK_CUDA(launch_pdl(causal_conv_kernel<E, 1>, grid, dim3(128), 0, (cudaStream_t)stream, *a, strip));
-        return 0;
+        auto go = [&](auto kern) -> int {
+            OVB_CHECK_CUDA(launch_pdl(kern, grid, dim3(128), 0, (cudaStream_t)stream, *a, strip));
+            return 0;
+        };
+        if (!vec) return go(causal_conv_kernel<E, 1, 0>);
+        return a->taps == 2 ? go(causal_conv_kernel<E, 4, 2>) : a->taps == 3 ? go(causal_conv_kernel<E, 4, 3>) : a->taps == 4 ? go(causal_conv_kernel<E, 4, 4>)
+                                                                                                             : go(causal_conv_kernel<E, 4, 0>);
     });
 }
 
@@ -506,15 +493,13 @@ int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream) {
     OVB_REQUIRE(a->y && a->gates && a->gate_b && a->log_decay && a->state && a->out, "ovb_lru_scan: null operand");
     return dispatch_store(a->dtype, "ovb_lru_scan", [&](auto e) -> int {
         using E = decltype(e);
-        const bool pair = a->bw % 2 == 0 && a->ldx % 2 == 0 && a->ldy % 2 == 0 && a->ldu % 2 == 0 && a->ldo % 2 == 0 && a->ldg % 2 == 0 &&
-                          a->gb_pitch % 2 == 0 && a->gi_off % 2 == 0 && a->ub_pitch % 2 == 0 && rec_aligned(a->x) && rec_aligned(a->y) && rec_aligned(a->u) &&
-                          rec_aligned(a->out) && rec_aligned(a->gates);
         auto go = [&](auto kern, int channels, int threads) -> int {
             OVB_CHECK_CUDA(launch_pdl(kern, dim3(ceil_div(a->N, channels), a->B), dim3(threads), 0, (cudaStream_t)stream, *a));
             return 0;
         };
-        if (a->max_q_len <= LRU_L) return pair && a->B * a->N > (1 << 17) ? go(lru_scan_kernel<E, 1, 2>, 256, 128) : go(lru_scan_kernel<E, 1, 1>, 128, 128);
-        return pair ? go(lru_scan_kernel<E, 16, 2>, 64, 512) : go(lru_scan_kernel<E, 16, 1>, 32, 512);
+        if (a->max_q_len <= LRU_L) return go(lru_scan_kernel<E, 1>, 128, 128);
+        // many groups: small CTAs, several per SM; few groups: more warps on each sequence
+        return (long long)ceil_div(a->N, 32) * a->B >= 4 * 148 ? go(lru_scan_kernel<E, 4>, 32, 128) : go(lru_scan_kernel<E, 16>, 32, 512);
     });
 }
 
