@@ -1,13 +1,14 @@
 // Latent attention in its absorbed form, and the expansion of cached rows for prefill.
 //
 // latent_attention_kernel: every query head attends to the same cached row per token; the first part of that row is also the value.
-// One CTA serves one token (decode: one sequence), 16 or 32 of its heads and one share of the visible keys. Key tiles of 64 rows
-// pass through two shared-memory stages, one bulk copy per row, and are read for both products:
-//   scores   the 8 warps split the row's columns in quarters and the tile's keys in halves; the queries' fragments of a warp's
-//            quarter stay in registers for the whole loop. The four partial sums meet in shared memory.
-//   softmax  8 or 16 neighbouring threads per head add the partials, mask, keep running maximum and sum; P as bf16.
-//   sums     every warp owns its own slice of the value columns for all 64 keys, so the accumulator needs no merge.
-// Rows are 16 bytes longer in shared memory than in the cache, which spreads ldmatrix over all banks.
+// One CTA of four warps serves one token (decode: one sequence), 16 of its heads and one share of the visible keys; two CTAs or
+// more share an SM and hide each other's barriers. Key tiles of 32 rows pass through two shared-memory stages, one bulk copy per
+// page, and are read for both products:
+//   scores   the warps split the row's columns in quarters; the queries' fragments of a warp's quarter stay in registers for the
+//            whole loop. The four partial sums meet in shared memory.
+//   softmax  8 neighbouring threads per head add the partials, mask, keep running maximum and sum; P as bf16.
+//   sums     every warp owns its own slice of the value columns for all keys of the tile, so the accumulator needs no merge.
+// Pages keep the cache's row pitch in shared memory: a pitch of an odd number of 16-byte pieces spreads ldmatrix over all banks.
 // With split keys the partial sums go to scratch and the decode kernels' merge finishes.
 //
 // latent_gather_kernel: the rows that the windows of a batch's new tokens reach, made contiguous, so that a plain product expands
@@ -27,7 +28,7 @@ OVB_DEBUG_LIMITS_DEFINE
 
 namespace {
 
-constexpr int kWarps = 8, kKeys = 64;
+constexpr int kWarps = 4, kKeys = 32, kHeads = 16;
 
 constexpr int kScorePitch = kKeys + 8;    // floats per row of partial scores
 
@@ -38,22 +39,24 @@ struct LatentKParams {
     int* status;
 };
 
-__device__ __forceinline__ uint32_t p_off(int r, int chunk) { return uint32_t(r * kKeys * 2 + ((chunk ^ (r & 7)) << 4)); }
+// Rows of 64 bytes: two rows share the 128 bytes of all banks.
+__device__ __forceinline__ uint32_t p_off(int r, int chunk) { return uint32_t(r * kKeys * 2 + ((chunk ^ ((r >> 1) & 3)) << 4)); }
 
-// MT: 16-head tiles; VT: 16-column pieces of the value per warp; KQ: most 16-column steps in a quarter of the row.
-template <int MT, int VT, int KQ>
-__global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(LatentKParams a) {
-    constexpr int R = MT * 16, TPR = kWarps * 32 / R, NQ = kKeys / (TPR * 4);    // rows, threads per row, quads of keys per thread
+// VT: 16-column pieces of the value per warp; KQ: most 16-column steps in a quarter of the row.
+template <int VT, int KQ>
+__global__ void __launch_bounds__(kWarps * 32, 2) latent_attention_kernel(LatentKParams a) {
+    constexpr int R = kHeads, TPR = kWarps * 32 / R;    // rows, threads per row (four keys each)
+    static_assert(TPR * 4 == kKeys, "softmax threads cover the tile");
     const PaKParams& p = a.p;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
-    const int row_bytes = a.row * 2, pitch = row_bytes + 16, ksteps = a.row / 16;
+    const int pitch = p.k_row * 2, ksteps = a.row / 16;
     const int stage = kKeys * pitch;
     const int shared_part = max(R * pitch, 4 * R * kScorePitch * 4);
     uint8_t* sK = smem;                                                  // two stages
     uint8_t* sQ = sK + 2 * stage;                                        // queries, then partial scores [4][R][kScorePitch]
     float* sS = reinterpret_cast<float*>(sQ);
-    uint8_t* sP = sQ + shared_part;                                      // [R][64] bf16
+    uint8_t* sP = sQ + shared_part;                                      // [R][32] bf16
     float* sCorr = reinterpret_cast<float*>(sP + R * kKeys * 2);         // [R]
     float* sMax = sCorr + R;                                             // [R]
     uint64_t* full = reinterpret_cast<uint64_t*>(sMax + R);              // [2]
@@ -87,19 +90,23 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
     const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int ntiles = k_hi > k_lo ? (k_hi - k_lo + kKeys - 1) / kKeys : 0;
     const int* blocks = p.block_indices + p.block_indices_begins[b];
-    // Eight lanes of every warp copy one row of a tile each; the row's place is looked up a tile ahead. Keys past the end repeat
-    // the last one (finite, and masked).
-    const uint8_t* next_row = nullptr;
+    // One lane of warp 0 copies each page (or the tile's part of it); its place is looked up a tile ahead. Pages past the last key
+    // repeat the last one, and rows of a page past it hold what the cache holds there: finite, and masked.
+    const int seg = min(p.block_size, kKeys), nseg = kKeys / seg;
+    const uint8_t* next_part = nullptr;
     auto look_up = [&](int tile) {
-        if (lane < 8 && tile < ntiles) {
-            const int j = min(k_lo + tile * kKeys + warp * 8 + lane, k_hi - 1);
+        if (warp == 0 && lane < nseg && tile < ntiles) {
+            int j = k_lo + tile * kKeys + lane * seg;
+            if (j >= k_hi) j = (k_hi - 1) / seg * seg;
             const int blk = OVB_DBG_BLOCK(blocks[j >> a.block_shift]);
-            next_row = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk << a.block_shift) + (j & (p.block_size - 1))) * p.k_row * 2;
+            next_part = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk << a.block_shift) + (j & (p.block_size - 1))) * pitch;
         }
     };
     auto load = [&](int tile, int st) {
-        if (tid == 0) mbar_arrive_expect_tx(&full[st], kKeys * row_bytes);
-        if (lane < 8) bulk_load_1d(sK + st * stage + (warp * 8 + lane) * pitch, next_row, row_bytes, &full[st]);
+        if (warp == 0) {
+            if (lane == 0) mbar_arrive_expect_tx(&full[st], stage);
+            if (lane < nseg) bulk_load_1d(sK + st * stage + lane * seg * pitch, next_part, seg * pitch, &full[st]);
+        }
         look_up(tile + 1);
     };
     look_up(0);
@@ -107,22 +114,17 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
     cp_async_wait<0>();
     __syncthreads();
     // ---- this warp's quarter of the queries, in registers
-    const int kq = warp & 3, kg = warp >> 2, per = (ksteps + 3) / 4;
+    const int kq = warp, per = (ksteps + 3) / 4;
     const int k0 = kq * per, kn = max(0, min(per, ksteps - k0));
-    uint32_t qf[MT][KQ][4];
+    uint32_t qf[KQ][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int i = 0; i < KQ; ++i) {
+        const int ks = min(k0 + min(i, max(kn - 1, 0)), ksteps - 1);     // (steps past the end are not used)
+        ldsm_x4(smem_u32(sQ + ((lane & 7) + 8 * ((lane >> 3) & 1)) * pitch + ks * 32 + (lane >> 4) * 16), qf[i][0], qf[i][1], qf[i][2], qf[i][3]);
+    }
+    float o[VT * 2][4];
 #pragma unroll
-        for (int i = 0; i < KQ; ++i) {
-            const int ks = k0 + min(i, max(kn - 1, 0));                  // (steps past the end are not used)
-            ldsm_x4(smem_u32(sQ + (m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * pitch + ks * 32 + (lane >> 4) * 16), qf[m][i][0], qf[m][i][1], qf[m][i][2],
-                    qf[m][i][3]);
-        }
-    float o[MT][VT * 2][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int i = 0; i < VT * 2; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
+    for (int i = 0; i < VT * 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const int srow = tid / TPR, sc = tid % TPR;                          // softmax: this thread's row and place in it
     float m_run = -CUDART_INF_F, l_run = 0.f;
     const int gm = lane >> 3;
@@ -133,103 +135,76 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
         if (tile + 1 < ntiles) load(tile + 1, st ^ 1);
         ok = mbar_wait(&full[st], (tile >> 1) & 1, abort_flag, a.status);
         const uint8_t* kS = sK + st * stage;
-        // ---- partial scores: 32 keys of half kg over the columns of quarter kq
-        float s[MT][4][4];
+        // ---- partial scores of the tile over the columns of this warp's quarter
+        float s[4][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int n = 0; n < 4; ++n) s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f;
+        for (int n = 0; n < 4; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
 #pragma unroll
         for (int i = 0; i < KQ; ++i) {
             if (i < kn) {
                 uint32_t kf[8];
 #pragma unroll
                 for (int g = 0; g < 2; ++g)
-                    ldsm_x4(smem_u32(kS + (kg * 32 + g * 16 + (gm >> 1) * 8 + (lane & 7)) * pitch + (k0 + i) * 32 + (gm & 1) * 16), kf[g * 4], kf[g * 4 + 1],
-                            kf[g * 4 + 2], kf[g * 4 + 3]);
+                    ldsm_x4(smem_u32(kS + (g * 16 + (gm >> 1) * 8 + (lane & 7)) * pitch + (k0 + i) * 32 + (gm & 1) * 16), kf[g * 4], kf[g * 4 + 1], kf[g * 4 + 2],
+                            kf[g * 4 + 3]);
 #pragma unroll
-                for (int m = 0; m < MT; ++m)
-#pragma unroll
-                    for (int n = 0; n < 4; ++n) mma16816<false>(s[m][n], qf[m][i], kf[n * 2], kf[n * 2 + 1]);
+                for (int n = 0; n < 4; ++n) mma16816<false>(s[n], qf[i], kf[n * 2], kf[n * 2 + 1]);
             }
         }
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+        for (int n = 0; n < 4; ++n)
 #pragma unroll
-            for (int n = 0; n < 4; ++n)
-#pragma unroll
-                for (int ri = 0; ri < 2; ++ri)
-                    *reinterpret_cast<float2*>(sS + (kq * R + m * 16 + ri * 8 + (lane >> 2)) * kScorePitch + kg * 32 + n * 8 + (lane & 3) * 2) =
-                        make_float2(s[m][n][ri * 2], s[m][n][ri * 2 + 1]);
+            for (int ri = 0; ri < 2; ++ri)
+                *reinterpret_cast<float2*>(sS + (kq * R + ri * 8 + (lane >> 2)) * kScorePitch + n * 8 + (lane & 3) * 2) = make_float2(s[n][ri * 2], s[n][ri * 2 + 1]);
         __syncthreads();
         // ---- softmax of a row by TPR neighbouring threads
-        float v[NQ][4];
+        const int key = sc * 4, j = k_lo + tile * kKeys + key;
+        float4 x = *reinterpret_cast<const float4*>(sS + srow * kScorePitch + key);
+#pragma unroll
+        for (int q = 1; q < 4; ++q) {
+            const float4 y = *reinterpret_cast<const float4*>(sS + (q * R + srow) * kScorePitch + key);
+            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+        }
+        float v[4] = {x.x, x.y, x.z, x.w};
         float mx = m_run;
 #pragma unroll
-        for (int g = 0; g < NQ; ++g) {
-            const int key = (g * TPR + sc) * 4;
-            float4 x = *reinterpret_cast<const float4*>(sS + srow * kScorePitch + key);
-#pragma unroll
-            for (int q = 1; q < 4; ++q) {
-                const float4 y = *reinterpret_cast<const float4*>(sS + (q * R + srow) * kScorePitch + key);
-                x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
-            }
-            const float xs[4] = {x.x, x.y, x.z, x.w};
-            const int j = k_lo + tile * kKeys + key;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                v[g][e] = j + e >= lo && j + e < k_hi ? xs[e] * p.scale_log2 : -CUDART_INF_F;
-                mx = fmaxf(mx, v[g][e]);
-            }
+        for (int e = 0; e < 4; ++e) {
+            v[e] = j + e >= lo && j + e < k_hi ? v[e] * p.scale_log2 : -CUDART_INF_F;
+            mx = fmaxf(mx, v[e]);
         }
 #pragma unroll
         for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
         const float base = mx == -CUDART_INF_F ? 0.f : mx;
         const float corr = exp2f(m_run - base);
         m_run = mx;
-        l_run *= corr;
 #pragma unroll
-        for (int g = 0; g < NQ; ++g) {
-            float e[4];
-#pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                e[k] = exp2f(v[g][k] - base);
-                l_run += e[k];
-            }
-            const int key = (g * TPR + sc) * 4;
-            *reinterpret_cast<uint2*>(sP + p_off(srow, key / 8) + (key & 4) * 2) = make_uint2(pack_bf16x2(e[0], e[1]), pack_bf16x2(e[2], e[3]));
-        }
+        for (int e = 0; e < 4; ++e) v[e] = exp2f(v[e] - base);
+        l_run = l_run * corr + (v[0] + v[1]) + (v[2] + v[3]);
+        *reinterpret_cast<uint2*>(sP + p_off(srow, key / 8) + (key & 4) * 2) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
         if (sc == 0) sCorr[srow] = corr;
         __syncthreads();
         // ---- O += P V for this warp's value columns
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+        for (int ri = 0; ri < 2; ++ri) {
+            const float c = sCorr[ri * 8 + (lane >> 2)];
 #pragma unroll
-            for (int ri = 0; ri < 2; ++ri) {
-                const float c = sCorr[m * 16 + ri * 8 + (lane >> 2)];
-#pragma unroll
-                for (int i = 0; i < VT * 2; ++i) {
-                    o[m][i][ri * 2] *= c;
-                    o[m][i][ri * 2 + 1] *= c;
-                }
+            for (int i = 0; i < VT * 2; ++i) {
+                o[i][ri * 2] *= c;
+                o[i][ri * 2 + 1] *= c;
             }
+        }
 #pragma unroll
         for (int kk = 0; kk < kKeys / 16; ++kk) {
-            uint32_t pf[MT][4];
-#pragma unroll
-            for (int m = 0; m < MT; ++m)
-                ldsm_x4(smem_u32(sP + p_off(m * 16 + (lane & 7) + 8 * ((lane >> 3) & 1), kk * 2 + (lane >> 4))), pf[m][0], pf[m][1], pf[m][2], pf[m][3]);
+            uint32_t pf[4];
+            ldsm_x4(smem_u32(sP + p_off((lane & 7) + 8 * ((lane >> 3) & 1), kk * 2 + (lane >> 4))), pf[0], pf[1], pf[2], pf[3]);
 #pragma unroll
             for (int w = 0; w < VT; ++w) {
                 const int col = (warp * VT + w) * 16;
                 if (col < a.cpad) {
                     uint32_t b0, b1, b2, b3;
                     ldsm_x4_t(smem_u32(kS + (kk * 16 + (gm & 1) * 8 + (lane & 7)) * pitch + col * 2 + (gm >> 1) * 16), b0, b1, b2, b3);
-#pragma unroll
-                    for (int m = 0; m < MT; ++m) {
-                        mma16816<false>(o[m][2 * w], pf[m], b0, b1);
-                        mma16816<false>(o[m][2 * w + 1], pf[m], b2, b3);
-                    }
+                    mma16816<false>(o[2 * w], pf, b0, b1);
+                    mma16816<false>(o[2 * w + 1], pf, b2, b3);
                 }
             }
         }
@@ -248,38 +223,39 @@ __global__ void __launch_bounds__(kWarps * 32, 1) latent_attention_kernel(Latent
         return;
     }
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int ri = 0; ri < 2; ++ri) {
+        const int r = ri * 8 + (lane >> 2), h = h0 + r;
+        if (h >= p.Hq) continue;
+        const float l = sCorr[r], inv = l > 0.f ? 1.f / l : 0.f;
+        float* scr = p.scratch + (((size_t)t * p.Hq + h) * p.nsplit + split) * (a.cpad + 2);
 #pragma unroll
-        for (int ri = 0; ri < 2; ++ri) {
-            const int r = m * 16 + ri * 8 + (lane >> 2), h = h0 + r;
-            if (h >= p.Hq) continue;
-            const float l = sCorr[r], inv = l > 0.f ? 1.f / l : 0.f;
-            float* scr = p.scratch + (((size_t)t * p.Hq + h) * p.nsplit + split) * (a.cpad + 2);
-#pragma unroll
-            for (int i = 0; i < VT * 2; ++i) {
-                const int col = warp * VT * 16 + i * 8 + (lane & 3) * 2;
-                if (col < a.cpad) {
-                    if (p.nsplit > 1)
-                        *reinterpret_cast<float2*>(scr + col) = make_float2(o[m][i][ri * 2], o[m][i][ri * 2 + 1]);
-                    else
-                        *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.o_head + col) =
-                            pack_bf16x2(o[m][i][ri * 2] * inv, o[m][i][ri * 2 + 1] * inv);
-                }
-            }
-            if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
-                scr[a.cpad] = sMax[r];
-                scr[a.cpad + 1] = l;
+        for (int i = 0; i < VT * 2; ++i) {
+            const int col = warp * VT * 16 + i * 8 + (lane & 3) * 2;
+            if (col < a.cpad) {
+                if (p.nsplit > 1)
+                    *reinterpret_cast<float2*>(scr + col) = make_float2(o[i][ri * 2], o[i][ri * 2 + 1]);
+                else
+                    *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.o_head + col) =
+                        pack_bf16x2(o[i][ri * 2] * inv, o[i][ri * 2 + 1] * inv);
             }
         }
+        if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
+            scr[a.cpad] = sMax[r];
+            scr[a.cpad + 1] = l;
+        }
+    }
 }
 
-template <int MT, int VT, int KQ>
+int latent_smem(int k_row) {
+    const int pitch = k_row * 2, partials = 4 * kHeads * kScorePitch * 4;
+    return 2 * kKeys * pitch + (kHeads * pitch > partials ? kHeads * pitch : partials) + kHeads * kKeys * 2 + 2 * kHeads * 4 + 64 + 128;
+}
+
+template <int VT, int KQ>
 int launch_latent(const LatentKParams& a, cudaStream_t stream) {
-    constexpr int R = MT * 16;
-    const int pitch = a.row * 2 + 16, shared_part = R * pitch > 4 * R * kScorePitch * 4 ? R * pitch : 4 * R * kScorePitch * 4;
-    const int smem = 2 * kKeys * pitch + shared_part + R * kKeys * 2 + 2 * R * 4 + 64 + 128;
+    const int smem = latent_smem(a.p.k_row);
     if (smem > 227 * 1024 || a.row / 16 > 4 * KQ) return ERR_UNSUPPORTED;
-    auto kern = latent_attention_kernel<MT, VT, KQ>;
+    auto kern = latent_attention_kernel<VT, KQ>;
     static std::atomic<uint64_t> configured{0};   // one bit per device; raised to the whole limit once
     int dev = 0;
     OVB_CHECK_CUDA(cudaGetDevice(&dev));
@@ -288,7 +264,7 @@ int launch_latent(const LatentKParams& a, cudaStream_t stream) {
         OVB_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         configured.fetch_or(bit, std::memory_order_release);
     }
-    OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.p.T, ceil_div(a.p.Hq, R), a.p.nsplit), dim3(kWarps * 32), (size_t)smem, stream, a));
+    OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.p.T, ceil_div(a.p.Hq, kHeads), a.p.nsplit), dim3(kWarps * 32), (size_t)smem, stream, a));
     return a.p.nsplit > 1 ? launch_decode_combine(a.p, a.cpad, stream) : 0;
 }
 
@@ -337,7 +313,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __res
 }  // namespace
 
 int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int max_ctx, long long scratch_bytes, cudaStream_t stream) {
-    if (row % 16 || cpad > 512 || (p.block_size & (p.block_size - 1)) || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
+    if (row % 16 || cpad > 512 || (p.block_size & (p.block_size - 1)) || p.k_row < row || p.k_row % 8 || p.ldq % 8 || p.q_head % 8 || p.ldo % 2 || p.o_head % 2 ||
         (reinterpret_cast<uintptr_t>(p.q) & 15) || (reinterpret_cast<uintptr_t>(p.k_cache) & 15) || (reinterpret_cast<uintptr_t>(p.out) & 3) || p.T > (1 << 30))
         return ERR_UNSUPPORTED;
     LatentKParams a;
@@ -348,16 +324,16 @@ int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int m
     while ((1 << a.block_shift) < p.block_size) ++a.block_shift;
     a.status = status_word();
     a.p.dv_store = cpad;
-    const int mt = p.Hq <= 16 ? 1 : 2;
     const int keys = p.sliding_window > 0 && p.sliding_window + kKeys - 1 < max_ctx ? p.sliding_window + kKeys - 1 : max_ctx;
-    const int tiles = ceil_div(keys, kKeys), ctas = p.T * ceil_div(p.Hq, mt * 16);
+    const int tiles = ceil_div(keys, kKeys), ctas = p.T * ceil_div(p.Hq, kHeads);
+    const int slots = 148 * (latent_smem(p.k_row) * 4 <= 220 * 1024 ? 4 : latent_smem(p.k_row) * 3 <= 222 * 1024 ? 3 : 2);   // CTAs that run at a time
     int best = 1;
     if (max_q_len == 1 && p.T == p.B && p.scratch != nullptr) {
-        // shares of the keys: whole waves of one CTA per SM, a fixed cost of about two key tiles per CTA and one for the merge
+        // shares of the keys: whole waves, a fixed cost of about five key tiles per CTA and a few more for the merge
         double best_cost = 1e30;
         for (int n = 1; n <= 32 && n <= tiles; ++n) {
-            if ((long long)ctas * 16 * mt * n * (cpad + 2) * 4 > scratch_bytes) break;
-            const double cost = ceil_div(ctas * n, 148) * (ceil_div(tiles, n) + 2.0) + (n > 1 ? 1.0 : 0.0);
+            if ((long long)p.T * p.Hq * n * (cpad + 2) * 4 > scratch_bytes) break;
+            const double cost = ceil_div(ctas * n, slots) * (ceil_div(tiles, n) + 5.0) + (n > 1 ? 4.0 + 0.25 * n : 0.0);
             if (cost < best_cost) {
                 best_cost = cost;
                 best = n;
@@ -366,9 +342,7 @@ int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int m
     }
     a.p.nsplit = best;
     a.p.keys_per_split = ceil_div(tiles, best) * kKeys;
-    const int vt = cpad <= 128 ? 1 : cpad <= 256 ? 2 : 4;
-    if (mt == 1) return vt == 1 ? launch_latent<1, 1, 3>(a, stream) : vt == 2 ? launch_latent<1, 2, 5>(a, stream) : launch_latent<1, 4, 9>(a, stream);
-    return vt == 1 ? launch_latent<2, 1, 3>(a, stream) : vt == 2 ? launch_latent<2, 2, 5>(a, stream) : launch_latent<2, 4, 9>(a, stream);
+    return cpad <= 128 ? launch_latent<2, 3>(a, stream) : cpad <= 256 ? launch_latent<4, 5>(a, stream) : launch_latent<8, 9>(a, stream);
 }
 
 }  // namespace ovb

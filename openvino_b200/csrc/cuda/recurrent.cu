@@ -314,13 +314,13 @@ __device__ __forceinline__ float rec_sqrt(float z) {
     return r;
 }
 
-constexpr int LRU_L = 8;    // tokens per warp and round
+constexpr int LRU_PIECE = 8;    // tokens per warp and round of a prompt
 
 // One group of 32 channels (a lane each) of one sequence. The NW warps of the group take consecutive pieces of LRU_L tokens: each
 // composes the affine maps S -> a S + b of its piece, the pieces' maps are chained through shared memory, and the piece is then
 // replayed from its true starting state. NW = 1 (decode): a CTA holds four independent groups.
-template <class E, int NW>
-__global__ void __launch_bounds__(NW == 1 ? 128 : NW * 32) lru_scan_kernel(ovb_rglru_args p) {
+template <class E, int NW, int LRU_L>
+__global__ void __launch_bounds__(NW == 1 ? 128 : NW * 32, NW == 4 ? 7 : 1) lru_scan_kernel(ovb_rglru_args p) {
     pdl_enter();
     __shared__ float sA[2][NW][32], sB[2][NW][32];        // (two sets: one barrier per round)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -497,9 +497,11 @@ int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream) {
             OVB_CHECK_CUDA(launch_pdl(kern, dim3(ceil_div(a->N, channels), a->B), dim3(threads), 0, (cudaStream_t)stream, *a));
             return 0;
         };
-        if (a->max_q_len <= LRU_L) return go(lru_scan_kernel<E, 1>, 128, 128);
+        if (a->max_q_len == 1) return go(lru_scan_kernel<E, 1, 1>, 128, 128);
+        if (a->max_q_len <= LRU_PIECE) return go(lru_scan_kernel<E, 1, LRU_PIECE>, 128, 128);
         // many groups: small CTAs, several per SM; few groups: more warps on each sequence
-        return (long long)ceil_div(a->N, 32) * a->B >= 4 * 148 ? go(lru_scan_kernel<E, 4>, 32, 128) : go(lru_scan_kernel<E, 16>, 32, 512);
+        return (long long)ceil_div(a->N, 32) * a->B >= 4 * 148 ? go(lru_scan_kernel<E, 4, LRU_PIECE>, 32, 128)
+                                                              : go(lru_scan_kernel<E, 16, LRU_PIECE>, 32, 512);
     });
 }
 

@@ -127,6 +127,7 @@ class LatentAttentionMixer:
         H, D, R, C, Dv = s.heads, s.dim, s.rot_dim, s.kv_rank, s.vdim
         self.dp, self.rp, self.cp, self.dv = _up(D, 16), _up(R, 16), _up(C, 16), _up(Dv, 16)
         self.q_pitch, self.row = self.dp + self.rp, self.cp + self.rp
+        self.pitch = self.row + 8         # a cached row: an odd number of 16-byte pieces, so that pages copied to shared memory as they are read without bank conflicts
         q = pk.raw("mix", "q").reshape(H, D + R, -1)
         q = torch.cat([_pad_rows(q[:, :D].reshape(H * D, -1), H, self.dp).reshape(H, self.dp, -1),
                        _pad_rows(q[:, D:].reshape(H * R, -1), H, self.rp).reshape(H, self.rp, -1)], 1).reshape(H * self.q_pitch, -1)
@@ -152,7 +153,7 @@ class LatentAttentionMixer:
         return rows if rows <= 2 * sb.Tcap else 0
 
     def allocate(self, ex: "LayeredExecutor") -> None:
-        self.cache = torch.zeros((ex.num_kv_blocks, ex.block_size, self.row), dtype=ex.dtype, device=ex.device)
+        self.cache = torch.zeros((ex.num_kv_blocks, ex.block_size, self.pitch), dtype=ex.dtype, device=ex.device)
 
     def state(self) -> List[torch.Tensor]:
         return []
@@ -170,7 +171,7 @@ class LatentAttentionMixer:
             dict(q_rot=q[:, self.cp:], ld_qr=q.stride(0), qr_pitch=self.row)
         K.latent_prepare(proj=proj, cache=self.cache, c_norm=self.c_norm, positions=sb.view("positions"), slot_map=sb.view("slot_map"), T=T,
                          H=H, C=s.kv_rank, R=s.rot_dim, q_pitch=self.q_pitch, q_rot_off=self.dp, c_off=self.c_off, kr_off=self.kr_off, ldp=proj.stride(0),
-                         row_pitch=self.row, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **q_rot, **self.rot.args())
+                         row_pitch=self.pitch, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **q_rot, **self.rot.args())
         attn = sb.scratch("attn", T, self.o.K)
         if rows:
             self._attend_expanded(ex, sb, shp, rows, proj, attn)
@@ -185,11 +186,11 @@ class LatentAttentionMixer:
                      block_indices_begins=sb.view("block_indices_begins"), B=shp.B, window=s.window, block_size=ex.block_size)
         lat = sb.scratch("latent_rows", rows, self.ukv.K, cap=2 * sb.Tcap)
         kv = sb.scratch("latent_kv", rows, self.ukv.N, cap=2 * sb.Tcap)
-        K.latent_gather(cache=self.cache, out=lat, kv_rows=sb.kv_rows, rows=rows, cols=self.cp, row_pitch=self.row, out_pitch=lat.stride(0), **batch)
+        K.latent_gather(cache=self.cache, out=lat, kv_rows=sb.kv_rows, rows=rows, cols=self.cp, row_pitch=self.pitch, out_pitch=lat.stride(0), **batch)
         K.gemm(lat, self.ukv, out=kv, ws=ex.ws)
         K.latent_prefill(q=proj, kv=kv, cache=self.cache, out=attn, kv_rows=sb.kv_rows, T=shp.T, H=H, rows=rows, R=s.rot_dim, Dv=self.dv, ldq=proj.stride(0),
                          q_head=self.q_pitch, q_rot_off=self.dp, ld_kv=kv.stride(0), k_head=self.k_head, v_off=H * self.k_head, v_head=self.v_head,
-                         row_pitch=self.row, key_off=self.cp, ldo=attn.stride(0), o_head=self.dv, scale=s.scale, **batch)
+                         row_pitch=self.pitch, key_off=self.cp, ldo=attn.stride(0), o_head=self.dv, scale=s.scale, **batch)
         ex.kernel_launches += 3
 
     def _attend_absorbed(self, ex, sb, shp: StepShape, proj: torch.Tensor, q: torch.Tensor, attn: torch.Tensor) -> None:
@@ -197,7 +198,7 @@ class LatentAttentionMixer:
         K.gemm_block_diag(proj[:, :self.c_off], self.uk, q, self.q_pitch, self.row, ws=ex.ws)
         lat = sb.scratch("latent_o", T, H * self.cp)
         ex.attention(sb, shp, q=q, k=self.cache, v=self.cache, out=lat, Hq=H, Hkv=1, Dk=self.row, Dv=s.kv_rank, ldq=q.stride(0), q_head=self.row,
-                     k_row=self.row, v_row=self.row, ldo=lat.stride(0), o_head=self.cp, window=s.window, scale=s.scale)
+                     k_row=self.pitch, v_row=self.pitch, ldo=lat.stride(0), o_head=self.cp, window=s.window, scale=s.scale)
         K.gemm_block_diag(lat[:, :H * self.cp], self.uv, attn, self.cp, self.dv, ws=ex.ws)
         ex.kernel_launches += 3
 

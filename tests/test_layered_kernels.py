@@ -253,7 +253,8 @@ def test_latent_attention_forms(sizes, which):
             rows = [torch.cat([torch.nn.functional.pad(c, (0, cp - C)), r], -1)[:, None] for c, r in zip(lat, key)]
             ws = torch.empty(1 << 23, device="cuda")
             for dtype in DTYPES:
-                cache = pb.fill(rows, row, dtype)
+                pitch = row + 8
+                cache = pb.fill(rows, pitch, dtype)
                 qd = torch.zeros(pb.T, H, dp + rp)
                 qd[..., :D], qd[..., dp:dp + R] = new[..., :D], new[..., D:]
                 qd = qd.reshape(pb.T, -1).cuda().to(dtype)
@@ -261,7 +262,7 @@ def test_latent_attention_forms(sizes, which):
                 qa.view(pb.T, H, row)[..., cp:cp + R] = new[..., D:].cuda().to(dtype)
                 K.gemm_block_diag(qd, K.BlockDiagWeight(uk.transpose(1, 2).cuda().to(dtype)), qa, dp + rp, row)
                 lo = torch.zeros(pb.T, H * cp, dtype=dtype, device="cuda")
-                K.window_attention(q=qa, k=cache, v=cache, out=lo, Hq=H, Hkv=1, Dk=row, Dv=C, ldq=H * row, q_head=row, k_row=row, v_row=row, ldo=H * cp, o_head=cp,
+                K.window_attention(q=qa, k=cache, v=cache, out=lo, Hq=H, Hkv=1, Dk=row, Dv=C, ldq=H * row, q_head=row, k_row=pitch, v_row=pitch, ldo=H * cp, o_head=cp,
                                    window=window, scale=scale, max_context_len=pb.max_ctx, max_q_len=pb.max_q_len, dtype=K.storage_type(dtype), scratch=ws,
                                    scratch_bytes=ws.nbytes, exact=1 if dtype == torch.float32 else 0, **pb.args)
                 out = torch.zeros(pb.T, H * dv, dtype=dtype, device="cuda")
@@ -275,13 +276,13 @@ def test_latent_attention_forms(sizes, which):
             batch = dict(pb.args, window=window)
             T = batch.pop("T")
             g, begins = torch.zeros(n, up(C, 64), dtype=bf, device="cuda"), torch.zeros(pb.B + 1, dtype=torch.int32, device="cuda")
-            K.latent_gather(cache=cache, out=g, kv_rows=begins, rows=n, cols=cp, row_pitch=row, out_pitch=g.stride(0), **batch)
+            K.latent_gather(cache=cache, out=g, kv_rows=begins, rows=n, cols=cp, row_pitch=pitch, out_pitch=g.stride(0), **batch)
             assert torch.equal(g[:, :C].float().cpu(), torch.cat([c[f:] for c, f in zip(lat, first)]))
             wk, wv = torch.nn.functional.pad(uk, (0, g.shape[1] - C, 0, kh - D)), torch.nn.functional.pad(uv, (0, g.shape[1] - C, 0, vh - Dv))
             kv = K.gemm(g, K.PackedWeight.from_dense(torch.cat([wk.reshape(H * kh, -1), wv.reshape(H * vh, -1)]).to(bf).cuda()))
             out = torch.zeros(T, H * dv, dtype=bf, device="cuda")
             K.latent_prefill(q=qd, kv=kv, cache=cache, out=out, kv_rows=begins, T=T, H=H, rows=n, R=R, Dv=dv, ldq=qd.stride(0), q_head=dp + rp, q_rot_off=dp,
-                             ld_kv=kv.stride(0), k_head=kh, v_off=H * kh, v_head=vh, row_pitch=row, key_off=cp, ldo=H * dv, o_head=dv, scale=scale, **batch)
+                             ld_kv=kv.stride(0), k_head=kh, v_off=H * kh, v_head=vh, row_pitch=pitch, key_off=cp, ldo=H * dv, o_head=dv, scale=scale, **batch)
             close(out.reshape(T, H, dv)[..., :Dv], want, 2.5e-2)
     K.check_status("latent attention")
 
