@@ -556,23 +556,32 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
     }
 }
 
-// Split-KV partials [Hq, nsplit, dv + 2] of every sequence (sums, then maximum and denominator) -> output rows.
-__global__ void pa_decode_combine_kernel(PaKParams p, int dv) {
+// Split-KV partials [Hq, nsplit, dv + 2] of every sequence (sums, then maximum and denominator) -> output rows. nsplit <= 32.
+__global__ void __launch_bounds__(128) pa_decode_combine_kernel(PaKParams p, int dv) {
     pdl_enter_attn();
+    __shared__ float w[32];
     const int b = blockIdx.x, hq = blockIdx.y;
-    const int tok = p.subsequence_begins[b];
     const float* base = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit) * (dv + 2);
-    for (int d = threadIdx.x; d < p.dv_store; d += blockDim.x) {
-        float m = -CUDART_INF_F;
-        for (int s = 0; s < p.nsplit; ++s) m = fmaxf(m, base[(size_t)s * (dv + 2) + dv]);
-        float l = 0.f, o = 0.f;
-        for (int s = 0; s < p.nsplit; ++s) {
-            const float* src = base + (size_t)s * (dv + 2);
-            const float sc = (src[dv] == -CUDART_INF_F) ? 0.f : exp2f(src[dv] - m);
-            l += src[dv + 1] * sc;
-            o += src[d] * sc;
-        }
-        store_decoded(p, tok, hq, d, l > 0.f ? o / l : 0.f);
+    if (threadIdx.x < 32) {
+        const bool has = (int)threadIdx.x < p.nsplit;
+        const float* row = base + (size_t)(has ? threadIdx.x : 0) * (dv + 2) + dv;
+        const float m = has ? row[0] : -CUDART_INF_F;
+        float l = has ? row[1] : 0.f, mx = m;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float sc = m == -CUDART_INF_F ? 0.f : exp2f(m - mx);
+        l *= sc;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+        w[threadIdx.x] = l > 0.f ? sc / l : 0.f;
+    }
+    const int tok = p.subsequence_begins[b];
+    __syncthreads();
+    for (int d = threadIdx.x; d < p.dv_store; d += 128) {
+        float o = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < p.nsplit; ++s) o += w[s] * base[(size_t)s * (dv + 2) + d];
+        store_decoded(p, tok, hq, d, o);
     }
 }
 

@@ -27,11 +27,7 @@ __global__ void __launch_bounds__(kThreads) attention_exact_kernel(ovb_wattn_arg
     __shared__ float sp[kThreads], red[kThreads / 32];
     __shared__ int s_b;
     const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
-    if (tid == 0) {
-        int b = 0;
-        while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
-        s_b = b;
-    }
+    find_sequence(p.subsequence_begins, p.B, t, &s_b);
     const E* q = reinterpret_cast<const E*>(p.q) + (size_t)t * p.ldq + (size_t)h * p.q_head;
     for (int i = tid; i < p.Dk; i += kThreads) sq[i] = ld_f32(q + i) * p.scale;
     __syncthreads();

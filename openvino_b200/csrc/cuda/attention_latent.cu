@@ -1,13 +1,15 @@
 // Latent attention in its absorbed form, and the expansion of cached rows for prefill.
 //
 // latent_attention_kernel: every query head attends to the same cached row per token; the first part of that row is also the value.
-// One CTA of four warps serves one token (decode: one sequence), 16 of its heads and one share of the visible keys; two CTAs or
-// more share an SM and hide each other's barriers. Key tiles of 32 rows pass through two shared-memory stages, one bulk copy per
-// page, and are read for both products:
+// One CTA of four warps serves one token (decode: one sequence), 16 of its heads and one share of the visible keys; several CTAs
+// share an SM and hide each other's barriers. Key tiles of 16 rows pass through three shared-memory stages, one bulk copy per page,
+// and are read for both products:
 //   scores   the warps split the row's columns in quarters; the queries' fragments of a warp's quarter stay in registers for the
 //            whole loop. The four partial sums meet in shared memory.
-//   softmax  8 neighbouring threads per head add the partials, mask, keep running maximum and sum; P as bf16.
+//   softmax  8 neighbouring threads per head add the partials, mask, keep running maximum and sum; P as bf16. The maximum is only
+//            raised when a tile exceeds it by more than a factor of 2^8, so the accumulators are rarely rescaled.
 //   sums     every warp owns its own slice of the value columns for all keys of the tile, so the accumulator needs no merge.
+// The products of a step are the scores of tile t + 1 and the sums of tile t: independent, between the same two barriers.
 // Pages keep the cache's row pitch in shared memory: a pitch of an odd number of 16-byte pieces spreads ldmatrix over all banks.
 // With split keys the partial sums go to scratch and the decode kernels' merge finishes.
 //
@@ -28,9 +30,9 @@ OVB_DEBUG_LIMITS_DEFINE
 
 namespace {
 
-constexpr int kWarps = 4, kKeys = 32, kHeads = 16;
-
+constexpr int kWarps = 4, kKeys = 16, kHeads = 16, kStages = 3;
 constexpr int kScorePitch = kKeys + 8;    // floats per row of partial scores
+constexpr int kPPitch = 48;               // bytes per row of P
 
 struct LatentKParams {
     PaKParams p;
@@ -39,43 +41,38 @@ struct LatentKParams {
     int* status;
 };
 
-// Rows of 64 bytes: two rows share the 128 bytes of all banks.
-__device__ __forceinline__ uint32_t p_off(int r, int chunk) { return uint32_t(r * kKeys * 2 + ((chunk ^ ((r >> 1) & 3)) << 4)); }
+// A thread's reads of a stage are done before a bulk copy that is issued after the next barrier may write it. (ldmatrix results that
+// are only needed later may otherwise still be outstanding: seen as wrong queries when they shared the first stage to be refilled.)
+__device__ __forceinline__ void fence_reads_before_copies() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
-// VT: 16-column pieces of the value per warp; KQ: most 16-column steps in a quarter of the row.
-template <int VT, int KQ>
-__global__ void __launch_bounds__(kWarps * 32, 2) latent_attention_kernel(LatentKParams a) {
-    constexpr int R = kHeads, TPR = kWarps * 32 / R;    // rows, threads per row (four keys each)
-    static_assert(TPR * 4 == kKeys, "softmax threads cover the tile");
+// VT: 16-column pieces of the value per warp; KQ: most 16-column steps in a quarter of the row; FULL: row and value fill them exactly.
+template <int VT, int KQ, bool FULL>
+__global__ void __launch_bounds__(kWarps * 32, 3) latent_attention_kernel(LatentKParams a) {
+    constexpr int R = kHeads, TPR = kWarps * 32 / R;                     // rows, threads per row (two keys each)
+    static_assert(TPR * 2 == kKeys, "softmax threads cover the tile");
     const PaKParams& p = a.p;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
     const int pitch = p.k_row * 2, ksteps = a.row / 16;
     const int stage = kKeys * pitch;
-    const int shared_part = max(R * pitch, 4 * R * kScorePitch * 4);
-    uint8_t* sK = smem;                                                  // two stages
-    uint8_t* sQ = sK + 2 * stage;                                        // queries, then partial scores [4][R][kScorePitch]
-    float* sS = reinterpret_cast<float*>(sQ);
-    uint8_t* sP = sQ + shared_part;                                      // [R][32] bf16
-    float* sCorr = reinterpret_cast<float*>(sP + R * kKeys * 2);         // [R]
+    uint8_t* sK = smem;
+    uint8_t* sQ = sK + 2 * stage;                                        // queries pass through the last stage
+    float* sS = reinterpret_cast<float*>(sK + kStages * stage);          // partial scores [4][R][kScorePitch]
+    uint8_t* sP = reinterpret_cast<uint8_t*>(sS + 4 * R * kScorePitch);
+    float* sCorr = reinterpret_cast<float*>(sP + R * kPPitch);           // [R]
     float* sMax = sCorr + R;                                             // [R]
-    uint64_t* full = reinterpret_cast<uint64_t*>(sMax + R);              // [2]
-    volatile int* abort_flag = reinterpret_cast<volatile int*>(full + 2);
+    uint64_t* full = reinterpret_cast<uint64_t*>(sMax + R);              // [kStages]
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(full + kStages);
     int* s_b = const_cast<int*>(abort_flag) + 1;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int t = blockIdx.x, h0 = blockIdx.y * R, split = blockIdx.z;
     if (tid == 0) {
-        mbar_init(&full[0], 1);
-        mbar_init(&full[1], 1);
+        for (int i = 0; i < kStages; ++i) mbar_init(&full[i], 1);
         mbar_fence_init();
         *abort_flag = 0;
     }
     pdl_enter_attn();
-    if (tid == 0) {
-        int b = 0;
-        while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
-        *s_b = b;
-    }
+    find_sequence(p.subsequence_begins, p.B, t, s_b);
     for (int r = warp; r < R; r += kWarps) {
         const bool valid = h0 + r < p.Hq;
         const uint8_t* src = reinterpret_cast<const uint8_t*>(p.q) + ((size_t)t * p.ldq + (size_t)(valid ? h0 + r : 0) * p.q_head) * 2;
@@ -90,36 +87,37 @@ __global__ void __launch_bounds__(kWarps * 32, 2) latent_attention_kernel(Latent
     const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int ntiles = k_hi > k_lo ? (k_hi - k_lo + kKeys - 1) / kKeys : 0;
     const int* blocks = p.block_indices + p.block_indices_begins[b];
-    // One lane of warp 0 copies each page (or the tile's part of it); its place is looked up a tile ahead. Pages past the last key
-    // repeat the last one, and rows of a page past it hold what the cache holds there: finite, and masked.
+    // One lane of warp 0 copies each page (or the tile's part of it); its place is looked up a tile ahead. Rows of a page past the
+    // last key hold what the cache holds there: finite, and masked.
     const int seg = min(p.block_size, kKeys), nseg = kKeys / seg;
     const uint8_t* next_part = nullptr;
     auto look_up = [&](int tile) {
         if (warp == 0 && lane < nseg && tile < ntiles) {
             int j = k_lo + tile * kKeys + lane * seg;
-            if (j >= k_hi) j = (k_hi - 1) / seg * seg;
+            if (j >= k_hi) j = (k_hi - 1) / seg * seg;                   // (pages shorter than a tile: the last one again)
             const int blk = OVB_DBG_BLOCK(blocks[j >> a.block_shift]);
             next_part = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)blk << a.block_shift) + (j & (p.block_size - 1))) * pitch;
         }
     };
-    auto load = [&](int tile, int st) {
-        if (warp == 0) {
+    auto load = [&](int tile) {
+        if (warp == 0 && tile < ntiles) {
+            const int st = tile % kStages;
             if (lane == 0) mbar_arrive_expect_tx(&full[st], stage);
             if (lane < nseg) bulk_load_1d(sK + st * stage + lane * seg * pitch, next_part, seg * pitch, &full[st]);
         }
         look_up(tile + 1);
     };
     look_up(0);
-    if (ntiles > 0) load(0, 0);
+    load(0);
+    load(1);
     cp_async_wait<0>();
     __syncthreads();
     // ---- this warp's quarter of the queries, in registers
-    const int kq = warp, per = (ksteps + 3) / 4;
-    const int k0 = kq * per, kn = max(0, min(per, ksteps - k0));
+    const int per = FULL ? KQ : (ksteps + 3) / 4, k0 = warp * per, kn = FULL ? KQ : max(0, min(per, ksteps - k0));
     uint32_t qf[KQ][4];
 #pragma unroll
     for (int i = 0; i < KQ; ++i) {
-        const int ks = min(k0 + min(i, max(kn - 1, 0)), ksteps - 1);     // (steps past the end are not used)
+        const int ks = FULL ? k0 + i : min(k0 + min(i, max(kn - 1, 0)), ksteps - 1);     // (steps past the end are not used)
         ldsm_x4(smem_u32(sQ + ((lane & 7) + 8 * ((lane >> 3) & 1)) * pitch + ks * 32 + (lane >> 4) * 16), qf[i][0], qf[i][1], qf[i][2], qf[i][3]);
     }
     float o[VT * 2][4];
@@ -127,87 +125,105 @@ __global__ void __launch_bounds__(kWarps * 32, 2) latent_attention_kernel(Latent
     for (int i = 0; i < VT * 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const int srow = tid / TPR, sc = tid % TPR;                          // softmax: this thread's row and place in it
     float m_run = -CUDART_INF_F, l_run = 0.f;
-    const int gm = lane >> 3;
     bool ok = true;
-    for (int tile = 0; tile < ntiles; ++tile) {
-        const int st = tile & 1;
-        __syncthreads();                                                 // the other stage, the partials and P are free
-        if (tile + 1 < ntiles) load(tile + 1, st ^ 1);
-        ok = mbar_wait(&full[st], (tile >> 1) & 1, abort_flag, a.status);
-        const uint8_t* kS = sK + st * stage;
-        // ---- partial scores of the tile over the columns of this warp's quarter
-        float s[4][4];
+    fence_reads_before_copies();
+    __syncthreads();                                                     // the queries are out of the last stage
+    load(2);
+    const int gm = lane >> 3;
+    const uint32_t k_off = ((gm >> 1) * 8 + (lane & 7)) * pitch + k0 * 32 + (gm & 1) * 16;               // score operand of step 0
+    const uint32_t v_off = ((gm & 1) * 8 + (lane & 7)) * pitch + warp * (VT * 32) + (gm >> 1) * 16;      // value operand of piece 0
+    for (int tile = -1; tile < ntiles; ++tile) {
+        // ---- products: scores of tile + 1, sums of tile
+        const bool more = tile + 1 < ntiles;
+        if (more) ok = mbar_wait(&full[(tile + 1) % kStages], ((tile + 1) / kStages) & 1, abort_flag, a.status);
+        const uint32_t kS = smem_u32(sK + (more ? (tile + 1) % kStages : 0) * stage) + k_off;
+        const uint32_t vS = smem_u32(sK + (tile < 0 ? 0 : tile % kStages) * stage) + v_off;
+        uint32_t pf[4];
+        if (tile >= 0) {
+            const float c0 = sCorr[lane >> 2], c1 = sCorr[8 + (lane >> 2)];
+            ldsm_x4(smem_u32(sP + ((lane & 7) + 8 * ((lane >> 3) & 1)) * kPPitch + (lane >> 4) * 16), pf[0], pf[1], pf[2], pf[3]);
+            if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-        for (int n = 0; n < 4; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-#pragma unroll
-        for (int i = 0; i < KQ; ++i) {
-            if (i < kn) {
-                uint32_t kf[8];
-#pragma unroll
-                for (int g = 0; g < 2; ++g)
-                    ldsm_x4(smem_u32(kS + (g * 16 + (gm >> 1) * 8 + (lane & 7)) * pitch + (k0 + i) * 32 + (gm & 1) * 16), kf[g * 4], kf[g * 4 + 1], kf[g * 4 + 2],
-                            kf[g * 4 + 3]);
-#pragma unroll
-                for (int n = 0; n < 4; ++n) mma16816<false>(s[n], qf[i], kf[n * 2], kf[n * 2 + 1]);
-            }
-        }
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-            for (int ri = 0; ri < 2; ++ri)
-                *reinterpret_cast<float2*>(sS + (kq * R + ri * 8 + (lane >> 2)) * kScorePitch + n * 8 + (lane & 3) * 2) = make_float2(s[n][ri * 2], s[n][ri * 2 + 1]);
-        __syncthreads();
-        // ---- softmax of a row by TPR neighbouring threads
-        const int key = sc * 4, j = k_lo + tile * kKeys + key;
-        float4 x = *reinterpret_cast<const float4*>(sS + srow * kScorePitch + key);
-#pragma unroll
-        for (int q = 1; q < 4; ++q) {
-            const float4 y = *reinterpret_cast<const float4*>(sS + (q * R + srow) * kScorePitch + key);
-            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
-        }
-        float v[4] = {x.x, x.y, x.z, x.w};
-        float mx = m_run;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            v[e] = j + e >= lo && j + e < k_hi ? v[e] * p.scale_log2 : -CUDART_INF_F;
-            mx = fmaxf(mx, v[e]);
-        }
-#pragma unroll
-        for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-        const float base = mx == -CUDART_INF_F ? 0.f : mx;
-        const float corr = exp2f(m_run - base);
-        m_run = mx;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) v[e] = exp2f(v[e] - base);
-        l_run = l_run * corr + (v[0] + v[1]) + (v[2] + v[3]);
-        *reinterpret_cast<uint2*>(sP + p_off(srow, key / 8) + (key & 4) * 2) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-        if (sc == 0) sCorr[srow] = corr;
-        __syncthreads();
-        // ---- O += P V for this warp's value columns
-#pragma unroll
-        for (int ri = 0; ri < 2; ++ri) {
-            const float c = sCorr[ri * 8 + (lane >> 2)];
-#pragma unroll
-            for (int i = 0; i < VT * 2; ++i) {
-                o[i][ri * 2] *= c;
-                o[i][ri * 2 + 1] *= c;
-            }
-        }
-#pragma unroll
-        for (int kk = 0; kk < kKeys / 16; ++kk) {
-            uint32_t pf[4];
-            ldsm_x4(smem_u32(sP + p_off((lane & 7) + 8 * ((lane >> 3) & 1), kk * 2 + (lane >> 4))), pf[0], pf[1], pf[2], pf[3]);
-#pragma unroll
-            for (int w = 0; w < VT; ++w) {
-                const int col = (warp * VT + w) * 16;
-                if (col < a.cpad) {
-                    uint32_t b0, b1, b2, b3;
-                    ldsm_x4_t(smem_u32(kS + (kk * 16 + (gm & 1) * 8 + (lane & 7)) * pitch + col * 2 + (gm >> 1) * 16), b0, b1, b2, b3);
-                    mma16816<false>(o[2 * w], pf, b0, b1);
-                    mma16816<false>(o[2 * w + 1], pf, b2, b3);
+                for (int i = 0; i < VT * 2; ++i) {
+                    o[i][0] *= c0; o[i][1] *= c0;
+                    o[i][2] *= c1; o[i][3] *= c1;
                 }
             }
         }
+        float s[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        if (FULL && more && tile >= 0) {
+#pragma unroll
+            for (int i = 0; i < (KQ > VT ? KQ : VT); ++i) {
+                uint32_t f[4], g[4];
+                if (i < KQ) ldsm_x4(kS + i * 32, f[0], f[1], f[2], f[3]);
+                if (i < VT) ldsm_x4_t(vS + i * 32, g[0], g[1], g[2], g[3]);
+                if (i < KQ) {
+                    mma16816<false>(s[0], qf[i], f[0], f[1]);
+                    mma16816<false>(s[1], qf[i], f[2], f[3]);
+                }
+                if (i < VT) {
+                    mma16816<false>(o[2 * i], pf, g[0], g[1]);
+                    mma16816<false>(o[2 * i + 1], pf, g[2], g[3]);
+                }
+            }
+        } else {
+            if (more) {
+#pragma unroll
+                for (int i = 0; i < KQ; ++i)
+                    if (i < kn) {
+                        uint32_t f[4];
+                        ldsm_x4(kS + i * 32, f[0], f[1], f[2], f[3]);
+                        mma16816<false>(s[0], qf[i], f[0], f[1]);
+                        mma16816<false>(s[1], qf[i], f[2], f[3]);
+                    }
+            }
+            if (tile >= 0) {
+#pragma unroll
+                for (int w = 0; w < VT; ++w)
+                    if ((warp * VT + w) * 16 < a.cpad) {
+                        uint32_t g[4];
+                        ldsm_x4_t(vS + w * 32, g[0], g[1], g[2], g[3]);
+                        mma16816<false>(o[2 * w], pf, g[0], g[1]);
+                        mma16816<false>(o[2 * w + 1], pf, g[2], g[3]);
+                    }
+            }
+        }
+        if (!more) break;
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int ri = 0; ri < 2; ++ri)
+                *reinterpret_cast<float2*>(sS + (warp * R + ri * 8 + (lane >> 2)) * kScorePitch + n * 8 + (lane & 3) * 2) = make_float2(s[n][ri * 2], s[n][ri * 2 + 1]);
+        fence_reads_before_copies();
+        __syncthreads();                                                 // partials written; the stage of `tile` is free
+        if (tile >= 0) load(tile + kStages);
+        // ---- softmax of tile + 1, a row by TPR neighbouring threads
+        const int key = sc * 2, j = k_lo + (tile + 1) * kKeys + key;
+        float2 x = *reinterpret_cast<const float2*>(sS + srow * kScorePitch + key);
+#pragma unroll
+        for (int q = 1; q < 4; ++q) {
+            const float2 y = *reinterpret_cast<const float2*>(sS + (q * R + srow) * kScorePitch + key);
+            x.x += y.x; x.y += y.y;
+        }
+        x.x = j >= lo && j < k_hi ? x.x * p.scale_log2 : -CUDART_INF_F;
+        x.y = j + 1 >= lo && j + 1 < k_hi ? x.y * p.scale_log2 : -CUDART_INF_F;
+        float mx = fmaxf(x.x, x.y);
+#pragma unroll
+        for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+        float corr = 1.f;
+        if (mx > m_run + 8.f) {                                          // (the same for the whole row)
+            corr = exp2f(m_run - mx);
+            m_run = mx;
+        }
+        const float base = m_run == -CUDART_INF_F ? 0.f : m_run;
+        x.x = exp2f(x.x - base);
+        x.y = exp2f(x.y - base);
+        l_run = l_run * corr + x.x + x.y;
+        *reinterpret_cast<uint32_t*>(sP + srow * kPPitch + key * 2) = pack_bf16x2(x.x, x.y);
+        if (sc == 0) sCorr[srow] = corr;
+        __syncthreads();
     }
     // ---- denominators
 #pragma unroll
@@ -246,16 +262,13 @@ __global__ void __launch_bounds__(kWarps * 32, 2) latent_attention_kernel(Latent
     }
 }
 
-int latent_smem(int k_row) {
-    const int pitch = k_row * 2, partials = 4 * kHeads * kScorePitch * 4;
-    return 2 * kKeys * pitch + (kHeads * pitch > partials ? kHeads * pitch : partials) + kHeads * kKeys * 2 + 2 * kHeads * 4 + 64 + 128;
-}
+int latent_smem(int k_row) { return kStages * kKeys * k_row * 2 + 4 * kHeads * kScorePitch * 4 + kHeads * kPPitch + 2 * kHeads * 4 + 64 + 128; }
 
-template <int VT, int KQ>
+template <int VT, int KQ, bool FULL>
 int launch_latent(const LatentKParams& a, cudaStream_t stream) {
     const int smem = latent_smem(a.p.k_row);
     if (smem > 227 * 1024 || a.row / 16 > 4 * KQ) return ERR_UNSUPPORTED;
-    auto kern = latent_attention_kernel<VT, KQ>;
+    auto kern = latent_attention_kernel<VT, KQ, FULL>;
     static std::atomic<uint64_t> configured{0};   // one bit per device; raised to the whole limit once
     int dev = 0;
     OVB_CHECK_CUDA(cudaGetDevice(&dev));
@@ -266,6 +279,11 @@ int launch_latent(const LatentKParams& a, cudaStream_t stream) {
     }
     OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.p.T, ceil_div(a.p.Hq, kHeads), a.p.nsplit), dim3(kWarps * 32), (size_t)smem, stream, a));
     return a.p.nsplit > 1 ? launch_decode_combine(a.p, a.cpad, stream) : 0;
+}
+
+template <int VT, int KQ>
+int launch_latent_sizes(const LatentKParams& a, cudaStream_t stream) {
+    return a.row == 64 * KQ && a.cpad == 64 * VT ? launch_latent<VT, KQ, true>(a, stream) : launch_latent<VT, KQ, false>(a, stream);
 }
 
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __restrict__ cache, uint8_t* __restrict__ out, int* __restrict__ kv_rows,
@@ -326,14 +344,14 @@ int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int m
     a.p.dv_store = cpad;
     const int keys = p.sliding_window > 0 && p.sliding_window + kKeys - 1 < max_ctx ? p.sliding_window + kKeys - 1 : max_ctx;
     const int tiles = ceil_div(keys, kKeys), ctas = p.T * ceil_div(p.Hq, kHeads);
-    const int slots = 148 * (latent_smem(p.k_row) * 4 <= 220 * 1024 ? 4 : latent_smem(p.k_row) * 3 <= 222 * 1024 ? 3 : 2);   // CTAs that run at a time
+    const int slots = 148 * 3;   // CTAs that run at a time (registers)
     int best = 1;
     if (max_q_len == 1 && p.T == p.B && p.scratch != nullptr) {
-        // shares of the keys: whole waves, a fixed cost of about five key tiles per CTA and a few more for the merge
+        // shares of the keys: whole waves, a fixed cost of about ten key tiles per CTA and a few more for the merge
         double best_cost = 1e30;
         for (int n = 1; n <= 32 && n <= tiles; ++n) {
             if ((long long)p.T * p.Hq * n * (cpad + 2) * 4 > scratch_bytes) break;
-            const double cost = ceil_div(ctas * n, slots) * (ceil_div(tiles, n) + 5.0) + (n > 1 ? 4.0 + 0.25 * n : 0.0);
+            const double cost = ceil_div(ctas * n, slots) * (ceil_div(tiles, n) + 10.0) + (n > 1 ? 8.0 + 0.5 * n : 0.0);
             if (cost < best_cost) {
                 best_cost = cost;
                 best = n;
@@ -342,7 +360,7 @@ int launch_latent_attention(PaKParams p, int row, int cpad, int max_q_len, int m
     }
     a.p.nsplit = best;
     a.p.keys_per_split = ceil_div(tiles, best) * kKeys;
-    return cpad <= 128 ? launch_latent<2, 3>(a, stream) : cpad <= 256 ? launch_latent<4, 5>(a, stream) : launch_latent<8, 9>(a, stream);
+    return cpad <= 128 ? launch_latent_sizes<2, 3>(a, stream) : cpad <= 256 ? launch_latent_sizes<4, 5>(a, stream) : launch_latent_sizes<8, 9>(a, stream);
 }
 
 }  // namespace ovb

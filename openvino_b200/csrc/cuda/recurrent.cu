@@ -253,11 +253,14 @@ constexpr int CONV_STRIP = 8;    // tokens per thread of a prompt
 template <class E, int V, int TAPS>
 __global__ void __launch_bounds__(128) causal_conv_kernel(ovb_rglru_args p, int strip) {
     pdl_enter();
+    __shared__ int s_b;
     const int c = (blockIdx.y * 128 + threadIdx.x) * V, keep = p.taps - 1;
-    if (c >= p.N) return;
-    int t = blockIdx.x * strip, b = 0;
+    int t = blockIdx.x * strip;
     const int t_end = min(p.T, t + strip);
-    while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) ++b;
+    find_sequence(p.subsequence_begins, p.B, t, &s_b);
+    __syncthreads();
+    if (c >= p.N) return;
+    int b = s_b;
     const E* x = reinterpret_cast<const E*>(p.x) + c;
     E* u = reinterpret_cast<E*>(p.u) + (c / p.bw) * p.ub_pitch + c % p.bw;
     auto put = [&](int tok, const float (&acc)[V]) {

@@ -68,6 +68,13 @@ __device__ __forceinline__ void pdl_enter_attn() {
     if (OVB_PDL_ATTN) pdl_trigger();
 }
 
+// The sequence of a ragged batch that token t belongs to, looked for by the whole CTA: the thread that finds it writes *found (in
+// shared memory; a barrier must follow).
+__device__ __forceinline__ void find_sequence(const int* begins, int B, int t, int* found) {
+    for (int b = threadIdx.x; b < B; b += blockDim.x)
+        if (begins[b] <= t && t < begins[b + 1]) *found = b;
+}
+
 // ---------------------------------------------------------------- mbarrier
 __device__ __forceinline__ void mbar_init(uint64_t* bar, uint32_t count) {
     asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
