@@ -257,6 +257,7 @@ def build_selective(stats_csv, out_dir, stems=None, link: bool = True) -> Path:
         return obj
 
     srcs = [s_ for s_ in cuda_sources() if stems is None or s_.stem in stems]
+    srcs.sort(key=lambda s_: -s_.stat().st_size)      # the long compilations first
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
     if not link:
@@ -265,6 +266,29 @@ def build_selective(stats_csv, out_dir, stems=None, link: bool = True) -> Path:
     vers.write_text("{ global: ovb_*; local: *; };\n")
     target = out_dir / "libovb_cuda.so"
     _run([nvcc, "-shared", "-o", str(target), *map(str, objs), "-cudart", "static", "-Xlinker", "--version-script=%s" % vers])
+    return target
+
+
+# Kernels that the program of layered decoders runs (runtime/layered_llm.py), and the GEMM variants it uses: bf16 weights.
+LAYERED_STEMS = ("attention", "attention_exact", "attention_heads", "attention_latent", "attention_sm100", "common", "elementwise", "gemm_f32", "gemm_sm100",
+                 "recurrent", "residual", "sampling")
+
+
+def layered_library() -> Path:
+    """A kernel library that serves layered decoders: the full one where it is built and current, else a selective build of the
+    kernels that they need (``lib/libovb_layered.so``), which takes a fraction of the time."""
+    hdrs = sorted((CSRC / "cuda").glob("*.cuh")) + sorted((CSRC / "cuda").glob("*.h"))
+    full = LIB / "libovb_cuda.so"
+    if not _stale(full, cuda_sources() + hdrs):
+        return full
+    target = LIB / "libovb_layered.so"
+    if _stale(target, [CSRC / "cuda" / (stem + ".cu") for stem in LAYERED_STEMS] + hdrs):
+        work = OBJ / "layered"
+        work.mkdir(parents=True, exist_ok=True)
+        LIB.mkdir(exist_ok=True)
+        variants = work / "variants.csv"
+        variants.write_text("".join("gemm,%d,0,0\n" % bt for bt in (16, 32, 64, 128, 256)))
+        shutil.copy(build_selective(variants, work, LAYERED_STEMS), target)
     return target
 
 

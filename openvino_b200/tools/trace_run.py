@@ -23,6 +23,10 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, default=8192, help="most tokens that live requests hold at any time")
     args = ap.parse_args(argv)
 
+    # a fresh checkout compiles only the kernels that these models need
+    from ..build import layered_library
+    os.environ.setdefault("OVB_CUDA_LIB", str(layered_library()))
+
     import torch
 
     from ..genai.replay import Replay

@@ -35,3 +35,14 @@ def test_decode_variants_fit_two_ctas_per_sm(gemm):
 def test_gemm_uses_no_static_shared_memory(gemm):
     # the kernel opts in to the whole dynamic shared-memory limit of the SM: one static __shared__ word makes the opt-in fail
     assert all(r["static_smem"] == 0 for r in gemm.values()), {n: r["static_smem"] for n, r in gemm.items() if r["static_smem"]}
+
+
+def test_layered_decoders_need_no_more_than_the_full_library(gemm):
+    assert all((build.CSRC / "cuda" / (stem + ".cu")).exists() for stem in build.LAYERED_STEMS)
+    assert build.layered_library() == build.LIB / "libovb_cuda.so"        # built and current: nothing else is compiled
+
+
+@pytest.mark.parametrize("stem", ["attention_latent", "attention_sm100", "residual", "attention_heads", "gemm_f32", "attention_exact"])
+def test_kernels_of_layered_decoders_do_not_spill(gemm, stem):
+    res = build.kernel_resources(stem)
+    assert res and all(r["spill_stores"] == 0 and r["stack"] == 0 for r in res.values()), {n: r for n, r in res.items() if r["spill_stores"] or r["stack"]}
