@@ -43,6 +43,7 @@ struct PaKParams {
     // read from the paged cache `shared` (rows of shared_row elements) at column shared_col, and meets the query's columns from q_shared on.
     const int* kv_rows;
     const void* shared;
+    int cache_rows;           // rows of the paged caches (0: not known); copies are bounded by it
     int kv_total, kv_ld, k_head, v_head, shared_row, shared_col, q_shared;
 };
 

@@ -133,6 +133,7 @@ extern "C" int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream
         p.past_lens = a->past_lens; p.subsequence_begins = a->subsequence_begins;
         p.block_indices = a->block_indices; p.block_indices_begins = a->block_indices_begins;
         p.scratch = a->scratch;
+        p.cache_rows = a->cache_rows;
         p.B = a->B; p.T = a->T; p.Hq = a->Hq; p.Hkv = a->Hkv; p.group = a->Hq / a->Hkv;
         p.ldq = a->ldq; p.q_head = a->q_head; p.ldo = a->ldo; p.o_head = a->o_head; p.k_row = a->k_row; p.v_row = a->v_row;
         p.ld_gate = a->ld_gate; p.gate_head = a->gate_head;

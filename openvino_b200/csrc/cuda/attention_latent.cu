@@ -405,6 +405,7 @@ int ovb_latent_prefill(const ovb_latent_prefill_args* a, ovb_stream_t stream) {
     p.ldq = a->ldq; p.q_head = a->q_head; p.ldo = a->ldo; p.o_head = a->o_head;
     p.k_row = p.v_row = 8;                     // (pages hold the shared part only)
     p.kv_rows = a->kv_rows; p.kv_total = a->rows; p.kv_ld = a->ld_kv; p.k_head = a->k_head; p.v_head = a->v_head;
+    p.cache_rows = a->cache_rows;
     p.shared = a->cache; p.shared_row = a->row_pitch; p.shared_col = a->key_off; p.q_shared = a->q_rot_off;
     p.block_size = a->block_size; p.sliding_window = a->window; p.causal = 1;
     p.scale_log2 = a->scale * 1.4426950408889634f;

@@ -28,9 +28,12 @@
 
 #include "attention.cuh"
 #include "common.cuh"
+#include "debug_bounds.cuh"
 #include "sm100_ptx.cuh"
 
 namespace ovb {
+
+OVB_DEBUG_LIMITS_DEFINE
 
 namespace {
 
@@ -190,7 +193,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                 const int part = u / npages, pg = u % npages;
                 int row = row_base + j0 + pg * kPage, col_k = h * p.k_head, col_v = h * p.v_head;
                 if (SRC == SRC_PAGED || (RH > 0 && part >= KH && part < KH + RH)) {
-                    const int blk = p.block_indices[blk_begin + j0 / kPage + pg];
+                    const int blk = OVB_DBG_BLOCK(p.block_indices[blk_begin + j0 / kPage + pg]);
                     row = SRC == SRC_PAGED ? (blk * p.Hkv + h) * kPage : blk * kPage;
                     col_k = col_v = 0;
                 }
@@ -411,15 +414,15 @@ int launch_tc_parts(const PaKParams& p, int num_q_tiles, cudaStream_t stream) {
     // Q rows are tokens; a box is the TOK tokens of a tile x 64 columns of one head (rows past T read as zeros)
     if (int rc = make_tmap_2d(&tmQ, p.q, dt, 2, (uint64_t)p.T, (uint64_t)p.ldq, (uint64_t)p.ldq * 2, TOK, 64, true)) return rc;
     if (SRC == SRC_PAGED) {
-        // the cache seen as rows of one head: row = (block * Hkv + head) * 16 + slot; the row count only bounds coordinates
-        const uint64_t rows = 1ull << 30;
+        // the cache seen as rows of one head: row = (block * Hkv + head) * 16 + slot
+        const uint64_t rows = p.cache_rows > 0 ? (uint64_t)p.cache_rows : 1ull << 30;
         if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, rows, p.k_row, (uint64_t)p.k_row * 2, kPage, 64, true)) return rc;
         if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, rows, p.v_row, (uint64_t)p.v_row * 2, kPage, 64, true)) return rc;
     } else if (SRC == SRC_LATENT) {
         // pages of 16 rows that reach past a sequence's last key read the next sequence's rows (masked) or zeros behind the last
-        const uint64_t rows = 1ull << 30;
-        if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.kv_ld, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
-        if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.kv_ld, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
+        const uint64_t rows = p.cache_rows > 0 ? (uint64_t)p.cache_rows : 1ull << 30;
+        if (int rc = make_tmap_2d(&tmK, p.k_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.Hkv * p.k_head, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
+        if (int rc = make_tmap_2d(&tmV, p.v_cache, dt, 2, (uint64_t)p.kv_total, (uint64_t)p.Hkv * p.v_head, (uint64_t)p.kv_ld * 2, kPage, 64, true)) return rc;
         if (int rc = make_tmap_2d(&tmR, p.shared, dt, 2, rows, p.shared_row, (uint64_t)p.shared_row * 2, kPage, 64, true)) return rc;
     } else {
         const uint64_t rows = (uint64_t)p.B * p.dense_S;
@@ -491,3 +494,10 @@ int launch_window_tc(PaKParams p, int dk, int dshared, int dv, cudaStream_t stre
 }
 
 }  // namespace ovb
+
+#ifdef OVB_DEBUG_BOUNDS
+extern "C" int ovb_debug_set_limits_attention_tc(const ovb::DebugLimits* l) {
+    OVB_CHECK_CUDA(cudaMemcpyToSymbol(ovb::g_dbg_limits, l, sizeof(*l)));
+    return 0;
+}
+#endif

@@ -121,6 +121,7 @@ int ovb_debug_set_limits_elementwise(const ovb::DebugLimits* l);
 int ovb_debug_set_limits_heads(const ovb::DebugLimits* l);
 int ovb_debug_set_limits_exact(const ovb::DebugLimits* l);
 int ovb_debug_set_limits_latent(const ovb::DebugLimits* l);
+int ovb_debug_set_limits_attention_tc(const ovb::DebugLimits* l);
 #endif
 
 int ovb_debug_bounds_enabled(void) {
@@ -141,6 +142,7 @@ int ovb_debug_set_limits(int kv_blocks, int vocab) {
     if (int rc = ovb_debug_set_limits_heads(&l)) return rc;
     if (int rc = ovb_debug_set_limits_exact(&l)) return rc;
     if (int rc = ovb_debug_set_limits_latent(&l)) return rc;
+    if (int rc = ovb_debug_set_limits_attention_tc(&l)) return rc;
     return ovb_debug_set_limits_elementwise(&l);
 #else
     (void)kv_blocks; (void)vocab;

@@ -385,6 +385,7 @@ typedef struct {
     int block_size, window, max_context_len, max_q_len, dtype;
     float scale;
     int exact;                // 1: fp32 arithmetic throughout (no tensor cores)
+    int cache_rows;           // rows of k (and of v), 0: not known
 } ovb_wattn_args;
 int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream);
 
@@ -405,6 +406,7 @@ typedef struct {
     const int* block_indices;
     const int* block_indices_begins;
     int B, T, H, rows, R, Dv, ldq, q_head, q_rot_off, ld_kv, k_head, v_off, v_head, row_pitch, key_off, ldo, o_head, block_size, window;
+    int cache_rows;           // rows of cache, 0: not known
     float scale;
 } ovb_latent_prefill_args;
 int ovb_latent_prefill(const ovb_latent_prefill_args* a, ovb_stream_t stream);

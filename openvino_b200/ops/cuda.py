@@ -75,13 +75,13 @@ class WindowAttnArgs(C.Structure):
     _fields_ = (_fields(("q", "k", "v", "out", "gate", "past_lens", "subsequence_begins", "block_indices", "block_indices_begins", "scratch"), ())
                 + [("scratch_bytes", C.c_longlong)]
                 + _fields((), ("B", "T", "Hq", "Hkv", "Dk", "Dv", "ldq", "q_head", "k_row", "v_row", "ldo", "o_head", "ld_gate", "gate_head", "block_size",
-                               "window", "max_context_len", "max_q_len", "dtype"), ("scale",)) + [("exact", C.c_int)])
+                               "window", "max_context_len", "max_q_len", "dtype"), ("scale",)) + [("exact", C.c_int), ("cache_rows", C.c_int)])
 
 
 class LatentPrefillArgs(C.Structure):
     _fields_ = _fields(("q", "kv", "cache", "out", "kv_rows", "past_lens", "subsequence_begins", "block_indices", "block_indices_begins"),
                        ("B", "T", "H", "rows", "R", "Dv", "ldq", "q_head", "q_rot_off", "ld_kv", "k_head", "v_off", "v_head", "row_pitch", "key_off", "ldo",
-                        "o_head", "block_size", "window"), ("scale",))
+                        "o_head", "block_size", "window", "cache_rows"), ("scale",))
 
 
 class RgLruArgs(C.Structure):
@@ -418,6 +418,7 @@ def latent_prepare(**kw) -> None:
 
 def window_attention(**kw) -> None:
     """Paged attention with separate key / value sizes, window and output gate; fields of ``ovb_wattn_args``."""
+    kw["cache_rows"] = kw["k"].numel() // kw["k_row"]
     _check(lib().ovb_window_attention(C.byref(_fill(WindowAttnArgs(), kw)), C.c_void_p(_stream())), "ovb_window_attention")
 
 
@@ -431,6 +432,7 @@ def latent_gather(cache, out, kv_rows, past_lens, subsequence_begins, block_indi
 
 def latent_prefill(**kw) -> None:
     """Latent attention over expanded rows; fields of ``ovb_latent_prefill_args``."""
+    kw["cache_rows"] = kw["cache"].numel() // kw["row_pitch"]
     _check(lib().ovb_latent_prefill(C.byref(_fill(LatentPrefillArgs(), kw)), C.c_void_p(_stream())), "ovb_latent_prefill")
 
 
