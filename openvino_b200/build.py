@@ -270,7 +270,7 @@ def build_selective(stats_csv, out_dir, stems=None, link: bool = True) -> Path:
 
 
 # Kernels that the program of layered decoders runs (runtime/layered_llm.py), and the GEMM variants it uses: bf16 weights.
-LAYERED_STEMS = ("attention", "attention_exact", "attention_heads", "attention_latent", "attention_sm100", "common", "elementwise", "gemm_f32", "gemm_sm100",
+LAYERED_STEMS = ("attention", "attention_exact", "attention_heads", "attention_latent", "attention_sm100", "common", "delta_rule", "elementwise", "gemm_f32", "gemm_sm100",
                  "recurrent", "residual", "sampling")
 
 

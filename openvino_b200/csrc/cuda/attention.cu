@@ -312,7 +312,8 @@ __global__ void __launch_bounds__(256, 1) pa_prefill_kernel(PaKParams p) {
 // One value of a decoded token's output, through the optional gate.
 __device__ __forceinline__ void store_decoded(const PaKParams& p, int tok, int hq, int d, float v) {
     if (p.gate != nullptr)
-        v /= 1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)tok * p.ld_gate + (size_t)hq * p.gate_head + d]));
+        v /= 1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)tok * p.ld_gate + (size_t)hq * p.gate_head +
+                                                                                          (p.gate_scalar ? 0 : d)]));
     reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.ldo + (size_t)hq * p.o_head + d] = __float2bfloat16_rn(v);
 }
 
@@ -353,13 +354,13 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
     const int tok = p.subsequence_begins[b];
     const int ctx = p.past_lens[b] + 1;
     const int blk_begin = p.block_indices_begins[b];
-    // the splits share the keys from the first page that the window touches
-    const int k_first = p.sliding_window > 0 ? max(0, (ctx - p.sliding_window) / PAGE * PAGE) : 0;
+    // the splits share the keys from the first page that the window or the chunk touches
+    const int win_lo = first_visible_key(ctx - 1, p.sliding_window, p.chunk);
+    const int k_first = win_lo / PAGE * PAGE;
     const int k_lo = k_first + split * p.keys_per_split;
     const int k_hi = min(ctx, k_lo + p.keys_per_split);
     const int page_lo = k_lo / PAGE;
     const int page_hi = (k_hi + PAGE - 1) / PAGE;         // exclusive
-    const int win_lo = p.sliding_window > 0 ? ctx - p.sliding_window : 0;
 
     // Q: G real rows, the rest zero
     for (int i = threadIdx.x; i < 16 * CHK; i += 128) {
@@ -547,6 +548,7 @@ __global__ void __launch_bounds__(128) pa_decode_kernel(PaKParams p) {
         }
         const int hq = hq0 + rr;
         if (p.nsplit == 1) {
+            if (p.sink != nullptr) l += exp2f(p.sink[hq] * 1.4426950408889634f - m);
             if (GT > 0 || d < p.dv_store) store_decoded(p, tok, hq, d, l > 0.f ? o / l : 0.f);
         } else {
             float* sc = p.scratch + (((size_t)b * p.Hq + hq) * p.nsplit + split) * (DV + 2);
@@ -573,6 +575,7 @@ __global__ void __launch_bounds__(128) pa_decode_combine_kernel(PaKParams p, int
         l *= sc;
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+        if (p.sink != nullptr) l += exp2f(p.sink[hq] * 1.4426950408889634f - mx);
         w[threadIdx.x] = l > 0.f ? sc / l : 0.f;
     }
     const int tok = p.subsequence_begins[b];
@@ -664,7 +667,9 @@ int launch_window_decode(PaKParams p, int dk, int dv, int max_ctx, long long scr
         !aligned(p.v_cache))
         return ERR_UNSUPPORTED;
     const int ck = dk <= 64 ? 64 : dk <= 128 ? 128 : 256, cv = dv <= 64 ? 64 : dv <= 128 ? 128 : 256;
-    const int keys = p.sliding_window > 0 && p.sliding_window + 15 < max_ctx ? p.sliding_window + 15 : max_ctx;   // a window may start inside a page
+    int keys = max_ctx;       // that the splits share (a window or a chunk may start inside a page)
+    if (p.sliding_window > 0 && p.sliding_window + 15 < keys) keys = p.sliding_window + 15;
+    if (p.chunk > 0 && p.chunk + 15 < keys) keys = p.chunk + 15;
     p.dv_store = dv;
     p.nsplit = decode_nsplit(p.B, p.Hkv * ((p.group + 7) / 8), keys);
     const long long per_split = (long long)p.B * p.Hq * (cv + 2) * 4;

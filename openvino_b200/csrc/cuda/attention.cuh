@@ -37,6 +37,9 @@ struct PaKParams {
     // optional output gate: out *= sigmoid(gate[t * ld_gate + head * gate_head + column])
     const void* gate;
     int ld_gate, gate_head;
+    int gate_scalar;          // 1: one gate value per head, gate[t * ld_gate + head * gate_head]
+    int chunk;                // > 0: a position sees only keys of its own chunk of this many positions (counted from position 0)
+    const float* sink;        // [Hq] or NULL: exp(sink[head]) is added to the softmax denominator (no key, no value, not scaled)
     int group;                // query heads per KV head where the kernel takes it at run time
     // Latent attention with expanded heads: keys and values of sequence b, from key kv_first(b) on, are the contiguous rows
     // kv_rows[b] .. of k_cache / v_cache (head h at column h * k_head / h * v_head); a second key part that all heads share is
@@ -46,6 +49,14 @@ struct PaKParams {
     int cache_rows;           // rows of the paged caches (0: not known); copies are bounded by it
     int kv_total, kv_ld, k_head, v_head, shared_row, shared_col, q_shared;
 };
+
+// First key that position `pos` sees under a sliding window and / or a chunk (0: off); it never decreases with the position.
+__host__ __device__ inline int first_visible_key(int pos, int window, int chunk) {
+    int lo = window > 0 ? pos - window + 1 : 0;
+    if (lo < 0) lo = 0;
+    const int start = chunk > 0 ? pos - pos % chunk : 0;
+    return lo > start ? lo : start;
+}
 
 // First key that is expanded for a sequence: what the window of its first new token reaches, rounded down to whole key tiles.
 __host__ __device__ inline int latent_first_key(int past, int window) {

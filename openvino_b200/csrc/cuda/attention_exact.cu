@@ -34,7 +34,7 @@ __global__ void __launch_bounds__(kThreads) attention_exact_kernel(ovb_wattn_arg
     const int b = s_b, kvh = h / (p.Hq / p.Hkv);
     const int pos = p.past_lens[b] + t - p.subsequence_begins[b];
     const int* blocks = p.block_indices + p.block_indices_begins[b];
-    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int lo = first_visible_key(pos, p.window, p.chunk);
     auto row_of = [&](int j) {
         const int blk = OVB_DBG_BLOCK(blocks[j / p.block_size]);
         return ((size_t)blk * p.Hkv + kvh) * p.block_size + j % p.block_size;
@@ -83,6 +83,7 @@ __global__ void __launch_bounds__(kThreads) attention_exact_kernel(ovb_wattn_arg
         }
         __syncthreads();
     }
+    if (p.sink) l += expf(p.sink[h] - m);
     E* out = reinterpret_cast<E*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.o_head;
     const E* gate = p.gate ? reinterpret_cast<const E*>(p.gate) + (size_t)t * p.ld_gate + (size_t)h * p.gate_head : nullptr;
 #pragma unroll
@@ -90,7 +91,7 @@ __global__ void __launch_bounds__(kThreads) attention_exact_kernel(ovb_wattn_arg
         const int d = tid + i * kThreads;
         if (d < p.Dv) {
             float o = acc[i] / l;
-            if (gate) o *= 1.f / (1.f + expf(-ld_f32(gate + d)));
+            if (gate) o *= 1.f / (1.f + expf(-ld_f32(gate + (p.gate_scalar ? 0 : d))));
             st_f32(out + d, o);
         }
     }
@@ -136,11 +137,11 @@ extern "C" int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream
         p.cache_rows = a->cache_rows;
         p.B = a->B; p.T = a->T; p.Hq = a->Hq; p.Hkv = a->Hkv; p.group = a->Hq / a->Hkv;
         p.ldq = a->ldq; p.q_head = a->q_head; p.ldo = a->ldo; p.o_head = a->o_head; p.k_row = a->k_row; p.v_row = a->v_row;
-        p.ld_gate = a->ld_gate; p.gate_head = a->gate_head;
-        p.block_size = a->block_size; p.sliding_window = a->window; p.causal = 1;
+        p.ld_gate = a->ld_gate; p.gate_head = a->gate_head; p.gate_scalar = a->gate_scalar;
+        p.block_size = a->block_size; p.sliding_window = a->window; p.chunk = a->chunk; p.sink = a->sink; p.causal = 1;
         p.scale_log2 = a->scale * 1.4426950408889634f;
         const bool decode = a->max_q_len == 1 && a->T == a->B;
-        const int rc = a->k == a->v ? (a->Hkv == 1 && a->gate == nullptr ? launch_latent_attention(p, a->Dk, (a->Dv + 15) / 16 * 16, a->max_q_len, a->max_context_len,
+        const int rc = a->k == a->v ? (a->Hkv == 1 && a->gate == nullptr && a->chunk == 0 && a->sink == nullptr ? launch_latent_attention(p, a->Dk, (a->Dv + 15) / 16 * 16, a->max_q_len, a->max_context_len,
                                                                                                    a->scratch_bytes, (cudaStream_t)stream) : ERR_UNSUPPORTED)
                      : decode ? launch_window_decode(p, a->Dk, a->Dv, a->max_context_len, a->scratch_bytes, (cudaStream_t)stream)
                               : a->scale > 0.f ? launch_window_tc(p, a->Dk, 0, (a->Dv + 15) / 16 * 16, (cudaStream_t)stream) : ERR_UNSUPPORTED;

@@ -1,8 +1,9 @@
 // From projections to what attention reads: per-head norms, rotary positions and the rows of the paged cache.
 //
-//   heads_prepare   grouped-query attention. Every query and key head may be RMS-normed over its dimensions (weights shared by
-//                   the heads) and its first dimensions turned by the position; queries are changed in place, key and value
-//                   rows go to the cache.
+//   heads_prepare   grouped-query attention. Every projected column may pass a short causal convolution; every query and key head
+//                   may be RMS-normed over its dimensions (weights shared by the heads) and its first dimensions turned by the
+//                   position; values may be mixed with those of an earlier layer. Queries are changed in place (or written to a
+//                   buffer of their own when there is a convolution), key and value rows go to the cache.
 //   latent_prepare  latent attention. The low-rank row of a token is normed and cached together with the one turned key part
 //                   that all heads share; the queries' turned part is written where the attention kernel reads it.
 //
@@ -10,6 +11,7 @@
 // the rotation; dimension i is paired with i + dims / 2. Norms, angles and sums are fp32. Rows of heads are padded to the pitch
 // that the attention kernels want; the padding is zero and is never written.
 #include "debug_bounds.cuh"
+#include "short_conv.cuh"
 #include "sm100_ptx.cuh"
 #include "store_types.cuh"
 
@@ -42,60 +44,198 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
-struct HeadsParams {
-    void* proj;              // [T, ldp]: query heads at column 0, key heads at k_off, value heads at v_off
-    void* k_cache;           // [blocks, G, block_size, dk_pad]
-    void* v_cache;           // [blocks, G, block_size, dv_pad]
-    const float* q_norm;     // [D] or NULL
-    const float* k_norm;
-    const int* positions;
-    const int* slot_map;
-    Rotation rot;
-    int T, H, G, D, Dv, dk_pad, dv_pad, ldp, k_off, v_off, block_size;
-    float eps;
+__device__ __forceinline__ void turn_by(float2 cs, float& u, float& v) {
+    const float a = u * cs.x - v * cs.y, b = v * cs.x + u * cs.y;
+    u = a;
+    v = b;
+}
+
+__global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, float2* __restrict__ table, int n, int half, float mult) {
+    pdl_enter();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    float s, c;
+    sincosf((float)positions[i / half] * inv_freq[i % half], &s, &c);
+    table[i] = make_float2(c * mult, s * mult);
+}
+
+struct HeadUnit {            // what one warp works on: a query, key or value head
+    bool is_q, is_k;
+    int kvh, n, col;         // KV head, columns, first column in proj
 };
+__device__ __forceinline__ HeadUnit head_unit(const ovb_heads_args& p, int head) {
+    HeadUnit u;
+    u.is_q = head < p.H;
+    u.is_k = !u.is_q && head < p.H + p.G;
+    u.kvh = u.is_q ? 0 : (head - p.H) % p.G;
+    u.n = u.is_q || u.is_k ? p.D : p.Dv;
+    u.col = u.is_q ? head * p.dk_pad : u.is_k ? p.k_off + u.kvh * p.dk_pad : p.v_off + u.kvh * p.dv_pad;
+    return u;
+}
+// Row of the paged cache (or of the query buffer) that takes token t of this head; NULL: no slot.
+template <class E>
+__device__ __forceinline__ E* head_row(const ovb_heads_args& p, const HeadUnit& u, int t) {
+    if (u.is_q) return p.q_out ? reinterpret_cast<E*>(p.q_out) + (size_t)t * p.ldq + u.col : reinterpret_cast<E*>(p.proj) + (size_t)t * p.ldp + u.col;
+    const int slot = OVB_DBG_SLOT(p.slot_map[t], p.block_size);
+    if (slot < 0) return nullptr;
+    const size_t row = ((size_t)(slot / p.block_size) * p.G + u.kvh) * p.block_size + slot % p.block_size;
+    return u.is_k ? reinterpret_cast<E*>(p.k_cache) + row * p.dk_pad : reinterpret_cast<E*>(p.v_cache) + row * p.dv_pad;
+}
 
 // One warp per (token, head); the row passes through shared memory because a rotation pairs elements of different lanes.
 template <class E>
-__global__ void __launch_bounds__(128) heads_prepare_kernel(HeadsParams p) {
+__global__ void __launch_bounds__(128) heads_prepare_kernel(ovb_heads_args p) {
     pdl_enter();
     extern __shared__ float rows[];
+    __shared__ int s_b;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x, head = blockIdx.y * 4 + warp;
+    if (p.taps > 0) {
+        find_sequence(p.subsequence_begins, p.B, t, &s_b);
+        __syncthreads();
+    }
     if (head >= p.H + 2 * p.G) return;
-    E* proj = reinterpret_cast<E*>(p.proj) + (size_t)t * p.ldp;
-    const bool is_q = head < p.H, is_k = !is_q && head < p.H + p.G;
-    const int kvh = is_q ? 0 : (head - p.H) % p.G;
-    E* src = is_q ? proj + head * p.dk_pad : is_k ? proj + p.k_off + kvh * p.dk_pad : proj + p.v_off + kvh * p.dv_pad;
-    E* dst = src;
-    if (!is_q) {
-        const int slot = OVB_DBG_SLOT(p.slot_map[t], p.block_size);
-        if (slot < 0) return;
-        const size_t row = ((size_t)(slot / p.block_size) * p.G + kvh) * p.block_size + slot % p.block_size;
-        dst = is_k ? reinterpret_cast<E*>(p.k_cache) + row * p.dk_pad : reinterpret_cast<E*>(p.v_cache) + row * p.dv_pad;
-    }
-    if (!is_q && !is_k) {
-        for (int i = lane; i < p.Dv; i += 32) dst[i] = src[i];
-        return;
-    }
-    float* r = rows + warp * p.D;
+    const HeadUnit u = head_unit(p, head);
+    const E* src = reinterpret_cast<const E*>(p.proj) + u.col;
+    E* dst = head_row<E>(p, u, t);
+    float* r = rows + warp * max(p.D, p.Dv);
+    const ShortConv cv = {p.conv_w, p.conv_ring, p.taps, p.conv_cols};
     float ss = 0.f;
-    for (int i = lane; i < p.D; i += 32) {
-        const float v = ld_f32(src + i);
+    for (int i = lane; i < u.n; i += 32) {
+        float v;
+        if (p.taps > 0) {
+            const int begin = p.subsequence_begins[s_b], pos = p.positions[t];
+            float* ring = cv.ring + (size_t)p.slots[s_b] * cv.taps * cv.cols + u.col + i;
+            v = 0.f;
+            for (int j = 0; j < cv.taps; ++j)
+                v = fmaf(cv.w[(size_t)j * cv.cols + u.col + i], conv_input(src + i, p.ldp, ring, cv, t, begin, pos, cv.taps - 1 - j), v);
+            if (p.max_q_len == 1 && cv.taps > 1) ring[(size_t)(pos % cv.taps) * cv.cols] = ld_f32(src + (size_t)t * p.ldp + i);
+        } else {
+            v = ld_f32(src + (size_t)t * p.ldp + i);
+        }
         r[i] = v;
         ss += v * v;
     }
-    const float* w = is_q ? p.q_norm : p.k_norm;
+    if (!u.is_q && !u.is_k) {
+        E* first = p.v_mode ? reinterpret_cast<E*>(p.v_first) + (size_t)t * p.ld_vf + u.kvh * p.Dv : nullptr;
+        for (int i = lane; i < u.n; i += 32) {
+            float v = r[i];
+            if (p.v_mode == 1) st_f32(first + i, v);
+            if (p.v_mode == 2) v = (1.f - p.v_mix) * v + p.v_mix * ld_f32(first + i);
+            if (dst) st_f32(dst + i, v);
+        }
+        return;
+    }
+    if (!dst) return;
+    const float* w = u.is_q ? p.q_norm : p.k_norm;
     if (w) {
         const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.D + p.eps);
         for (int i = lane; i < p.D; i += 32) r[i] *= inv * w[i];
     }
     __syncwarp();
-    const int half = p.rot.dims / 2;
+    const int half = p.rot_dims / 2;
+    const Rotation rot = {p.inv_freq, p.rot_dims, p.rot_mult};
     const float pos = (float)p.positions[t];
-    for (int i = lane; i < half; i += 32) turn(p.rot, pos, i, r[i], r[i + half]);
+    for (int i = lane; i < half; i += 32) {
+        if (p.rope) turn_by(reinterpret_cast<const float2*>(p.rope)[(size_t)t * half + i], r[i], r[i + half]);
+        else turn(rot, pos, i, r[i], r[i + half]);
+    }
     __syncwarp();
     for (int i = lane; i < p.D; i += 32) st_f32(dst + i, r[i]);
+}
+
+constexpr int HEADS_STRIP = 8;      // tokens per warp of a prompt
+
+// The same for heads of up to 128 columns in pieces of four: a warp walks a strip of tokens of one head with its columns in registers
+// (lane l: columns 4 l ..), so that every projected value is fetched once; rotation partners sit in other lanes. TAPS 0: no convolution.
+template <class E, int TAPS>
+__global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int strip) {
+    pdl_enter();
+    __shared__ int s_b;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * strip, t_end = min(p.T, t0 + strip), head = blockIdx.y * 4 + warp;
+    if (TAPS > 0) {
+        find_sequence(p.subsequence_begins, p.B, t0, &s_b);
+        __syncthreads();
+    }
+    if (head >= p.H + 2 * p.G) return;
+    constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 0;
+    const HeadUnit u = head_unit(p, head);
+    const bool is_v = !u.is_q && !u.is_k;
+    const int c = lane * 4;
+    const bool live = c < u.n;
+    const E* src = reinterpret_cast<const E*>(p.proj) + u.col + (live ? c : 0);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 w[TAPS > 0 ? TAPS : 1], hist[KEEP > 0 ? KEEP : 1], raw[HEADS_STRIP];
+#pragma unroll
+    for (int k = 0; k < HEADS_STRIP; ++k) raw[k] = (live && t0 + k < t_end) ? ld4_f32(src + (size_t)(t0 + k) * p.ldp) : zero;
+    if (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = live ? ld4_f32(p.conv_w + (size_t)j * p.conv_cols + u.col + c) : zero;
+    }
+    const float* nw = u.is_q ? p.q_norm : u.is_k ? p.k_norm : nullptr;
+    const float4 gain = nw && live ? make_float4(nw[c], nw[c + 1], nw[c + 2], nw[c + 3]) : zero;
+    // the partner of column c is c + half (in the lower half) or c - half
+    const int half = is_v ? 0 : p.rot_dims / 2;
+    const bool lower = c < half, turned = c < 2 * half;
+    const int partner = turned ? (lower ? lane + half / 4 : lane - half / 4) : lane;
+    const ShortConv cv = {p.conv_w, p.conv_ring, TAPS, p.conv_cols};
+    int b = TAPS > 0 ? s_b : 0, begin = TAPS > 0 ? p.subsequence_begins[b] : 0;
+#pragma unroll
+    for (int k = 0; k < HEADS_STRIP; ++k) {
+        const int t = t0 + k;
+        if (t >= t_end) break;
+        float4 v = raw[k];
+        if (TAPS > 0) {
+            const int pos = p.positions[t];
+            bool fresh = k == 0;
+            while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) {
+                ++b;
+                begin = t;
+                fresh = true;
+            }
+            float* ring = cv.ring + (size_t)p.slots[b] * TAPS * cv.cols + u.col + c;
+            if (fresh) {
+#pragma unroll
+                for (int j = 0; j < KEEP; ++j) hist[j] = live ? conv_input4(src, p.ldp, ring, cv, t, begin, pos, KEEP - j) : zero;
+            }
+            if (p.max_q_len == 1 && TAPS > 1 && live) st4_f32(ring + (size_t)(pos % TAPS) * cv.cols, v);
+            float4 acc = zero;
+#pragma unroll
+            for (int j = 0; j < KEEP; ++j) acc = fma4(w[j], hist[j], acc);
+            acc = fma4(w[TAPS > 0 ? TAPS - 1 : 0], v, acc);
+#pragma unroll
+            for (int j = 0; j + 1 < KEEP; ++j) hist[j] = hist[j + 1];
+            if (KEEP > 0) hist[KEEP - 1] = v;
+            v = acc;
+        }
+        if (nw) {
+            const float inv = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)p.D + p.eps);
+            v = make_float4(v.x * inv * gain.x, v.y * inv * gain.y, v.z * inv * gain.z, v.w * inv * gain.w);
+        }
+        if (half > 0) {
+            const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, partner), __shfl_sync(0xffffffffu, v.y, partner), __shfl_sync(0xffffffffu, v.z, partner),
+                                         __shfl_sync(0xffffffffu, v.w, partner));
+            if (turned) {
+                const float4* cs = reinterpret_cast<const float4*>(p.rope + ((size_t)t * half + (lower ? c : c - half)) * 2);
+                const float4 a = cs[0], d = cs[1];       // (cos, sin) of four pairs
+                const float sg = lower ? -1.f : 1.f;     // lower: u cos - v sin, upper: v cos + u sin
+                v = make_float4(v.x * a.x + sg * (o.x * a.y), v.y * a.z + sg * (o.y * a.w), v.z * d.x + sg * (o.z * d.y), v.w * d.z + sg * (o.w * d.w));
+            }
+        }
+        if (is_v && p.v_mode && live) {
+            E* first = reinterpret_cast<E*>(p.v_first) + (size_t)t * p.ld_vf + u.kvh * p.Dv + c;
+            if (p.v_mode == 1) {
+                st4_f32(first, v);
+            } else {
+                const float4 f = ld4_f32(first);
+                const float a = 1.f - p.v_mix;
+                v = make_float4(a * v.x + p.v_mix * f.x, a * v.y + p.v_mix * f.y, a * v.z + p.v_mix * f.z, a * v.w + p.v_mix * f.w);
+            }
+        }
+        E* dst = head_row<E>(p, u, t);
+        if (dst && live) st4_f32(dst + c, v);
+    }
 }
 
 struct LatentParams {
@@ -178,17 +318,48 @@ extern "C" int ovb_debug_set_limits_heads(const ovb::DebugLimits* l) {
 extern "C" {
 using namespace ovb;
 
+int ovb_rope_table(const int* positions, const float* inv_freq, float* table, int T, int half, float mult, ovb_stream_t stream) {
+    OVB_REQUIRE(positions && inv_freq && table && T > 0 && half > 0, "ovb_rope_table: bad arguments");
+    OVB_CHECK_CUDA(launch_pdl(rope_table_kernel, dim3(ceil_div(T * half, 256)), dim3(256), 0, (cudaStream_t)stream, positions, inv_freq,
+                              reinterpret_cast<float2*>(table), T * half, half, mult));
+    return 0;
+}
+
 int ovb_heads_prepare(const ovb_heads_args* a, ovb_stream_t stream) {
     OVB_REQUIRE(a && a->proj && a->k_cache && a->v_cache && a->positions && a->slot_map, "ovb_heads_prepare: null operand");
     OVB_REQUIRE(a->T > 0 && a->H > 0 && a->G > 0 && a->D > 0 && a->Dv > 0 && a->dk_pad >= a->D && a->dv_pad >= a->Dv && a->block_size > 0,
                 "ovb_heads_prepare: bad sizes");
     OVB_REQUIRE(a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->D && (a->rot_dims == 0 || a->inv_freq), "ovb_heads_prepare: bad rotation");
-    OVB_REQUIRE(a->D <= 2048, "ovb_heads_prepare: head size %d above 2048", a->D);
-    HeadsParams p = {a->proj, a->k_cache, a->v_cache, a->q_norm, a->k_norm, a->positions, a->slot_map, {a->inv_freq, a->rot_dims, a->rot_mult},
-                     a->T, a->H, a->G, a->D, a->Dv, a->dk_pad, a->dv_pad, a->ldp, a->k_off, a->v_off, a->block_size, a->eps};
+    OVB_REQUIRE(a->D <= 2048 && a->Dv <= 2048, "ovb_heads_prepare: head sizes %d, %d above 2048", a->D, a->Dv);
+    OVB_REQUIRE(a->taps == 0 || (a->taps > 0 && a->conv_w && a->conv_ring && a->subsequence_begins && a->past_lens && a->slots && a->q_out && a->B > 0 &&
+                                 a->conv_cols >= a->v_off + a->G * a->dv_pad), "ovb_heads_prepare: bad short convolution");
+    OVB_REQUIRE(a->v_mode == 0 || (a->v_first && a->ld_vf >= a->G * a->Dv && (a->v_mode == 1 || a->v_mode == 2)), "ovb_heads_prepare: bad value mixing");
+    auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    const int units = a->H + 2 * a->G;
+    // heads in registers: whole pieces of four columns everywhere, rotation partners at whole lanes, angles from the table
+    const bool strip_form = a->D <= 128 && a->Dv <= 128 && a->D % 4 == 0 && a->Dv % 4 == 0 && a->rot_dims % 8 == 0 && (a->rot_dims == 0 || a->rope) && a->taps <= 4 &&
+                            a->ldp % 4 == 0 && a->dk_pad % 4 == 0 && a->dv_pad % 4 == 0 && a->k_off % 4 == 0 && a->v_off % 4 == 0 && a->conv_cols % 4 == 0 &&
+                            a->ldq % 4 == 0 && a->ld_vf % 4 == 0 && aligned(a->proj) && aligned(a->q_out) && aligned(a->k_cache) && aligned(a->v_cache) &&
+                            aligned(a->conv_w) && aligned(a->conv_ring) && aligned(a->v_first) && aligned(a->rope);
     return dispatch_store(a->dtype, "ovb_heads_prepare", [&](auto e) -> int {
         using E = decltype(e);
-        OVB_CHECK_CUDA(launch_pdl(heads_prepare_kernel<E>, dim3(p.T, ceil_div(p.H + 2 * p.G, 4)), dim3(128), (size_t)4 * p.D * 4, (cudaStream_t)stream, p));
+        if (strip_form) {
+            // few tokens: a warp each; many: strips that share the inputs of the convolution
+            const int strip = (long long)a->T * units <= 148 * 32 || a->max_q_len == 1 ? 1 : HEADS_STRIP;
+            auto go = [&](auto kern) -> int {
+                OVB_CHECK_CUDA(launch_pdl(kern, dim3(ceil_div(a->T, strip), ceil_div(units, 4)), dim3(128), 0, (cudaStream_t)stream, *a, strip));
+                return 0;
+            };
+            switch (a->taps) {
+                case 0: return go(heads_strip_kernel<E, 0>);
+                case 1: return go(heads_strip_kernel<E, 1>);
+                case 2: return go(heads_strip_kernel<E, 2>);
+                case 3: return go(heads_strip_kernel<E, 3>);
+                default: return go(heads_strip_kernel<E, 4>);
+            }
+        }
+        const int width = a->D > a->Dv ? a->D : a->Dv;
+        OVB_CHECK_CUDA(launch_pdl(heads_prepare_kernel<E>, dim3(a->T, ceil_div(units, 4)), dim3(128), (size_t)4 * width * 4, (cudaStream_t)stream, *a));
         return 0;
     });
 }

@@ -161,9 +161,8 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int tq1 = min(q_len, tq0 + TOK);
     const int kv_total = PAGED ? past + q_len : p.dense_S;
     const int kv_end = p.causal ? min(kv_total, past + tq1) : kv_total;
-    int kv_start = 0;
-    if (p.sliding_window > 0) kv_start = max(0, past + tq0 - p.sliding_window + 1);
-    kv_start = (kv_start / kBK) * kBK;
+    const int kv_start = PAGED ? first_visible_key(past + tq0, p.sliding_window, p.chunk) / kBK * kBK : 0;
+    const int lo_last = PAGED ? first_visible_key(past + tq1 - 1, p.sliding_window, p.chunk) : 0;   // of the tile's last token
     const int ntiles = (kv_end - kv_start + kBK - 1) / kBK;
 
     if (warp == 4) {
@@ -246,6 +245,7 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         const int g = r / TOK, tl = r % TOK;
         const int qpos = past + tq0 + tl;
         const bool row_valid = (tq0 + tl) < q_len && (GT > 0 || g < G);
+        const int lo_row = PAGED ? first_visible_key(qpos, p.sliding_window, p.chunk) : 0;
         const uint32_t lane_base = tmem + (uint32_t(warp * 32) << 16);
         float m_used = -CUDART_INF_F, l_sum = 0.f;
         bool ok = true;
@@ -257,12 +257,12 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
             const int j0 = kv_start + j * kBK;
             // does any row of the tile need a mask? (uniform over the CTA)
             const bool need_mask = (j0 + kBK > kv_end) || (p.causal && (j0 + kBK - 1 > past + tq0)) ||
-                                   (p.sliding_window > 0 && (j0 <= past + tq1 - 1 - p.sliding_window));
+                                   j0 < lo_last;
             int hi = kBK, lo = 0;                        // keys [lo, hi) of the tile are visible to this row
             if (need_mask) {
                 hi = min(hi, kv_end - j0);
                 if (p.causal) hi = min(hi, qpos - j0 + 1);
-                if (p.sliding_window > 0) lo = max(lo, qpos - p.sliding_window + 1 - j0);
+                lo = max(lo, lo_row - j0);
                 if (!row_valid) hi = 0;
             }
             // The whole row of S goes to registers in one round trip to tensor memory (eight loads in flight, one wait);
@@ -337,7 +337,15 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         }
         // ---- epilogue: O / l. The gate's row is requested before the last product is waited for.
         uint4 gw[DV / 8];
-        const bool gated = p.gate != nullptr && row_valid;
+        const bool gated = p.gate != nullptr && !p.gate_scalar && row_valid;
+        float head_gate = 1.f, sink = -CUDART_INF_F;
+        if (row_valid) {
+            if (p.gate != nullptr && p.gate_scalar) {
+                const __nv_bfloat16 gv = reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)(tok_begin + tq0 + tl) * p.ld_gate + (size_t)(h * G + g) * p.gate_head];
+                head_gate = __fdividef(1.f, 1.f + __expf(-__bfloat162float(gv)));
+            }
+            if (p.sink != nullptr) sink = p.sink[h * G + g] * 1.4426950408889634f;
+        }
         if (gated) {
             const uint4* gate = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.gate) + (size_t)(tok_begin + tq0 + tl) * p.ld_gate +
                                                                (size_t)(h * G + g) * p.gate_head);
@@ -348,7 +356,8 @@ pa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (ok && ntiles > 0) ok = mbar_wait(&pv_done[(ntiles - 1) & 1], ((ntiles - 1) >> 1) & 1, abort_flag, status);
         if (ok) {
             tc_fence_after_sync();
-            const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+            if (sink != -CUDART_INF_F && m_used != -CUDART_INF_F) l_sum += exp2f(sink - m_used);
+            const float inv = l_sum > 0.f ? head_gate / l_sum : 0.f;
             uint8_t* dst = reinterpret_cast<uint8_t*>(p.out) + ((size_t)(tok_begin + tq0 + tl) * p.ldo + (size_t)(h * G + g) * p.o_head) * 2;
 #pragma unroll
             for (int c = 0; c < DV; c += 16) {
@@ -474,8 +483,9 @@ int launch_window_tc(PaKParams p, int dk, int dshared, int dv, cudaStream_t stre
     const int kh = ceil_div(dk, 64), rh = ceil_div(dshared, 64), vh = ceil_div(dv, 64);
     if (p.block_size != kPage || p.group < 1 || p.group > 16 || kh + rh > 3 || rh > 1 || vh > 2) return ERR_UNSUPPORTED;
     auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-    if (!aligned(p.q) || !aligned(p.k_cache) || !aligned(p.v_cache) || !aligned(p.out) || !aligned(p.gate) || !aligned(p.shared)) return ERR_UNSUPPORTED;
-    if (p.ldq % 8 || p.q_head % 8 || p.ldo % 8 || p.o_head % 8 || p.ld_gate % 8 || p.gate_head % 8 || dv % 16 || p.k_row % 8 || p.v_row % 8) return ERR_UNSUPPORTED;
+    if (!aligned(p.q) || !aligned(p.k_cache) || !aligned(p.v_cache) || !aligned(p.out) || !aligned(p.shared)) return ERR_UNSUPPORTED;
+    if (!p.gate_scalar && (!aligned(p.gate) || p.ld_gate % 8 || p.gate_head % 8)) return ERR_UNSUPPORTED;
+    if (p.ldq % 8 || p.q_head % 8 || p.ldo % 8 || p.o_head % 8 || dv % 16 || p.k_row % 8 || p.v_row % 8) return ERR_UNSUPPORTED;
     p.dv_store = dv;
     const int tiles = p.T / tile_tokens(p.group) + p.B;      // upper bound of the tiles of all sequences
     if (rh > 0) {

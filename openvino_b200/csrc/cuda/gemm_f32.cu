@@ -16,6 +16,7 @@ struct GemmF32Params {
     float* out;
     long long sx, sw, sb, so;     // elements between the batch members' operands
     int T, N, K, ldx, ldw, ldo, act;
+    float limit;                  // OVB_ACT_SOFTCAP
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Params p) {
@@ -60,6 +61,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Params p) {
             if (p.act == OVB_ACT_GELU_TANH) v = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
             else if (p.act == OVB_ACT_SILU) v = v / (1.f + expf(-v));
             else if (p.act == OVB_ACT_RELU) v = fmaxf(v, 0.f);
+            else if (p.act == OVB_ACT_RELU2) v = fmaxf(v, 0.f) * v;
+            else if (p.act == OVB_ACT_SOFTCAP) v = p.limit * tanhf(v / p.limit);
             out[(size_t)t * p.ldo + n] = v;
         }
 }
@@ -69,12 +72,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Params p) {
 }  // namespace ovb
 
 extern "C" int ovb_gemm_f32(const float* x, const float* w, const float* bias, float* out, int batch, long long sx, long long sw, long long sb, long long so,
-                            int T, int N, int K, int ldx, int ldw, int ldo, int act, ovb_stream_t stream) {
+                            int T, int N, int K, int ldx, int ldw, int ldo, int act, float act_limit, ovb_stream_t stream) {
     using namespace ovb;
     OVB_REQUIRE(x && w && out && batch > 0 && T > 0 && N > 0 && K > 0 && batch <= 65535, "ovb_gemm_f32: bad arguments");
     OVB_REQUIRE(ceil_div(T, FT) <= 65535, "ovb_gemm_f32: %d rows are too many", T);
-    OVB_REQUIRE(act == OVB_ACT_NONE || act == OVB_ACT_GELU_TANH || act == OVB_ACT_SILU || act == OVB_ACT_RELU, "ovb_gemm_f32: activation %d is not served", act);
-    GemmF32Params p = {x, w, bias, out, sx, sw, sb, so, T, N, K, ldx, ldw, ldo, act};
+    OVB_REQUIRE(act == OVB_ACT_NONE || act == OVB_ACT_GELU_TANH || act == OVB_ACT_SILU || act == OVB_ACT_RELU || act == OVB_ACT_RELU2 ||
+                    (act == OVB_ACT_SOFTCAP && act_limit > 0.f), "ovb_gemm_f32: activation %d is not served", act);
+    GemmF32Params p = {x, w, bias, out, sx, sw, sb, so, T, N, K, ldx, ldw, ldo, act, act_limit};
     OVB_CHECK_CUDA(launch_pdl(gemm_f32_kernel, dim3(ceil_div(N, FT), ceil_div(T, FT), batch), dim3(256), 0, (cudaStream_t)stream, p));
     return 0;
 }

@@ -96,7 +96,7 @@ struct GemmKParams {
     int num_groups;
     int group_mode;           // 3: block-diagonal, no offsets (group g reads x at column g * group_ldx and writes out at column g * group_ldo)
     int group_ldx, group_ldo;
-    float act_limit, act_slope, act_shift;   // OVB_ACT_GLU_LIMITED
+    float act_limit, act_slope, act_shift;   // OVB_ACT_GLU_LIMITED; OVB_ACT_SOFTCAP: act_limit
 };
 
 // polls of a peer flag (~0.25 us apart) before a wait gives up: GemmKParams::spin_limit, set per launch from peer_spin_limit()
@@ -123,8 +123,8 @@ __device__ __forceinline__ __half from_float<__half>(float v) {
     return __float2half_rn(v);
 }
 
-__device__ __forceinline__ float apply_act(float v, int act) {
-    switch (act) {
+__device__ __forceinline__ float apply_act(float v, const GemmKParams& p) {
+    switch (p.act) {
         case OVB_ACT_GELU_ERF: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
         case OVB_ACT_RELU: return v > 0.f ? v : 0.f;
         case OVB_ACT_SILU: return v / (1.0f + __expf(-v));
@@ -132,6 +132,8 @@ __device__ __forceinline__ float apply_act(float v, int act) {
             float u = 0.7978845608028654f * (v + 0.044715f * v * v * v);
             return 0.5f * v * (1.0f + tanhf(u));
         }
+        case OVB_ACT_RELU2: return v > 0.f ? v * v : 0.f;
+        case OVB_ACT_SOFTCAP: return p.act_limit * tanhf(v / p.act_limit);
         default: return v;
     }
 }
@@ -651,7 +653,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                           ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0) &&
                           out_col % 8 == 0 && (p.residual == nullptr || ((p.ldr % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.residual) & 15) == 0)));
         // plain 16-bit output of the larger tiles: straight from the accumulator's registers
-        const bool direct16 = OVB_GEMM_DIRECT && BT >= 128 && fast && p.act == OVB_ACT_NONE && p.residual == nullptr;
+        const bool direct16 = OVB_GEMM_DIRECT && BT >= 128 && fast && (p.act == OVB_ACT_NONE || p.act == OVB_ACT_RELU2) && p.residual == nullptr;
         // fp32 output of a tile inside N: the lanes of a warp hold 32 consecutive columns of a token, stored as they are
         const bool plain32 = !QUANT && p.world <= 1 && p.splits == 1 && p.out_f32 && n0 + TILE_N <= p.N && p.residual == nullptr && p.act == OVB_ACT_NONE;
         // fp32 staging keeps a single rounding (after the residual add): BT x 128 x 4 bytes <= 2 * STAGE_BYTES
@@ -1071,7 +1073,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             const int tok = t0 + col;
             if (tok < T_end && oc < p.N) {
                 v += bias_v;
-                v = apply_act(v, p.act);
+                v = apply_act(v, p);
                 if (p.residual) v += to_float(reinterpret_cast<const E*>(p.residual)[(size_t)tok * p.ldr + oc]);
                 if (p.out_f32)
                     reinterpret_cast<float*>(p.out)[(size_t)tok * p.ldo + out_col + oc] = v;
@@ -1101,7 +1103,11 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                     E* o = reinterpret_cast<E*>(p.out) + (size_t)(t0 + c0 + odd) * p.ldo + out_col + (oc & ~1);
 #pragma unroll
                     for (int j = 0; j < 16; j += 2) {
-                        const float v0 = __uint_as_float(r[j]) + bias_v, v1 = __uint_as_float(r[j + 1]) + bias_v;
+                        float v0 = __uint_as_float(r[j]) + bias_v, v1 = __uint_as_float(r[j + 1]) + bias_v;
+                        if (p.act == OVB_ACT_RELU2) {
+                            v0 = fmaxf(v0, 0.f) * v0;
+                            v1 = fmaxf(v1, 0.f) * v1;
+                        }
                         const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
                         E pair[2] = {from_float<E>(odd ? got : v0), from_float<E>(odd ? v1 : got)};
                         if (t0 + c0 + j + odd < T_end) *reinterpret_cast<uint32_t*>(o + (size_t)j * p.ldo) = *reinterpret_cast<uint32_t*>(pair);
@@ -1109,7 +1115,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 } else if (fast) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        stage_out[(c0 + j) * TILE_N + row] = apply_act(__uint_as_float(r[j]) + bias_v, p.act);
+                        stage_out[(c0 + j) * TILE_N + row] = apply_act(__uint_as_float(r[j]) + bias_v, p);
                 } else if (plain32) {
                     float* o = reinterpret_cast<float*>(p.out) + (size_t)(t0 + c0) * p.ldo + out_col + oc;
 #pragma unroll
@@ -1220,7 +1226,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                             if (oc4 + j < p.N) {
                                 float v = vv[j];
                                 if (p.bias) v += to_float(reinterpret_cast<const E*>(p.bias)[oc4 + j]);
-                                v = apply_act(v, p.act);
+                                v = apply_act(v, p);
                                 if (p.residual) v += to_float(reinterpret_cast<const E*>(p.residual)[(size_t)tok * p.ldr + oc4 + j]);
                                 vv[j] = v;
                             }

@@ -52,6 +52,8 @@ enum {
     OVB_ACT_GELU_TANH = 5,
     OVB_ACT_GLU_LIMITED = 6,   // rows of W as for SWIGLU; g = min(gate, act_limit), u = clamp(up, -act_limit, act_limit);
                                // out [T, N/2] = g * sigmoid(act_slope * g) * (u + act_shift)
+    OVB_ACT_RELU2 = 7,         // square of relu
+    OVB_ACT_SOFTCAP = 8,       // act_limit * tanh(v / act_limit)
 };
 
 typedef struct {
@@ -321,21 +323,43 @@ int ovb_comm_allreduce(const ovb_comm* c, void* data, int64_t n, int dtype, ovb_
 // h[r] = table[ids[r]] (fp32), x[r] = the same in the storage type (may be NULL).
 int ovb_stream_embed(const int* ids, const void* table, float* h, void* x, int rows, int cols, int vocab, int ldt, int ldh, int ldx, int dtype,
                      ovb_stream_t stream);
-// s = alpha * h[row_idx ? row_idx[r] : r] (+ y[r], fp32, may be NULL); out = s / sqrt(mean(s^2) + eps) * (w_offset + w) to h_out (fp32)
-// and / or x_out (storage type). h_out may be h when row_idx is NULL.
-int ovb_sum_rmsnorm(const float* h, const int* row_idx, const float* y, const float* w, float* h_out, void* x_out, int rows, int cols, int ldh, int ldy,
-                    int ldho, int ldx, float alpha, float w_offset, float eps, int dtype, ovb_stream_t stream);
+// s = alpha * h[src] (+ y[src], fp32, may be NULL), src = row_idx ? row_idx[r] : r; out = s / sqrt(mean(s^2) + eps) * (w_offset + w) to
+// h_out (fp32) and / or x_out (storage type); the same with w2 to x2_out; s itself to s_out. h_out and s_out may be h when row_idx is
+// NULL. Weights are padded with zeros to a multiple of four.
+typedef struct {
+    const float* h;
+    const int* row_idx;
+    const float* y;
+    const float* w;
+    const float* w2;
+    float* h_out;
+    float* s_out;
+    void* x_out;
+    void* x2_out;
+    int rows, cols, ldh, ldy, ldho, lds, ldx, ldx2, dtype;
+    float alpha, w_offset, eps;
+} ovb_sum_rmsnorm_args;
+int ovb_sum_rmsnorm(const ovb_sum_rmsnorm_args* a, ovb_stream_t stream);
 // g = min(gate, limit), u = clamp(up, -limit, limit); out = g * sigmoid(slope * g) * (u + shift); up starts up_off columns after gate.
 int ovb_glu_limited(const void* gu, void* out, int rows, int F, int up_off, int ldg, int ldo, float limit, float slope, float shift, int dtype,
                     ovb_stream_t stream);
 // fp32 products without tensor cores: out[b] = act(x[b] w[b]^T + bias[b]); s* = elements between batch members.
 int ovb_gemm_f32(const float* x, const float* w, const float* bias, float* out, int batch, long long sx, long long sw, long long sb, long long so, int T, int N,
-                 int K, int ldx, int ldw, int ldo, int act, ovb_stream_t stream);
+                 int K, int ldx, int ldw, int ldo, int act, float act_limit, ovb_stream_t stream);
 int ovb_argmax_f32(const float* logits, int ld, int rows, int vocab, void* out_ids, int ids_i32, float* out_max, ovb_stream_t stream);
 int ovb_sample_f32(const float* logits, int ld, int rows, int vocab, float temperature, int top_k, float top_p, uint64_t seed, const int* step, int* out_ids,
                    ovb_stream_t stream);
 
-// Query / key norms, rotary positions and cache rows of grouped-query attention (attention_heads.cu).
+// cos and sin of the rotation angles of every token: table[t, i] = (cos, sin)(positions[t] * inv_freq[i]) * mult, i < half.
+int ovb_rope_table(const int* positions, const float* inv_freq, float* table, int T, int half, float mult, ovb_stream_t stream);
+
+// Short causal convolutions (short_conv.cuh): the inputs of a step, proj [T, ldp] columns 0 .. cols, go to the rings of their slots. Only
+// for steps with more than one token per sequence; the kernels below do it themselves when max_q_len is 1.
+int ovb_conv_ring_update(const void* proj, float* ring, const int* subsequence_begins, const int* past_lens, const int* slots, int B, int cols, int taps, int ldp,
+                         int dtype, ovb_stream_t stream);
+
+// Short convolution, query / key norms, rotary positions, value mixing and cache rows of grouped-query attention (attention_heads.cu).
+// With taps > 0 every column of q, k and v passes the convolution first and the queries go to q_out (not their place in proj).
 typedef struct {
     void* proj;              // [T, ldp]: H query heads (pitch dk_pad), G key heads at k_off (pitch dk_pad), G value heads at v_off (pitch dv_pad)
     void* k_cache;           // [blocks, G, block_size, dk_pad]
@@ -347,6 +371,16 @@ typedef struct {
     const int* slot_map;
     int T, H, G, D, Dv, dk_pad, dv_pad, ldp, k_off, v_off, block_size, rot_dims, dtype;
     float rot_mult, eps;
+    const float* rope;       // [T, rot_dims / 2] (cos, sin) pairs (ovb_rope_table), or NULL: computed here
+    void* q_out;             // [T, ldq], heads at a pitch of dk_pad; NULL: in place
+    const float* conv_w;     // [taps, conv_cols]: a channel is a column of proj
+    float* conv_ring;        // [slots, taps, conv_cols]
+    const int* subsequence_begins;
+    const int* past_lens;
+    const int* slots;
+    void* v_first;           // [T, ld_vf] values (heads of Dv columns) that later layers mix in, or NULL
+    int B, taps, conv_cols, ldq, ld_vf, v_mode, max_q_len;      // v_mode 1: write v_first, 2: v <- (1 - v_mix) v + v_mix v_first
+    float v_mix;
 } ovb_heads_args;
 int ovb_heads_prepare(const ovb_heads_args* a, ovb_stream_t stream);
 
@@ -366,8 +400,10 @@ typedef struct {
 int ovb_latent_prepare(const ovb_latent_args* a, ovb_stream_t stream);
 
 // Causal attention over a paged cache with key and value sizes of their own, an optional sliding window (a position sees itself and
-// the window - 1 positions before it; 0 = off) and an optional sigmoid gate on the output. Key rows: ((block * Hkv + kv head) *
-// block_size + slot) * k_row, value rows likewise with v_row (v may point into the key rows).
+// the window - 1 positions before it; 0 = off), optional chunks (a position sees only its own chunk of `chunk` positions counted from
+// position 0; 0 = off), an optional sink per query head (exp(sink) joins the softmax denominator) and an optional sigmoid gate on the
+// output, per column or per head. Key rows: ((block * Hkv + kv head) * block_size + slot) * k_row, value rows likewise with v_row (v may
+// point into the key rows).
 typedef struct {
     const void* q;            // + t * ldq + head * q_head
     const void* k;
@@ -386,6 +422,8 @@ typedef struct {
     float scale;
     int exact;                // 1: fp32 arithmetic throughout (no tensor cores)
     int cache_rows;           // rows of k (and of v), 0: not known
+    int chunk, gate_scalar;   // gate_scalar 1: one gate value per head
+    const float* sink;        // [Hq] or NULL
 } ovb_wattn_args;
 int ovb_window_attention(const ovb_wattn_args* a, ovb_stream_t stream);
 
@@ -433,6 +471,29 @@ typedef struct {
 } ovb_rglru_args;
 int ovb_causal_conv(const ovb_rglru_args* a, ovb_stream_t stream);
 int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream);
+
+// Gated delta rule with a decay per key channel, from the projections to the heads that the output projection reads (delta_rule.cu).
+// Per head: q, k, v pass their short convolution and silu; q and k become unit vectors (q also times q_scale);
+// g = exp(-decay_a * softplus(low + dt_bias)); S <- g S; S <- S + k (beta (v - S^T k))^T; o = S^T q; out = rms_norm(o) * norm * sigmoid(gate).
+// Everything behind the convolutions is fp32. D and Dv are the true sizes, dk and dv the pitches of heads (multiples of 16, zeros in
+// projections, convolution weights and norm behind the true size).
+typedef struct {
+    const void* proj;        // [T, ldp]: G query heads at column 0, G key heads at k_off, H value heads at v_off, H beta logits at b_off
+    const float* low;        // [T, ld_low]: decay inputs [H, dk] at column 0, output gate logits [H, dv] at gate_off
+    const float* conv_w;     // [taps, conv_cols]: a channel is a column of proj
+    float* conv_ring;        // [slots, taps, conv_cols]
+    const float* decay_a;    // [H]
+    const float* dt_bias;    // [H, dk]
+    const float* norm;       // [dv]
+    float* state;            // [slots, H, dk, dv]
+    void* out;               // [T, ldo], heads at a pitch of o_head
+    const int* subsequence_begins;
+    const int* past_lens;
+    const int* slots;
+    int B, T, H, G, D, Dv, dk, dv, ldp, k_off, v_off, b_off, ld_low, gate_off, conv_cols, taps, ldo, o_head, max_q_len, dtype;
+    float q_scale, eps;
+} ovb_delta_args;
+int ovb_channel_delta(const ovb_delta_args* a, ovb_stream_t stream);
 
 #ifdef __cplusplus
 }

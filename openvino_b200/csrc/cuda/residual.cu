@@ -1,4 +1,5 @@
-// A residual stream kept in fp32: token embedding, "sum, then norm" and the clamped gated MLP activation.
+// A residual stream kept in fp32: token embedding, "sum, then norm" (one or two norms of the same sum) and the clamped gated MLP
+// activation.
 //
 // The stream h is [rows, ldh] fp32; x is the copy of it in the storage type of the matrix products (bf16, or none when the
 // products themselves run in fp32 and read h). Row pitches are multiples of four elements; columns between the width and
@@ -33,15 +34,14 @@ __global__ void stream_embed_kernel(const int* __restrict__ ids, const E* __rest
     }
 }
 
-// s = alpha * h[src row] (+ y);  out = s / sqrt(mean(s^2) + eps) * (w_offset + w).  One CTA per row, the row stays in registers.
+// s = alpha * h[src row] (+ y[src row]);  out = s / sqrt(mean(s^2) + eps) * (w_offset + w), for up to two weights.  One CTA per row,
+// the row stays in registers.
 template <class E, int MAXV>
-__global__ void __launch_bounds__(kNormThreads)
-sum_rmsnorm_kernel(const float* __restrict__ h, const int* __restrict__ row_idx, const float* __restrict__ y, const float* __restrict__ w, float* h_out,
-                   E* __restrict__ x_out, int cols, int ldh, int ldy, int ldho, int ldx, float alpha, float w_offset, float eps) {
+__global__ void __launch_bounds__(kNormThreads) sum_rmsnorm_kernel(ovb_sum_rmsnorm_args p) {
     pdl_enter();
     __shared__ float red[kNormThreads / 32];
-    const int row = blockIdx.x, src = row_idx ? row_idx[row] : row;
-    const int nvec = (cols + 3) / 4;
+    const int row = blockIdx.x, src = p.row_idx ? p.row_idx[row] : row;
+    const int nvec = (p.cols + 3) / 4;
     float4 v[MAXV];
     float ss = 0.f;
 #pragma unroll
@@ -49,10 +49,10 @@ sum_rmsnorm_kernel(const float* __restrict__ h, const int* __restrict__ row_idx,
         const int k = threadIdx.x + i * kNormThreads;
         v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (k < nvec) {
-            const float4 a = ld4_f32(h + (size_t)src * ldh + k * 4);
-            v[i] = make_float4(alpha * a.x, alpha * a.y, alpha * a.z, alpha * a.w);
-            if (y) {
-                const float4 b = ld4_f32(y + (size_t)row * ldy + k * 4);
+            const float4 a = ld4_f32(p.h + (size_t)src * p.ldh + k * 4);
+            v[i] = make_float4(p.alpha * a.x, p.alpha * a.y, p.alpha * a.z, p.alpha * a.w);
+            if (p.y) {
+                const float4 b = ld4_f32(p.y + (size_t)src * p.ldy + k * 4);
                 v[i].x += b.x; v[i].y += b.y; v[i].z += b.z; v[i].w += b.w;
             }
             ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
@@ -65,16 +65,23 @@ sum_rmsnorm_kernel(const float* __restrict__ h, const int* __restrict__ row_idx,
     float tot = 0.f;
 #pragma unroll
     for (int i = 0; i < kNormThreads / 32; ++i) tot += red[i];
-    const float inv = 1.f / sqrtf(tot / (float)cols + eps);
+    const float inv = 1.f / sqrtf(tot / (float)p.cols + p.eps);
+    E* x_out = reinterpret_cast<E*>(p.x_out);
+    E* x2_out = reinterpret_cast<E*>(p.x2_out);
 #pragma unroll
     for (int i = 0; i < MAXV; ++i) {
         const int k = threadIdx.x + i * kNormThreads;
         if (k < nvec) {
-            const float4 g = ld4_f32(w + k * 4);
-            const float4 o = make_float4(v[i].x * inv * (w_offset + g.x), v[i].y * inv * (w_offset + g.y), v[i].z * inv * (w_offset + g.z),
-                                         v[i].w * inv * (w_offset + g.w));
-            if (h_out) st4_f32(h_out + (size_t)row * ldho + k * 4, o);
-            if (x_out) st4_f32(x_out + (size_t)row * ldx + k * 4, o);
+            if (p.s_out) st4_f32(p.s_out + (size_t)row * p.lds + k * 4, v[i]);
+            auto weighted = [&](const float* w) {
+                const float4 g = ld4_f32(w + k * 4);
+                return make_float4(v[i].x * inv * (p.w_offset + g.x), v[i].y * inv * (p.w_offset + g.y), v[i].z * inv * (p.w_offset + g.z),
+                                   v[i].w * inv * (p.w_offset + g.w));
+            };
+            const float4 o = weighted(p.w);
+            if (p.h_out) st4_f32(p.h_out + (size_t)row * p.ldho + k * 4, o);
+            if (x_out) st4_f32(x_out + (size_t)row * p.ldx + k * 4, o);
+            if (x2_out) st4_f32(x2_out + (size_t)row * p.ldx2 + k * 4, weighted(p.w2));
         }
     }
 }
@@ -95,20 +102,18 @@ __global__ void glu_limited_kernel(const E* __restrict__ gu, E* __restrict__ out
 }
 
 template <class E>
-int launch_sum_rmsnorm(const float* h, const int* row_idx, const float* y, const float* w, float* h_out, E* x_out, int rows, int cols, int ldh, int ldy,
-                       int ldho, int ldx, float alpha, float w_offset, float eps, cudaStream_t stream) {
+int launch_sum_rmsnorm(const ovb_sum_rmsnorm_args& a, cudaStream_t stream) {
     auto go = [&](auto kern) -> int {
-        OVB_CHECK_CUDA(launch_pdl(kern, dim3(rows), dim3(kNormThreads), 0, stream, h, row_idx, y, w, h_out, x_out, cols, ldh, ldy, ldho, ldx, alpha,
-                                  w_offset, eps));
+        OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.rows), dim3(kNormThreads), 0, stream, a));
         return 0;
     };
-    const int per = ceil_div(ceil_div(cols, 4), kNormThreads);
+    const int per = ceil_div(ceil_div(a.cols, 4), kNormThreads);
     if (per <= 1) return go(sum_rmsnorm_kernel<E, 1>);
     if (per <= 2) return go(sum_rmsnorm_kernel<E, 2>);
     if (per <= 4) return go(sum_rmsnorm_kernel<E, 4>);
     if (per <= 8) return go(sum_rmsnorm_kernel<E, 8>);
     if (per <= 16) return go(sum_rmsnorm_kernel<E, 16>);
-    set_error("ovb_sum_rmsnorm: width %d above %d", cols, 16 * 4 * kNormThreads);
+    set_error("ovb_sum_rmsnorm: width %d above %d", a.cols, 16 * 4 * kNormThreads);
     return ERR_UNSUPPORTED;
 }
 
@@ -130,13 +135,13 @@ int ovb_stream_embed(const int* ids, const void* table, float* h, void* x, int r
     });
 }
 
-int ovb_sum_rmsnorm(const float* h, const int* row_idx, const float* y, const float* w, float* h_out, void* x_out, int rows, int cols, int ldh, int ldy,
-                    int ldho, int ldx, float alpha, float w_offset, float eps, int dtype, ovb_stream_t stream) {
-    OVB_REQUIRE(h && w && (h_out || x_out) && rows > 0 && cols > 0, "ovb_sum_rmsnorm: bad arguments");
-    OVB_REQUIRE(ldh % 4 == 0 && ldy % 4 == 0 && ldho % 4 == 0 && ldx % 4 == 0, "ovb_sum_rmsnorm: row pitches must be multiples of 4 elements");
-    return dispatch_store(dtype, "ovb_sum_rmsnorm", [&](auto e) -> int {
+int ovb_sum_rmsnorm(const ovb_sum_rmsnorm_args* a, ovb_stream_t stream) {
+    OVB_REQUIRE(a && a->h && a->w && (a->h_out || a->x_out) && a->rows > 0 && a->cols > 0 && (a->x2_out == nullptr || a->w2), "ovb_sum_rmsnorm: bad arguments");
+    OVB_REQUIRE(a->ldh % 4 == 0 && a->ldy % 4 == 0 && a->ldho % 4 == 0 && a->lds % 4 == 0 && a->ldx % 4 == 0 && a->ldx2 % 4 == 0,
+                "ovb_sum_rmsnorm: row pitches must be multiples of 4 elements");
+    return dispatch_store(a->dtype, "ovb_sum_rmsnorm", [&](auto e) -> int {
         using E = decltype(e);
-        return launch_sum_rmsnorm<E>(h, row_idx, y, w, h_out, (E*)x_out, rows, cols, ldh, ldy, ldho, ldx, alpha, w_offset, eps, (cudaStream_t)stream);
+        return launch_sum_rmsnorm<E>(*a, (cudaStream_t)stream);
     });
 }
 

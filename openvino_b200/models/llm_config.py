@@ -54,7 +54,7 @@ NAMED = {c.name: c for c in (LLAMA3_8B, LLAMA3_70B, MIXTRAL_8X7B, TINY_LLAMA, TI
 
 # ----------------------------------------------------------------------------------------- layered decoders
 # A decoder whose layers are listed one by one: every layer names its token mixer and its feed-forward, each with sizes of its
-# own. The residual stream is fp32. The serving program of these configurations is runtime/layered_llm.py.
+# own. The residual stream is fp32; how sublayers and norms meet it is the configuration's ``block``. The serving program of these configurations is runtime/layered_llm.py.
 @dataclass(frozen=True)
 class RotarySpec:
     """Rotation of the first ``dims`` dimensions by the position (dimension i paired with i + dims / 2). ``yarn`` = (factor,
@@ -83,7 +83,8 @@ class RotarySpec:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Grouped-query attention; ``window`` 0 = full causal attention, else a position sees itself and window - 1 before it."""
+    """Grouped-query attention; ``window`` 0 = full causal attention, else a position sees itself and window - 1 before it;
+    ``chunk`` > 0: a position sees only keys of its own chunk of that many positions, counted from position 0."""
     heads: int
     kv_heads: int
     dim: int
@@ -93,6 +94,15 @@ class AttentionSpec:
     qk_norm: bool = False          # RMS norm of every query / key head, one weight of size dim for all heads
     gated: bool = False            # heads times sigmoid(W_g x) before the output projection
     rotary: Optional[RotarySpec] = None
+    head_gate: bool = False        # the gate is one number per head instead of one per column
+    chunk: int = 0
+    sink: bool = False             # exp(sink), a number per head, joins the softmax denominator
+    taps: int = 0                  # > 0: short causal convolution on every column of q, k and v, ahead of the rotation
+    v_mix: bool = False            # values are mixed with those of the first layer that has this set
+
+    @property
+    def carries_state(self) -> bool:
+        return self.taps > 1
 
 
 @dataclass(frozen=True)
@@ -107,6 +117,22 @@ class LatentAttentionSpec:
     scale: float
     rotary: RotarySpec
     window: int = 0
+    carries_state = False
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """Gated delta rule with a decay per head and key channel, short convolutions with silu on q, k and v, unit-norm queries and keys, a
+    norm and a low-rank sigmoid gate on every head's read-out. ``decay_rank`` / ``gate_rank``: inner sizes of the two low-rank
+    projections, 0 = whatever the checkpoint's tensors have."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int = 0
+    gate_rank: int = 0
+    carries_state = True
 
 
 @dataclass(frozen=True)
@@ -116,6 +142,7 @@ class RgLruSpec:
     blocks: int
     taps: int
     decay: float = 8.0             # log a = -decay * r * softplus(lambda)
+    carries_state = True
 
 
 @dataclass(frozen=True)
@@ -128,21 +155,35 @@ class LimitedGluSpec:
 
 
 @dataclass(frozen=True)
+class SquaredReluSpec:
+    """W_down relu(W_up x)^2."""
+    ff: int
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec, RgLruSpec]
-    mlp: Optional[LimitedGluSpec] = None
+    mixer: Union[AttentionSpec, LatentAttentionSpec, RgLruSpec, ChannelDeltaSpec]
+    mlp: Optional[Union[LimitedGluSpec, SquaredReluSpec]] = None
+
+
+# How a layer meets the residual stream x.
+POST_NORM = "post_norm"            # x <- norm1(scale * x + mixer(x)), then x <- norm2(scale * x + mlp(x))
+PARALLEL_NORM = "parallel_norm"    # x <- x + mixer(norm1(x)) + mlp(norm2(x))
 
 
 @dataclass(frozen=True)
 class LayeredConfig:
-    """Layers with the norm after each sum: x <- norm(residual_scale * x + sublayer(x)), norm weight = norm_offset + stored."""
+    """Layers in one of the two forms above; a norm's weight is norm_offset + what is stored."""
     name: str
     vocab_size: int
     hidden_size: int
     layers: Tuple[LayerSpec, ...]
     norm_eps: float = 1e-5
-    residual_scale: float = 1.0
+    residual_scale: float = 1.0    # POST_NORM only
     norm_offset: float = 0.0
+    block: str = POST_NORM
+    embed_norm: bool = False       # the embedding passes a norm of its own
+    logit_softcap: float = 0.0     # > 0: logits <- cap * tanh(logits / cap)
 
     @property
     def num_layers(self) -> int:
@@ -150,4 +191,5 @@ class LayeredConfig:
 
     @property
     def has_recurrent_state(self) -> bool:
-        return any(isinstance(l.mixer, RgLruSpec) for l in self.layers)
+        """True when a request holds state that is not rows of the paged cache."""
+        return any(l.mixer.carries_state for l in self.layers)

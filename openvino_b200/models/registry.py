@@ -10,7 +10,7 @@ from dataclasses import dataclass
 from typing import Callable, Dict
 
 from ..utils.safetensors import SafetensorsFile
-from . import busatar
+from . import busatar, sapasun
 from .llm_config import LayeredConfig
 
 
@@ -21,7 +21,8 @@ class Architecture:
     tensor_shapes: Callable[[LayeredConfig], dict]
 
 
-ARCHITECTURES: Dict[str, Architecture] = {"Busatar": Architecture(busatar.read_config, busatar.tensor_name, busatar.tensor_shapes)}
+ARCHITECTURES: Dict[str, Architecture] = {"Busatar": Architecture(busatar.read_config, busatar.tensor_name, busatar.tensor_shapes),
+                                          "Sapasun": Architecture(sapasun.read_config, sapasun.tensor_name, sapasun.tensor_shapes)}
 
 
 def register(name: str, arch: Architecture) -> None:
@@ -44,8 +45,9 @@ class Checkpoint:
             t = self.tensors[name]
         except KeyError:
             raise KeyError("the checkpoint has no tensor '%s'" % name) from None
-        if tuple(t.shape) != tuple(self._shapes[name]):
-            raise ValueError("tensor '%s' has the shape %s, its configuration asks for %s" % (name, tuple(t.shape), tuple(self._shapes[name])))
+        want = tuple(self._shapes[name])      # None: a size that the configuration leaves to the tensor
+        if len(t.shape) != len(want) or any(w is not None and n != w for n, w in zip(t.shape, want)):
+            raise ValueError("tensor '%s' has the shape %s, its configuration asks for %s" % (name, tuple(t.shape), want))
         return t
 
 

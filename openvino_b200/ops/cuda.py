@@ -22,7 +22,7 @@ _LIB_PATH = Path(os.environ["OVB_CUDA_LIB"]) if os.environ.get("OVB_CUDA_LIB") e
 W_BF16, W_U4, W_U8, W_F16, W_F8 = 0, 1, 2, 3, 4
 W_F32 = 16                     # fp32 weights: products without tensor cores (ovb_gemm_f32)
 DT_F32, DT_BF16 = 0, 2         # storage types of the layered decoders' kernels
-ACT_NONE, ACT_GELU_ERF, ACT_RELU, ACT_SILU, ACT_SWIGLU, ACT_GELU_TANH, ACT_GLU_LIMITED = 0, 1, 2, 3, 4, 5, 6
+ACT_NONE, ACT_GELU_ERF, ACT_RELU, ACT_SILU, ACT_SWIGLU, ACT_GELU_TANH, ACT_GLU_LIMITED, ACT_RELU2, ACT_SOFTCAP = 0, 1, 2, 3, 4, 5, 6, 7, 8
 
 STATUS_NAMES = {0: "ok", 1: "mbarrier wait timed out", 2: "peer flag wait timed out", 3: "bad argument seen on device",
                 4: "local flag wait timed out", 5: "index out of range (debug build; the access was skipped)"}
@@ -62,7 +62,9 @@ def _fields(pointers, ints, floats=()):
 
 class HeadsArgs(C.Structure):
     _fields_ = _fields(("proj", "k_cache", "v_cache", "q_norm", "k_norm", "inv_freq", "positions", "slot_map"),
-                       ("T", "H", "G", "D", "Dv", "dk_pad", "dv_pad", "ldp", "k_off", "v_off", "block_size", "rot_dims", "dtype"), ("rot_mult", "eps"))
+                       ("T", "H", "G", "D", "Dv", "dk_pad", "dv_pad", "ldp", "k_off", "v_off", "block_size", "rot_dims", "dtype"), ("rot_mult", "eps")) + \
+        _fields(("rope", "q_out", "conv_w", "conv_ring", "subsequence_begins", "past_lens", "slots", "v_first"),
+                ("B", "taps", "conv_cols", "ldq", "ld_vf", "v_mode", "max_q_len"), ("v_mix",))
 
 
 class LatentArgs(C.Structure):
@@ -75,7 +77,19 @@ class WindowAttnArgs(C.Structure):
     _fields_ = (_fields(("q", "k", "v", "out", "gate", "past_lens", "subsequence_begins", "block_indices", "block_indices_begins", "scratch"), ())
                 + [("scratch_bytes", C.c_longlong)]
                 + _fields((), ("B", "T", "Hq", "Hkv", "Dk", "Dv", "ldq", "q_head", "k_row", "v_row", "ldo", "o_head", "ld_gate", "gate_head", "block_size",
-                               "window", "max_context_len", "max_q_len", "dtype"), ("scale",)) + [("exact", C.c_int), ("cache_rows", C.c_int)])
+                               "window", "max_context_len", "max_q_len", "dtype"), ("scale",))
+                + _fields((), ("exact", "cache_rows", "chunk", "gate_scalar")) + _fields(("sink",), ()))
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = _fields(("proj", "low", "conv_w", "conv_ring", "decay_a", "dt_bias", "norm", "state", "out", "subsequence_begins", "past_lens", "slots"),
+                       ("B", "T", "H", "G", "D", "Dv", "dk", "dv", "ldp", "k_off", "v_off", "b_off", "ld_low", "gate_off", "conv_cols", "taps", "ldo", "o_head",
+                        "max_q_len", "dtype"), ("q_scale", "eps"))
+
+
+class SumNormArgs(C.Structure):
+    _fields_ = _fields(("h", "row_idx", "y", "w", "w2", "h_out", "s_out", "x_out", "x2_out"),
+                       ("rows", "cols", "ldh", "ldy", "ldho", "lds", "ldx", "ldx2", "dtype"), ("alpha", "w_offset", "eps"))
 
 
 class LatentPrefillArgs(C.Structure):
@@ -284,18 +298,18 @@ class PackedWeight:
 # ------------------------------------------------------------------------------------------ ops
 def gemm(x: torch.Tensor, w: PackedWeight, out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None,
          act: int = ACT_NONE, out_f32: bool = False, ws: Optional[Workspace] = None, splits: int = 0,
-         block_t: int = 0, comm=None, glu=None) -> torch.Tensor:
+         block_t: int = 0, comm=None, glu=None, cap: float = 0.0) -> torch.Tensor:
     """out[T, N] = act(x[T, K] @ dequant(W)^T + bias) + residual  on the tcgen05 GEMM.
 
     ``comm`` (a ``parallel.comm.CommStruct``): sum the product over the tensor-parallel ranks inside the epilogue.
-    ``glu`` (limit, slope, shift): parameters of ``ACT_GLU_LIMITED``. fp32 weights (``W_F32``) take the product without
+    ``glu`` (limit, slope, shift): parameters of ``ACT_GLU_LIMITED``; ``cap``: bound of ``ACT_SOFTCAP``. fp32 weights (``W_F32``) take the product without
     tensor cores; ``x`` and ``out`` are then fp32."""
     assert x.dim() == 2 and x.stride(1) == 1
     T, K = x.shape
     assert K == w.K, (K, w.K)
     if w.mode == W_F32:
         assert residual is None and comm is None
-        return _gemm_f32(x, w, out, act)
+        return _gemm_f32(x, w, out, act, cap)
     if out is None:
         out = torch.empty((T, w.N // 2 if act in (ACT_SWIGLU, ACT_GLU_LIMITED) else w.N), dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
     if ws is None:
@@ -317,17 +331,19 @@ def gemm(x: torch.Tensor, w: PackedWeight, out: Optional[torch.Tensor] = None, r
     a.comm = C.addressof(comm) if comm is not None else None
     if act == ACT_GLU_LIMITED:
         a.act_limit, a.act_slope, a.act_shift = glu
+    elif act == ACT_SOFTCAP:
+        a.act_limit = cap
     _check(lib().ovb_gemm(C.byref(a), C.c_void_p(_stream())), "ovb_gemm")
     return out
 
 
-def _gemm_f32(x: torch.Tensor, w: "PackedWeight", out: Optional[torch.Tensor], act: int = ACT_NONE) -> torch.Tensor:
+def _gemm_f32(x: torch.Tensor, w: "PackedWeight", out: Optional[torch.Tensor], act: int = ACT_NONE, limit: float = 0.0) -> torch.Tensor:
     T, K = x.shape
     if out is None:
         out = torch.empty((T, w.N), dtype=torch.float32, device=x.device)
     _check(lib().ovb_gemm_f32(C.c_void_p(x.data_ptr()), C.c_void_p(w.w.data_ptr()), C.c_void_p(_ptr(w.bias)), C.c_void_p(out.data_ptr()), C.c_int(1),
                               C.c_longlong(0), C.c_longlong(0), C.c_longlong(0), C.c_longlong(0), C.c_int(T), C.c_int(w.N), C.c_int(K), C.c_int(x.stride(0)),
-                              C.c_int(K), C.c_int(out.stride(0)), C.c_int(act), C.c_void_p(_stream())), "ovb_gemm_f32")
+                              C.c_int(K), C.c_int(out.stride(0)), C.c_int(act), C.c_float(limit), C.c_void_p(_stream())), "ovb_gemm_f32")
     return out
 
 
@@ -354,8 +370,8 @@ def gemm_block_diag(x: torch.Tensor, w: BlockDiagWeight, out: torch.Tensor, x_pi
     if w.mode == W_F32:
         _check(lib().ovb_gemm_f32(C.c_void_p(x.data_ptr()), C.c_void_p(w.w.data_ptr()), C.c_void_p(None), C.c_void_p(out.data_ptr()), C.c_int(w.G),
                                   C.c_longlong(x_pitch), C.c_longlong(w.N * w.K), C.c_longlong(0), C.c_longlong(out_pitch), C.c_int(T), C.c_int(w.N),
-                                  C.c_int(w.K), C.c_int(x.stride(0)), C.c_int(w.K), C.c_int(out.stride(0)), C.c_int(ACT_NONE), C.c_void_p(_stream())),
-               "ovb_gemm_f32 (block-diagonal)")
+                                  C.c_int(w.K), C.c_int(x.stride(0)), C.c_int(w.K), C.c_int(out.stride(0)), C.c_int(ACT_NONE), C.c_float(0.0),
+                                  C.c_void_p(_stream())), "ovb_gemm_f32 (block-diagonal)")
         return out
     if ws is None:
         ws = default_workspace(x.device)
@@ -382,15 +398,37 @@ def stream_embed(ids, table, h, x=None):
                                   C.c_int(storage_type(table.dtype)), C.c_void_p(_stream())), "ovb_stream_embed")
 
 
-def sum_rmsnorm(h, w, eps, cols, rows=None, y=None, alpha=1.0, w_offset=0.0, h_out=None, x_out=None, row_idx=None):
-    """s = alpha * h (+ y); s / sqrt(mean(s^2) + eps) * (w_offset + w) to ``h_out`` (fp32) and / or ``x_out``. ``w`` is padded with
-    zeros to a multiple of four; ``row_idx`` gathers rows of h."""
-    rows = (row_idx if row_idx is not None else h).shape[0] if rows is None else rows
-    ld = lambda t: C.c_int(t.stride(0) if t is not None else 0)
-    _check(lib().ovb_sum_rmsnorm(C.c_void_p(h.data_ptr()), C.c_void_p(_ptr(row_idx)), C.c_void_p(_ptr(y)), C.c_void_p(w.data_ptr()), C.c_void_p(_ptr(h_out)),
-                                 C.c_void_p(_ptr(x_out)), C.c_int(rows), C.c_int(cols), ld(h), ld(y), ld(h_out), ld(x_out), C.c_float(alpha), C.c_float(w_offset),
-                                 C.c_float(eps), C.c_int(storage_type(x_out.dtype if x_out is not None else torch.float32)), C.c_void_p(_stream())),
-           "ovb_sum_rmsnorm")
+def sum_rmsnorm(h, w, eps, cols, y=None, alpha=1.0, w_offset=0.0, h_out=None, x_out=None, row_idx=None, s_out=None, w2=None, x2_out=None):
+    """s = alpha * h (+ y); s / sqrt(mean(s^2) + eps) * (w_offset + w) to ``h_out`` (fp32) and / or ``x_out``, the same with ``w2`` to
+    ``x2_out``, s itself to ``s_out``. Weights are padded with zeros to a multiple of four; ``row_idx`` gathers rows of h and y."""
+    a = SumNormArgs()
+    for name, t, ld in (("h", h, "ldh"), ("y", y, "ldy"), ("h_out", h_out, "ldho"), ("s_out", s_out, "lds"), ("x_out", x_out, "ldx"), ("x2_out", x2_out, "ldx2")):
+        if t is not None:
+            setattr(a, name, t.data_ptr())
+            setattr(a, ld, t.stride(0))
+    a.row_idx, a.w, a.w2 = _ptr(row_idx), w.data_ptr(), _ptr(w2)
+    a.rows, a.cols = (row_idx if row_idx is not None else h).shape[0], cols
+    a.dtype = storage_type(x_out.dtype if x_out is not None else torch.float32)
+    a.alpha, a.w_offset, a.eps = alpha, w_offset, eps
+    _check(lib().ovb_sum_rmsnorm(C.byref(a), C.c_void_p(_stream())), "ovb_sum_rmsnorm")
+
+
+def rope_table(positions, inv_freq, out, mult=1.0) -> None:
+    """out[t, i] = (cos, sin)(positions[t] * inv_freq[i]) * mult; out: fp32 [T, 2 * half]."""
+    _check(lib().ovb_rope_table(C.c_void_p(positions.data_ptr()), C.c_void_p(inv_freq.data_ptr()), C.c_void_p(out.data_ptr()), C.c_int(out.shape[0]),
+                                C.c_int(inv_freq.numel()), C.c_float(mult), C.c_void_p(_stream())), "ovb_rope_table")
+
+
+def conv_ring_update(proj, ring, subsequence_begins, past_lens, slots, B) -> None:
+    """Last taps - 1 inputs of every sequence of a step -> ``ring`` [slots, taps, cols] (columns 0 .. cols of ``proj``)."""
+    _check(lib().ovb_conv_ring_update(C.c_void_p(proj.data_ptr()), C.c_void_p(ring.data_ptr()), C.c_void_p(subsequence_begins.data_ptr()),
+                                      C.c_void_p(past_lens.data_ptr()), C.c_void_p(slots.data_ptr()), C.c_int(B), C.c_int(ring.shape[2]), C.c_int(ring.shape[1]),
+                                      C.c_int(proj.stride(0)), C.c_int(storage_type(proj.dtype)), C.c_void_p(_stream())), "ovb_conv_ring_update")
+
+
+def channel_delta(**kw) -> None:
+    """Gated delta rule with a decay per key channel, from projections to gated heads; fields of ``ovb_delta_args``."""
+    _check(lib().ovb_channel_delta(C.byref(_fill(DeltaArgs(), kw)), C.c_void_p(_stream())), "ovb_channel_delta")
 
 
 def glu_limited(gu, out, F, up_off, limit, slope=1.702, shift=1.0):

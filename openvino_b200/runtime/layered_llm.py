@@ -1,9 +1,11 @@
 """Serving program of layered decoders (``LayeredConfig``): every layer is a token mixer and an optional feed-forward with sizes of
-their own, the residual stream is fp32 and each sum is followed by a norm.
+their own on an fp32 residual stream. Either each sum is followed by a norm (``POST_NORM``), or mixer and feed-forward read two norms of
+the same stream and are added to it together (``PARALLEL_NORM``); their output projections are then one product over the concatenated
+heads and activations.
 
 The executor shares step descriptors, paging, CUDA graphs, sampling and token feedback with the other programs (``LlmExecutor``)
 and adds per-layer caches: key / value pages of grouped-query attention, one row per token of latent attention, and fp32
-recurrent state per request slot. Matrix products and activations are bf16 (fp32 accumulation), or everything is fp32 with
+recurrent state and inputs of short convolutions per request slot. Matrix products and activations are bf16 (fp32 accumulation), or everything is fp32 with
 ``dtype=torch.float32``.
 
 Layout rules. Row pitches are multiples of 64 elements and heads are padded to 16, so that the tensor-core kernels read whole
@@ -15,7 +17,8 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..models.llm_config import AttentionSpec, LatentAttentionSpec, LayeredConfig, LimitedGluSpec, RgLruSpec, RotarySpec
+from ..models.llm_config import (PARALLEL_NORM, AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, LayeredConfig, LimitedGluSpec, RgLruSpec, RotarySpec,
+                                 SquaredReluSpec)
 from ..models.registry import Checkpoint
 from ..ops import cuda as K
 from .cuda_llm import LlmExecutor, StepBuffers, StepShape
@@ -65,55 +68,99 @@ class _Rotation:
     def __init__(self, rot: Optional[RotarySpec], device):
         self.dims = rot.dims if rot else 0
         self.mult = rot.multiplier() if rot else 1.0
-        self.inv_freq = torch.tensor(rot.inv_freq(), dtype=torch.float64).float().to(device) if rot else None
+        self.freq = tuple(rot.inv_freq()) if rot else ()
+        self.inv_freq = torch.tensor(self.freq, dtype=torch.float64).float().to(device) if rot else None
 
     def args(self) -> dict:
         return dict(rot_dims=self.dims, rot_mult=self.mult, inv_freq=self.inv_freq)
 
 
+class _ShortConv:
+    """Filters of short causal convolutions on the first columns of a projection, and the ring of inputs of every request slot."""
+
+    def __init__(self, filters: List[torch.Tensor]):
+        self.w = torch.cat([f.float() for f in filters], 0).t().contiguous()      # [taps, columns]
+        self.taps, self.cols = self.w.shape
+
+    def allocate(self, ex: "LayeredExecutor") -> None:
+        self.ring = torch.zeros((ex.num_slots, self.taps, self.cols), dtype=torch.float32, device=ex.device)
+
+    def args(self, sb: "LayeredStepBuffers", shp: StepShape) -> dict:
+        return dict(conv_w=self.w, conv_ring=self.ring, conv_cols=self.cols, taps=self.taps, subsequence_begins=sb.view("subsequence_begins"),
+                    past_lens=sb.view("past_lens"), slots=sb.view("state_slots"), B=shp.B, max_q_len=shp.max_q_len)
+
+    def advance(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, proj: torch.Tensor) -> None:
+        """Behind the kernel that convolves: the step's last inputs go to the rings (a decode step's kernel does that itself)."""
+        if shp.max_q_len > 1 and self.taps > 1:
+            K.conv_ring_update(proj, self.ring, sb.view("subsequence_begins"), sb.view("past_lens"), sb.view("state_slots"), shp.B)
+            ex.kernel_launches += 1
+
+
+# A mixer's ``run`` writes the columns that the output projection ``out_weight`` [width, columns] reads; a feed-forward likewise.
 class AttentionMixer:
-    """Grouped-query attention: one product for q, k, v and the gate, norms + rotation + cache write, attention with the gate in
-    its epilogue, output projection."""
+    """Grouped-query attention: one product for q, k, v and the gate, short convolution + norms + rotation + value mixing + cache write in
+    one kernel, attention with sink and gate in its epilogue."""
 
     def __init__(self, s: AttentionSpec, pk: _Packer):
         self.s, self.rot = s, _Rotation(s.rotary, pk.device)
         self.dk, self.dv = _up(s.dim, 16), _up(s.vdim, 16)
-        parts = [_pad_rows(pk.raw("mix", "q"), s.heads, self.dk), _pad_rows(pk.raw("mix", "k"), s.kv_heads, self.dk),
-                 _pad_rows(pk.raw("mix", "v"), s.kv_heads, self.dv)]
-        if s.gated:
+        pads = {"q": (s.heads, self.dk), "k": (s.kv_heads, self.dk), "v": (s.kv_heads, self.dv)}
+        parts = [_pad_rows(pk.raw("mix", key), *pad) for key, pad in pads.items()]
+        if s.head_gate:
+            parts.append(pk.raw("mix", "g"))
+        elif s.gated:
             parts.append(_pad_rows(pk.raw("mix", "g"), s.heads, self.dv))
         self.k_off = s.heads * self.dk
         self.v_off = self.k_off + s.kv_heads * self.dk
         self.g_off = self.v_off + s.kv_heads * self.dv
         self.proj = pk.linear(torch.cat(parts, 0))
-        self.o = pk.linear(_pad_cols(pk.raw("mix", "o"), s.heads, self.dv))
+        self.out_weight = _pad_cols(pk.raw("mix", "o"), s.heads, self.dv)
         self.q_norm = pk.f32("mix", "q.norm") if s.qk_norm else None
         self.k_norm = pk.f32("mix", "k.norm") if s.qk_norm else None
+        self.sink = pk.f32("mix", "sink") if s.sink else None
+        self.conv = _ShortConv([_pad_rows(pk.raw("mix", key + ".conv"), *pad) for key, pad in pads.items()]) if s.taps else None
+        self.v_mode, self.v_mix = 0, 0.0           # set by the executor's weights: 1 = first layer that mixes values, 2 = a later one
+        if s.v_mix:
+            self.v_mode, self.v_mix = 2, float(pk.raw("mix", "vmix").float())
 
     def allocate(self, ex: "LayeredExecutor") -> None:
         shape = (ex.num_kv_blocks, self.s.kv_heads, ex.block_size)
         self.k_cache = torch.zeros(shape + (self.dk,), dtype=ex.dtype, device=ex.device)
         self.v_cache = torch.zeros(shape + (self.dv,), dtype=ex.dtype, device=ex.device)
+        if self.conv:
+            self.conv.allocate(ex)
 
     def state(self) -> List[torch.Tensor]:
-        return []
+        return [self.conv.ring] if self.conv else []
 
     def cache_bytes(self) -> int:
-        return self.k_cache.nbytes + self.v_cache.nbytes
+        return self.k_cache.nbytes + self.v_cache.nbytes + sum(t.nbytes for t in self.state())
 
-    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, out: torch.Tensor) -> None:
         s, T = self.s, shp.T
         proj = sb.scratch("proj", T, self.proj.N)
         K.gemm(x, self.proj, out=proj, ws=ex.ws)
+        q, extra = proj, {}
+        if self.conv:
+            q = sb.scratch("queries", T, self.k_off)
+            extra.update(self.conv.args(sb, shp), q_out=q, ldq=q.stride(0))
+        if self.v_mode:
+            first = sb.scratch("v_first", T, s.kv_heads * s.vdim)
+            extra.update(v_first=first, ld_vf=first.stride(0), v_mode=self.v_mode, v_mix=self.v_mix)
+        if self.rot.dims:
+            extra.update(rope=ex.rope(sb, shp, self.rot))
         K.heads_prepare(proj=proj, k_cache=self.k_cache, v_cache=self.v_cache, q_norm=self.q_norm, k_norm=self.k_norm, positions=sb.view("positions"),
                         slot_map=sb.view("slot_map"), T=T, H=s.heads, G=s.kv_heads, D=s.dim, Dv=s.vdim, dk_pad=self.dk, dv_pad=self.dv, ldp=proj.stride(0),
-                        k_off=self.k_off, v_off=self.v_off, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **self.rot.args())
-        attn = sb.scratch("attn", T, self.o.K)
-        gate = dict(gate=proj[:, self.g_off:], ld_gate=proj.stride(0), gate_head=self.dv) if s.gated else {}
-        ex.attention(sb, shp, q=proj, k=self.k_cache, v=self.v_cache, out=attn, Hq=s.heads, Hkv=s.kv_heads, Dk=self.dk, Dv=s.vdim, ldq=proj.stride(0),
-                     q_head=self.dk, k_row=self.dk, v_row=self.dv, ldo=attn.stride(0), o_head=self.dv, window=s.window, scale=s.scale, **gate)
-        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
-        ex.kernel_launches += 4
+                        k_off=self.k_off, v_off=self.v_off, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **self.rot.args(), **extra)
+        if self.conv:
+            self.conv.advance(ex, sb, shp, proj)
+        gate = {}
+        if s.gated or s.head_gate:
+            gate = dict(gate=proj[:, self.g_off:], ld_gate=proj.stride(0), gate_head=1 if s.head_gate else self.dv, gate_scalar=int(s.head_gate))
+        ex.attention(sb, shp, q=q, k=self.k_cache, v=self.v_cache, out=out, Hq=s.heads, Hkv=s.kv_heads, Dk=self.dk, Dv=s.vdim, ldq=q.stride(0),
+                     q_head=self.dk, k_row=self.dk, v_row=self.dv, ldo=out.stride(0), o_head=self.dv, window=s.window, chunk=s.chunk, sink=self.sink,
+                     scale=s.scale, **gate)
+        ex.kernel_launches += 3
 
 
 class LatentAttentionMixer:
@@ -138,7 +185,7 @@ class LatentAttentionMixer:
         self.c_norm = pk.f32("mix", "dkv.norm")
         self.uk = pk.block_diag(pk.raw("mix", "uk").reshape(H, D, C).transpose(1, 2))
         self.uv = pk.block_diag(pk.raw("mix", "uv").reshape(H, Dv, C))
-        self.o = pk.linear(_pad_cols(pk.raw("mix", "o"), H, self.dv))
+        self.out_weight = _pad_cols(pk.raw("mix", "o"), H, self.dv)
         self.k_head, self.v_head = _up(D, 64), _up(Dv, 64)
         self.ukv = None
         if pk.dtype == torch.bfloat16 and self.k_head <= 128 and R <= 64 and self.v_head <= 128 and s.scale > 0:
@@ -161,7 +208,7 @@ class LatentAttentionMixer:
     def cache_bytes(self) -> int:
         return self.cache.nbytes
 
-    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, out: torch.Tensor) -> None:
         s, T, H = self.s, shp.T, self.s.heads
         proj = sb.scratch("proj", T, self.proj.N)
         K.gemm(x, self.proj, out=proj, ws=ex.ws)
@@ -172,13 +219,11 @@ class LatentAttentionMixer:
         K.latent_prepare(proj=proj, cache=self.cache, c_norm=self.c_norm, positions=sb.view("positions"), slot_map=sb.view("slot_map"), T=T,
                          H=H, C=s.kv_rank, R=s.rot_dim, q_pitch=self.q_pitch, q_rot_off=self.dp, c_off=self.c_off, kr_off=self.kr_off, ldp=proj.stride(0),
                          row_pitch=self.pitch, key_off=self.cp, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **q_rot, **self.rot.args())
-        attn = sb.scratch("attn", T, self.o.K)
         if rows:
-            self._attend_expanded(ex, sb, shp, rows, proj, attn)
+            self._attend_expanded(ex, sb, shp, rows, proj, out)
         else:
-            self._attend_absorbed(ex, sb, shp, proj, q, attn)
-        K.gemm(attn, self.o, out=y, out_f32=True, ws=ex.ws)
-        ex.kernel_launches += 3
+            self._attend_absorbed(ex, sb, shp, proj, q, out)
+        ex.kernel_launches += 2
 
     def _attend_expanded(self, ex, sb, shp: StepShape, rows: int, proj: torch.Tensor, attn: torch.Tensor) -> None:
         s, H = self.s, self.s.heads
@@ -217,6 +262,7 @@ class RgLruMixer:
         pad = lambda t: torch.nn.functional.pad(t, (0, self.np - N))
         self.proj = pk.linear(torch.cat([_pad_rows(pk.raw("mix", "y"), 1, self.np), _pad_rows(pk.raw("mix", "x"), 1, self.np)], 0),
                               torch.cat([pad(pk.raw("mix", "y.b")), pad(pk.raw("mix", "x.b"))]))
+        self.out_weight = pk.raw("mix", "o")
         self.conv_w = pk.raw("mix", "conv").float().t().contiguous()          # [taps, N]
         self.conv_b = pk.f32("mix", "conv.b")
         ra, ri = pk.raw("mix", "ra"), pk.raw("mix", "ri")
@@ -224,7 +270,6 @@ class RgLruMixer:
         self.gates = pk.block_diag(torch.cat([grow(ra), grow(ri)], 1))        # [B, 2 * bp, bw]
         self.gate_b = torch.stack([pk.f32("mix", "ra.b"), pk.f32("mix", "ri.b")]).contiguous()
         self.log_decay = (s.decay * torch.nn.functional.softplus(pk.raw("mix", "lam").double())).float().contiguous()
-        self.o = pk.linear(pk.raw("mix", "o"))
 
     def allocate(self, ex: "LayeredExecutor") -> None:
         self.lru_state = torch.zeros((ex.num_slots, self.s.width), dtype=torch.float32, device=ex.device)
@@ -236,13 +281,12 @@ class RgLruMixer:
     def cache_bytes(self) -> int:
         return self.lru_state.nbytes + self.conv_state.nbytes
 
-    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, out: torch.Tensor) -> None:
         s, T = self.s, shp.T
         proj = sb.scratch("proj", T, self.proj.N)
         K.gemm(x, self.proj, out=proj, ws=ex.ws)
         u = sb.scratch("lru_u", T, s.blocks * self.bp)
         gates = sb.scratch("lru_gates", T, s.blocks * 2 * self.bp, torch.float32)
-        out = sb.scratch("lru_out", T, self.o.K)
         args = dict(x=proj[:, self.np:], y=proj, u=u, out=out, gates=gates, gate_b=self.gate_b, log_decay=self.log_decay, conv_w=self.conv_w,
                     conv_b=self.conv_b, state=self.lru_state, conv_state=self.conv_state, subsequence_begins=sb.view("subsequence_begins"),
                     past_lens=sb.view("past_lens"), slots=sb.view("state_slots"), B=shp.B, T=T, N=s.width, taps=s.taps, bw=self.bw, ub_pitch=self.bp,
@@ -251,8 +295,60 @@ class RgLruMixer:
         K.causal_conv(**args)
         K.gemm_block_diag(u, self.gates, gates, self.bp, 2 * self.bp, ws=ex.ws)
         K.lru_scan(**args)
-        K.gemm(out, self.o, out=y, out_f32=True, ws=ex.ws)
-        ex.kernel_launches += 5
+        ex.kernel_launches += 4
+
+
+class ChannelDeltaMixer:
+    """Gated delta rule with a decay per key channel: one product for q, k, v, step sizes and the inner halves of the two low-rank
+    projections, one block-diagonal product for their outer halves (fp32), one kernel for everything else."""
+
+    def __init__(self, s: ChannelDeltaSpec, pk: _Packer):
+        self.s = s
+        self.dk, self.dv = _up(s.dim, 16), _up(s.vdim, 16)
+        H, G = s.heads, s.kv_heads
+        pads = {"q": (G, self.dk), "k": (G, self.dk), "v": (H, self.dv)}
+        self.k_off = G * self.dk
+        self.v_off = 2 * self.k_off
+        self.b_off = self.v_off + H * self.dv
+        self.low_off = self.b_off + _up(H, 16)
+        a1, a2, g1, g2 = (pk.raw("mix", key) for key in ("a1", "a2", "g1", "g2"))
+        if a1.shape[0] != a2.shape[1] or g1.shape[0] != g2.shape[1]:
+            raise ValueError("layer %d: the halves of a low-rank projection do not fit each other" % pk.layer)
+        self.rank = _up(max(a1.shape[0], g1.shape[0]), 16)                         # columns of an inner half
+        self.proj = pk.linear(torch.cat([_pad_rows(pk.raw("mix", key), *pad) for key, pad in pads.items()] + [
+            _pad_rows(pk.raw("mix", "b"), 1, _up(H, 16)), _pad_rows(a1, 1, self.rank), _pad_rows(g1, 1, self.rank)], 0))
+        a2, g2 = _pad_rows(a2, H, self.dk), _pad_rows(g2, H, self.dv)
+        self.low_n = max(a2.shape[0], g2.shape[0])
+        grow = lambda w: torch.nn.functional.pad(w, (0, self.rank - w.shape[1], 0, self.low_n - w.shape[0]))
+        self.low = pk.block_diag(torch.stack([grow(a2), grow(g2)]))               # [2, low_n, rank]
+        self.out_weight = _pad_cols(pk.raw("mix", "o"), H, self.dv)
+        self.conv = _ShortConv([_pad_rows(pk.raw("mix", key + ".conv"), *pad) for key, pad in pads.items()])
+        self.decay_a = pk.raw("mix", "A_log").float().exp().contiguous()
+        self.dt_bias = torch.nn.functional.pad(pk.raw("mix", "dt_bias").float().reshape(H, s.dim), (0, self.dk - s.dim)).contiguous()
+        self.norm = pk.f32("mix", "norm", 16)
+
+    def allocate(self, ex: "LayeredExecutor") -> None:
+        self.delta_state = torch.zeros((ex.num_slots, self.s.heads, self.dk, self.dv), dtype=torch.float32, device=ex.device)
+        self.conv.allocate(ex)
+
+    def state(self) -> List[torch.Tensor]:
+        return [self.delta_state, self.conv.ring]
+
+    def cache_bytes(self) -> int:
+        return sum(t.nbytes for t in self.state())
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, out: torch.Tensor) -> None:
+        s, T = self.s, shp.T
+        proj = sb.scratch("proj", T, self.proj.N)
+        K.gemm(x, self.proj, out=proj, ws=ex.ws)
+        low = sb.scratch("delta_low", T, 2 * self.low_n, torch.float32)
+        K.gemm_block_diag(proj[:, self.low_off:], self.low, low, self.rank, self.low_n, ws=ex.ws)
+        K.channel_delta(proj=proj, low=low, decay_a=self.decay_a, dt_bias=self.dt_bias, norm=self.norm, state=self.delta_state, out=out, T=T, H=s.heads,
+                        G=s.kv_heads, D=s.dim, Dv=s.vdim, dk=self.dk, dv=self.dv, ldp=proj.stride(0), k_off=self.k_off, v_off=self.v_off, b_off=self.b_off,
+                        ld_low=low.stride(0), gate_off=self.low_n, ldo=out.stride(0), o_head=self.dv, dtype=ex.storage, q_scale=s.dim ** -0.5,
+                        eps=ex.cfg.norm_eps, **self.conv.args(sb, shp))
+        self.conv.advance(ex, sb, shp, proj)
+        ex.kernel_launches += 3
 
 
 class LimitedGlu:
@@ -263,10 +359,10 @@ class LimitedGlu:
         gate, up = _pad_rows(pk.raw("mlp", "gate"), 1, self.fp), _pad_rows(pk.raw("mlp", "up"), 1, self.fp)
         self.fused = pk.dtype == torch.bfloat16
         self.gate_up = pk.linear(K.interleave_gate_up(gate, up) if self.fused else torch.cat([gate, up], 0))
-        self.down = pk.linear(pk.raw("mlp", "down"))
+        self.out_weight = pk.raw("mlp", "down")
 
-    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, y: torch.Tensor) -> None:
-        s, act = self.s, sb.scratch("mlp_act", shp.T, self.fp)
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, act: torch.Tensor) -> None:
+        s = self.s
         if self.fused:
             K.gemm(x, self.gate_up, out=act, act=K.ACT_GLU_LIMITED, glu=(s.limit, s.slope, s.shift), ws=ex.ws)
         else:
@@ -274,19 +370,43 @@ class LimitedGlu:
             K.gemm(x, self.gate_up, out=gu, ws=ex.ws)
             K.glu_limited(gu, act, s.ff, self.fp, s.limit, s.slope, s.shift)
             ex.kernel_launches += 1
-        K.gemm(act, self.down, out=y, out_f32=True, ws=ex.ws)
-        ex.kernel_launches += 2
+        ex.kernel_launches += 1
 
 
-MIXERS = {AttentionSpec: AttentionMixer, LatentAttentionSpec: LatentAttentionMixer, RgLruSpec: RgLruMixer}
+class SquaredRelu:
+    """MLP with relu(up)^2; the activation runs in the epilogue of the up product."""
+
+    def __init__(self, s: SquaredReluSpec, pk: _Packer):
+        self.fp = _up(s.ff, 64)
+        self.up = pk.linear(_pad_rows(pk.raw("mlp", "up"), 1, self.fp))
+        self.out_weight = pk.raw("mlp", "down")
+
+    def run(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, x: torch.Tensor, act: torch.Tensor) -> None:
+        K.gemm(x, self.up, out=act, act=K.ACT_RELU2, ws=ex.ws)
+        ex.kernel_launches += 1
+
+
+MIXERS = {AttentionSpec: AttentionMixer, LatentAttentionSpec: LatentAttentionMixer, RgLruSpec: RgLruMixer, ChannelDeltaSpec: ChannelDeltaMixer}
+MLPS = {LimitedGluSpec: LimitedGlu, SquaredReluSpec: SquaredRelu}
 
 
 class _Layer:
-    def __init__(self, spec, pk: _Packer):
+    """``out``: one output product over [mixer columns | feed-forward columns] of a parallel layer, else the mixer's (``down``: the
+    feed-forward's). ``mix_cols`` / ``mlp_cols``: columns that mixer and feed-forward write, whole k-blocks of the product."""
+
+    def __init__(self, spec, pk: _Packer, parallel: bool):
         self.mixer = MIXERS[type(spec.mixer)](spec.mixer, pk)
+        self.mlp = MLPS[type(spec.mlp)](spec.mlp, pk) if spec.mlp is not None else None
         self.norm1 = pk.f32("norm", "1", 4)
-        self.mlp = LimitedGlu(spec.mlp, pk) if spec.mlp is not None else None
         self.norm2 = pk.f32("norm", "2", 4) if spec.mlp is not None else None
+        subs = [self.mixer] + ([self.mlp] if self.mlp is not None else [])
+        widths = [_up(sub.out_weight.shape[1], 64) for sub in subs]
+        weights = [torch.nn.functional.pad(sub.out_weight, (0, n - sub.out_weight.shape[1])) for sub, n in zip(subs, widths)]
+        for sub in subs:
+            sub.out_weight = None
+        self.mix_cols, self.mlp_cols = widths[0], sum(widths[1:])
+        self.out = pk.linear(torch.cat(weights, 1) if parallel else weights[0])
+        self.down = pk.linear(weights[1]) if self.mlp is not None and not parallel else None
 
 
 class LayeredWeights:
@@ -295,24 +415,34 @@ class LayeredWeights:
     def __init__(self, ckpt: Checkpoint, device, dtype: torch.dtype = torch.bfloat16):
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("layered decoders are served in bfloat16 or float32")
-        self.config, self.dtype = ckpt.config, dtype
-        self.layers = [_Layer(spec, _Packer(ckpt, i, device, dtype)) for i, spec in enumerate(ckpt.config.layers)]
+        cfg = self.config = ckpt.config
+        self.dtype = dtype
+        self.layers = [_Layer(spec, _Packer(ckpt, i, device, dtype), cfg.block == PARALLEL_NORM) for i, spec in enumerate(cfg.layers)]
+        mixing = [layer.mixer for layer in self.layers if getattr(layer.mixer, "v_mode", 0)]
+        if any(m.s.kv_heads * m.s.vdim != mixing[0].s.kv_heads * mixing[0].s.vdim for m in mixing):
+            raise ValueError("layers that mix values must have the same number of value columns")
+        for m in mixing[:1]:
+            m.v_mode = 1
         pk = _Packer(ckpt, -1, device, dtype)
         self.embed = pk.raw("", "embed").to(dtype).contiguous()
+        self.embed_norm = pk.f32("", "embed.norm", 4) if cfg.embed_norm else None
         self.final_norm = pk.f32("", "final.norm", 4)
         self.head = pk.linear(pk.raw("", "head"))
 
 
 class LayeredStepBuffers(StepBuffers):
-    """Descriptor, fp32 residual stream ``h``, its copy ``x`` in the compute type (``h`` itself in fp32), sublayer output ``y`` and
-    named scratch that layers share."""
+    """Descriptor, fp32 residual stream ``h``, what the products of a layer read in the compute type (``x``: its copy, or ``h`` itself in
+    fp32; ``x`` and ``x2``: its two norms in parallel layers), sublayer output ``y`` and named scratch that layers share."""
 
     def __init__(self, cfg: LayeredConfig, dtype: torch.dtype, Tcap: int, Bcap: int, max_blocks_per_seq: int, device):
         super().__init__(Tcap, Bcap, max_blocks_per_seq, device, cfg.vocab_size, logits_dtype=torch.float32, state_slots=True)
         width = _up(cfg.hidden_size, 64)
         zeros = lambda rows, dt: torch.zeros((rows, width), dtype=dt, device=device)
         self.h, self.y = zeros(Tcap, torch.float32), zeros(Tcap, torch.float32)
-        self.x = self.h if dtype == torch.float32 else zeros(Tcap, dtype)
+        parallel = cfg.block == PARALLEL_NORM
+        self.x = self.h if dtype == torch.float32 and not parallel else zeros(Tcap, dtype)
+        self.x2 = zeros(Tcap, dtype) if parallel else None
+        self.ropes: Dict[tuple, torch.Tensor] = {}      # angle tables of the step, by rotation
         self.last_x = zeros(Bcap, dtype)
         self.kv_rows = torch.zeros(Bcap + 1, dtype=torch.int32, device=device)
         self.device, self.dtype = device, dtype
@@ -354,6 +484,17 @@ class LayeredExecutor(LlmExecutor):
                            max_context_len=shp.max_ctx, max_q_len=shp.max_q_len, dtype=self.storage, scratch=self.ws.pa_scratch,
                            scratch_bytes=self.ws.pa_scratch.nbytes, exact=1 if self.dtype == torch.float32 else 0, **kw)
 
+    def rope(self, sb: LayeredStepBuffers, shp: StepShape, rot: _Rotation) -> torch.Tensor:
+        """(cos, sin) of the step's positions for a rotation; computed by the first layer that asks for it."""
+        key = (rot.dims, rot.mult, rot.freq)
+        if key not in sb.ropes:
+            table = sb.scratch("rope %s" % (key,), shp.T, rot.dims, torch.float32)
+            table = table.as_strided((shp.T, rot.dims), (rot.dims, 1))            # no gaps between tokens
+            K.rope_table(sb.view("positions"), rot.inv_freq, table, rot.mult)
+            self.kernel_launches += 1
+            sb.ropes[key] = table
+        return sb.ropes[key]
+
     def _norm(self, sb: LayeredStepBuffers, T: int, w: torch.Tensor) -> None:
         """x <- norm(residual_scale * x + y), in fp32, plus the copy that the next products read."""
         cfg = self.cfg
@@ -364,23 +505,56 @@ class LayeredExecutor(LlmExecutor):
         T, B = shp.T, shp.B
         ids = sb.view("ids")[:T]
         K.resolve_ids(ids, sb.view("tok_src")[:T], self.last_token)
-        K.stream_embed(ids, self.w.embed, sb.h, None if sb.x is sb.h else sb.x)
-        x, y = sb.x[:T], sb.y[:T]
-        for i, layer in enumerate(self.w.layers):
-            layer.mixer.run(self, sb, shp, x, y)
-            self._norm(sb, T, layer.norm1)
-            if layer.mlp is not None:
-                layer.mlp.run(self, sb, shp, x, y)
-                self._norm(sb, T, layer.norm2)
-                self.kernel_launches += 1
+        copy = None if sb.x is sb.h or self.cfg.block == PARALLEL_NORM else sb.x       # (parallel layers start with their norms)
+        K.stream_embed(ids, self.w.embed, sb.h, copy)
+        sb.ropes.clear()
+        if self.w.embed_norm is not None:
+            K.sum_rmsnorm(sb.h[:T], self.w.embed_norm, self.cfg.norm_eps, self.cfg.hidden_size, w_offset=self.cfg.norm_offset, h_out=sb.h[:T],
+                          x_out=None if copy is None else copy[:T])
+            self.kernel_launches += 1
+        if self.cfg.block == PARALLEL_NORM:
+            self._parallel_layers(sb, shp)
+        else:
+            self._post_norm_layers(sb, shp)
         self._logits(sb, sb.view("logit_idx")[:B], sb.logits[:B])
-        self.kernel_launches += 2 + len(self.w.layers) + 3
+        self.kernel_launches += 2 + 3
         self._sample(sb, B)
+
+    def _post_norm_layers(self, sb: LayeredStepBuffers, shp: StepShape) -> None:
+        T = shp.T
+        x, y = sb.x[:T], sb.y[:T]
+        for layer in self.w.layers:
+            heads = sb.scratch("heads", T, layer.mix_cols)
+            layer.mixer.run(self, sb, shp, x, heads)
+            K.gemm(heads, layer.out, out=y, out_f32=True, ws=self.ws)
+            self._norm(sb, T, layer.norm1)
+            self.kernel_launches += 2
+            if layer.mlp is not None:
+                act = sb.scratch("mlp_act", T, layer.mlp_cols)
+                layer.mlp.run(self, sb, shp, x, act)
+                K.gemm(act, layer.down, out=y, out_f32=True, ws=self.ws)
+                self._norm(sb, T, layer.norm2)
+                self.kernel_launches += 2
+
+    def _parallel_layers(self, sb: LayeredStepBuffers, shp: StepShape) -> None:
+        """The output of a layer stays in ``y`` until the next layer's norms (or the final one) add it to the stream."""
+        cfg, T = self.cfg, shp.T
+        h, x, x2, y = sb.h[:T], sb.x[:T], sb.x2[:T], sb.y[:T]
+        for i, layer in enumerate(self.w.layers):
+            second = dict(w2=layer.norm2, x2_out=x2) if layer.mlp is not None else {}
+            K.sum_rmsnorm(h, layer.norm1, cfg.norm_eps, cfg.hidden_size, y=y if i else None, w_offset=cfg.norm_offset, s_out=h if i else None, x_out=x, **second)
+            both = sb.scratch("heads", T, layer.mix_cols + layer.mlp_cols)
+            layer.mixer.run(self, sb, shp, x, both[:, :layer.mix_cols])
+            if layer.mlp is not None:
+                layer.mlp.run(self, sb, shp, x2, both[:, layer.mix_cols:])
+            K.gemm(both, layer.out, out=y, out_f32=True, ws=self.ws)
+            self.kernel_launches += 2
 
     def _logits(self, sb: LayeredStepBuffers, rows: torch.Tensor, out: torch.Tensor) -> None:
         cfg, x = self.cfg, sb.last_x[:rows.shape[0]]
-        K.sum_rmsnorm(sb.h, self.w.final_norm, cfg.norm_eps, cfg.hidden_size, w_offset=cfg.norm_offset, x_out=x, row_idx=rows)
-        K.gemm(x, self.w.head, out=out, out_f32=True, ws=self.ws)
+        y = sb.y if cfg.block == PARALLEL_NORM and self.w.layers else None
+        K.sum_rmsnorm(sb.h, self.w.final_norm, cfg.norm_eps, cfg.hidden_size, y=y, w_offset=cfg.norm_offset, x_out=x, row_idx=rows)
+        K.gemm(x, self.w.head, out=out, out_f32=True, act=K.ACT_SOFTCAP if cfg.logit_softcap > 0 else K.ACT_NONE, cap=cfg.logit_softcap, ws=self.ws)
 
     def logits_at(self, sb: LayeredStepBuffers, rows: List[int]) -> torch.Tensor:
         """Logits (fp32) after the step that ``sb`` holds, at the given token rows of its batch."""
