@@ -42,7 +42,7 @@ def test_layered_decoders_need_no_more_than_the_full_library(gemm):
     assert build.layered_library() == build.LIB / "libovb_cuda.so"        # built and current: nothing else is compiled
 
 
-@pytest.mark.parametrize("stem", ["attention_latent", "attention_sm100", "residual", "attention_heads", "gemm_f32", "attention_exact"])
+@pytest.mark.parametrize("stem", ["attention_latent", "attention_sm100", "residual", "attention_heads", "gemm_f32", "attention_exact", "delta_rule"])
 def test_kernels_of_layered_decoders_do_not_spill(gemm, stem):
     res = build.kernel_resources(stem)
     assert res and all(r["spill_stores"] == 0 and r["stack"] == 0 for r in res.values()), {n: r for n, r in res.items() if r["spill_stores"] or r["stack"]}

@@ -108,10 +108,19 @@ ROT = [None, dict(dims=16, base=1e4), dict(dims=24, base=5e5, scaling=dict(facto
        dict(dims=32, base=1e4, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0))]
 
 
-def rotary(rot):
+def rotation(rot):
     from openvino_b200.models.busatar import _rotary
     from openvino_b200.runtime.layered_llm import _Rotation
-    return _Rotation(_rotary(rot) if rot else None, "cuda").args()
+    return _Rotation(_rotary(rot) if rot else None, "cuda")
+
+
+def rope(rot, positions):
+    r = rotation(rot)
+    if not r.dims:
+        return {}
+    table = torch.zeros(positions.numel(), r.dims, device="cuda")
+    k().rope_table(positions, r.inv_freq, table, r.mult)
+    return dict(rot_dims=r.dims, rope=table)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -128,7 +137,7 @@ def test_heads_prepare(dtype, rot, norm):
     kc, vc = torch.zeros(pb.num_blocks, G, 16, dk, dtype=dtype, device="cuda"), torch.zeros(pb.num_blocks, G, 16, dv, dtype=dtype, device="cuda")
     K.heads_prepare(proj=proj, k_cache=kc, v_cache=vc, q_norm=wq.cuda() if norm else None, k_norm=wk.cuda() if norm else None, positions=pb.positions,
                     slot_map=pb.slot_map, T=pb.T, H=H, G=G, D=D, Dv=Dv, dk_pad=dk, dv_pad=dv, ldp=proj.stride(0), k_off=H * dk, v_off=(H + G) * dk,
-                    block_size=16, dtype=K.storage_type(dtype), eps=eps, **rotary(rot))
+                    block_size=16, dtype=K.storage_type(dtype), eps=eps, **rope(rot, pb.positions))
     tol = 1e-5 if dtype == torch.float32 else 1e-2
     for b, (past, n) in enumerate(pb.spans):
         rows = slice(pb.begins[b], pb.begins[b] + n)
@@ -160,7 +169,7 @@ def test_latent_prepare(dtype, rot):
     out = torch.zeros(pb.T, H * (cp + rp), dtype=dtype, device="cuda")
     K.latent_prepare(proj=proj, q_rot=out[:, cp:], cache=cache, c_norm=w.cuda(), positions=pb.positions, slot_map=pb.slot_map, T=pb.T, H=H, C=C, R=R,
                      q_pitch=dp + rp, q_rot_off=dp, c_off=H * (dp + rp), kr_off=H * (dp + rp) + cp, ldp=proj.stride(0), ld_qr=out.stride(0), qr_pitch=cp + rp,
-                     row_pitch=cp + rp, key_off=cp, block_size=16, dtype=K.storage_type(dtype), eps=eps, **rotary(rot))
+                     row_pitch=cp + rp, key_off=cp, block_size=16, dtype=K.storage_type(dtype), eps=eps, **rotation(rot).args())
     tol = 2e-4 if dtype == torch.float32 else 1e-2           # fp32 angles of a few thousand turns
     for b, (past, n) in enumerate(pb.spans):
         rows = slice(pb.begins[b], pb.begins[b] + n)
