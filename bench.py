@@ -92,7 +92,7 @@ def parse():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch"])
     ap.add_argument("--model", default="llama-3-8b",
-                    help="llama-3-8b (headline) | llama-3-70b | mixtral-8x7b | tiny-llama | tiny-moe (serving); bert-large | resnet18 (graph API); busatar (layered decoder beside a Llama of equal size)")
+                    help="llama-3-8b (headline) | llama-3-70b | mixtral-8x7b | tiny-llama | tiny-moe (serving); bert-large | resnet18 (graph API); busatar (layered decoder beside a Llama of equal size), sapasun (beside Busatar)")
     ap.add_argument("--kernels", action="store_true", help="busatar: also time every kernel call of a step with its roofline fraction")
     ap.add_argument("--sizes", default="", help="busatar: sizes to run, with commas between them (default: all of ops/bench_layers.py)")
     ap.add_argument("--requests", type=int, default=0, help="concurrent requests (default: the benchmark's number for the model)")
@@ -209,13 +209,13 @@ def graph_api_bench(args):
 
 
 def layered_bench(args):
-    """Prefill and decode throughput of the layered decoder beside the Llama program at equal size (ops/bench_layers.py), one GPU."""
+    """Prefill and decode throughput of a layered decoder beside the closest other model at equal size (ops/bench_layers.py), one GPU."""
     import torch
     from openvino_b200.ops import bench_layers
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    rows = bench_layers.main([x for x in args.sizes.split(",") if x] or list(bench_layers.SIZES), args.steps, args.warmup, args.kernels)
+    rows = bench_layers.main([x for x in args.sizes.split(",") if x], args.steps, args.warmup, args.kernels, args.model)
     clocks = sampler.stop()
     print(json.dumps({"metric": "tokens/s of one step", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "higher_is_better": True,
                       "dtype": "bf16", "data": "synthetic: uniform token ids, random weights", "peaks": bench_layers._peaks(), "clocks": clocks, "sizes": rows}))
@@ -228,7 +228,7 @@ def main():
         return reference_arm(args)
     if args.model in ("resnet18", "bert-large"):
         return graph_api_bench(args)
-    if args.model == "busatar":
+    if args.model in ("busatar", "sapasun"):
         return layered_bench(args)
     dr, dp, do = SERVING_DEFAULTS.get(args.model, (64, 1024, 256))
     args.requests, args.prompt_len, args.output_len = args.requests or dr, args.prompt_len or dp, args.output_len or do

@@ -8,7 +8,7 @@
 //                   that all heads share; the queries' turned part is written where the attention kernel reads it.
 //
 // A table of inverse frequencies (fp32, made by the host, whatever scaling it follows) and a multiplier of cos and sin describe
-// the rotation; dimension i is paired with i + dims / 2. Norms, angles and sums are fp32. Rows of heads are padded to the pitch
+// the rotation; heads_prepare takes the cosines and sines of the step's positions from a table (ovb_rope_table) that all layers share; dimension i is paired with i + dims / 2. Norms, angles and sums are fp32. Rows of heads are padded to the pitch
 // that the attention kernels want; the padding is zero and is never written.
 #include "debug_bounds.cuh"
 #include "short_conv.cuh"
@@ -27,7 +27,7 @@ struct Rotation {
     float mult;
 };
 
-// Turn the pair (u, v) = (r[i], r[i + dims / 2]) of a row by pos * inv_freq[i].
+// Turn the pair (u, v) = (r[i], r[i + dims / 2]) of a row by pos * inv_freq[i], or by an angle of the table (cos, sin).
 __device__ __forceinline__ void turn(const Rotation& rot, float pos, int i, float& u, float& v) {
     float s, c;
     sincosf(pos * rot.inv_freq[i], &s, &c);
@@ -76,7 +76,7 @@ __device__ __forceinline__ HeadUnit head_unit(const ovb_heads_args& p, int head)
 template <class E>
 __device__ __forceinline__ E* head_row(const ovb_heads_args& p, const HeadUnit& u, int t) {
     if (u.is_q) return p.q_out ? reinterpret_cast<E*>(p.q_out) + (size_t)t * p.ldq + u.col : reinterpret_cast<E*>(p.proj) + (size_t)t * p.ldp + u.col;
-    const int slot = OVB_DBG_SLOT(p.slot_map[t], p.block_size);
+    const int slot = OVB_DBG_SLOT(__ldg(p.slot_map + t), p.block_size);
     if (slot < 0) return nullptr;
     const size_t row = ((size_t)(slot / p.block_size) * p.G + u.kvh) * p.block_size + slot % p.block_size;
     return u.is_k ? reinterpret_cast<E*>(p.k_cache) + row * p.dk_pad : reinterpret_cast<E*>(p.v_cache) + row * p.dv_pad;
@@ -134,17 +134,12 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(ovb_heads_args p) {
     }
     __syncwarp();
     const int half = p.rot_dims / 2;
-    const Rotation rot = {p.inv_freq, p.rot_dims, p.rot_mult};
-    const float pos = (float)p.positions[t];
-    for (int i = lane; i < half; i += 32) {
-        if (p.rope) turn_by(reinterpret_cast<const float2*>(p.rope)[(size_t)t * half + i], r[i], r[i + half]);
-        else turn(rot, pos, i, r[i], r[i + half]);
-    }
+    for (int i = lane; i < half; i += 32) turn_by(reinterpret_cast<const float2*>(p.rope)[(size_t)t * half + i], r[i], r[i + half]);
     __syncwarp();
     for (int i = lane; i < p.D; i += 32) st_f32(dst + i, r[i]);
 }
 
-constexpr int HEADS_STRIP = 8;      // tokens per warp of a prompt
+constexpr int HEADS_STRIP = 4;      // tokens per warp of a prompt
 
 // The same for heads of up to 128 columns in pieces of four: a warp walks a strip of tokens of one head with its columns in registers
 // (lane l: columns 4 l ..), so that every projected value is fetched once; rotation partners sit in other lanes. TAPS 0: no convolution.
@@ -166,9 +161,13 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
     const bool live = c < u.n;
     const E* src = reinterpret_cast<const E*>(p.proj) + u.col + (live ? c : 0);
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    float4 w[TAPS > 0 ? TAPS : 1], hist[KEEP > 0 ? KEEP : 1], raw[HEADS_STRIP];
+    float4 w[TAPS > 0 ? TAPS : 1];
+    Raw4<E> hist[KEEP > 0 ? KEEP : 1], raw[HEADS_STRIP];
 #pragma unroll
-    for (int k = 0; k < HEADS_STRIP; ++k) raw[k] = (live && t0 + k < t_end) ? ld4_f32(src + (size_t)(t0 + k) * p.ldp) : zero;
+    for (int k = 0; k < HEADS_STRIP; ++k) {
+        raw[k].set(zero);
+        if (live && t0 + k < t_end) raw[k].load(src + (size_t)(t0 + k) * p.ldp);
+    }
     if (TAPS > 0) {
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[j] = live ? ld4_f32(p.conv_w + (size_t)j * p.conv_cols + u.col + c) : zero;
@@ -185,9 +184,9 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
     for (int k = 0; k < HEADS_STRIP; ++k) {
         const int t = t0 + k;
         if (t >= t_end) break;
-        float4 v = raw[k];
+        float4 v = raw[k].get();
         if (TAPS > 0) {
-            const int pos = p.positions[t];
+            const int pos = __ldg(p.positions + t);
             bool fresh = k == 0;
             while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) {
                 ++b;
@@ -197,16 +196,16 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
             float* ring = cv.ring + (size_t)p.slots[b] * TAPS * cv.cols + u.col + c;
             if (fresh) {
 #pragma unroll
-                for (int j = 0; j < KEEP; ++j) hist[j] = live ? conv_input4(src, p.ldp, ring, cv, t, begin, pos, KEEP - j) : zero;
+                for (int j = 0; j < KEEP; ++j) hist[j].set(live ? conv_input4(src, p.ldp, ring, cv, t, begin, pos, KEEP - j) : zero);
             }
             if (p.max_q_len == 1 && TAPS > 1 && live) st4_f32(ring + (size_t)(pos % TAPS) * cv.cols, v);
             float4 acc = zero;
 #pragma unroll
-            for (int j = 0; j < KEEP; ++j) acc = fma4(w[j], hist[j], acc);
+            for (int j = 0; j < KEEP; ++j) acc = fma4(w[j], hist[j].get(), acc);
             acc = fma4(w[TAPS > 0 ? TAPS - 1 : 0], v, acc);
 #pragma unroll
             for (int j = 0; j + 1 < KEEP; ++j) hist[j] = hist[j + 1];
-            if (KEEP > 0) hist[KEEP - 1] = v;
+            if (KEEP > 0) hist[KEEP - 1] = raw[k];
             v = acc;
         }
         if (nw) {
@@ -218,7 +217,7 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
                                          __shfl_sync(0xffffffffu, v.w, partner));
             if (turned) {
                 const float4* cs = reinterpret_cast<const float4*>(p.rope + ((size_t)t * half + (lower ? c : c - half)) * 2);
-                const float4 a = cs[0], d = cs[1];       // (cos, sin) of four pairs
+                const float4 a = __ldg(cs), d = __ldg(cs + 1);       // (cos, sin) of four pairs
                 const float sg = lower ? -1.f : 1.f;     // lower: u cos - v sin, upper: v cos + u sin
                 v = make_float4(v.x * a.x + sg * (o.x * a.y), v.y * a.z + sg * (o.y * a.w), v.z * d.x + sg * (o.z * d.y), v.w * d.z + sg * (o.w * d.w));
             }
@@ -329,15 +328,15 @@ int ovb_heads_prepare(const ovb_heads_args* a, ovb_stream_t stream) {
     OVB_REQUIRE(a && a->proj && a->k_cache && a->v_cache && a->positions && a->slot_map, "ovb_heads_prepare: null operand");
     OVB_REQUIRE(a->T > 0 && a->H > 0 && a->G > 0 && a->D > 0 && a->Dv > 0 && a->dk_pad >= a->D && a->dv_pad >= a->Dv && a->block_size > 0,
                 "ovb_heads_prepare: bad sizes");
-    OVB_REQUIRE(a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->D && (a->rot_dims == 0 || a->inv_freq), "ovb_heads_prepare: bad rotation");
+    OVB_REQUIRE(a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->D && (a->rot_dims == 0 || a->rope), "ovb_heads_prepare: bad rotation");
     OVB_REQUIRE(a->D <= 2048 && a->Dv <= 2048, "ovb_heads_prepare: head sizes %d, %d above 2048", a->D, a->Dv);
     OVB_REQUIRE(a->taps == 0 || (a->taps > 0 && a->conv_w && a->conv_ring && a->subsequence_begins && a->past_lens && a->slots && a->q_out && a->B > 0 &&
                                  a->conv_cols >= a->v_off + a->G * a->dv_pad), "ovb_heads_prepare: bad short convolution");
     OVB_REQUIRE(a->v_mode == 0 || (a->v_first && a->ld_vf >= a->G * a->Dv && (a->v_mode == 1 || a->v_mode == 2)), "ovb_heads_prepare: bad value mixing");
     auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
     const int units = a->H + 2 * a->G;
-    // heads in registers: whole pieces of four columns everywhere, rotation partners at whole lanes, angles from the table
-    const bool strip_form = a->D <= 128 && a->Dv <= 128 && a->D % 4 == 0 && a->Dv % 4 == 0 && a->rot_dims % 8 == 0 && (a->rot_dims == 0 || a->rope) && a->taps <= 4 &&
+    // heads in registers: whole pieces of four columns everywhere, rotation partners at whole lanes
+    const bool strip_form = a->D <= 128 && a->Dv <= 128 && a->D % 4 == 0 && a->Dv % 4 == 0 && a->rot_dims % 8 == 0 && a->taps <= 4 &&
                             a->ldp % 4 == 0 && a->dk_pad % 4 == 0 && a->dv_pad % 4 == 0 && a->k_off % 4 == 0 && a->v_off % 4 == 0 && a->conv_cols % 4 == 0 &&
                             a->ldq % 4 == 0 && a->ld_vf % 4 == 0 && aligned(a->proj) && aligned(a->q_out) && aligned(a->k_cache) && aligned(a->v_cache) &&
                             aligned(a->conv_w) && aligned(a->conv_ring) && aligned(a->v_first) && aligned(a->rope);
@@ -346,21 +345,20 @@ int ovb_heads_prepare(const ovb_heads_args* a, ovb_stream_t stream) {
         if (strip_form) {
             // few tokens: a warp each; many: strips that share the inputs of the convolution
             const int strip = (long long)a->T * units <= 148 * 32 || a->max_q_len == 1 ? 1 : HEADS_STRIP;
-            auto go = [&](auto kern) -> int {
-                OVB_CHECK_CUDA(launch_pdl(kern, dim3(ceil_div(a->T, strip), ceil_div(units, 4)), dim3(128), 0, (cudaStream_t)stream, *a, strip));
-                return 0;
-            };
-            switch (a->taps) {
-                case 0: return go(heads_strip_kernel<E, 0>);
-                case 1: return go(heads_strip_kernel<E, 1>);
-                case 2: return go(heads_strip_kernel<E, 2>);
-                case 3: return go(heads_strip_kernel<E, 3>);
-                default: return go(heads_strip_kernel<E, 4>);
-            }
+            auto kern = a->taps == 0   ? heads_strip_kernel<E, 0>
+                        : a->taps == 1 ? heads_strip_kernel<E, 1>
+                        : a->taps == 2 ? heads_strip_kernel<E, 2>
+                        : a->taps == 3 ? heads_strip_kernel<E, 3>
+                                       : heads_strip_kernel<E, 4>;
+            OVB_CHECK_CUDA(launch_pdl(kern, dim3(ceil_div(a->T, strip), ceil_div(units, 4)), dim3(128), 0, (cudaStream_t)stream, *a, strip));
+        } else {
+            const int width = a->D > a->Dv ? a->D : a->Dv;
+            OVB_CHECK_CUDA(launch_pdl(heads_prepare_kernel<E>, dim3(a->T, ceil_div(units, 4)), dim3(128), (size_t)4 * width * 4, (cudaStream_t)stream, *a));
         }
-        const int width = a->D > a->Dv ? a->D : a->Dv;
-        OVB_CHECK_CUDA(launch_pdl(heads_prepare_kernel<E>, dim3(a->T, ceil_div(units, 4)), dim3(128), (size_t)4 * width * 4, (cudaStream_t)stream, *a));
-        return 0;
+        // (a decode step's kernel has written the ring itself)
+        if (a->taps == 0 || a->max_q_len == 1) return 0;
+        return update_conv_ring<E>(a->proj, a->ldp, {a->conv_w, a->conv_ring, a->taps, a->conv_cols}, a->subsequence_begins, a->past_lens, a->slots, a->B,
+                                   (cudaStream_t)stream);
     });
 }
 

@@ -123,6 +123,9 @@ __device__ __forceinline__ __half from_float<__half>(float v) {
     return __float2half_rn(v);
 }
 
+// cap * tanh(v / cap); the error is of the order of an ulp of cap.
+__device__ __forceinline__ float soft_cap(float v, float cap) { return cap - __fdividef(2.0f * cap, 1.0f + __expf(__fdividef(2.0f * v, cap))); }
+
 __device__ __forceinline__ float apply_act(float v, const GemmKParams& p) {
     switch (p.act) {
         case OVB_ACT_GELU_ERF: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
@@ -133,7 +136,7 @@ __device__ __forceinline__ float apply_act(float v, const GemmKParams& p) {
             return 0.5f * v * (1.0f + tanhf(u));
         }
         case OVB_ACT_RELU2: return v > 0.f ? v * v : 0.f;
-        case OVB_ACT_SOFTCAP: return p.act_limit * tanhf(v / p.act_limit);
+        case OVB_ACT_SOFTCAP: return soft_cap(v, p.act_limit);
         default: return v;
     }
 }
@@ -655,7 +658,8 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         // plain 16-bit output of the larger tiles: straight from the accumulator's registers
         const bool direct16 = OVB_GEMM_DIRECT && BT >= 128 && fast && (p.act == OVB_ACT_NONE || p.act == OVB_ACT_RELU2) && p.residual == nullptr;
         // fp32 output of a tile inside N: the lanes of a warp hold 32 consecutive columns of a token, stored as they are
-        const bool plain32 = !QUANT && p.world <= 1 && p.splits == 1 && p.out_f32 && n0 + TILE_N <= p.N && p.residual == nullptr && p.act == OVB_ACT_NONE;
+        const bool plain32 = !QUANT && p.world <= 1 && p.splits == 1 && p.out_f32 && n0 + TILE_N <= p.N && p.residual == nullptr &&
+                             (p.act == OVB_ACT_NONE || p.act == OVB_ACT_SOFTCAP);
         // fp32 staging keeps a single rounding (after the residual add): BT x 128 x 4 bytes <= 2 * STAGE_BYTES
         float* stage_out = reinterpret_cast<float*>(smem);
 
@@ -1119,8 +1123,11 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 } else if (plain32) {
                     float* o = reinterpret_cast<float*>(p.out) + (size_t)(t0 + c0) * p.ldo + out_col + oc;
 #pragma unroll
-                    for (int j = 0; j < 16; ++j)
-                        if (t0 + c0 + j < T_end) o[(size_t)j * p.ldo] = __uint_as_float(r[j]) + bias_v;
+                    for (int j = 0; j < 16; ++j) {
+                        float v = __uint_as_float(r[j]) + bias_v;
+                        if (p.act == OVB_ACT_SOFTCAP) v = soft_cap(v, p.act_limit);
+                        if (t0 + c0 + j < T_end) o[(size_t)j * p.ldo] = v;
+                    }
                 } else if (p.splits == 1) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j) finish(c0 + j, __uint_as_float(r[j]));

@@ -353,25 +353,20 @@ int ovb_sample_f32(const float* logits, int ld, int rows, int vocab, float tempe
 // cos and sin of the rotation angles of every token: table[t, i] = (cos, sin)(positions[t] * inv_freq[i]) * mult, i < half.
 int ovb_rope_table(const int* positions, const float* inv_freq, float* table, int T, int half, float mult, ovb_stream_t stream);
 
-// Short causal convolutions (short_conv.cuh): the inputs of a step, proj [T, ldp] columns 0 .. cols, go to the rings of their slots. Only
-// for steps with more than one token per sequence; the kernels below do it themselves when max_q_len is 1.
-int ovb_conv_ring_update(const void* proj, float* ring, const int* subsequence_begins, const int* past_lens, const int* slots, int B, int cols, int taps, int ldp,
-                         int dtype, ovb_stream_t stream);
-
 // Short convolution, query / key norms, rotary positions, value mixing and cache rows of grouped-query attention (attention_heads.cu).
-// With taps > 0 every column of q, k and v passes the convolution first and the queries go to q_out (not their place in proj).
+// With taps > 0 every column of q, k and v passes the convolution first, the step's last inputs go to the rings of their slots
+// (short_conv.cuh), and the queries go to q_out (not their place in proj).
 typedef struct {
     void* proj;              // [T, ldp]: H query heads (pitch dk_pad), G key heads at k_off (pitch dk_pad), G value heads at v_off (pitch dv_pad)
     void* k_cache;           // [blocks, G, block_size, dk_pad]
     void* v_cache;           // [blocks, G, block_size, dv_pad]
     const float* q_norm;     // [D] or NULL
     const float* k_norm;
-    const float* inv_freq;   // [rot_dims / 2] or NULL
     const int* positions;
     const int* slot_map;
     int T, H, G, D, Dv, dk_pad, dv_pad, ldp, k_off, v_off, block_size, rot_dims, dtype;
-    float rot_mult, eps;
-    const float* rope;       // [T, rot_dims / 2] (cos, sin) pairs (ovb_rope_table), or NULL: computed here
+    float eps;
+    const float* rope;       // [T, rot_dims / 2] (cos, sin) pairs (ovb_rope_table), or NULL without a rotation
     void* q_out;             // [T, ldq], heads at a pitch of dk_pad; NULL: in place
     const float* conv_w;     // [taps, conv_cols]: a channel is a column of proj
     float* conv_ring;        // [slots, taps, conv_cols]
@@ -475,7 +470,7 @@ int ovb_lru_scan(const ovb_rglru_args* a, ovb_stream_t stream);
 // Gated delta rule with a decay per key channel, from the projections to the heads that the output projection reads (delta_rule.cu).
 // Per head: q, k, v pass their short convolution and silu; q and k become unit vectors (q also times q_scale);
 // g = exp(-decay_a * softplus(low + dt_bias)); S <- g S; S <- S + k (beta (v - S^T k))^T; o = S^T q; out = rms_norm(o) * norm * sigmoid(gate).
-// Everything behind the convolutions is fp32. D and Dv are the true sizes, dk and dv the pitches of heads (multiples of 16, zeros in
+// Everything behind the convolutions is fp32; state and convolution rings are brought up to date. D and Dv are the true sizes, dk and dv the pitches of heads (multiples of 16, zeros in
 // projections, convolution weights and norm behind the true size).
 typedef struct {
     const void* proj;        // [T, ldp]: G query heads at column 0, G key heads at k_off, H value heads at v_off, H beta logits at b_off

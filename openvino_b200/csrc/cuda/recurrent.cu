@@ -308,18 +308,6 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ovb_rglru_args p, int 
     }
 }
 
-// Inputs of a step's last taps - 1 positions of every sequence -> rings (short_conv.cuh).
-template <class E>
-__global__ void __launch_bounds__(128) conv_ring_update_kernel(const E* __restrict__ proj, float* __restrict__ ring, const int* __restrict__ begins,
-                                                               const int* __restrict__ past_lens, const int* __restrict__ slots, int cols, int taps, int ldp) {
-    pdl_enter();
-    const int b = blockIdx.y, c = blockIdx.x * 128 + threadIdx.x;
-    if (c >= cols) return;
-    const int begin = begins[b], end = begins[b + 1], past = past_lens[b];
-    float* mine = ring + (size_t)slots[b] * taps * cols + c;
-    for (int t = max(begin, end - (taps - 1)); t < end; ++t) mine[(size_t)((past + t - begin) % taps) * cols] = ld_f32(proj + (size_t)t * ldp + c);
-}
-
 __device__ __forceinline__ float rec_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 // gelu of the other branch: 0.5 z (1 + tanh(v)) = z * sigmoid(2 v)
 __device__ __forceinline__ float rec_gelu_tanh(float z) { return z * rec_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
@@ -499,19 +487,6 @@ int ovb_causal_conv(const ovb_rglru_args* a, ovb_stream_t stream) {
         if (!vec) return go(causal_conv_kernel<E, 1, 0>);
         return a->taps == 2 ? go(causal_conv_kernel<E, 4, 2>) : a->taps == 3 ? go(causal_conv_kernel<E, 4, 3>) : a->taps == 4 ? go(causal_conv_kernel<E, 4, 4>)
                                                                                                              : go(causal_conv_kernel<E, 4, 0>);
-    });
-}
-
-int ovb_conv_ring_update(const void* proj, float* ring, const int* subsequence_begins, const int* past_lens, const int* slots, int B, int cols, int taps, int ldp,
-                         int dtype, ovb_stream_t stream) {
-    using namespace ovb;
-    OVB_REQUIRE(proj && ring && subsequence_begins && past_lens && slots && B > 0 && B <= 65535 && cols > 0 && taps > 0 && ldp >= cols, "ovb_conv_ring_update: bad arguments");
-    if (taps == 1) return 0;
-    return dispatch_store(dtype, "ovb_conv_ring_update", [&](auto e) -> int {
-        using E = decltype(e);
-        OVB_CHECK_CUDA(launch_pdl(conv_ring_update_kernel<E>, dim3(ceil_div(cols, 128), B), dim3(128), 0, (cudaStream_t)stream, reinterpret_cast<const E*>(proj), ring,
-                                  subsequence_begins, past_lens, slots, cols, taps, ldp));
-        return 0;
     });
 }
 

@@ -28,6 +28,26 @@ __device__ __forceinline__ void st4_f32(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = r;
 }
 
+// Four elements as they lie in memory.
+template <class E>
+struct Raw4;
+template <>
+struct Raw4<float> {
+    float4 v;
+    __device__ __forceinline__ float4 get() const { return v; }
+    __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
+    __device__ __forceinline__ void set(float4 x) { v = x; }
+};
+template <>
+struct Raw4<__nv_bfloat16> {
+    uint2 v;
+    __device__ __forceinline__ float4 get() const {
+        return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+    }
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
+    __device__ __forceinline__ void set(float4 x) { st4_f32(reinterpret_cast<__nv_bfloat16*>(&v), x); }
+};
+
 // Host side: call `f` with a value of the element type that `dtype` (OVB_DT_F32 / OVB_DT_BF16) names.
 template <class F>
 inline int dispatch_store(int dtype, const char* what, F f) {

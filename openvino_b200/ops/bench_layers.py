@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of layered decoders beside the Llama-family program at equal size (random weights, bf16), and the
-device time of every kernel call of a step with its roofline fraction.
+"""Prefill and decode throughput of layered decoders beside the closest other model at equal size (random weights, bf16), and the
+device time of every kernel call of a step with its roofline fraction: Busatar beside the Llama-family program, Sapasun beside Busatar.
 
     python bench.py --model busatar [--kernels] [--sizes gqa-4k,latent-4k]
+    python bench.py --model sapasun [--kernels] [--sizes chunked-4k,delta-4k]
 
 Both programs run through their executors: a prefill step is launched as the scheduler would (ragged batch, paged cache), a decode
 step is replayed as its CUDA graph. Weights of a few layers exceed the L2 many times over. ``--kernels`` wraps every kernel entry
@@ -14,7 +15,8 @@ from typing import Dict, List, Tuple
 
 import torch
 
-from ..models.llm_config import AttentionSpec, LatentAttentionSpec, LayeredConfig, LayerSpec, LimitedGluSpec, LlmConfig, RgLruSpec, RotarySpec
+from ..models.llm_config import (PARALLEL_NORM, AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, LayeredConfig, LayerSpec, LimitedGluSpec, LlmConfig, RgLruSpec,
+                                 RotarySpec, SquaredReluSpec)
 from ..models.registry import ARCHITECTURES, Checkpoint
 from ..runtime.cuda_llm import CudaLlmExecutor, LlmWeights
 from ..runtime.layered_llm import LayeredExecutor, LayeredWeights
@@ -49,6 +51,28 @@ SIZES: Dict[str, Tuple[LayeredConfig, LlmConfig]] = OrderedDict([
 ])
 
 
+def _parallel(width: int, mixers, ff: int, vocab: int = 32000) -> LayeredConfig:
+    layers = tuple(LayerSpec(m, SquaredReluSpec(ff) if mlp else None) for m, mlp in mixers)
+    return LayeredConfig("Sapasun", vocab, width, layers, block=PARALLEL_NORM, embed_norm=True, logit_softcap=30.0)
+
+
+def _chunked(heads, kv, chunk):
+    return AttentionSpec(heads, kv, 128, 128, 128 ** -0.5, rotary=RotarySpec(64, 10000.0), head_gate=True, chunk=chunk, sink=True, taps=4, v_mix=True)
+
+
+def _delta(heads):
+    return ChannelDeltaSpec(heads, heads, 128, 128, 4, decay_rank=128, gate_rank=128)
+
+
+# name -> (Sapasun, Busatar of the same width, heads, window, layers and feed-forward parameters: a gated one has two input matrices)
+SAPASUN_SIZES: Dict[str, Tuple[LayeredConfig, LayeredConfig]] = OrderedDict([
+    ("chunked-4k", (_parallel(4096, [(_chunked(32, 8, 4096), True)] * 4, 21504), SIZES["gqa-4k"][0])),
+    ("delta-4k", (_parallel(4096, [(_delta(32), True)] * 4, 21504), SIZES["rglru-4k"][0])),
+    ("mixed-2k", (_parallel(2048, [(_chunked(16, 4, 1024), True), (_delta(16), False), (_chunked(16, 4, 1024), True), (_chunked(16, 4, 1024), True),
+                                   (_delta(16), True), (_chunked(16, 4, 1024), True)], 12288), SIZES["mixed-2k"][0])),
+])
+
+
 class _RandomTensors:
     """Random tensors of a checkpoint's shapes, made on the device when they are asked for."""
 
@@ -58,15 +82,17 @@ class _RandomTensors:
     def __getitem__(self, name):
         shape = self.shapes[name]
         t = torch.randn(shape, device="cuda", generator=self.g)
-        if name.endswith(".lam"):
+        if name.endswith(".lam") or name.endswith(".dt_bias"):
             return (t - 3.0).to(torch.bfloat16)
+        if len(shape) == 0:
+            return torch.tensor(0.5, dtype=torch.bfloat16, device="cuda")
         if len(shape) == 1:
             return (1.0 + 0.1 * t if name.endswith("q.norm") or name.endswith("k.norm") or name.endswith("dkv.norm") else 0.1 * t).to(torch.bfloat16)
         return (t * shape[-1] ** -0.5).to(torch.bfloat16)
 
 
 def make_layered(cfg: LayeredConfig, **kw) -> LayeredExecutor:
-    arch = ARCHITECTURES["Busatar"]
+    arch = ARCHITECTURES[cfg.name]
     return LayeredExecutor(LayeredWeights(Checkpoint(cfg, arch, _RandomTensors(arch.tensor_shapes(cfg))), torch.device("cuda")), **kw)
 
 
@@ -160,10 +186,18 @@ def run(executor, steps: int, warmup: int, kernels: bool) -> dict:
 
 
 # ------------------------------------------------------------------------------------------------ kernels of a step
-def _pairs(spans, window):
+# fp32 arithmetic outside the tensor cores: 148 SMs x 128 multiply-adds a clock at 1.9 GHz (nominal)
+FP32_TFLOPS = 148 * 128 * 2 * 1.9e-3
+
+
+def _pairs(spans, window, chunk=0):
     """(query, key) pairs and distinct keys that a batch's tokens see."""
     pairs = keys = 0
     for past, new in spans:
+        if chunk:
+            pairs += sum(p % chunk + 1 for p in range(past, past + new))
+            keys += past % chunk + new
+            continue
         w = window or past + new
         pairs += sum(min(p + 1, w) for p in range(past, past + new))
         keys += min(past + new, new + w - 1)
@@ -171,11 +205,14 @@ def _pairs(spans, window):
 
 
 def _cost(name, args, kw, spans):
-    """(label, bytes, flops) of a kernel call."""
+    """(label, bytes, flops on the tensor cores[, flops of fp32 arithmetic]) of a kernel call."""
     if name == "gemm":
         x, w = args[0], args[1]
         T, N = x.shape[0], w.N
         glu = kw.get("act", 0) in (K.ACT_SWIGLU, K.ACT_GLU_LIMITED)
+        if kw.get("act", 0) in (K.ACT_RELU2, K.ACT_SOFTCAP):
+            return "gemm N=%d K=%d +%s" % (N, w.K, "relu2" if kw["act"] == K.ACT_RELU2 else "softcap"), (N * w.K + T * w.K) * 2 + T * N * kw["out"].element_size(), \
+                2.0 * T * N * w.K
         outb = T * N * (2 if glu is False and not kw.get("out_f32") else 4 if kw.get("out_f32") else 1)
         return "gemm N=%d K=%d%s" % (N, w.K, " +glu" if glu else ""), (N * w.K + T * w.K) * 2 + outb, 2.0 * T * N * w.K
     if name == "gemm_block_diag":
@@ -186,11 +223,11 @@ def _cost(name, args, kw, spans):
         if name == "paged_attention":
             Hq, Hkv, D = args[7:10]
             Dk = Dv = row = D
-            T, latent, window = args[0].shape[0], False, kw["sliding_window"]
+            T, latent, window, chunk = args[0].shape[0], False, kw["sliding_window"], 0
         else:
             Hq, Hkv, Dk, Dv, T, window = kw["Hq"], kw["Hkv"], kw["Dk"], kw["Dv"], kw["T"], kw["window"]
-            latent = kw["k"] is kw["v"]
-        pairs, keys = _pairs(spans, window)
+            latent, chunk = kw["k"] is kw["v"], kw.get("chunk", 0)
+        pairs, keys = _pairs(spans, window, chunk)
         kv = keys * Hkv * (Dk if latent else Dk + Dv) * 2
         kind = "decode" if all(n == 1 for _, n in spans) else "prefill"
         return "%s attention %s" % ("latent" if latent else "paged", kind), kv + T * Hq * (Dk + Dv) * 2, 2.0 * pairs * Hq * (Dk + Dv)
@@ -203,14 +240,18 @@ def _cost(name, args, kw, spans):
     if name == "rmsnorm":
         return "norm", args[0].numel() * 4, 0.0
     if name == "sum_rmsnorm":
-        x = kw.get("x_out")
         rows = (kw["row_idx"] if kw.get("row_idx") is not None else args[0]).shape[0]
-        return "norm", rows * args[3] * (4 + (4 if kw.get("y") is not None else 0) + (4 if kw.get("h_out") is not None else 0) + (2 if x is not None else 0)), 0.0
+        extra = [4 for key in ("y", "h_out", "s_out") if kw.get(key) is not None] + [2 for key in ("x_out", "x2_out") if kw.get(key) is not None]
+        return "norm", rows * args[3] * (4 + sum(extra)), 0.0
     if name == "rope_kv_write":
         qkv, Hq, Hkv, D = args[0], args[5], args[6], args[7]
         return "head preparation", qkv.shape[0] * (Hq * 2 + Hkv * 4) * D * 2, 0.0
     if name == "heads_prepare":
         return "head preparation", kw["T"] * (kw["H"] * 2 * kw["D"] + kw["G"] * 2 * (kw["D"] + kw["Dv"])) * 2, 0.0
+    if name == "channel_delta":
+        # state: a decay (multiplication) and three multiply-adds per element and token, in fp32 by design
+        T, H, G, dk, dv = kw["T"], kw["H"], kw["G"], kw["dk"], kw["dv"]
+        return "recurrence", T * ((2 * G * dk + 2 * H * dv) * 2 + H * (dk + dv) * 4) + kw["B"] * H * dk * dv * 8, 0.0, 7.0 * T * H * dk * dv
     if name == "latent_prepare":
         return "head preparation (latent)", kw["T"] * (kw["H"] * 2 * kw["R"] + 2 * (kw["C"] + kw["R"])) * 2, 0.0
     if name == "causal_conv":
@@ -221,7 +262,7 @@ def _cost(name, args, kw, spans):
 
 
 _NAMES = ("gemm", "gemm_block_diag", "window_attention", "paged_attention", "latent_prefill", "latent_gather", "rmsnorm", "sum_rmsnorm", "rope_kv_write",
-          "heads_prepare", "latent_prepare", "causal_conv", "lru_scan", "stream_embed", "embedding", "argmax", "resolve_ids", "scatter_tokens")
+          "heads_prepare", "latent_prepare", "causal_conv", "lru_scan", "channel_delta", "rope_table", "stream_embed", "embedding", "argmax", "resolve_ids", "scatter_tokens")
 
 
 def profile(executor, step, spans, repeats: int = 3) -> List[dict]:
@@ -231,13 +272,13 @@ def profile(executor, step, spans, repeats: int = 3) -> List[dict]:
 
     def wrap(name, fn):
         def timed(*args, **kw):
-            label, nbytes, flops = _cost(name, args, kw, spans)
+            label, nbytes, flops, *fp32 = _cost(name, args, kw, spans)
             flush.sum()
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             a.record()
             out = fn(*args, **kw)
             b.record()
-            calls.append((label, nbytes, flops, a, b))
+            calls.append((label, nbytes, flops, fp32[0] if fp32 else 0.0, a, b))
             return out
         return timed
     step()
@@ -252,27 +293,32 @@ def profile(executor, step, spans, repeats: int = 3) -> List[dict]:
             setattr(K, n, fn)
     torch.cuda.synchronize()
     groups: Dict[str, list] = OrderedDict()
-    for label, nbytes, flops, a, b in calls:
-        groups.setdefault(label, []).append((a.elapsed_time(b), nbytes, flops))
+    for label, nbytes, flops, fp32, a, b in calls:
+        groups.setdefault(label, []).append((a.elapsed_time(b), nbytes, flops, fp32))
     peaks, rows = _peaks(), []
     for label, v in groups.items():
-        us = sorted(t for t, _, _ in v)[len(v) // 2] * 1e3
-        nbytes, flops = v[0][1], v[0][2]
-        bound = max(nbytes / (peaks["hbm_gbs"] * 1e3), flops / (peaks["bf16_tflops"] * 1e6))
-        rows.append({"kernel": label, "calls": len(v) // repeats, "us": round(us, 1), "roofline_us": round(bound, 1), "fraction": round(bound / us, 3),
-                     "bound": "hbm" if nbytes / (peaks["hbm_gbs"] * 1e3) >= bound else "tensor"})
+        ms, nbytes, flops, fp32 = sorted(v)[len(v) // 2]          # (calls of equal label may differ in size)
+        us = ms * 1e3
+        bounds = {"hbm": nbytes / (peaks["hbm_gbs"] * 1e3), "tensor": flops / (peaks["bf16_tflops"] * 1e6), "fp32": fp32 / (FP32_TFLOPS * 1e6)}
+        kind = max(bounds, key=bounds.get)
+        rows.append({"kernel": label, "calls": len(v) // repeats, "us": round(us, 1), "roofline_us": round(bounds[kind], 1),
+                     "fraction": round(bounds[kind] / us, 3), "bound": kind})
     return sorted(rows, key=lambda r: -r["us"] * r["calls"])
 
 
-def main(sizes: List[str], steps: int, warmup: int, kernels: bool) -> dict:
-    rows = OrderedDict()
-    for name in sizes:
-        layered, llama = SIZES[name]
+def main(sizes: List[str], steps: int, warmup: int, kernels: bool, model: str = "busatar") -> dict:
+    """Rows of the sizes that are named (all, if none is): {size: {model: ..., what it stands beside: ...}}."""
+    rows, pairs = OrderedDict(), SAPASUN_SIZES if model == "sapasun" else SIZES
+    for name in sizes or list(pairs):
+        layered, other = pairs[name]
         limits = dict(num_kv_blocks=64 * (2048 // 16 + 2) + 64, block_size=16, max_batch_tokens=8192, max_seqs=64, max_blocks_per_seq=514)
         rows[name] = {}
-        for arm, make in (("layered", lambda: make_layered(layered, **limits)),
-                          ("llama", lambda: CudaLlmExecutor(llama, LlmWeights.random(llama, torch.device("cuda")), device="cuda", **limits))):
-            ex = make()
+        arms = ("sapasun", "busatar") if model == "sapasun" else ("layered", "llama")
+        for arm, cfg in zip(arms, (layered, other)):
+            if isinstance(cfg, LayeredConfig):
+                ex = make_layered(cfg, **limits)
+            else:
+                ex = CudaLlmExecutor(cfg, LlmWeights.random(cfg, torch.device("cuda")), device="cuda", **limits)
             rows[name][arm] = run(ex, steps, warmup, kernels)
             del ex
             torch.cuda.empty_cache()

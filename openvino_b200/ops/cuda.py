@@ -61,8 +61,8 @@ def _fields(pointers, ints, floats=()):
 
 
 class HeadsArgs(C.Structure):
-    _fields_ = _fields(("proj", "k_cache", "v_cache", "q_norm", "k_norm", "inv_freq", "positions", "slot_map"),
-                       ("T", "H", "G", "D", "Dv", "dk_pad", "dv_pad", "ldp", "k_off", "v_off", "block_size", "rot_dims", "dtype"), ("rot_mult", "eps")) + \
+    _fields_ = _fields(("proj", "k_cache", "v_cache", "q_norm", "k_norm", "positions", "slot_map"),
+                       ("T", "H", "G", "D", "Dv", "dk_pad", "dv_pad", "ldp", "k_off", "v_off", "block_size", "rot_dims", "dtype"), ("eps",)) + \
         _fields(("rope", "q_out", "conv_w", "conv_ring", "subsequence_begins", "past_lens", "slots", "v_first"),
                 ("B", "taps", "conv_cols", "ldq", "ld_vf", "v_mode", "max_q_len"), ("v_mix",))
 
@@ -417,13 +417,6 @@ def rope_table(positions, inv_freq, out, mult=1.0) -> None:
     """out[t, i] = (cos, sin)(positions[t] * inv_freq[i]) * mult; out: fp32 [T, 2 * half]."""
     _check(lib().ovb_rope_table(C.c_void_p(positions.data_ptr()), C.c_void_p(inv_freq.data_ptr()), C.c_void_p(out.data_ptr()), C.c_int(out.shape[0]),
                                 C.c_int(inv_freq.numel()), C.c_float(mult), C.c_void_p(_stream())), "ovb_rope_table")
-
-
-def conv_ring_update(proj, ring, subsequence_begins, past_lens, slots, B) -> None:
-    """Last taps - 1 inputs of every sequence of a step -> ``ring`` [slots, taps, cols] (columns 0 .. cols of ``proj``)."""
-    _check(lib().ovb_conv_ring_update(C.c_void_p(proj.data_ptr()), C.c_void_p(ring.data_ptr()), C.c_void_p(subsequence_begins.data_ptr()),
-                                      C.c_void_p(past_lens.data_ptr()), C.c_void_p(slots.data_ptr()), C.c_int(B), C.c_int(ring.shape[2]), C.c_int(ring.shape[1]),
-                                      C.c_int(proj.stride(0)), C.c_int(storage_type(proj.dtype)), C.c_void_p(_stream())), "ovb_conv_ring_update")
 
 
 def channel_delta(**kw) -> None:

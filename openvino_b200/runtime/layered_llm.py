@@ -89,12 +89,6 @@ class _ShortConv:
         return dict(conv_w=self.w, conv_ring=self.ring, conv_cols=self.cols, taps=self.taps, subsequence_begins=sb.view("subsequence_begins"),
                     past_lens=sb.view("past_lens"), slots=sb.view("state_slots"), B=shp.B, max_q_len=shp.max_q_len)
 
-    def advance(self, ex: "LayeredExecutor", sb: "LayeredStepBuffers", shp: StepShape, proj: torch.Tensor) -> None:
-        """Behind the kernel that convolves: the step's last inputs go to the rings (a decode step's kernel does that itself)."""
-        if shp.max_q_len > 1 and self.taps > 1:
-            K.conv_ring_update(proj, self.ring, sb.view("subsequence_begins"), sb.view("past_lens"), sb.view("state_slots"), shp.B)
-            ex.kernel_launches += 1
-
 
 # A mixer's ``run`` writes the columns that the output projection ``out_weight`` [width, columns] reads; a feed-forward likewise.
 class AttentionMixer:
@@ -148,19 +142,17 @@ class AttentionMixer:
             first = sb.scratch("v_first", T, s.kv_heads * s.vdim)
             extra.update(v_first=first, ld_vf=first.stride(0), v_mode=self.v_mode, v_mix=self.v_mix)
         if self.rot.dims:
-            extra.update(rope=ex.rope(sb, shp, self.rot))
+            extra.update(rot_dims=self.rot.dims, rope=ex.rope(sb, shp, self.rot))
         K.heads_prepare(proj=proj, k_cache=self.k_cache, v_cache=self.v_cache, q_norm=self.q_norm, k_norm=self.k_norm, positions=sb.view("positions"),
                         slot_map=sb.view("slot_map"), T=T, H=s.heads, G=s.kv_heads, D=s.dim, Dv=s.vdim, dk_pad=self.dk, dv_pad=self.dv, ldp=proj.stride(0),
-                        k_off=self.k_off, v_off=self.v_off, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **self.rot.args(), **extra)
-        if self.conv:
-            self.conv.advance(ex, sb, shp, proj)
+                        k_off=self.k_off, v_off=self.v_off, block_size=ex.block_size, dtype=ex.storage, eps=ex.cfg.norm_eps, **extra)
         gate = {}
         if s.gated or s.head_gate:
             gate = dict(gate=proj[:, self.g_off:], ld_gate=proj.stride(0), gate_head=1 if s.head_gate else self.dv, gate_scalar=int(s.head_gate))
         ex.attention(sb, shp, q=q, k=self.k_cache, v=self.v_cache, out=out, Hq=s.heads, Hkv=s.kv_heads, Dk=self.dk, Dv=s.vdim, ldq=q.stride(0),
                      q_head=self.dk, k_row=self.dk, v_row=self.dv, ldo=out.stride(0), o_head=self.dv, window=s.window, chunk=s.chunk, sink=self.sink,
                      scale=s.scale, **gate)
-        ex.kernel_launches += 3
+        ex.kernel_launches += 3 + (self.conv is not None and shp.max_q_len > 1 and self.conv.taps > 1)
 
 
 class LatentAttentionMixer:
@@ -347,8 +339,7 @@ class ChannelDeltaMixer:
                         G=s.kv_heads, D=s.dim, Dv=s.vdim, dk=self.dk, dv=self.dv, ldp=proj.stride(0), k_off=self.k_off, v_off=self.v_off, b_off=self.b_off,
                         ld_low=low.stride(0), gate_off=self.low_n, ldo=out.stride(0), o_head=self.dv, dtype=ex.storage, q_scale=s.dim ** -0.5,
                         eps=ex.cfg.norm_eps, **self.conv.args(sb, shp))
-        self.conv.advance(ex, sb, shp, proj)
-        ex.kernel_launches += 3
+        ex.kernel_launches += 3 + (shp.max_q_len > 1 and self.conv.taps > 1)
 
 
 class LimitedGlu:

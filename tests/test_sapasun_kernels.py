@@ -208,8 +208,6 @@ def test_short_convolution_rotation_and_value_mixing(dtype, H, G, D, Dv, rot, ta
             K.heads_prepare(proj=proj, k_cache=kc, v_cache=vc, positions=pos, slot_map=smap, H=H, G=G, D=D, Dv=Dv, dk_pad=dk, dv_pad=dv, ldp=proj.stride(0),
                             k_off=H * dk, v_off=(H + G) * dk, block_size=16, dtype=K.storage_type(dtype), eps=1e-5, q_out=q_out, ldq=H * dk, conv_w=filt,
                             conv_ring=ring, conv_cols=filt.shape[1], taps=taps, v_first=vf if mode else None, ld_vf=vf.stride(0), v_mode=mode, v_mix=lam, **extra, **args)
-            if args["max_q_len"] > 1:
-                K.conv_ring_update(proj, ring, args["subsequence_begins"], args["past_lens"], args["slots"], args["B"])
             for (b, s, m), lo in zip(batch, begins):
                 got_q[b].append(q_out[lo:lo + m].reshape(m, H, dk)[..., :D].float().cpu())
                 if mode == 1:
@@ -269,8 +267,6 @@ def test_channel_delta_in_portions(dtype, H, G, D, Dv, taps):
         out = torch.zeros(T, H * dv, dtype=dtype, device="cuda")
         K.channel_delta(proj=proj, low=lows, out=out, H=H, G=G, D=D, Dv=Dv, dk=dk, dv=dv, ldp=proj.stride(0), k_off=G * dk, v_off=2 * G * dk, b_off=b_off,
                         ld_low=lows.stride(0), gate_off=H * dk, ldo=H * dv, o_head=dv, dtype=K.storage_type(dtype), q_scale=D ** -0.5, eps=eps, **const, **args)
-        if args["max_q_len"] > 1:
-            K.conv_ring_update(proj, ring, args["subsequence_begins"], args["past_lens"], args["slots"], args["B"])
         for (b, _, m), lo in zip(batch, begins):
             got[b].append(out[lo:lo + m].float().cpu().reshape(m, H, dv)[..., :Dv])
     for g, v in zip(got, want):
