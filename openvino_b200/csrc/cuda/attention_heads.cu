@@ -139,7 +139,7 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(ovb_heads_args p) {
     for (int i = lane; i < p.D; i += 32) st_f32(dst + i, r[i]);
 }
 
-constexpr int HEADS_STRIP = 4;      // tokens per warp of a prompt
+constexpr int HEADS_STRIP = 16, HEADS_BATCH = 4;      // tokens per warp of a prompt, and of those in registers at a time
 
 // The same for heads of up to 128 columns in pieces of four: a warp walks a strip of tokens of one head with its columns in registers
 // (lane l: columns 4 l ..), so that every projected value is fetched once; rotation partners sit in other lanes. TAPS 0: no convolution.
@@ -148,12 +148,7 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
     pdl_enter();
     __shared__ int s_b;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t0 = blockIdx.x * strip, t_end = min(p.T, t0 + strip), head = blockIdx.y * 4 + warp;
-    if (TAPS > 0) {
-        find_sequence(p.subsequence_begins, p.B, t0, &s_b);
-        __syncthreads();
-    }
-    if (head >= p.H + 2 * p.G) return;
+    const int t0 = blockIdx.x * strip, t_end = min(p.T, t0 + strip), head = min(blockIdx.y * 4 + warp, p.H + 2 * p.G - 1);   // (the last head once more)
     constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 0;
     const HeadUnit u = head_unit(p, head);
     const bool is_v = !u.is_q && !u.is_k;
@@ -162,12 +157,7 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
     const E* src = reinterpret_cast<const E*>(p.proj) + u.col + (live ? c : 0);
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     float4 w[TAPS > 0 ? TAPS : 1];
-    Raw4<E> hist[KEEP > 0 ? KEEP : 1], raw[HEADS_STRIP];
-#pragma unroll
-    for (int k = 0; k < HEADS_STRIP; ++k) {
-        raw[k].set(zero);
-        if (live && t0 + k < t_end) raw[k].load(src + (size_t)(t0 + k) * p.ldp);
-    }
+    float4 hist[KEEP > 0 ? KEEP : 1];
     if (TAPS > 0) {
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[j] = live ? ld4_f32(p.conv_w + (size_t)j * p.conv_cols + u.col + c) : zero;
@@ -179,61 +169,70 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
     const bool lower = c < half, turned = c < 2 * half;
     const int partner = turned ? (lower ? lane + half / 4 : lane - half / 4) : lane;
     const ShortConv cv = {p.conv_w, p.conv_ring, TAPS, p.conv_cols};
-    int b = TAPS > 0 ? s_b : 0, begin = TAPS > 0 ? p.subsequence_begins[b] : 0;
+    int b = 0, next = 0;                          // sequence, its end
+    if (TAPS > 0) {
+        find_sequence(p.subsequence_begins, p.B, t0, &s_b);
+        __syncthreads();
+        b = s_b;
+        next = p.subsequence_begins[b + 1];
+    }
+    for (int tb = t0; tb < t_end; tb += HEADS_BATCH) {
+        Raw4<E> raw[HEADS_BATCH];
 #pragma unroll
-    for (int k = 0; k < HEADS_STRIP; ++k) {
-        const int t = t0 + k;
-        if (t >= t_end) break;
-        float4 v = raw[k].get();
-        if (TAPS > 0) {
-            const int pos = __ldg(p.positions + t);
-            bool fresh = k == 0;
-            while (b + 1 < p.B && t >= p.subsequence_begins[b + 1]) {
-                ++b;
-                begin = t;
-                fresh = true;
-            }
-            float* ring = cv.ring + (size_t)p.slots[b] * TAPS * cv.cols + u.col + c;
-            if (fresh) {
+        for (int k = 0; k < HEADS_BATCH; ++k) {
+            raw[k].set(zero);
+            if (live && tb + k < t_end) raw[k].load(src + (size_t)(tb + k) * p.ldp);
+        }
 #pragma unroll
-                for (int j = 0; j < KEEP; ++j) hist[j].set(live ? conv_input4(src, p.ldp, ring, cv, t, begin, pos, KEEP - j) : zero);
-            }
-            if (p.max_q_len == 1 && TAPS > 1 && live) st4_f32(ring + (size_t)(pos % TAPS) * cv.cols, v);
-            float4 acc = zero;
+        for (int k = 0; k < HEADS_BATCH; ++k) {
+            const int t = tb + k;
+            if (t >= t_end) break;
+            float4 v = raw[k].get();
+            if (TAPS > 0) {
+                if (KEEP > 0 && (t == t0 || t >= next)) {      // what came before: this step's tokens, or the ring
+                    while (t >= next) next = p.subsequence_begins[++b + 1];
+                    const int begin = p.subsequence_begins[b], pos = p.positions[t];
+                    float* ring = cv.ring + (size_t)p.slots[b] * TAPS * cv.cols + u.col + c;
 #pragma unroll
-            for (int j = 0; j < KEEP; ++j) acc = fma4(w[j], hist[j].get(), acc);
-            acc = fma4(w[TAPS > 0 ? TAPS - 1 : 0], v, acc);
+                    for (int j = 0; j < KEEP; ++j) hist[j] = live ? conv_input4(src, p.ldp, ring, cv, t, begin, pos, KEEP - j) : zero;
+                    if (p.max_q_len == 1 && live) st4_f32(ring + (size_t)(pos % TAPS) * cv.cols, v);
+                }
+                float4 acc = zero;
 #pragma unroll
-            for (int j = 0; j + 1 < KEEP; ++j) hist[j] = hist[j + 1];
-            if (KEEP > 0) hist[KEEP - 1] = raw[k];
-            v = acc;
-        }
-        if (nw) {
-            const float inv = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)p.D + p.eps);
-            v = make_float4(v.x * inv * gain.x, v.y * inv * gain.y, v.z * inv * gain.z, v.w * inv * gain.w);
-        }
-        if (half > 0) {
-            const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, partner), __shfl_sync(0xffffffffu, v.y, partner), __shfl_sync(0xffffffffu, v.z, partner),
-                                         __shfl_sync(0xffffffffu, v.w, partner));
-            if (turned) {
-                const float4* cs = reinterpret_cast<const float4*>(p.rope + ((size_t)t * half + (lower ? c : c - half)) * 2);
-                const float4 a = __ldg(cs), d = __ldg(cs + 1);       // (cos, sin) of four pairs
-                const float sg = lower ? -1.f : 1.f;     // lower: u cos - v sin, upper: v cos + u sin
-                v = make_float4(v.x * a.x + sg * (o.x * a.y), v.y * a.z + sg * (o.y * a.w), v.z * d.x + sg * (o.z * d.y), v.w * d.z + sg * (o.w * d.w));
+                for (int j = 0; j < KEEP; ++j) acc = fma4(w[j], hist[j], acc);
+                acc = fma4(w[TAPS > 0 ? TAPS - 1 : 0], v, acc);
+#pragma unroll
+                for (int j = 0; j + 1 < KEEP; ++j) hist[j] = hist[j + 1];
+                if (KEEP > 0) hist[KEEP - 1] = v;
+                v = acc;
             }
-        }
-        if (is_v && p.v_mode && live) {
-            E* first = reinterpret_cast<E*>(p.v_first) + (size_t)t * p.ld_vf + u.kvh * p.Dv + c;
-            if (p.v_mode == 1) {
-                st4_f32(first, v);
-            } else {
-                const float4 f = ld4_f32(first);
-                const float a = 1.f - p.v_mix;
-                v = make_float4(a * v.x + p.v_mix * f.x, a * v.y + p.v_mix * f.y, a * v.z + p.v_mix * f.z, a * v.w + p.v_mix * f.w);
+            if (nw) {
+                const float inv = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)p.D + p.eps);
+                v = make_float4(v.x * inv * gain.x, v.y * inv * gain.y, v.z * inv * gain.z, v.w * inv * gain.w);
             }
+            if (half > 0) {
+                const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, partner), __shfl_sync(0xffffffffu, v.y, partner), __shfl_sync(0xffffffffu, v.z, partner),
+                                             __shfl_sync(0xffffffffu, v.w, partner));
+                if (turned) {
+                    const float4* cs = reinterpret_cast<const float4*>(p.rope + ((size_t)t * half + (lower ? c : c - half)) * 2);
+                    const float4 a = __ldg(cs), d = __ldg(cs + 1);       // (cos, sin) of four pairs
+                    const float sg = lower ? -1.f : 1.f;     // lower: u cos - v sin, upper: v cos + u sin
+                    v = make_float4(v.x * a.x + sg * (o.x * a.y), v.y * a.z + sg * (o.y * a.w), v.z * d.x + sg * (o.z * d.y), v.w * d.z + sg * (o.w * d.w));
+                }
+            }
+            if (is_v && p.v_mode && live) {
+                E* first = reinterpret_cast<E*>(p.v_first) + (size_t)t * p.ld_vf + u.kvh * p.Dv + c;
+                if (p.v_mode == 1) {
+                    st4_f32(first, v);
+                } else {
+                    const float4 f = ld4_f32(first);
+                    const float a = 1.f - p.v_mix;
+                    v = make_float4(a * v.x + p.v_mix * f.x, a * v.y + p.v_mix * f.y, a * v.z + p.v_mix * f.z, a * v.w + p.v_mix * f.w);
+                }
+            }
+            E* dst = head_row<E>(p, u, t);
+            if (dst && live) st4_f32(dst + c, v);
         }
-        E* dst = head_row<E>(p, u, t);
-        if (dst && live) st4_f32(dst + c, v);
     }
 }
 

@@ -1,19 +1,26 @@
 // Gated delta rule with a decay per key channel, fused with everything between its projections and the output projection: short
 // convolutions, silu, unit norms, decays, step sizes, the recurrence, the norm of its read-out and the output gate.
 //
-// The state S [dk, dv] of a head stays in registers for the whole piece of a sequence that a step brings and touches memory twice. Its
-// columns are independent: lane l of a consumer warp holds CPT columns (column group l % 8) at RL rows (row group l / 8), so that the dot
-// products over the rows are sums within a lane plus two shuffles, and no barrier stands in a token's chain
+// The state S [dk, dv] of a head lives in registers and touches memory twice per step. A token reads it, then changes it:
 //
-//     S <- g S;  m = S^T k;  o = S^T q;  u = beta (v - m);  S <- S + k u^T;  o += (k . q) u
+//     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //
-// (the read-out after the update, written with the dot product k . q so that both sums run side by side). Rows are taken two at a time
-// with the packed fp32 instructions of sm_100.
+// Prompts take four tokens at a time. With c_t = g_1 .. g_t (products of decays, never quotients: nothing overflows),
 //
-// One CTA works on (sequence, head, part of the columns). Consumer warps run the recurrence over a stage of up to 16 tokens in shared
-// memory; producer warps meanwhile fetch the raw inputs two stages ahead (cp.async), prepare the next stage (convolution, silu, norms,
-// decays: one warp per token) and finish the previous one (norm of the read-out, gate, store). When there are too few (sequence, head) pairs to fill the machine, a cluster of CTAs shares a
-// head's columns and reads each other's read-outs through distributed shared memory for the norm. Decode steps have a kernel of their own.
+//     u_t = beta_t (v_t - S^T (c_t k_t) - sum_{s<t} A_ts u_s),      A_ts = k_t . (g_{s+1} .. g_t k_s)
+//     o_t = S^T (c_t q_t) + sum_{s<=t} B_ts u_s,                    B_ts = q_t . (g_{s+1} .. g_t k_s)
+//     S   <- c_4 S + sum_s (g_{s+1} .. g_4 k_s) u_s^T
+//
+// which is the same sum in another order, entirely in fp32: 13 operations per state element for four tokens instead of 16, and one
+// reduction over the rows instead of four behind one another. Everything that does not depend on the state (convolutions, silu, unit
+// norms, decays, the vectors and coefficients above) is prepared by a kernel that works on all groups of four at once
+// (delta_prepare_kernel); the recurrence itself (delta_scan_kernel) walks the groups of a sequence.
+//
+// Columns of the state are independent. In the scan, lane l of a consumer warp holds CPT columns at RL of the rows, so that the dot
+// products are sums within a lane plus a few shuffles and no barrier stands in a group's chain; rows are taken two at a time with the
+// packed fp32 instructions of sm_100. Producer warps fetch the next stage of four groups (cp.async) and finish the previous one (norm of
+// the read-out, gate, store). When there are too few (sequence, head) pairs to fill the machine, a cluster of CTAs shares a head's
+// columns and reads each other's read-outs through distributed shared memory for the norm. Decode steps have a kernel of their own.
 #include <cooperative_groups.h>
 
 #include <atomic>
@@ -22,6 +29,7 @@
 #include "short_conv.cuh"
 #include "sm100_ptx.cuh"
 #include "store_types.cuh"
+#include "warp_sums.cuh"
 
 namespace ovb {
 
@@ -51,12 +59,6 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
-__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
-    f32x2 r;
-    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-
 __device__ __forceinline__ float delta_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -93,17 +95,148 @@ __device__ __forceinline__ float4 decay4(float a, float4 low, float4 bias) {
                        expf(-a * Fn<E>::softplus(low.w + bias.w)));
 }
 
+constexpr int GROUP = 4;                // tokens taken at a time
+constexpr int GROUP_VECTORS = 3 * GROUP + 1;                      // c_t k_t, c_t q_t, decayed k_s, c_4
+constexpr int GROUP_SCALARS = GROUP * (GROUP - 1) / 2 + GROUP * (GROUP + 1) / 2 + GROUP;      // A, B (row by row), beta
+static_assert(GROUP_SCALARS == 20, "whole 16-byte pieces");
+
+// Floats of the record of one (group, head): vectors [13][dk], values [4][dv], scalars. A sequence whose tokens of this step begin at row
+// t has its groups in rows t / 4 + b, ... (they do not overlap: T / 4 + B rows are enough).
+__host__ __device__ inline int record_floats(int dk, int dv) { return GROUP_VECTORS * dk + GROUP * dv + GROUP_SCALARS; }
+__device__ __forceinline__ int first_group(const int* begins, int b) { return begins[b] / GROUP + b; }
+
+// One warp per (group, head). TAPS 0: any number of taps.
+template <class E, int NV, int TAPS>
+__global__ void __launch_bounds__(128) delta_prepare_kernel(ovb_delta_args p) {
+    pdl_enter();
+    __shared__ int s_b;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x, h = blockIdx.y * 4 + warp;
+    for (int b = threadIdx.x; b < p.B; b += 128)
+        if (first_group(p.subsequence_begins, b) <= row && row < first_group(p.subsequence_begins, b + 1)) s_b = b;
+    __syncthreads();
+    const int b = s_b, begin = p.subsequence_begins[b], len = p.subsequence_begins[b + 1] - begin;
+    const int t0 = (row - first_group(p.subsequence_begins, b)) * GROUP, n = min(GROUP, len - t0);      // tokens of the group
+    if (n <= 0 || h >= p.H) return;
+    const int past = p.past_lens[b], kvh = h / (p.H / p.G);
+    const E* proj = reinterpret_cast<const E*>(p.proj);
+    const ShortConv cv = {p.conv_w, p.conv_ring, TAPS > 0 ? TAPS : p.taps, p.conv_cols};
+    const float* ring = p.conv_ring + (size_t)p.slots[b] * cv.taps * cv.cols;
+    float* rec = p.records + ((size_t)row * p.H + h) * record_floats(p.dk, p.dv);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+
+    // convolution and silu of four columns for the tokens of the group; zeros behind the last token
+    auto conv = [&](int col, float4 (&y)[GROUP]) {
+        if constexpr (TAPS > 0) {
+            Raw4<E> in[TAPS + GROUP - 1];
+            float4 w[TAPS];
+#pragma unroll
+            for (int j = 0; j < TAPS + GROUP - 1; ++j) {
+                const int rel = t0 + j - (TAPS - 1);
+                if (rel >= 0 && rel < len) in[j].load(proj + (size_t)(begin + rel) * p.ldp + col);
+                else if (rel < 0 && past + rel >= 0) in[j].set(ld4_f32(ring + (size_t)((past + rel) % TAPS) * cv.cols + col));
+                else in[j].set(zero);
+            }
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j] = ld4_f32(p.conv_w + (size_t)j * cv.cols + col);
+#pragma unroll
+            for (int t = 0; t < GROUP; ++t) {
+                float4 acc = zero;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fma4(w[j], in[t + j].get(), acc);
+                y[t] = t < n ? silu4<E>(acc) : zero;
+            }
+        } else {
+#pragma unroll
+            for (int t = 0; t < GROUP; ++t) {
+                float4 acc = zero;
+                if (t < n)
+                    for (int j = 0; j < cv.taps; ++j)
+                        acc = fma4(ld4_f32(cv.w + (size_t)j * cv.cols + col),
+                                   conv_input4(proj + col, p.ldp, ring + col, cv, begin + t0 + t, begin, past + t0 + t, cv.taps - 1 - j), acc);
+                y[t] = silu4<E>(acc);
+            }
+        }
+    };
+    float4 q[NV][GROUP], k[NV][GROUP];
+    float sums[2 * GROUP] = {};
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = i * 128 + lane * 4;
+        if (c < p.dk) {
+            conv(kvh * p.dk + c, q[i]);
+            conv(p.k_off + kvh * p.dk + c, k[i]);
+        } else {
+#pragma unroll
+            for (int t = 0; t < GROUP; ++t) q[i][t] = k[i][t] = zero;
+        }
+#pragma unroll
+        for (int t = 0; t < GROUP; ++t) {
+            sums[t] += dot4(q[i][t], q[i][t]);
+            sums[GROUP + t] += dot4(k[i][t], k[i][t]);
+        }
+    }
+    const float total = rec_reduce8(sums, lane);
+    float scale[2 * GROUP];
+#pragma unroll
+    for (int j = 0; j < 2 * GROUP; ++j)
+        scale[j] = (j < GROUP ? p.q_scale : 1.f) / sqrtf(__shfl_sync(0xffffffffu, total, ((j & 1) << 4) | ((j >> 1 & 1) << 3) | ((j >> 2 & 1) << 2)) + 1e-6f);
+    float ab[16] = {};                            // A then B
+    const float a = p.decay_a[h];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = i * 128 + lane * 4;
+        if (c >= p.dk) continue;
+        const float4 bias = ld4_f32(p.dt_bias + (size_t)h * p.dk + c);
+        float4 g[GROUP], r[GROUP], all = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+        for (int t = 0; t < GROUP; ++t)
+            g[t] = t < n ? decay4<E>(a, ld4_f32(p.low + (size_t)(begin + t0 + t) * p.ld_low + (size_t)h * p.dk + c), bias) : make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+        for (int t = 0; t < GROUP; ++t) {
+            const float4 kt = scale4(k[i][t], scale[GROUP + t]), qt = scale4(q[i][t], scale[t]);
+            all = mul4(all, g[t]);
+            st4_f32(rec + t * p.dk + c, mul4(all, kt));
+            st4_f32(rec + (GROUP + t) * p.dk + c, mul4(all, qt));
+#pragma unroll
+            for (int s = 0; s < t; ++s) {
+                r[s] = mul4(r[s], g[t]);
+                ab[t * (t - 1) / 2 + s] += dot4(kt, r[s]);
+                ab[6 + t * (t + 1) / 2 + s] += dot4(qt, r[s]);
+            }
+            r[t] = kt;
+            ab[6 + t * (t + 1) / 2 + t] += dot4(qt, kt);
+        }
+#pragma unroll
+        for (int s = 0; s < GROUP; ++s) st4_f32(rec + (2 * GROUP + s) * p.dk + c, r[s]);
+        st4_f32(rec + 3 * GROUP * p.dk + c, all);
+    }
+    float* scalars = rec + GROUP_VECTORS * p.dk + GROUP * p.dv;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = ab[half * 8 + j];
+        const float sum = rec_reduce8(v, lane);
+        if ((lane & 3) == 0) scalars[half * 8 + rec_owned_value8(lane)] = sum;
+    }
+    if (lane < GROUP) scalars[16 + lane] = lane < n ? Fn<E>::sigmoid(ld_f32(proj + (size_t)(begin + t0 + lane) * p.ldp + p.b_off + h)) : 0.f;
+    for (int c = lane * 4; c < p.dv; c += 128) {
+        float4 v[GROUP];
+        conv(p.v_off + h * p.dv + c, v);
+#pragma unroll
+        for (int t = 0; t < GROUP; ++t) st4_f32(rec + GROUP_VECTORS * p.dk + t * p.dv + c, v[t]);
+    }
+}
+
 struct DeltaShape {
     int parts;               // CTAs that share a head's columns (a cluster)
-    int cols;                // columns per CTA, a multiple of 8 CPT (the last part may reach past dv)
-    int consumers;           // warps that run the recurrence: cols / (8 CPT)
-    int chunk;               // tokens per stage
+    int cols;                // columns per CTA, whole consumer warps (the last part may reach past dv)
+    int consumers;           // warps that run the recurrence
+    int groups;              // groups per stage
 };
 
-// Floats of one stage: K, Q, G [chunk][DP], V [chunk][cols], beta and k . q [chunk] (padded to whole 16-byte pieces).
-__host__ __device__ inline int stage_floats(int dp, int cols, int chunk) { return chunk * (3 * dp + cols) + (2 * chunk + 3) / 4 * 4; }
-// Bytes of the raw inputs of one stage: rows of the head's q, k and of this CTA's v columns (chunk + taps - 1 tokens), decay inputs (chunk tokens).
-__host__ __device__ inline int raw_bytes(int dk, int cols, int chunk, int taps, int elem) { return (chunk + taps - 1) * (2 * dk + cols) * elem + chunk * dk * 4; }
+// Floats of a group in a stage: as its record, with DP rows and this CTA's columns.
+__host__ __device__ inline int staged_floats(int dp, int cols) { return GROUP_VECTORS * dp + GROUP * cols + GROUP_SCALARS; }
 
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
@@ -114,26 +247,21 @@ __device__ __forceinline__ void copy_wait() {
     asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
-// Warps of a CTA: fewer where the state takes more registers.
-constexpr int max_warps(int rl) { return rl >= 64 ? 10 : 12; }
+constexpr int scan_warps(int state) { return state >= 64 ? 12 : 16; }      // at most, by the state's registers per lane
 
-template <class E, int RL, int CPT>
-__global__ void __launch_bounds__(max_warps(RL) * 32, 1) channel_delta_kernel(ovb_delta_args p, DeltaShape s) {
-    constexpr int DP = RL * 4;                     // rows, zero behind p.dk
-    constexpr int NV = (DP + 127) / 128;           // pieces of four rows per lane
+// RGS row groups of RL rows: a warp has 32 / RGS lanes side by side, CPT columns each.
+template <class E, int RGS, int RL, int CPT>
+__global__ void __launch_bounds__(scan_warps(RL * CPT) * 32, 1) delta_scan_kernel(ovb_delta_args p, DeltaShape s) {
+    constexpr int DP = RGS * RL;                   // rows, zero behind p.dk
+    constexpr int LANES = 32 / RGS, WARP_COLS = LANES * CPT;
     extern __shared__ __align__(16) float smem[];
-    const int stage_len = stage_floats(DP, s.cols, s.chunk);
-    float* y_buf = smem + 2 * stage_len;           // [2][chunk][cols] read-outs
-    float* s_conv = y_buf + 2 * s.chunk * s.cols;  // [taps][2 DP + cols] filters of the head's q, k and of this CTA's v columns
-    const int conv_len = 2 * DP + s.cols;
-    float* s_bias = s_conv + p.taps * conv_len;    // [DP]
-    float* s_norm = s_bias + DP;                   // [cols]
-    uint8_t* raw_buf = reinterpret_cast<uint8_t*>(s_norm + s.cols);      // [2] raw inputs
-    const int raw_len = raw_bytes(p.dk, s.cols, s.chunk, p.taps, sizeof(E)), raw_pitch = 2 * p.dk + s.cols, keep = p.taps - 1;
+    const int group_len = staged_floats(DP, s.cols), stage_len = s.groups * group_len, tokens = s.groups * GROUP;      // of a stage
+    float* y_buf = smem + 2 * stage_len;           // [2][tokens][cols] read-outs
+    float* s_norm = y_buf + 2 * tokens * s.cols;   // [cols]
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int part = blockIdx.x % s.parts, h = blockIdx.x / s.parts, b = blockIdx.y;
-    const int c0 = part * s.cols, kvh = h / (p.H / p.G);
+    const int c0 = part * s.cols, v_cols = max(0, min(s.cols, p.dv - c0));
     const bool consumer = warp < s.consumers;
     const int pw = warp - s.consumers, npw = (blockDim.x >> 5) - s.consumers;       // producer warps
     const int pt = threadIdx.x - s.consumers * 32, npt = npw * 32;
@@ -142,152 +270,98 @@ __global__ void __launch_bounds__(max_warps(RL) * 32, 1) channel_delta_kernel(ov
         if (s.parts > 1) cluster.sync();
         else __syncthreads();
     };
-
-    // constants of the head (weights: no earlier kernel of the stream writes them)
-    for (int i = threadIdx.x; i < p.taps * conv_len; i += blockDim.x) {
-        const int j = i / conv_len, c = i % conv_len;
-        const bool is_v = c >= 2 * DP;
-        const int r = is_v ? c0 + c - 2 * DP : c % DP;                       // column within the head
-        const int col = is_v ? p.v_off + h * p.dv + r : (c < DP ? 0 : p.k_off) + kvh * p.dk + r;
-        s_conv[i] = r < (is_v ? p.dv : p.dk) ? p.conv_w[(size_t)j * p.conv_cols + col] : 0.f;
-    }
-    for (int i = threadIdx.x; i < DP; i += blockDim.x) s_bias[i] = i < p.dk ? p.dt_bias[(size_t)h * p.dk + i] : 0.f;
     for (int i = threadIdx.x; i < s.cols; i += blockDim.x) s_norm[i] = c0 + i < p.dv ? p.norm[c0 + i] : 0.f;
-    const float decay_a = p.decay_a[h];
+    if (p.dk < DP || v_cols < s.cols)              // what the copies leave out stays zero
+        for (int i = threadIdx.x; i < 2 * stage_len; i += blockDim.x) smem[i] = 0.f;
+    __syncthreads();
     pdl_enter();
 
     const int begin = p.subsequence_begins[b], len = p.subsequence_begins[b + 1] - begin, past = p.past_lens[b], slot = p.slots[b];
-    const int chunks = (len + s.chunk - 1) / s.chunk;
-    const E* proj = reinterpret_cast<const E*>(p.proj);
-    const int q_col = kvh * p.dk, k_col = p.k_off + kvh * p.dk, v_col = p.v_off + h * p.dv + c0;
-    const int v_cols = max(0, min(s.cols, p.dv - c0));
-    __syncthreads();
+    const int groups = (len + GROUP - 1) / GROUP, stages = (groups + s.groups - 1) / s.groups;
+    const int rec_len = record_floats(p.dk, p.dv);
+    const float* records = p.records + ((size_t)first_group(p.subsequence_begins, b) * p.H + h) * rec_len;
 
-    // raw inputs of stage c, on their way: row r of the buffer is token c * chunk - keep + r of the piece
     auto fetch = [&](int c) {
-        constexpr int EPC = 16 / sizeof(E);        // elements per 16-byte piece
-        E* rows = reinterpret_cast<E*>(raw_buf + (c & 1) * raw_len);
-        float* low = reinterpret_cast<float*>(rows + (s.chunk + keep) * raw_pitch);
-        const int first = c * s.chunk - keep, n = min(s.chunk, len - c * s.chunk);
-        const int nk = p.dk / EPC, per_row = 2 * nk + v_cols / EPC;
-        for (int i = pt; i < (n + keep) * per_row; i += npt) {
-            const int r = i / per_row, x = i % per_row, rel = first + r;
-            const int dst = x < 2 * nk ? x * EPC : 2 * p.dk + (x - 2 * nk) * EPC;
-            const int col = x < nk ? q_col + x * EPC : x < 2 * nk ? k_col + (x - nk) * EPC : v_col + (x - 2 * nk) * EPC;
-            E* d = rows + r * raw_pitch + dst;
-            if (rel >= 0) {
-                copy16(d, proj + (size_t)(begin + rel) * p.ldp + col);
-            } else {                               // before this piece: what earlier steps left, or zeros before position 0
-                const int pos = past + rel;
-                const float* ring = p.conv_ring + ((size_t)slot * p.taps + (pos >= 0 ? pos % p.taps : 0)) * p.conv_cols + col;
-#pragma unroll
-                for (int e = 0; e < EPC; ++e) st_f32(d + e, pos >= 0 ? ring[e] : 0.f);
+        const int n = min(s.groups, groups - c * s.groups), nk = p.dk / 4, nv = v_cols / 4;
+        for (int g = 0; g < n; ++g) {
+            const float* src = records + (size_t)(c * s.groups + g) * p.H * rec_len;
+            float* dst = smem + (c & 1) * stage_len + g * group_len;
+            if (p.dk == DP) {
+                for (int i = pt; i < GROUP_VECTORS * nk; i += npt) copy16(dst + i * 4, src + i * 4);
+            } else {
+                for (int i = pt; i < GROUP_VECTORS * nk; i += npt) copy16(dst + i / nk * DP + i % nk * 4, src + i * 4);
             }
-        }
-        const int nl = p.dk / 4;
-        for (int i = pt; i < n * nl; i += npt)
-            copy16(low + (i / nl) * p.dk + (i % nl) * 4, p.low + (size_t)(begin + c * s.chunk + i / nl) * p.ld_low + (size_t)h * p.dk + (i % nl) * 4);
-    };
-    // stage c from its raw inputs, a warp per token
-    auto stage = [&](int c) {
-        const E* rows = reinterpret_cast<const E*>(raw_buf + (c & 1) * raw_len);
-        const float* low = reinterpret_cast<const float*>(rows + (s.chunk + keep) * raw_pitch);
-        float* st = smem + (c & 1) * stage_len;
-        const int n = min(s.chunk, len - c * s.chunk);
-        for (int tt = pw; tt < n; tt += npw) {
-            const float bl = lane == 0 ? ld_f32(proj + (size_t)(begin + c * s.chunk + tt) * p.ldp + p.b_off + h) : 0.f;
-            const E* in = rows + tt * raw_pitch;
-            float4 q[NV], k[NV];
-            float qq = 0.f, kk = 0.f, qk = 0.f;
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-                const int x = i * 128 + lane * 4;
-                q[i] = k[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (x < p.dk) {
-#pragma unroll 2
-                    for (int j = 0; j < p.taps; ++j) {
-                        q[i] = fma4(ld4_f32(s_conv + j * conv_len + x), ld4_f32(in + j * raw_pitch + x), q[i]);
-                        k[i] = fma4(ld4_f32(s_conv + j * conv_len + DP + x), ld4_f32(in + j * raw_pitch + p.dk + x), k[i]);
-                    }
-                    q[i] = silu4<E>(q[i]);
-                    k[i] = silu4<E>(k[i]);
-                }
-                qq += dot4(q[i], q[i]);
-                kk += dot4(k[i], k[i]);
-                qk += dot4(q[i], k[i]);
-            }
-            const float iq = p.q_scale / sqrtf(delta_sum(qq) + 1e-6f), ik = 1.f / sqrtf(delta_sum(kk) + 1e-6f);
-            qk = delta_sum(qk) * iq * ik;
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-                const int x = i * 128 + lane * 4;
-                if (x < DP) {
-                    const float4 g = x < p.dk ? decay4<E>(decay_a, ld4_f32(low + tt * p.dk + x), ld4_f32(s_bias + x)) : make_float4(1.f, 1.f, 1.f, 1.f);
-                    st4_f32(st + tt * DP + x, scale4(k[i], ik));
-                    st4_f32(st + (s.chunk + tt) * DP + x, scale4(q[i], iq));
-                    st4_f32(st + (2 * s.chunk + tt) * DP + x, g);
-                }
-            }
-            for (int x = lane * 4; x < s.cols; x += 128) {
-                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (x < v_cols) {
-#pragma unroll 4
-                    for (int j = 0; j < p.taps; ++j)
-                        v = fma4(ld4_f32(s_conv + j * conv_len + 2 * DP + x), ld4_f32(in + j * raw_pitch + 2 * p.dk + x), v);
-                    v = silu4<E>(v);
-                }
-                st4_f32(st + 3 * s.chunk * DP + tt * s.cols + x, v);
-            }
-            if (lane == 0) {
-                st[s.chunk * (3 * DP + s.cols) + tt] = Fn<E>::sigmoid(bl);
-                st[s.chunk * (3 * DP + s.cols) + s.chunk + tt] = qk;
-            }
+            src += GROUP_VECTORS * p.dk;
+            dst += GROUP_VECTORS * DP;
+            for (int i = pt; i < GROUP * nv; i += npt) copy16(dst + i / nv * s.cols + i % nv * 4, src + i / nv * p.dv + c0 + i % nv * 4);
+            if (pt < GROUP_SCALARS / 4) copy16(dst + GROUP * s.cols + pt * 4, src + GROUP * p.dv + pt * 4);
         }
     };
-    // norm, gate and store of the read-outs of stage c; columns of the other parts of the cluster are read for the norm only
+    // norm, gate and store of the read-outs of stage c, up to four tokens of a warp side by side; columns of the other parts of the
+    // cluster are read for the norm only
     auto finish = [&](int c) {
-        const int n = min(s.chunk, len - c * s.chunk);
-        const float* ys = y_buf + (c & 1) * s.chunk * s.cols;
-        const float* gate = p.low + (size_t)(begin + c * s.chunk) * p.ld_low + p.gate_off + (size_t)h * p.dv + c0;
-        E* out = reinterpret_cast<E*>(p.out) + (size_t)(begin + c * s.chunk) * p.ldo + (size_t)h * p.o_head + c0;
-        const int x = lane * 4;
-        float4 g = pw < n && x < v_cols ? ld4_f32(gate + (size_t)pw * p.ld_low + x) : make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int tt = pw; tt < n; tt += npw) {
-            const float4 g_now = g;
-            if (tt + npw < n && x < v_cols) g = ld4_f32(gate + (size_t)(tt + npw) * p.ld_low + x);        // (the next token's, ahead of its use)
-            float ss = 0.f;
-            for (int col = x; col < s.parts * s.cols; col += 128) {
-                const int from = col / s.cols;
-                const float* row = ys + tt * s.cols + (col - from * s.cols);
-                const float4 y = ld4_f32(from == part ? row : cluster.map_shared_rank(row, from));
-                ss += dot4(y, y);
+        constexpr int SIDE = 4;
+        const int n = min(tokens, len - c * tokens), x = lane * 4;
+        const float* ys = y_buf + (c & 1) * tokens * s.cols;
+        const float* gate = p.low + (size_t)(begin + c * tokens) * p.ld_low + p.gate_off + (size_t)h * p.dv + c0;
+        E* out = reinterpret_cast<E*>(p.out) + (size_t)(begin + c * tokens) * p.ldo + (size_t)h * p.o_head + c0;
+        for (int first = pw; first < n; first += SIDE * npw) {
+            float4 g[SIDE];
+            float ss[SIDE];
+#pragma unroll
+            for (int i = 0; i < SIDE; ++i) {
+                const int tt = first + i * npw;
+                g[i] = tt < n && x < v_cols ? ld4_f32(gate + (size_t)tt * p.ld_low + x) : make_float4(0.f, 0.f, 0.f, 0.f);
+                ss[i] = 0.f;
             }
-            const float inv = 1.f / sqrtf(delta_sum(ss) / (float)p.Dv + p.eps);
-            for (int col = x; col < v_cols; col += 128) {
-                const float4 gv = col == x ? g_now : ld4_f32(gate + (size_t)tt * p.ld_low + col);
-                st4_f32(out + (size_t)tt * p.ldo + col, mul4(scale4(mul4(ld4_f32(ys + tt * s.cols + col), ld4_f32(s_norm + col)), inv), sigmoid4<E>(gv)));
+            for (int col = x; col < s.parts * s.cols; col += 128) {
+                const int from = s.parts > 1 ? col / s.cols : 0;
+                const float* rows = ys + (col - from * s.cols);
+                if (from != part) rows = cluster.map_shared_rank(rows, from);
+#pragma unroll
+                for (int i = 0; i < SIDE; ++i) {
+                    const int tt = first + i * npw;
+                    if (tt < n) {
+                        const float4 y = ld4_f32(rows + tt * s.cols);
+                        ss[i] += dot4(y, y);
+                    }
+                }
+            }
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1)
+#pragma unroll
+                for (int i = 0; i < SIDE; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], d);
+#pragma unroll
+            for (int i = 0; i < SIDE; ++i) {
+                const int tt = first + i * npw;
+                if (tt >= n) break;
+                const float inv = 1.f / sqrtf(ss[i] / (float)p.Dv + p.eps);
+                for (int col = x; col < v_cols; col += 128) {
+                    const float4 gv = col == x ? g[i] : ld4_f32(gate + (size_t)tt * p.ld_low + col);
+                    st4_f32(out + (size_t)tt * p.ldo + col, mul4(scale4(mul4(ld4_f32(ys + tt * s.cols + col), ld4_f32(s_norm + col)), inv), sigmoid4<E>(gv)));
+                }
             }
         }
     };
-    auto producers_meet = [&]() { asm volatile("bar.sync 1, %0;" ::"r"(npt) : "memory"); };
 
-    // rows 16 j + 4 rg + e, columns cc .. cc + CPT - 1 of this CTA; two rows packed
-    const int rg = lane >> 3, cc = warp * 8 * CPT + (lane & 7) * CPT;
+    // rows (j * RGS + rg) * 4 + e, columns cc .. cc + CPT - 1 of this CTA; two rows packed
+    const int rg = lane / LANES, cc = warp * WARP_COLS + lane % LANES * CPT;
     f32x2 S[RL / 2][CPT];
     float* state = p.state + ((size_t)slot * p.H + h) * p.dk * p.dv + c0 + cc;
-    const bool mine = consumer && c0 + cc < p.dv;      // (dv is a multiple of 16: whole column groups)
+    const bool mine = consumer && c0 + cc < p.dv;      // (dv is a multiple of 16: whole pieces of CPT columns)
+    auto row_of = [&](int i) { return ((i >> 1) * RGS + rg) * 4 + (i & 1) * 2; };
     if (consumer) {
         const bool load = mine && past > 0;
 #pragma unroll
         for (int i = 0; i < RL / 2; ++i) {
-            const int r = (i >> 1) * 16 + rg * 4 + (i & 1) * 2;
+            const int r = row_of(i);
             float lo[CPT], hi[CPT];
 #pragma unroll
             for (int c = 0; c < CPT; ++c) lo[c] = hi[c] = 0.f;
             if (load && r < p.dk) {
                 if constexpr (CPT == 2) {
-                    const float2 a = *reinterpret_cast<const float2*>(state + (size_t)r * p.dv), d = *reinterpret_cast<const float2*>(state + (size_t)(r + 1) * p.dv);
-                    lo[0] = a.x; lo[1] = a.y; hi[0] = d.x; hi[1] = d.y;
+                    const float2 x = *reinterpret_cast<const float2*>(state + (size_t)r * p.dv), y = *reinterpret_cast<const float2*>(state + (size_t)(r + 1) * p.dv);
+                    lo[0] = x.x; lo[1] = x.y; hi[0] = y.x; hi[1] = y.y;
                 } else {
                     lo[0] = state[(size_t)r * p.dv];
                     hi[0] = state[(size_t)(r + 1) * p.dv];
@@ -299,78 +373,105 @@ __global__ void __launch_bounds__(max_warps(RL) * 32, 1) channel_delta_kernel(ov
     } else {
         fetch(0);
         copy_commit();
-        if (chunks > 1) fetch(1);
-        copy_commit();
-        copy_wait<1>();
-        producers_meet();
-        stage(0);
+        copy_wait<0>();
     }
     barrier();
-    for (int c = 0; c < chunks; ++c) {
+    for (int c = 0; c < stages; ++c) {
         if (consumer) {
-            const float* st = smem + (c & 1) * stage_len;
-            const float* sk = st + rg * 4;
-            const float* sq = sk + s.chunk * DP;
-            const float* sg = sq + s.chunk * DP;
-            const float* sv = st + 3 * s.chunk * DP + cc;
-            const float* sb = st + s.chunk * (3 * DP + s.cols);
-            float* ys = y_buf + (c & 1) * s.chunk * s.cols + cc;
-            const int n = min(s.chunk, len - c * s.chunk);
-            for (int tt = 0; tt < n; ++tt) {
-                f32x2 m2[CPT][2], o2[CPT][2], k2[RL / 2];
+            const int n = min(s.groups, groups - c * s.groups);
+            for (int gi = 0; gi < n; ++gi) {
+                const float* st = smem + (c & 1) * stage_len + gi * group_len;
+                const float* vec = st + rg * 4;                                   // + vector * DP + j * 4 RGS
+                const float* sv = st + GROUP_VECTORS * DP + cc;
+                const float* sc = st + GROUP_VECTORS * DP + GROUP * s.cols;
+                f32x2 m2[GROUP][CPT], o2[GROUP][CPT];
 #pragma unroll
-                for (int x = 0; x < CPT; ++x) m2[x][0] = m2[x][1] = o2[x][0] = o2[x][1] = 0ull;
+                for (int t = 0; t < GROUP; ++t)
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) m2[t][x] = o2[t][x] = 0ull;
 #pragma unroll
                 for (int j = 0; j < RL / 4; ++j) {
-                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(sk + tt * DP + j * 16);
-                    const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(sq + tt * DP + j * 16);
-                    const ulonglong2 gg = *reinterpret_cast<const ulonglong2*>(sg + tt * DP + j * 16);
-                    k2[2 * j] = kk.x;
-                    k2[2 * j + 1] = kk.y;
+#pragma unroll
+                    for (int t = 0; t < GROUP; ++t) {
+                        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(vec + t * DP + j * 4 * RGS);
+                        const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(vec + (GROUP + t) * DP + j * 4 * RGS);
+#pragma unroll
+                        for (int x = 0; x < CPT; ++x) {
+                            m2[t][x] = fma2(S[2 * j][x], kk.x, m2[t][x]);
+                            m2[t][x] = fma2(S[2 * j + 1][x], kk.y, m2[t][x]);
+                            o2[t][x] = fma2(S[2 * j][x], qq.x, o2[t][x]);
+                            o2[t][x] = fma2(S[2 * j + 1][x], qq.y, o2[t][x]);
+                        }
+                    }
+                }
+                float co[GROUP_SCALARS], u[GROUP][CPT], o[GROUP][CPT];
+#pragma unroll
+                for (int i = 0; i < GROUP_SCALARS; i += 4) {
+                    const float4 f = ld4_f32(sc + i);
+                    co[i] = f.x; co[i + 1] = f.y; co[i + 2] = f.z; co[i + 3] = f.w;
+                }
+#pragma unroll
+                for (int t = 0; t < GROUP; ++t) {
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) {
+                        const float2 ms = unpack2(m2[t][x]), os = unpack2(o2[t][x]);
+                        float m = ms.x + ms.y;
+                        o[t][x] = os.x + os.y;
+#pragma unroll
+                        for (int d = LANES; d < 32; d *= 2) {
+                            m += __shfl_xor_sync(0xffffffffu, m, d);
+                            o[t][x] += __shfl_xor_sync(0xffffffffu, o[t][x], d);
+                        }
+                        u[t][x] = sv[t * s.cols + x] - m;
+                    }
+                }
+                float* ys = y_buf + (c & 1) * tokens * s.cols + gi * GROUP * s.cols + cc;
+#pragma unroll
+                for (int t = 0; t < GROUP; ++t) {
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) {
+#pragma unroll
+                        for (int r = 0; r < t; ++r) {
+                            u[t][x] = fmaf(-co[t * (t - 1) / 2 + r], u[r][x], u[t][x]);
+                            o[t][x] = fmaf(co[6 + t * (t + 1) / 2 + r], u[r][x], o[t][x]);
+                        }
+                        u[t][x] *= co[16 + t];
+                        o[t][x] = fmaf(co[6 + t * (t + 1) / 2 + t], u[t][x], o[t][x]);
+                    }
+                    if (rg == 0) {
+                        if constexpr (CPT == 2) *reinterpret_cast<float2*>(ys + t * s.cols) = make_float2(o[t][0], o[t][1]);
+                        else ys[t * s.cols] = o[t][0];
+                    }
+                }
+                f32x2 uu[GROUP][CPT];
+#pragma unroll
+                for (int t = 0; t < GROUP; ++t)
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) uu[t][x] = pack2(u[t][x], u[t][x]);
+#pragma unroll
+                for (int j = 0; j < RL / 4; ++j) {
+                    const ulonglong2 gg = *reinterpret_cast<const ulonglong2*>(vec + 3 * GROUP * DP + j * 4 * RGS);
 #pragma unroll
                     for (int x = 0; x < CPT; ++x) {
                         S[2 * j][x] = mul2(S[2 * j][x], gg.x);
                         S[2 * j + 1][x] = mul2(S[2 * j + 1][x], gg.y);
-                        m2[x][0] = fma2(S[2 * j][x], kk.x, m2[x][0]);
-                        m2[x][1] = fma2(S[2 * j + 1][x], kk.y, m2[x][1]);
-                        o2[x][0] = fma2(S[2 * j][x], qq.x, o2[x][0]);
-                        o2[x][1] = fma2(S[2 * j + 1][x], qq.y, o2[x][1]);
                     }
-                }
-                const float beta = sb[tt], kq = sb[s.chunk + tt];
-                float u[CPT], o[CPT];
 #pragma unroll
-                for (int x = 0; x < CPT; ++x) {
-                    const float2 ms = unpack2(add2(m2[x][0], m2[x][1])), os = unpack2(add2(o2[x][0], o2[x][1]));
-                    float m = ms.x + ms.y;
-                    o[x] = os.x + os.y;
-                    m += __shfl_xor_sync(0xffffffffu, m, 8);
-                    o[x] += __shfl_xor_sync(0xffffffffu, o[x], 8);
-                    m += __shfl_xor_sync(0xffffffffu, m, 16);
-                    o[x] += __shfl_xor_sync(0xffffffffu, o[x], 16);
-                    u[x] = beta * (sv[tt * s.cols + x] - m);
-                    o[x] = fmaf(kq, u[x], o[x]);
-                }
+                    for (int t = 0; t < GROUP; ++t) {
+                        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(vec + (2 * GROUP + t) * DP + j * 4 * RGS);
 #pragma unroll
-                for (int x = 0; x < CPT; ++x) {
-                    const f32x2 uu = pack2(u[x], u[x]);
-#pragma unroll
-                    for (int i = 0; i < RL / 2; ++i) S[i][x] = fma2(k2[i], uu, S[i][x]);
-                }
-                if (rg == 0) {
-                    if constexpr (CPT == 2) *reinterpret_cast<float2*>(ys + tt * s.cols) = make_float2(o[0], o[1]);
-                    else ys[tt * s.cols] = o[0];
+                        for (int x = 0; x < CPT; ++x) {
+                            S[2 * j][x] = fma2(kk.x, uu[t][x], S[2 * j][x]);
+                            S[2 * j + 1][x] = fma2(kk.y, uu[t][x], S[2 * j + 1][x]);
+                        }
+                    }
                 }
             }
         } else {
-            if (c + 2 < chunks) fetch(c + 2);      // (into the buffer of stage c, which is finished)
+            if (c + 1 < stages) fetch(c + 1);
             copy_commit();
-            if (c + 1 < chunks) {
-                copy_wait<1>();
-                producers_meet();
-                stage(c + 1);
-            }
             if (c > 0) finish(c - 1);
+            copy_wait<0>();
         }
         barrier();
     }
@@ -378,22 +479,22 @@ __global__ void __launch_bounds__(max_warps(RL) * 32, 1) channel_delta_kernel(ov
         if (mine) {
 #pragma unroll
             for (int i = 0; i < RL / 2; ++i) {
-                const int r = (i >> 1) * 16 + rg * 4 + (i & 1) * 2;
+                const int r = row_of(i);
                 if (r < p.dk) {
                     if constexpr (CPT == 2) {
-                        const float2 a = unpack2(S[i][0]), d = unpack2(S[i][1]);
-                        *reinterpret_cast<float2*>(state + (size_t)r * p.dv) = make_float2(a.x, d.x);
-                        *reinterpret_cast<float2*>(state + (size_t)(r + 1) * p.dv) = make_float2(a.y, d.y);
+                        const float2 x = unpack2(S[i][0]), y = unpack2(S[i][1]);
+                        *reinterpret_cast<float2*>(state + (size_t)r * p.dv) = make_float2(x.x, y.x);
+                        *reinterpret_cast<float2*>(state + (size_t)(r + 1) * p.dv) = make_float2(x.y, y.y);
                     } else {
-                        const float2 a = unpack2(S[i][0]);
-                        state[(size_t)r * p.dv] = a.x;
-                        state[(size_t)(r + 1) * p.dv] = a.y;
+                        const float2 x = unpack2(S[i][0]);
+                        state[(size_t)r * p.dv] = x.x;
+                        state[(size_t)(r + 1) * p.dv] = x.y;
                     }
                 }
             }
         }
     } else {
-        finish(chunks - 1);
+        finish(stages - 1);
     }
     if (s.parts > 1) cluster.sync();       // the other parts may still read this CTA's read-outs
 }
@@ -564,31 +665,37 @@ int launch_channel_delta_step(const ovb_delta_args& a, cudaStream_t stream) {
     return ERR_UNSUPPORTED;
 }
 
-template <class E, int RL, int CPT>
-int launch_channel_delta(const ovb_delta_args& a, cudaStream_t stream) {
+template <class E, int NV>
+int launch_prepare(const ovb_delta_args& a, cudaStream_t stream) {
+    auto kern = a.taps == 1   ? delta_prepare_kernel<E, NV, 1>
+                : a.taps == 2 ? delta_prepare_kernel<E, NV, 2>
+                : a.taps == 3 ? delta_prepare_kernel<E, NV, 3>
+                : a.taps == 4 ? delta_prepare_kernel<E, NV, 4>
+                              : delta_prepare_kernel<E, NV, 0>;
+    OVB_CHECK_CUDA(launch_pdl(kern, dim3(a.T / GROUP + a.B, ceil_div(a.H, 4)), dim3(128), 0, stream, a));
+    return 0;
+}
+
+template <class E, int RGS, int RL, int CPT>
+int launch_scan(const ovb_delta_args& a, int parts, cudaStream_t stream) {
+    constexpr int DP = RGS * RL, MAX_WARPS = scan_warps(RL * CPT);
+    const int unit = 32 / RGS * CPT, units = ceil_div(a.dv, unit);       // columns of a warp
+    while (parts < 8 && ceil_div(units, parts) > MAX_WARPS - 2) parts *= 2;
     DeltaShape s;
-    const int unit = 8 * CPT, groups = ceil_div(a.dv, unit);       // column groups of a warp each
-    // one CTA per (sequence, head) when those fill the machine, else up to eight that share the columns
-    s.parts = 1;
-    while (s.parts < 8 && a.B * a.H * s.parts * 2 <= 148 && ceil_div(groups, s.parts * 2) * unit * (s.parts * 2 - 1) < a.dv) s.parts *= 2;
-    while (ceil_div(groups, s.parts) > 8) s.parts *= 2;
-    s.consumers = ceil_div(groups, s.parts);
-    s.cols = s.consumers * unit;
-    if (s.parts > 8) {
+    s.parts = parts;
+    s.consumers = ceil_div(units, parts);
+    if (s.consumers > MAX_WARPS - 2) {
         set_error("ovb_channel_delta: value size %d is too large", a.dv);
         return ERR_UNSUPPORTED;
     }
-    const int dp = RL * 4;
-    auto bytes = [&]() {
-        return 4 * ((size_t)2 * stage_floats(dp, s.cols, s.chunk) + 2 * s.chunk * s.cols + a.taps * (2 * dp + s.cols) + dp + s.cols) +
-               2 * (size_t)raw_bytes(a.dk, s.cols, s.chunk, a.taps, sizeof(E));
-    };
-    s.chunk = a.max_q_len == 1 ? 1 : 16;
-    while (s.chunk > 1 && bytes() > 227 * 1024) s.chunk /= 2;
+    s.cols = s.consumers * unit;
+    auto bytes = [&]() { return 4 * ((size_t)2 * s.groups * (staged_floats(DP, s.cols) + GROUP * s.cols) + s.cols); };
+    s.groups = 4;
+    while (s.groups > 1 && (bytes() > 227 * 1024 || s.groups * GROUP >= 2 * a.max_q_len)) s.groups /= 2;
     const size_t smem = bytes();
-    OVB_REQUIRE(smem <= 227 * 1024, "ovb_channel_delta: %d taps need too much shared memory", a.taps);
-    const int producers = a.max_q_len == 1 ? 2 : max_warps(RL) - s.consumers < 8 ? max_warps(RL) - s.consumers : 8;
-    auto kern = channel_delta_kernel<E, RL, CPT>;
+    OVB_REQUIRE(smem <= 227 * 1024, "ovb_channel_delta: heads of %d x %d need too much shared memory", a.dk, a.dv);
+    const int producers = MAX_WARPS - s.consumers < 4 ? MAX_WARPS - s.consumers : 4;
+    auto kern = delta_scan_kernel<E, RGS, RL, CPT>;
     static std::atomic<uint64_t> configured{0};
     int dev = 0;
     OVB_CHECK_CUDA(cudaGetDevice(&dev));
@@ -619,12 +726,32 @@ int launch_channel_delta(const ovb_delta_args& a, cudaStream_t stream) {
     cfg.attrs = attr;
     cfg.numAttrs = n;
     OVB_CHECK_CUDA(cudaLaunchKernelEx(&cfg, kern, a, s));
+    return 0;
+}
+
+template <class E>
+int launch_channel_delta(const ovb_delta_args& a, cudaStream_t stream) {
+    OVB_REQUIRE(a.records && (reinterpret_cast<uintptr_t>(a.records) & 15) == 0, "ovb_channel_delta: no room for the groups' records");
+    if (int rc = a.dk <= 128 ? launch_prepare<E, 1>(a, stream) : launch_prepare<E, 2>(a, stream)) return rc;
+    // one CTA per (sequence, head) when those fill the machine, else up to eight that share the columns
+    int parts = 1;
+    while (parts < 8 && a.B * a.H * parts * 2 <= 148 && a.dv >= 16 * parts * 2) parts *= 2;
+    int rc;
+    if (a.dk <= 32) rc = launch_scan<E, 4, 8, 2>(a, parts, stream);
+    else if (a.dk <= 64) rc = parts > 1 ? launch_scan<E, 8, 8, 2>(a, parts, stream) : launch_scan<E, 4, 16, 2>(a, parts, stream);
+    else if (a.dk <= 128) rc = parts > 1 ? launch_scan<E, 8, 16, 2>(a, parts, stream) : launch_scan<E, 4, 32, 2>(a, parts, stream);
+    else rc = launch_scan<E, 8, 32, 2>(a, parts, stream);
+    if (rc) return rc;
     return update_conv_ring<E>(a.proj, a.ldp, {a.conv_w, a.conv_ring, a.taps, a.conv_cols}, a.subsequence_begins, a.past_lens, a.slots, a.B, stream);
 }
 
 }  // namespace
 
 }  // namespace ovb
+
+extern "C" int64_t ovb_channel_delta_record_floats(int T, int B, int H, int dk, int dv) {
+    return (int64_t)(T / ovb::GROUP + B) * H * ovb::record_floats(dk, dv);
+}
 
 extern "C" int ovb_channel_delta(const ovb_delta_args* a, ovb_stream_t stream_) {
     using namespace ovb;
@@ -643,11 +770,10 @@ extern "C" int ovb_channel_delta(const ovb_delta_args* a, ovb_stream_t stream_) 
         using E = decltype(e);
         const int rc = launch_channel_delta_step<E>(*a, stream);
         if (rc != ERR_UNSUPPORTED) return rc;
-        if (a->dk <= 32) return launch_channel_delta<E, 8, 2>(*a, stream);
-        if (a->dk <= 64) return launch_channel_delta<E, 16, 2>(*a, stream);
-        if (a->dk <= 128) return launch_channel_delta<E, 32, 2>(*a, stream);
-        if (a->dk <= 256) return launch_channel_delta<E, 64, 1>(*a, stream);
-        set_error("ovb_channel_delta: key size %d above 256", a->dk);
-        return ERR_UNSUPPORTED;
+        if (a->dk > 256) {
+            set_error("ovb_channel_delta: key size %d above 256", a->dk);
+            return ERR_UNSUPPORTED;
+        }
+        return launch_channel_delta<E>(*a, stream);
     });
 }

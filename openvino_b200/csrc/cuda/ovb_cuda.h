@@ -485,9 +485,11 @@ typedef struct {
     const int* subsequence_begins;
     const int* past_lens;
     const int* slots;
+    float* records;          // scratch of ovb_channel_delta_record_floats(T, B, H, dk, dv) floats
     int B, T, H, G, D, Dv, dk, dv, ldp, k_off, v_off, b_off, ld_low, gate_off, conv_cols, taps, ldo, o_head, max_q_len, dtype;
     float q_scale, eps;
 } ovb_delta_args;
+int64_t ovb_channel_delta_record_floats(int T, int B, int H, int dk, int dv);
 int ovb_channel_delta(const ovb_delta_args* a, ovb_stream_t stream);
 
 #ifdef __cplusplus

@@ -82,7 +82,7 @@ class WindowAttnArgs(C.Structure):
 
 
 class DeltaArgs(C.Structure):
-    _fields_ = _fields(("proj", "low", "conv_w", "conv_ring", "decay_a", "dt_bias", "norm", "state", "out", "subsequence_begins", "past_lens", "slots"),
+    _fields_ = _fields(("proj", "low", "conv_w", "conv_ring", "decay_a", "dt_bias", "norm", "state", "out", "subsequence_begins", "past_lens", "slots", "records"),
                        ("B", "T", "H", "G", "D", "Dv", "dk", "dv", "ldp", "k_off", "v_off", "b_off", "ld_low", "gate_off", "conv_cols", "taps", "ldo", "o_head",
                         "max_q_len", "dtype"), ("q_scale", "eps"))
 
@@ -130,6 +130,7 @@ def lib():
         l.ovb_status_ptr.restype = C.c_void_p
         l.ovb_gemm_ws_bytes.restype = C.c_int64
         l.ovb_pa_scratch_bytes.restype = C.c_int64
+        l.ovb_channel_delta_record_floats.restype = C.c_int64
         l.ovb_gemm.argtypes = [C.POINTER(GemmArgs), C.c_void_p]
         l.ovb_paged_attention.argtypes = [C.POINTER(PaArgs), C.c_void_p]
         l.ovb_status_read.argtypes = [C.c_void_p]
@@ -417,6 +418,11 @@ def rope_table(positions, inv_freq, out, mult=1.0) -> None:
     """out[t, i] = (cos, sin)(positions[t] * inv_freq[i]) * mult; out: fp32 [T, 2 * half]."""
     _check(lib().ovb_rope_table(C.c_void_p(positions.data_ptr()), C.c_void_p(inv_freq.data_ptr()), C.c_void_p(out.data_ptr()), C.c_int(out.shape[0]),
                                 C.c_int(inv_freq.numel()), C.c_float(mult), C.c_void_p(_stream())), "ovb_rope_table")
+
+
+def channel_delta_record_floats(T: int, B: int, H: int, dk: int, dv: int) -> int:
+    """fp32 scratch that ``channel_delta`` needs for a step of T tokens in B sequences."""
+    return int(lib().ovb_channel_delta_record_floats(C.c_int(T), C.c_int(B), C.c_int(H), C.c_int(dk), C.c_int(dv)))
 
 
 def channel_delta(**kw) -> None:

@@ -335,7 +335,9 @@ class ChannelDeltaMixer:
         K.gemm(x, self.proj, out=proj, ws=ex.ws)
         low = sb.scratch("delta_low", T, 2 * self.low_n, torch.float32)
         K.gemm_block_diag(proj[:, self.low_off:], self.low, low, self.rank, self.low_n, ws=ex.ws)
-        K.channel_delta(proj=proj, low=low, decay_a=self.decay_a, dt_bias=self.dt_bias, norm=self.norm, state=self.delta_state, out=out, T=T, H=s.heads,
+        # (what the kernel prepares for all groups of tokens at once; the largest step decides the size)
+        records = sb.scratch("delta_records", 1, K.channel_delta_record_floats(sb.Tcap, sb.Bcap, s.heads, self.dk, self.dv), torch.float32, cap=1)
+        K.channel_delta(proj=proj, low=low, records=records, decay_a=self.decay_a, dt_bias=self.dt_bias, norm=self.norm, state=self.delta_state, out=out, T=T, H=s.heads,
                         G=s.kv_heads, D=s.dim, Dv=s.vdim, dk=self.dk, dv=self.dv, ldp=proj.stride(0), k_off=self.k_off, v_off=self.v_off, b_off=self.b_off,
                         ld_low=low.stride(0), gate_off=self.low_n, ldo=out.stride(0), o_head=self.dv, dtype=ex.storage, q_scale=s.dim ** -0.5,
                         eps=ex.cfg.norm_eps, **self.conv.args(sb, shp))

@@ -258,6 +258,7 @@ def test_channel_delta_in_portions(dtype, H, G, D, Dv, taps):
     const = dict(conv_w=filt, conv_ring=ring, conv_cols=filt.shape[1], taps=taps, decay_a=a_log.exp().cuda(), state=state,
                  dt_bias=torch.nn.functional.pad(dt.reshape(H, D), (0, dk - D)).contiguous().cuda(), norm=torch.nn.functional.pad(norm, (0, dv - Dv)).cuda())
     got, b_off = [[] for _ in LENS], filt.shape[1]
+    const["records"] = torch.full((K.channel_delta_record_floats(sum(LENS), len(LENS), H, dk, dv),), float("nan"), device="cuda")
     for batch, begins, args in Portions():
         T = args["T"]
         cat = lambda f: torch.cat([f(b, slice(s, s + m)) for b, s, m in batch])
@@ -287,9 +288,10 @@ def test_decay_is_per_channel_and_exact_over_many_tokens():
     low[:, D:] = 30.0
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
     out, silu = torch.zeros(L, D, device="cuda"), lambda z: oracle.silu(torch.tensor(z, dtype=torch.float64))
+    records = torch.empty(K.channel_delta_record_floats(L, 1, 1, D, D), device="cuda")
     K.channel_delta(proj=proj.cuda(), low=low.cuda(), conv_w=torch.ones(1, 3 * D, device="cuda"), conv_ring=torch.zeros(1, 1, 3 * D, device="cuda"),
                     decay_a=torch.ones(1, device="cuda"), dt_bias=torch.zeros(1, D, device="cuda"), norm=torch.ones(D, device="cuda"),
-                    state=torch.zeros(1, 1, D, D, device="cuda"), out=out, subsequence_begins=i32([0, L]), past_lens=i32([0]), slots=i32([0]), B=1, T=L, H=1, G=1, D=D,
+                    state=torch.zeros(1, 1, D, D, device="cuda"), out=out, records=records, subsequence_begins=i32([0, L]), past_lens=i32([0]), slots=i32([0]), B=1, T=L, H=1, G=1, D=D,
                     Dv=D, dk=D, dv=D, ldp=proj.stride(0), k_off=D, v_off=2 * D, b_off=3 * D, ld_low=2 * D, gate_off=D, conv_cols=3 * D, taps=1, ldo=D, o_head=D,
                     max_q_len=L, dtype=K.DT_F32, q_scale=1.0, eps=1.0)
     dt = torch.nn.functional.softplus(torch.tensor([-6.0, -8.0], dtype=torch.float64))
