@@ -144,7 +144,7 @@ constexpr int HEADS_STRIP = 16, HEADS_BATCH = 4;      // tokens per warp of a pr
 // The same for heads of up to 128 columns in pieces of four: a warp walks a strip of tokens of one head with its columns in registers
 // (lane l: columns 4 l ..), so that every projected value is fetched once; rotation partners sit in other lanes. TAPS 0: no convolution.
 template <class E, int TAPS>
-__global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int strip) {
+__global__ void __launch_bounds__(128, sizeof(E) == 2 ? 7 : 4) heads_strip_kernel(ovb_heads_args p, int strip) {
     pdl_enter();
     __shared__ int s_b;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -163,7 +163,6 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
         for (int j = 0; j < TAPS; ++j) w[j] = live ? ld4_f32(p.conv_w + (size_t)j * p.conv_cols + u.col + c) : zero;
     }
     const float* nw = u.is_q ? p.q_norm : u.is_k ? p.k_norm : nullptr;
-    const float4 gain = nw && live ? make_float4(nw[c], nw[c + 1], nw[c + 2], nw[c + 3]) : zero;
     // the partner of column c is c + half (in the lower half) or c - half
     const int half = is_v ? 0 : p.rot_dims / 2;
     const bool lower = c < half, turned = c < 2 * half;
@@ -176,13 +175,20 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
         b = s_b;
         next = p.subsequence_begins[b + 1];
     }
+    Raw4<E> ahead[HEADS_BATCH];
+    auto request = [&](int tb) {
+#pragma unroll
+        for (int k = 0; k < HEADS_BATCH; ++k) {
+            ahead[k].set(zero);
+            if (live && tb + k < t_end) ahead[k].load(src + (size_t)(tb + k) * p.ldp);
+        }
+    };
+    request(t0);
     for (int tb = t0; tb < t_end; tb += HEADS_BATCH) {
         Raw4<E> raw[HEADS_BATCH];
 #pragma unroll
-        for (int k = 0; k < HEADS_BATCH; ++k) {
-            raw[k].set(zero);
-            if (live && tb + k < t_end) raw[k].load(src + (size_t)(tb + k) * p.ldp);
-        }
+        for (int k = 0; k < HEADS_BATCH; ++k) raw[k] = ahead[k];
+        request(tb + HEADS_BATCH);
 #pragma unroll
         for (int k = 0; k < HEADS_BATCH; ++k) {
             const int t = tb + k;
@@ -208,7 +214,7 @@ __global__ void __launch_bounds__(128) heads_strip_kernel(ovb_heads_args p, int 
             }
             if (nw) {
                 const float inv = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)p.D + p.eps);
-                v = make_float4(v.x * inv * gain.x, v.y * inv * gain.y, v.z * inv * gain.z, v.w * inv * gain.w);
+                if (live) v = make_float4(v.x * inv * __ldg(nw + c), v.y * inv * __ldg(nw + c + 1), v.z * inv * __ldg(nw + c + 2), v.w * inv * __ldg(nw + c + 3));
             }
             if (half > 0) {
                 const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, partner), __shfl_sync(0xffffffffu, v.y, partner), __shfl_sync(0xffffffffu, v.z, partner),
