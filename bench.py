@@ -93,8 +93,8 @@ def parse():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch"])
     ap.add_argument("--model", default="llama-3-8b",
                     help="llama-3-8b (headline) | llama-3-70b | mixtral-8x7b | tiny-llama | tiny-moe (serving); bert-large | resnet18 (graph API); busatar (layered decoder beside a Llama of equal size), sapasun (beside Busatar)")
-    ap.add_argument("--kernels", action="store_true", help="busatar: also time every kernel call of a step with its roofline fraction")
-    ap.add_argument("--sizes", default="", help="busatar: sizes to run, with commas between them (default: all of ops/bench_layers.py)")
+    ap.add_argument("--kernels", action="store_true", help="busatar, sapasun: also time every kernel call of a step with its roofline fraction")
+    ap.add_argument("--sizes", default="", help="busatar, sapasun: sizes to run, with commas between them (default: all of ops/bench_layers.py)")
     ap.add_argument("--requests", type=int, default=0, help="concurrent requests (default: the benchmark's number for the model)")
     ap.add_argument("--prompt-len", type=int, default=0)
     ap.add_argument("--output-len", type=int, default=0)
